@@ -235,8 +235,27 @@ def _load_ffn(lw: LayerWeights, view: NameView, cfg: ModelConfig, prefix: str, q
         lw.gate_up, lw.down = mlp(prefix + ".mlp", cfg.ffn)
 
 
+def load_listed(st: SafetensorsSet, cfg: ModelConfig, device, dtype: str = "bfloat16") -> ModelWeights:
+    """A model that lists its layers: unquantised tensors under the design's own names, checked against the
+    configuration before anything is assembled; ``dtype`` float32 keeps everything in 32-bit."""
+    from ..models.latent import assemble, tensor_shapes
+    bad = []
+    for name, shape in tensor_shapes(cfg).items():
+        if not st.has(name):
+            bad.append(f"{name}: missing")
+        elif tuple(st.shape(name)) != shape:
+            bad.append(f"{name}: shape {st.shape(name)}, expected {list(shape)}")
+        elif st.dtype(name) not in ("BF16", "F16", "F32"):
+            bad.append(f"{name}: element type {st.dtype(name)}")
+    if bad:
+        raise ValueError(f"{st.dir}: the tensors do not fit config.json:\n  " + "\n  ".join(bad))
+    return assemble(cfg, lambda name: st.get(name, copy=torch.device(device).type == "cpu"), device,
+                    torch.float32 if dtype == "float32" else torch.bfloat16)
+
+
 def load(snapshot: str, device="cuda", mtp: bool = True, int8_head: bool = False, tp: Tuple[int, int] = (0, 1),
-         report=sys.stderr) -> ModelWeights:
+         report=sys.stderr, dtype: str = "bfloat16") -> ModelWeights:
+    """``dtype``: "bfloat16", or "float32" for families that are served in 32-bit."""
     t0 = time.time()
     snap = resolve_snapshot(snapshot)
     with open(os.path.join(snap, "config.json")) as f:
@@ -244,6 +263,15 @@ def load(snapshot: str, device="cuda", mtp: bool = True, int8_head: bool = False
     if "text_config" in hf:
         hf = {**hf["text_config"], "quantization_config": hf.get("quantization_config", hf["text_config"].get("quantization_config"))}
     cfg = ModelConfig.from_hf_config(hf)
+    if cfg.layer_specs:
+        if tp[1] != 1 or int8_head:
+            raise ValueError(f"{cfg.name}: models that list their layers run on one GPU with an unquantised head")
+        w = load_listed(SafetensorsSet(snap), cfg, device, dtype)
+        if report is not None:
+            report.write(f"load: {cfg.name} {dtype} from {snap}: {w.nbytes() / 1e9:.3f} GB resident, {time.time() - t0:.1f} s\n")
+        return w
+    if dtype != "bfloat16":
+        raise ValueError(f"{cfg.name}: this family is served in bfloat16 only")
     qc = QuantConfig.parse(hf)
     st = SafetensorsSet(snap)
     view = NameView(st, copy=torch.device(device).type == "cpu")

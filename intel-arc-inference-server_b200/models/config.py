@@ -22,6 +22,48 @@ class LinearDesc:
 
 
 @dataclass(frozen=True)
+class LatentAttention:
+    """Attention whose queries and keys / values go through low-rank latents; the cache holds the key-value latent and
+    one rotated key part shared by the heads."""
+    heads: int
+    dim: int                      # unrotated query / key dimensions of a head
+    rot_dim: int                  # rotated query / key dimensions of a head
+    vdim: int                     # value dimensions of a head
+    kv_rank: int
+    q_rank: int
+    scale: float
+    rope_dims: int                # rotated leading dimensions of the rot_dim part
+    rope_base: float
+    window: int = 0               # a position sees itself and the window - 1 positions before it (0: all)
+
+
+@dataclass(frozen=True)
+class ExpertFfn:
+    """Routed SwiGLU experts.  ``score``: "softmax" over all experts or a "sigmoid" each; with ``groups`` > 1 only
+    experts of the ``keep`` groups with the largest sums of their two best scores can be chosen; ``renorm``: the chosen
+    scores are divided by their sum."""
+    experts: int
+    top: int
+    ff: int
+    score: str = "sigmoid"
+    groups: int = 1
+    keep: int = 1
+    renorm: bool = False
+
+    @property
+    def rule(self) -> tuple:
+        return (int(self.score == "sigmoid"), self.groups, self.keep, int(self.renorm))
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    """One layer of a model that lists its layers: a mixer and a feed-forward (or none), each followed by a layer norm
+    of its output, added to an fp32 residual stream."""
+    mixer: LatentAttention
+    ffn: Optional[ExpertFfn]
+
+
+@dataclass(frozen=True)
 class ModelConfig:
     name: str
     n_layers: int
@@ -55,6 +97,9 @@ class ModelConfig:
     gdn_k_heads: int = 0
     gdn_v_heads: int = 0
     gdn_head_dim: int = 128
+    # models that list their layers one by one (unquantised weights, fp32 residual stream, norms on sublayer outputs);
+    # the scalar fields above then hold the largest values over the layers
+    layer_specs: tuple = ()
 
     @property
     def q_dim(self) -> int:
@@ -120,6 +165,8 @@ class ModelConfig:
         The reference's ``tp_card_desc`` does this for its two cards (src/model/model_desc.cc:252-285)."""
         if world == 1:
             return self
+        if self.layer_specs:
+            raise ValueError("models that list their layers are not sliced for tensor parallelism")
         if self.n_q_heads % world or self.n_kv_heads % world:
             raise ValueError(f"tensor parallel {world} does not divide {self.n_q_heads} q / {self.n_kv_heads} kv heads")
         if self.ffn % (64 * world) or (self.shared_ffn and self.shared_ffn % (64 * world)):
@@ -153,8 +200,21 @@ class ModelConfig:
         gdn = self.gdn_proj_dim * h + h * self.gdn_value_dim
         return (g * gdn + (self.n_layers - g) * attn) / self.n_layers
 
+    def layer_linears(self, spec: LayerSpec):
+        """(weights a token's step reads, weights held) of one listed layer."""
+        a, h = spec.mixer, self.hidden
+        mix = (a.q_rank + a.kv_rank + a.rot_dim) * h + a.heads * (a.dim + a.rot_dim) * a.q_rank \
+            + a.heads * (a.dim + a.vdim) * a.kv_rank + h * a.heads * a.vdim
+        if spec.ffn is None:
+            return mix, mix
+        f = spec.ffn
+        one = 3 * f.ff * h
+        return mix + f.experts * h + f.top * one, mix + f.experts * (h + one)
+
     def param_count(self) -> int:
         h = self.hidden
+        if self.layer_specs:
+            return int(sum(self.layer_linears(s)[1] for s in self.layer_specs) + 2 * self.vocab * h)
         per = self._mixer_params()
         if self.is_moe:
             per += self.n_experts * 3 * self.expert_ffn * h + self.n_experts * h
@@ -169,6 +229,8 @@ class ModelConfig:
         perf model, docs/05-perf-model.md:35-39): int4 nibbles + fp16 group scales
         for every linear that is touched, plus the head."""
         h = self.hidden
+        if self.layer_specs:
+            return 2.0 * sum(self.layer_linears(s)[0] for s in self.layer_specs) + self.vocab * h * lm_head_bytes_per_weight
         int4 = 0.5 + 2.0 / self.group_size
         per = self._mixer_params() * int4
         if self.is_moe:
@@ -180,10 +242,28 @@ class ModelConfig:
         return self.n_layers * per + self.vocab * h * lm_head_bytes_per_weight
 
     def kv_bytes_per_token(self, kv_dtype: str = "bf16") -> int:
+        if self.layer_specs:
+            return sum((s.mixer.kv_rank + s.mixer.rot_dim) * (4 if kv_dtype == "f32" else 2) for s in self.layer_specs)
         per_head = self.head_dim * (2 if kv_dtype == "bf16" else 1) + (4 if kv_dtype == "int8" else 0)
         return (self.n_layers - self.n_gdn_layers) * 2 * self.n_kv_heads * per_head
 
+    def to_listed_config(self) -> dict:
+        """The inverse of the listed designs' readers."""
+        def layer(s):
+            m, f = s.mixer, s.ffn
+            mixer = {"dim": m.dim, "heads": m.heads, "kv_rank": m.kv_rank, "q_rank": m.q_rank, "rot_dim": m.rot_dim,
+                     "vdim": m.vdim, "scale": m.scale, "rot": {"base": m.rope_base, "dims": m.rope_dims}}
+            if m.window:
+                mixer["mask"] = {"size": m.window}
+            mlp = None if f is None else {"kind": "moe", "expert": {"ff": f.ff}, "router": {
+                "experts": f.experts, "top": f.top, "groups": {"count": f.groups, "keep": f.keep}}}
+            return {"type": "latent_attention", "mixer": mixer, "mlp": mlp}
+        return {"architecture": self.architecture, "name": self.name, "width": self.hidden, "vocab": self.vocab,
+                "norm": {"eps": self.rms_eps}, "layers": [layer(s) for s in self.layer_specs]}
+
     def to_hf_config(self) -> dict:
+        if self.layer_specs:
+            return self.to_listed_config()
         d = {
             "architectures": [self.architecture],
             "model_type": "b200_moe" if self.is_moe else "b200_dense",
@@ -217,6 +297,11 @@ class ModelConfig:
 
     @staticmethod
     def from_hf_config(d: dict) -> "ModelConfig":
+        """The configuration of a checkpoint's ``config.json``; a name in ``LISTED_ARCHITECTURES`` under "architecture"
+        selects the reader of that design's keys."""
+        reader = LISTED_ARCHITECTURES.get(d.get("architecture"))
+        if reader is not None:
+            return reader(d)
         return ModelConfig(
             name=d.get("name", d.get("_name_or_path", "model")),
             n_layers=d["num_hidden_layers"], hidden=d["hidden_size"],
@@ -234,6 +319,44 @@ class ModelConfig:
             gdn_head_dim=d.get("linear_key_head_dim", 128) or 128,
             architecture=(d.get("architectures") or ["B200DenseForCausalLM"])[0],
         )
+
+
+def listed_config(name: str, architecture: str, specs, hidden: int, vocab: int, eps: float) -> ModelConfig:
+    """A model given by its layers; the scalar fields other parts of the framework read hold the largest values."""
+    specs = tuple(specs)
+    ffns = [s.ffn for s in specs if s.ffn is not None]
+    return ModelConfig(name, len(specs), hidden, max(s.mixer.heads for s in specs), 1, max(s.mixer.dim + s.mixer.rot_dim for s in specs),
+                       0, vocab, rms_eps=eps, n_experts=max((f.experts for f in ffns), default=0),
+                       top_k=max((f.top for f in ffns), default=0), expert_ffn=max((f.ff for f in ffns), default=0),
+                       architecture=architecture, layer_specs=specs)
+
+
+def mumusun_config(d: dict) -> ModelConfig:
+    """``config.json`` of a Mumusun checkpoint: "layers" lists every layer's mixer and feed-forward."""
+    specs = []
+    for i, layer in enumerate(d["layers"]):
+        if layer["type"] != "latent_attention":
+            raise ValueError(f"layer {i}: mixer {layer['type']!r} is not part of Mumusun")
+        m, f = layer["mixer"], layer["mlp"]
+        rot = m["rot"]
+        if rot["dims"] % 2 or rot["dims"] > m["rot_dim"]:
+            raise ValueError(f"layer {i}: {rot['dims']} rotated dimensions do not fit a part of {m['rot_dim']}")
+        mixer = LatentAttention(m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], m["q_rank"], float(m["scale"]),
+                                rot["dims"], float(rot["base"]), (m.get("mask") or {}).get("size", 0) or 0)
+        ffn = None
+        if f is not None:
+            if f["kind"] != "moe":
+                raise ValueError(f"layer {i}: feed-forward {f['kind']!r} is not part of Mumusun")
+            r = f["router"]
+            g = r.get("groups") or {"count": 1, "keep": 1}
+            if r["experts"] % g["count"] or r["top"] > g["keep"] * (r["experts"] // g["count"]):
+                raise ValueError(f"layer {i}: {r['experts']} experts, {g} and top {r['top']} do not fit together")
+            ffn = ExpertFfn(r["experts"], r["top"], f["expert"]["ff"], "sigmoid", g["count"], g["keep"], False)
+        specs.append(LayerSpec(mixer, ffn))
+    return listed_config(d.get("name", "mumusun"), "Mumusun", specs, d["width"], d["vocab"], float(d["norm"]["eps"]))
+
+
+LISTED_ARCHITECTURES = {"Mumusun": mumusun_config}
 
 
 def tiny_dense() -> ModelConfig:
@@ -287,6 +410,25 @@ def moe_35b_a3b() -> ModelConfig:
                        expert_ffn=512, shared_ffn=512, architecture="B200MoeForCausalLM")
 
 
+def mumusun_mini() -> ModelConfig:
+    """Small Mumusun: four layers of unequal sizes, windows and experts, the last one without a feed-forward."""
+    def mix(heads, dim, rot, vdim, rank, q_rank, window):
+        return LatentAttention(heads, dim, rot, vdim, rank, q_rank, (dim + rot) ** -0.5, rot, 1e5, window)
+    return listed_config("mumusun-mini", "Mumusun", (
+        LayerSpec(mix(4, 64, 32, 64, 192, 160, 96), ExpertFfn(16, 4, 96, groups=4, keep=2)),
+        LayerSpec(mix(8, 48, 24, 56, 136, 120, 0), ExpertFfn(9, 2, 72, groups=3, keep=1)),
+        LayerSpec(mix(20, 40, 16, 96, 256, 200, 33), ExpertFfn(6, 3, 128, groups=1, keep=1)),
+        LayerSpec(mix(3, 96, 40, 112, 320, 88, 160), None)), 320, 1000, 1e-5)
+
+
+def mumusun_16b() -> ModelConfig:
+    """A Mumusun of real layer sizes: 27 layers, hidden 2048, 16 heads of 128 + 64 over a latent of 512 with a window of
+    4096, 64 experts of 1408 in 8 groups, 6 per token."""
+    mix = LatentAttention(16, 128, 64, 128, 512, 1536, 192 ** -0.5, 64, 1e6, 4096)
+    return listed_config("mumusun-16b", "Mumusun", (LayerSpec(mix, ExpertFfn(64, 6, 1408, groups=8, keep=4)),) * 27, 2048,
+                         102400, 1e-6)
+
+
 def dflash_drafter(target: ModelConfig) -> ModelConfig:
     """DFlash-style block drafter: a 2-layer W4A16 decoder at the target's width."""
     return replace(target, name=target.name + "-dflash", n_layers=2, n_experts=0, top_k=0, expert_ffn=0,
@@ -296,6 +438,7 @@ def dflash_drafter(target: ModelConfig) -> ModelConfig:
 
 PRESETS = {
     "tiny-dense": tiny_dense, "tiny-moe": tiny_moe, "small-dense": small_dense, "small-windowed": small_windowed, "small-hybrid": small_hybrid, "small-moe": small_moe, "dense-27b": dense_27b, "hybrid-27b": hybrid_27b, "moe-35b-a3b": moe_35b_a3b,
+    "mumusun-mini": mumusun_mini, "mumusun-16b": mumusun_16b,
 }
 
 

@@ -82,14 +82,40 @@ def attn_splits(n_kv_heads: int, depth: int) -> int:
     return max(4, min(64, 296 // max(1, n_kv_heads), max(depth, 64) // 64))
 
 
+class ListedBuffers:
+    """What the engine and the head read of a listed model's step; the layers' activations are in ``scratch``."""
+
+    def __init__(self, cfg: ModelConfig, max_rows: int, wp: int, device, dtype):
+        from .latent import ListedScratch
+        self.max_rows = max_rows
+        self.scratch = ListedScratch(device, dtype, fixed=max_rows)
+        self.resid = torch.zeros(max_rows, wp, dtype=torch.float32, device=device)
+        self.logits = torch.zeros(max_rows, cfg.vocab, dtype=torch.float32, device=device)
+        self.ncand = K.head_ncand(cfg.vocab) if dtype == torch.bfloat16 else 1
+        self.cand_val = torch.zeros(max_rows * self.ncand, dtype=torch.float32, device=device)
+        self.cand_idx = torch.zeros(max_rows * self.ncand, dtype=torch.int32, device=device)
+        self.flag = torch.zeros(4, dtype=torch.int32, device=device)
+
+
 class KVCache:
-    """Paged KV: per layer ``[page][kv_head][16][D]`` for K and for V (bf16 or int8 + fp32 scales)."""
+    """Paged KV: per layer ``[page][kv_head][16][D]`` for K and for V (bf16 or int8 + fp32 scales); latent-attention layers
+    hold one latent row per position instead, ``[page][16][lc]`` (``latent[layer]``)."""
 
     def __init__(self, cfg: ModelConfig, n_layers: int, num_pages: int, device, kv_dtype: str = "bf16", n_slots: int = 1):
         self.kv_int8 = kv_dtype == "int8"
         dt = torch.int8 if self.kv_int8 else torch.bfloat16
         self.num_pages = num_pages
         self.n_layers = n_layers                # layers addressed by ``layer`` (trunk + draft-head layers)
+        self.latent = []
+        if cfg.layer_specs:
+            from .latent import LatentGeometry
+            if kv_dtype not in ("bf16", "f32"):
+                raise ValueError(f"latent-attention layers keep a bf16 (or, served in 32-bit, fp32) cache, not {kv_dtype}")
+            ldt = torch.float32 if kv_dtype == "f32" else torch.bfloat16
+            self.latent = [torch.zeros(num_pages, cfg.page_size, LatentGeometry.of(sp.mixer).lc, dtype=ldt, device=device)
+                           for sp in cfg.layer_specs]
+            self.k = self.v = self.k_scale = self.v_scale = self.gdn_conv = self.gdn_state = None
+            return
         # gated delta-net layers hold no KV: only the others get a plane of the cache
         self._plane = {}
         for li in range(n_layers):
@@ -116,6 +142,15 @@ class KVCache:
             self.gdn_conv[:, slot].zero_()
             self.gdn_state[:, slot].zero_()
 
+    def page_tensors(self) -> dict:
+        """Everything that belongs to a page, by name, as tensors ``[planes][page]...``."""
+        if self.latent:
+            return {f"latent{i}": t.unsqueeze(0) for i, t in enumerate(self.latent)}
+        out = {"k": self.k, "v": self.v}
+        if self.kv_int8:
+            out.update({"k_scale": self.k_scale, "v_scale": self.v_scale})
+        return out
+
     def layer(self, li: int):
         j = self._plane[li]
         ks = self.k_scale[j] if self.kv_int8 else None
@@ -133,6 +168,17 @@ class DecoderModel:
         self.device = weights.embed.device
         self.max_rows = max_rows
         self.nsplit_attn = nsplit_attn
+        self.listed = None
+        if cfg.layer_specs:
+            from .latent import ListedLayers
+            if tp is not None and tp.world > 1 or nccl is not None or int8_head:
+                raise ValueError("models that list their layers run on one GPU with an unquantised head")
+            self.listed = ListedLayers(weights, max_pos)
+            self.buf = ListedBuffers(cfg, max_rows, self.listed.wp, self.device, self.listed.dtype)
+            self.tp = self.nccl = None
+            self.head_rows, self.vocab_offset, self.max_pos, self.int8_head = cfg.vocab, 0, max_pos, False
+            self._mega_shared = None
+            return
         self.tp = tp if tp is not None and tp.world > 1 else None
         # ``nccl`` = (rank, world, group): the comparison path -- the same kernels, unfused, with NCCL
         # all-reduces after the row-parallel linears and an NCCL gather for the arg-max
@@ -522,6 +568,46 @@ class DecoderModel:
             pend = self._nccl_reduce(pend[0], pend[1], m)
         return pend if pend is not None else (None, 0)
 
+    # ------------------------------------------------------------------ models that list their layers
+    def listed_walk(self, m: int, rows, block_table, kv: KVCache, scratch, resid, plan=None):
+        """All layers of a listed model for ``m`` rows (``rows``: ``models.latent.StepRows``): the fp32 residual rows are
+        left in ``resid[:m]``.  ``plan``: how a mixed batch's rows are attended (None: every row on its own).
+
+        Per layer: the mixer's slices, folded by the kernel that norms them and adds them to the residual; the experts'
+        slots, weighted and folded by the same kernel."""
+        from ..ops import latent as L
+        ll, cfg = self.listed, self.cfg
+        h = scratch.get("h", m, ll.wp)
+        L.embed_rows(self.w.embed, rows.token, m, resid, h, self.buf.flag)
+        for li, (spec, lw) in enumerate(zip(cfg.layer_specs, self.w.layers)):
+            part, s = ll.mixer(scratch, li, m, rows, block_table, kv.latent[li], plan)
+            L.sublayer_norm(part, m, cfg.hidden, lw.input_norm, cfg.rms_eps, resid, h, slices=s, slice_elems=m * ll.wp,
+                            row_elems=ll.wp)
+            if spec.ffn is not None:
+                L.sublayer_norm(m=m, width=cfg.hidden, w=lw.post_norm, eps=cfg.rms_eps, x=resid, h=h,
+                                **ll.experts(scratch, spec.ffn, lw.moe, m))
+
+    def listed_logits(self, resid, sel, n: int, scratch, logits):
+        """Output norm and head of residual rows ``sel[:n]`` (None: rows 0..n - 1) into ``logits[:n]``."""
+        from ..ops import latent as L
+        ll, cfg, b = self.listed, self.cfg, self.buf
+        x = scratch.get("head_x", n, ll.wp)
+        L.layer_norm_rows(resid, sel, self.w.final_norm, cfg.rms_eps, n, cfg.hidden, x)
+        if ll.f32:
+            L.linear_f32(x, self.w.lm_head, logits, n)
+            L.row_argmax(logits, n, cfg.vocab, b.cand_val, b.cand_idx)
+        else:
+            K.head_gemv(self.w.lm_head, x, logits, n, cfg.vocab, ll.wp, b.cand_val, b.cand_idx)
+
+    def _listed_step(self, m: int, ctrl, block_table, kv: KVCache, advance: bool):
+        from .latent import StepRows
+        b = self.buf
+        rows = StepRows(ctrl[K.CTRL_ROW_REQ: K.CTRL_ROW_REQ + m], ctrl[K.CTRL_ROW_POS: K.CTRL_ROW_POS + m],
+                        ctrl[K.CTRL_CUR_TOKEN: K.CTRL_CUR_TOKEN + m])
+        self.listed_walk(m, rows, block_table, kv, b.scratch, b.resid)
+        self.listed_logits(b.resid, None, m, b.scratch, b.logits)
+        K.argmax_finish(b.cand_val, b.cand_idx, b.ncand, m, ctrl, advance)
+
     def _nccl_reduce(self, part, splits: int, m: int):
         """Comparison path: sum the split slices, all-reduce the ranks' partial sums with NCCL."""
         if self.nccl is None:
@@ -583,5 +669,7 @@ class DecoderModel:
         ``ctrl[out_token]``; with ``advance`` the rows' tokens and positions move on for the next replay.
         ``one_request``: the rows are consecutive positions of one request (plain decode, verify rows)."""
         assert 1 <= m <= self.max_rows
+        if self.listed is not None:
+            return self._listed_step(m, ctrl, block_table, kv, advance)
         pend = self.layers_walk(self.w.layers, m, ctrl, block_table, max_blocks, kv, one_request=one_request)
         self.head(m, pend, ctrl, advance)

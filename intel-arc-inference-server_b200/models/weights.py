@@ -85,6 +85,26 @@ class GdnWeights:
 
 
 @dataclass
+class LatentWeights:
+    """A latent-attention mixer, unquantised (bf16, or fp32 for models served in 32-bit), padded to whole 64s."""
+    down: torch.Tensor             # [qp + kvp + rp][Wp]: query latent, key-value latent, shared rotated key part
+    q_norm: torch.Tensor           # fp32 [q_rank]
+    kv_norm: torch.Tensor          # fp32 [kv_rank]
+    uq: torch.Tensor               # [heads * (dn + rp)][qp]
+    uk: torch.Tensor               # [heads * dn][kvp]
+    uv: torch.Tensor               # [heads * dv][kvp]
+    o: torch.Tensor                # [Wp][heads * dv]
+
+
+@dataclass
+class ExpertStack:
+    """Unquantised routed experts of one layer, padded to whole 64s."""
+    router: torch.Tensor           # [E rounded up to 8][Wp]
+    gate_up: torch.Tensor          # [E][2 * ffp][Wp], interleave16
+    down: torch.Tensor             # [E][Wp][ffp]
+
+
+@dataclass
 class LayerWeights:
     input_norm: torch.Tensor       # fp32 [hidden]
     post_norm: torch.Tensor        # fp32 [hidden]
@@ -100,6 +120,9 @@ class LayerWeights:
     experts_gate_up_w4b: Optional[torch.Tensor] = None
     experts_down_w4b: Optional[torch.Tensor] = None
     gdn: Optional[GdnWeights] = None               # set instead of qkv / o on gated delta-net layers
+    # listed layers: input_norm / post_norm then belong to the mixer's and the feed-forward's OUTPUT
+    latent: Optional[LatentWeights] = None
+    moe: Optional[ExpertStack] = None
 
 
 @dataclass
@@ -135,6 +158,9 @@ class ModelWeights:
                 tot += lw.experts_gate_up_w4b.numel() + lw.experts_down_w4b.numel()
             if lw.shared is not None:
                 tot += lw.shared.gate_up.nbytes + lw.shared.down.nbytes
+            for part in (lw.latent, lw.moe):
+                if part is not None:
+                    tot += sum(t.numel() * t.element_size() for t in vars(part).values())
         return tot
 
 
@@ -206,6 +232,9 @@ def random_weights(cfg: ModelConfig, device="cpu", seed: int = 0, exact: Optiona
     ``head_rows``: rows of the lm_head this rank holds (vocabulary-parallel head)."""
     if exact is None:
         exact = cfg.param_count() < 100_000_000
+    if cfg.layer_specs:
+        from .latent import random_listed_weights
+        return random_listed_weights(cfg, device, seed, std)
     h = cfg.hidden
     hr = cfg.vocab if head_rows is None else head_rows
     if exact:

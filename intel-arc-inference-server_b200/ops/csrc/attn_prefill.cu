@@ -1,4 +1,5 @@
-// Causal flash attention for prompt chunks over the paged KV cache, on tcgen05 / TMEM (head_dim 128).
+// Causal flash attention for prompt chunks on tcgen05 / TMEM: over the paged KV cache (head_dim 128), and over contiguous
+// key / value rows with their own head sizes (latent attention, whose keys and values are expanded before).
 //
 //   O[r] = softmax( q[r] . K[0 .. pos(r)]^T / sqrt(D) ) V[0 .. pos(r)]      pos(r) = pos0 + r
 //
@@ -19,7 +20,7 @@ using namespace b2;
 
 namespace {
 
-constexpr int D = 128;
+constexpr int D = 128;    // head size of the paged form
 constexpr int BQ = 128;   // rows of a query tile
 
 struct AttnPfParams {
@@ -31,7 +32,12 @@ struct AttnPfParams {
   int window;      // > 0: a row attends to its last `window` positions only; key tiles before the CTA's first window are skipped
   float scale_log2;
   __nv_bfloat16* out;  // [C][n_q * D]
+  // contiguous form: one entry per CTA column (blockIdx.x) of kTileWords ints: first row in q and out, rows (<= 128 per
+  // query tile), position of the first row and key row of position 0, both counted from the segment's first key
+  const int* tiles;
+  int dn;              // columns of a head in the key matrix (a multiple of 64; the shared part fills up the head)
 };
+constexpr int kTileWords = 4;
 
 #ifdef B2_ATTN_PROF
 // measurement build: cycles per phase, summed over tiles and CTAs by one softmax thread and the MMA thread
@@ -60,10 +66,20 @@ __device__ unsigned long long g_attn_prof[16];
 constexpr int BK2 = 64;
 constexpr int kThreads2 = 608;    // TMA warp, MMA warp of tile 0, 2 tiles x 2 column halves x 4 softmax warps, MMA warp of tile 1
 constexpr int kMmaWarp1 = 18;
-constexpr int Q2_BYTES = 2 * BQ * D * 2;          // two query tiles, each [2 d-blocks][128 rows][64]
-constexpr int KV2_BYTES = BK2 * D * 2;            // 16 KB per K or V tile: [2 d-blocks][64 keys][64]
-constexpr int KVS = 4;                            // K / V ring depth (tiles in flight)
-constexpr int SMEM2 = Q2_BYTES + 2 * KVS * KV2_BYTES + 1024 + 256 + 2 * 2 * 2 * 128 * 4;   // + alignment, barriers, exchange slots
+// A form of the kernel: blocks of 64 dims of a query / key (NDK) and of a value (NDV), query tiles per CTA (NW; one where
+// two do not fit), ring depth (KVS: K / V tiles in flight), K / V from pages or from contiguous rows.
+template <int NDK_, int NDV_, int NW_, int KVS_, bool PAGED_>
+struct Form {
+  static constexpr int NDK = NDK_, NDV = NDV_, NW = NW_, KVS = KVS_, DV = NDV_ * 64;
+  static constexpr bool PAGED = PAGED_;
+  static constexpr int QT_BYTES = BQ * NDK * 128;           // a query tile: [d-blocks][128 rows][64]
+  static constexpr int Q_BYTES = NW * QT_BYTES;
+  static constexpr int K_BYTES = BK2 * NDK * 128;           // a K tile: [d-blocks][64 keys][64]
+  static constexpr int V_BYTES = BK2 * NDV * 128;
+  static constexpr int SMEM = Q_BYTES + KVS * (K_BYTES + V_BYTES) + 1024 + 256 + 2 * 2 * 2 * 128 * 4;   // + alignment, barriers, exchange slots
+  static_assert(SMEM <= 227 * 1024, "shared memory of one CTA");
+  static_assert(NW == 1 || NDV <= 2, "tensor memory: 256 score columns + NW x DV accumulator columns");
+};
 
 // smem descriptor for the MN-major V operand: rows are keys (128 B = 64 dims, 128-byte swizzle), 8-key groups are
 // 1024 B apart (stride byte offset); the next block of 64 dims is a whole tile half away (leading byte offset).
@@ -77,12 +93,17 @@ __device__ __forceinline__ uint64_t make_desc_v2(uint32_t smem_addr) {
   return d;
 }
 
+// map_r: contiguous form, the key part shared by all heads [rows][64 x blocks]; a head's key is dn columns of map_k
+// followed by it
+template <class F>
 __global__ void __launch_bounds__(kThreads2, 1)
 attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
-                         const __grid_constant__ CUtensorMap map_v, const AttnPfParams p) {
+                         const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_r,
+                         const AttnPfParams p) {
+  constexpr int KVS = F::KVS, NDK = F::NDK, NDV = F::NDV;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
-  const uint32_t q_s = base, k_s0 = base + Q2_BYTES, v_s0 = k_s0 + KVS * KV2_BYTES, bars = v_s0 + KVS * KV2_BYTES;
+  const uint32_t q_s = base, k_s0 = base + F::Q_BYTES, v_s0 = k_s0 + KVS * F::K_BYTES, bars = v_s0 + KVS * F::V_BYTES;
   // barriers (8 bytes each): q_full; k_full, k_empty, v_full, v_empty [KVS each]; per tile w: s_full[w][2],
   // p_full[w], o_done[w][2]
   const uint32_t b_qfull = bars, b_kfull = bars + 8, b_kempty = b_kfull + 8 * KVS, b_vfull = b_kempty + 8 * KVS,
@@ -95,13 +116,19 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int qt = gridDim.x - 1 - blockIdx.x;   // heavy (late) pairs first
-  const int head = blockIdx.y, kh = head / (p.n_q / p.n_kv);
-  const int row0 = qt * 2 * BQ;
+  const int head = blockIdx.y, kh = F::PAGED ? head / (p.n_q / p.n_kv) : head;
+  // row0: first row inside the chunk (segment); C rows; pos0: position of chunk row 0, counted from the first key;
+  // qrow: row of q / out that holds chunk row 0; krow: key row of position 0 (contiguous form)
+  int row0 = qt * F::NW * BQ, C = p.C, pos0 = p.pos0, qrow = 0, krow = 0;
+  if (!F::PAGED) {
+    const int* tile = p.tiles + blockIdx.x * kTileWords;
+    row0 = 0; qrow = tile[0]; C = tile[1]; pos0 = tile[2]; krow = tile[3];
+  }
   // key tiles each query tile needs, counted from the first tile any of the CTA's rows needs
-  const int t0 = p.window > 0 ? max(0, p.pos0 + row0 - p.window + 1) / BK2 : 0;
+  const int t0 = p.window > 0 ? max(0, pos0 + row0 - p.window + 1) / BK2 : 0;
   int n_w[2];
-  n_w[0] = (p.pos0 + min(row0 + BQ, p.C) - 1) / BK2 + 1 - t0;
-  n_w[1] = row0 + BQ < p.C ? (p.pos0 + min(row0 + 2 * BQ, p.C) - 1) / BK2 + 1 - t0 : 0;
+  n_w[0] = (pos0 + min(row0 + BQ, C) - 1) / BK2 + 1 - t0;
+  n_w[1] = F::NW > 1 && row0 + BQ < C ? (pos0 + min(row0 + 2 * BQ, C) - 1) / BK2 + 1 - t0 : 0;
   const int n_all = max(n_w[0], n_w[1]);
 
   if (threadIdx.x == 0) {
@@ -130,53 +157,70 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
   auto t_s = [&](int w, int b) { return tmem_base + (uint32_t)(w * 2 + b) * BK2; };
-  auto t_o = [&](int w) { return tmem_base + 256 + (uint32_t)w * D; };
+  auto t_o = [&](int w) { return tmem_base + 256 + (uint32_t)w * F::DV; };
 
   if (warp == 0) {
     if (lane == 0) {
       prefetch_tmap(&map_q);
       prefetch_tmap(&map_k);
       prefetch_tmap(&map_v);
+      if (!F::PAGED) prefetch_tmap(&map_r);
       const int nq = n_w[1] > 0 ? 2 : 1;
-      mbar_expect_tx(b_qfull, nq * BQ * D * 2);
-      for (int w = 0; w < nq; ++w) {
-        tma_load_2d(q_s + w * (BQ * D * 2), &map_q, head * D, row0 + w * BQ, b_qfull);
-        tma_load_2d(q_s + w * (BQ * D * 2) + BQ * 128, &map_q, head * D + 64, row0 + w * BQ, b_qfull);
-      }
+      mbar_expect_tx(b_qfull, nq * F::QT_BYTES);
+      for (int w = 0; w < nq; ++w)
+#pragma unroll
+        for (int c = 0; c < NDK; ++c)
+          tma_load_2d(q_s + w * F::QT_BYTES + c * (BQ * 128), &map_q, (head * NDK + c) * 64, qrow + row0 + w * BQ, b_qfull);
       bool ok = true;
       int issued = 0;
       for (int i = 0; i < n_all && ok; ++i) {
         const int s = i % KVS, ph = (i / KVS) & 1;
-        const uint32_t k_s = k_s0 + s * KV2_BYTES, v_s = v_s0 + s * KV2_BYTES;
+        const uint32_t k_s = k_s0 + s * F::K_BYTES, v_s = v_s0 + s * F::V_BYTES;
         // Always 4 pages: table entries past the sequence point at pages that hold finite data (page 0 is the
         // never-allocated zero page) and those keys are masked out; an unfilled part of a tile could hold NaN bit
         // patterns, and 0 * NaN in P V would poison the row.
         constexpr int n_pages = BK2 / 16;
         int rowc[n_pages];
 #pragma unroll
-        for (int pg = 0; pg < n_pages; ++pg) {
+        for (int pg = 0; pg < n_pages && F::PAGED; ++pg) {
           const int pi = (t0 + i) * n_pages + pg;
           const int page = pi < p.max_blocks ? __ldg(p.block_table + pi) : 0;
           rowc[pg] = (page * p.n_kv + kh) * 16;
         }
+        // contiguous rows: those past the segment are another's, or rows the workspace keeps finite, and masked out
+        const int kr = krow + (t0 + i) * BK2;
         if (i >= KVS) ok = mbar_wait(b_kempty + 8 * s, ph ^ 1, ERR_ATTN_WAIT);
         if (!ok) break;
-        mbar_expect_tx(b_kfull + 8 * s, KV2_BYTES);
+        mbar_expect_tx(b_kfull + 8 * s, F::K_BYTES);
+        if (F::PAGED) {
 #pragma unroll
-        for (int pg = 0; pg < n_pages; ++pg) {
-          tma_load_2d(k_s + pg * 2048, &map_k, 0, rowc[pg], b_kfull + 8 * s);
-          tma_load_2d(k_s + BK2 * 128 + pg * 2048, &map_k, 64, rowc[pg], b_kfull + 8 * s);
+          for (int pg = 0; pg < n_pages; ++pg) {
+            tma_load_2d(k_s + pg * 2048, &map_k, 0, rowc[pg], b_kfull + 8 * s);
+            tma_load_2d(k_s + BK2 * 128 + pg * 2048, &map_k, 64, rowc[pg], b_kfull + 8 * s);
+          }
+        } else {
+          const int cn = p.dn >> 6;
+#pragma unroll
+          for (int c = 0; c < NDK; ++c) {
+            if (c < cn) tma_load_2d(k_s + c * (BK2 * 128), &map_k, head * p.dn + c * 64, kr, b_kfull + 8 * s);
+            else tma_load_2d(k_s + c * (BK2 * 128), &map_r, (c - cn) * 64, kr, b_kfull + 8 * s);
+          }
         }
         if (i >= KVS) ok = mbar_wait(b_vempty + 8 * s, ph ^ 1, ERR_ATTN_WAIT);
         if (!ok) {
           mbar_wait(b_kfull + 8 * s, ph, ERR_ATTN_WAIT);  // drain the K copies just issued
           break;
         }
-        mbar_expect_tx(b_vfull + 8 * s, KV2_BYTES);
+        mbar_expect_tx(b_vfull + 8 * s, F::V_BYTES);
+        if (F::PAGED) {
 #pragma unroll
-        for (int pg = 0; pg < n_pages; ++pg) {
-          tma_load_2d(v_s + pg * 2048, &map_v, 0, rowc[pg], b_vfull + 8 * s);
-          tma_load_2d(v_s + BK2 * 128 + pg * 2048, &map_v, 64, rowc[pg], b_vfull + 8 * s);
+          for (int pg = 0; pg < n_pages; ++pg) {
+            tma_load_2d(v_s + pg * 2048, &map_v, 0, rowc[pg], b_vfull + 8 * s);
+            tma_load_2d(v_s + BK2 * 128 + pg * 2048, &map_v, 64, rowc[pg], b_vfull + 8 * s);
+          }
+        } else {
+#pragma unroll
+          for (int c = 0; c < NDV; ++c) tma_load_2d(v_s + c * (BK2 * 128), &map_v, (head * NDV + c) * 64, kr, b_vfull + 8 * s);
         }
         issued = i + 1;
       }
@@ -195,13 +239,13 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       const int w = warp == 1 ? 0 : 1;
       const int nt = n_w[w];
       constexpr uint32_t idesc_qk = make_idesc(1, 1, BQ, BK2);
-      constexpr uint32_t idesc_pv = make_idesc(1, 1, BQ, D) | (1u << 16);  // B (V) is MN-major
+      constexpr uint32_t idesc_pv = make_idesc(1, 1, BQ, F::DV) | (1u << 16);  // B (V) is MN-major
       bool ok = mbar_wait(b_qfull, 0, ERR_ATTN_WAIT);
       // Descriptor words: every 128-byte-swizzled K-major operand shares one high word, V (MN-major) has its own; the
       // low word is (address >> 4) plus the leading-offset field, so an operand piece is one integer add away.
       const uint32_t hi_k = (uint32_t)(make_desc_sw128(0) >> 32), hi_v = (uint32_t)(make_desc_v2(0) >> 32);
-      const uint32_t ql = (uint32_t)make_desc_sw128(q_s + w * (BQ * D * 2));
-      const uint32_t k_lo0 = (uint32_t)make_desc_sw128(k_s0), v_lo0 = (uint32_t)make_desc_v2(v_s0);   // ring stage 0; a stage is KV2_BYTES >> 4 further
+      const uint32_t ql = (uint32_t)make_desc_sw128(q_s + (F::NW > 1 ? w : 0) * F::QT_BYTES);
+      const uint32_t k_lo0 = (uint32_t)make_desc_sw128(k_s0), v_lo0 = (uint32_t)make_desc_v2(v_s0);   // ring stage 0; a stage is K_BYTES / V_BYTES >> 4 further
       const uint32_t to = t_o(w);
       auto issue_qk = [&](int j) -> bool {
         const int s = j & 1, ks = j % KVS;
@@ -209,9 +253,9 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         // the buffer's first 32 columns hold P(j - 2) until that tile's P V product has read them
         if (j >= 2 && !mbar_wait(b_odone(w, s), ((j >> 1) - 1) & 1, ERR_ATTN_WAIT)) return false;
         tc_fence_after();
-        const uint32_t kl = k_lo0 + ks * (KV2_BYTES >> 4), ts = t_s(w, s);
+        const uint32_t kl = k_lo0 + ks * (F::K_BYTES >> 4), ts = t_s(w, s);
 #pragma unroll
-        for (int k = 0; k < 8; ++k)   // 8 x 16 dims; dims 64.. live in the operands' second block
+        for (int k = 0; k < 4 * NDK; ++k)   // steps of 16 dims; every 64 dims live in a block of their own
           umma_f16_w(ts, ql + (((k >> 2) * (BQ * 128) + (k & 3) * 32) >> 4), hi_k,
                      kl + (((k >> 2) * (BK2 * 128) + (k & 3) * 32) >> 4), hi_k, idesc_qk, k != 0);
         tc_commit(b_sfull(w, s));
@@ -243,7 +287,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         APROF_T(m3);
         APROF_ADD(8, m0, m1); APROF_ADD(9, m1, m2); APROF_ADD(10, m2, m3); APROF_ADD(11, m0, m0 + 1);
         tc_fence_after();
-        const uint32_t vl = v_lo0 + ks * (KV2_BYTES >> 4), tp = t_s(w, s);
+        const uint32_t vl = v_lo0 + ks * (F::V_BYTES >> 4), tp = t_s(w, s);
 #pragma unroll
         for (int k = 0; k < 4; ++k)   // 4 x 16 keys: P comes from tensor memory, 8 columns (16 bf16) per step
           umma_f16_ts_w(to, tp + 8 * k, vl + ((k * 16 * 128) >> 4), hi_v, idesc_pv, (i | k) != 0);
@@ -262,11 +306,11 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const int quarter = warp & 3;         // TMEM lane quarter this warp may touch
     const int r = quarter * 32 + lane;    // row inside the tile
     const int rowg = row0 + w * BQ + r;   // row inside the chunk
-    const int qpos = p.pos0 + rowg;
+    const int qpos = pos0 + rowg;
     const int qlo = p.window > 0 ? qpos - p.window + 1 : 0;   // the row's keys: qlo <= key <= qpos
-    const bool row_ok = rowg < p.C;
+    const bool row_ok = rowg < C;
     const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
-    const int first_pos = p.pos0 + row0 + w * BQ;             // position of the tile's first row
+    const int first_pos = pos0 + row0 + w * BQ;             // position of the tile's first row
     const int nt = n_w[w];
     // float [tile w][tile parity][half][128 rows]: the halves of a row exchange their maxima (and, at the end, sums)
     const uint32_t xch = bars + 256 + (uint32_t)w * (2 * 2 * 128 * 4);
@@ -327,7 +371,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         tc_fence_after();
         if (ok && resc) {
 #pragma unroll 1
-          for (int c = 2 * half; c < 2 * half + 2; ++c) {   // this thread's half of the row's accumulator
+          for (int c = NDV * half; c < NDV * half + NDV; ++c) {   // this thread's half of the row's accumulator
             uint32_t o[32];
             B2_TMEM_LD_32(t_o(w) + lane_addr + c * 32, o);
             tmem_ld_wait();
@@ -407,9 +451,9 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     if (ok && nt > 0) {
       tc_fence_after();
       const float inv = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* dst = p.out + (size_t)rowg * (p.n_q * D) + head * D;
+      __nv_bfloat16* dst = p.out + (size_t)(qrow + rowg) * (p.n_q * F::DV) + head * F::DV;
 #pragma unroll 1
-      for (int c = 2 * half; c < 2 * half + 2; ++c) {
+      for (int c = NDV * half; c < NDV * half + NDV; ++c) {
         uint32_t o[32];
         B2_TMEM_LD_32(t_o(w) + lane_addr + c * 32, o);
         tmem_ld_wait();
@@ -461,6 +505,21 @@ int make_map_bf16(CUtensorMap* map, const void* ptr, uint64_t rows, uint64_t col
   return r == CUDA_SUCCESS ? 0 : -101 - (int)r;
 }
 
+template <class F>
+int launch_form(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mr,
+                const AttnPfParams& p, int columns, int heads, cudaStream_t st) {
+  static bool configured[64] = {};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (!configured[dev & 63]) {
+    cudaError_t e = cudaFuncSetAttribute(attn_prefill_pair_kernel<F>, cudaFuncAttributeMaxDynamicSharedMemorySize, F::SMEM);
+    if (e != cudaSuccess) return (int)e;
+    configured[dev & 63] = true;
+  }
+  attn_prefill_pair_kernel<F><<<dim3(columns, heads), kThreads2, F::SMEM, st>>>(mq, mk, mv, mr, p);
+  return (int)cudaGetLastError();
+}
+
 }  // namespace
 
 // q: bf16 [C][n_q*128]; k_cache / v_cache: bf16 [num_pages][n_kv][16][128]; block_table: the sequence's
@@ -488,21 +547,51 @@ extern "C" int b2_attn_prefill(const void* q, const void* k_cache, const void* v
   if (rc) return rc;
   rc = make_map_bf16(&mv, v_cache, (uint64_t)num_pages * n_kv * 16, D, 16);
   if (rc) return rc;
-  static bool configured[64] = {};
-  int dev = 0;
-  cudaGetDevice(&dev);
-  if (!configured[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_pair_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM2);
-    if (e != cudaSuccess) return (int)e;
-    configured[dev & 63] = true;
-  }
-  AttnPfParams p;
+  AttnPfParams p = {};
   p.block_table = block_table; p.n_q = n_q; p.n_kv = n_kv; p.C = C; p.pos0 = pos0; p.max_blocks = max_blocks;
   p.scale_log2 = scale * 1.4426950408889634f; p.out = (__nv_bfloat16*)out;
   p.window = window > 0 ? window : 0;
-  dim3 grid((C + 2 * BQ - 1) / (2 * BQ), n_q);
-  attn_prefill_pair_kernel<<<grid, kThreads2, SMEM2, (cudaStream_t)stream>>>(mq, mk, mv, p);
-  return (int)cudaGetLastError();
+  return launch_form<Form<2, 2, 2, 4, true>>(mq, mk, mv, mv, p, (C + 2 * BQ - 1) / (2 * BQ), n_q, (cudaStream_t)stream);
+}
+
+// Query rows per CTA column of the contiguous form for dk / dv dims of a key / value (multiples of 64): 256, 128, or 0
+// when no form covers the sizes.
+extern "C" int b2_attn_rows_per_tile(int dk, int dv) {
+  const int ndk = dk / 64, ndv = dv / 64;
+  if (dk % 64 || dv % 64 || ndk < 2 || ndk > 4 || (ndv != 1 && ndv != 2 && ndv != 4)) return 0;
+  return ndk <= 3 && ndv <= 2 ? 256 : 128;
+}
+
+// q: bf16 [q_rows][H * dk]; k: [k_rows][H * dn] and the shared part kr: [k_rows][dk - dn]; v: [k_rows][H * dv]; out
+// [q_rows][H * dv].  tiles: n_tiles x 4 ints (device): first row of q, rows, position of that row, key row of position
+// 0 -- positions counted from the first key row of the tile's segment.
+extern "C" int b2_attn_prefill_rows(const void* q, const void* k, const void* kr, const void* v, void* out, const int* tiles,
+                                    int n_tiles, int q_rows, int k_rows, int H, int dn, int dk, int dv, float scale,
+                                    int window, void* stream) {
+  const int rpt = b2_attn_rows_per_tile(dk, dv);
+  if (!rpt || dn % 64 || dn < 64 || dn >= dk || n_tiles < 1 || H < 1) return -1;
+  CUtensorMap mq, mk, mr, mv;
+  int rc = make_map_bf16(&mq, q, (uint64_t)q_rows, (uint64_t)H * dk, BQ);
+  if (!rc) rc = make_map_bf16(&mk, k, (uint64_t)k_rows, (uint64_t)H * dn, BK2);
+  if (!rc) rc = make_map_bf16(&mr, kr, (uint64_t)k_rows, (uint64_t)(dk - dn), BK2);
+  if (!rc) rc = make_map_bf16(&mv, v, (uint64_t)k_rows, (uint64_t)H * dv, BK2);
+  if (rc) return rc;
+  AttnPfParams p = {};
+  p.n_q = p.n_kv = H; p.scale_log2 = scale * 1.4426950408889634f; p.out = (__nv_bfloat16*)out;
+  p.window = window > 0 ? window : 0; p.tiles = tiles; p.dn = dn;
+  cudaStream_t st = (cudaStream_t)stream;
+  switch (dk / 64 * 10 + dv / 64) {
+    case 21: return launch_form<Form<2, 1, 2, 4, false>>(mq, mk, mv, mr, p, n_tiles, H, st);
+    case 22: return launch_form<Form<2, 2, 2, 4, false>>(mq, mk, mv, mr, p, n_tiles, H, st);
+    case 31: return launch_form<Form<3, 1, 2, 3, false>>(mq, mk, mv, mr, p, n_tiles, H, st);
+    case 32: return launch_form<Form<3, 2, 2, 3, false>>(mq, mk, mv, mr, p, n_tiles, H, st);
+    case 41: return launch_form<Form<4, 1, 1, 3, false>>(mq, mk, mv, mr, p, n_tiles, H, st);
+    case 42: return launch_form<Form<4, 2, 1, 3, false>>(mq, mk, mv, mr, p, n_tiles, H, st);
+    case 24: return launch_form<Form<2, 4, 1, 3, false>>(mq, mk, mv, mr, p, n_tiles, H, st);
+    case 34: return launch_form<Form<3, 4, 1, 3, false>>(mq, mk, mv, mr, p, n_tiles, H, st);
+    case 44: return launch_form<Form<4, 4, 1, 2, false>>(mq, mk, mv, mr, p, n_tiles, H, st);
+  }
+  return -1;
 }
 
 B2_DEFINE_STATUS(attn)

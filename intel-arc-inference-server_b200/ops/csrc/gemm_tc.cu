@@ -536,17 +536,17 @@ EncodeTiledFn encode_fn() {
   return fn;
 }
 
-// rows x cols (cols contiguous) matrix, optionally a stack of `batch` of them; box = box_rows x 128 bytes
+// rows x cols (cols contiguous) matrix (batch 0), or a stack of `batch` of them; box = box_rows x 128 bytes
 int make_map(CUtensorMap* map, const void* ptr, bool i8, uint64_t rows, uint64_t cols, uint64_t batch,
              uint32_t box_rows) {
   EncodeTiledFn fn = encode_fn();
   if (!fn) return -100;
   const uint64_t esz = i8 ? 1 : 2;
-  cuuint64_t dims[3] = {cols, rows, batch};
+  cuuint64_t dims[3] = {cols, rows, batch ? batch : 1};
   cuuint64_t strides[2] = {cols * esz, rows * cols * esz};
   cuuint32_t box[3] = {(cuuint32_t)(BKB / esz), box_rows, 1};
   cuuint32_t estr[3] = {1, 1, 1};
-  const int rank = batch > 1 ? 3 : 2;
+  const int rank = batch ? 3 : 2;
   CUresult r = fn(map, i8 ? CU_TENSOR_MAP_DATA_TYPE_UINT8 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, rank,
                   const_cast<void*>(ptr), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
                   CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
@@ -610,7 +610,7 @@ extern "C" int b2_gemm_w4(const void* a, const void* w4b, void* c, int M, int N,
   p.w4_expert_bytes = (long long)((N + 127) / 128) * (K / 64) * kW4Block;
   if (bn != 128 && bn != 256) bn = (N >= 256 && (N % 256 == 0 || N > 2048)) ? 256 : 128;
   CUtensorMap ma;
-  int rc = make_map(&ma, a, false, (uint64_t)M, (uint64_t)K, 1, BM);
+  int rc = make_map(&ma, a, false, (uint64_t)M, (uint64_t)K, 0, BM);
   if (rc) return rc;
   const int tiles_m = blk_expert ? max_blk : (M + BM - 1) / BM;
   const int n_tiles = tiles_m * ((N + bn - 1) / bn);
@@ -641,9 +641,9 @@ static int gemm_tc_impl(const void* a, const void* b, void* c, int M, int N, int
   p.blk_expert = blk_expert; p.blk_row0 = blk_row0; p.blk_rows = blk_rows; p.n_blk = n_blk; p.max_blk = max_blk;
   if (bn != 128 && bn != 256) bn = (N >= 256 && (N % 256 == 0 || N > 2048)) ? 256 : 128;
   CUtensorMap ma, mb;
-  int rc = make_map(&ma, a, i8 != 0, (uint64_t)M, (uint64_t)K, 1, BM);
+  int rc = make_map(&ma, a, i8 != 0, (uint64_t)M, (uint64_t)K, 0, BM);
   if (rc) return rc;
-  rc = make_map(&mb, b, i8 != 0, (uint64_t)N, (uint64_t)K, blk_expert ? (uint64_t)n_experts : 1, (uint32_t)bn);
+  rc = make_map(&mb, b, i8 != 0, (uint64_t)N, (uint64_t)K, blk_expert ? (uint64_t)n_experts : 0, (uint32_t)bn);
   if (rc) return rc;
   const int tiles_m = blk_expert ? max_blk : (M + BM - 1) / BM;
   const int n_tiles = tiles_m * ((N + bn - 1) / bn);

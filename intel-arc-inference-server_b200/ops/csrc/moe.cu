@@ -1,7 +1,8 @@
 // Mixture-of-experts glue kernels: routing, expert-major sorting with a device-side block table,
 // gather, and the weighted combine.
 //
-//   moe_route     softmax over all experts -> top-k (ties to the lower id) -> renormalise
+//   moe_route     scores of all experts (softmax or sigmoid) -> optional choice of expert groups -> top-k (ties to the
+//                 lower id) -> weights (renormalised over the chosen, or the scores)
 //   moe_count     per-expert histogram + the rank of every (token, slot) inside its expert
 //   moe_plan      prefix over experts padded to 128-row blocks -> block table for the grouped GEMM
 //   moe_scatter   (token, slot) -> sorted row; gather of the activation rows in sorted order
@@ -19,11 +20,19 @@ using namespace b2;
 namespace {
 
 // ---------------------------------------------------------------- route: one warp per token
+// How logits become a choice of experts and their weights.
+struct RouteRule {
+  int sigmoid;   // 0: softmax over all experts, 1: a sigmoid per expert
+  int groups;    // > 1: experts form this many equal groups of neighbours; only the `keep` groups with the largest sums
+  int keep;      //      of their two best scores stay eligible
+  int renorm;    // 1: weights divided by their sum over the chosen experts, 0: the scores themselves
+};
+
 // logits fp32 [T][ld], the first E columns are the experts (E <= 512).  topk_idx int32 [T][k], topk_w fp32 [T][k].
-// One row's routing by a whole warp: softmax over E logits, top-k by repeated arg-max (ties to the lower id), weights
-// renormalised over the chosen k.  `stride` >= k entries per row in topk_idx / topk_w.
-__device__ __forceinline__ void route_row(const float* __restrict__ lrow, int E, int k, int* __restrict__ idx_out,
-                                          float* __restrict__ w_out, int lane) {
+// One row's routing by a whole warp: scores of E logits, top-k by repeated arg-max (ties to the lower id).
+// `stride` >= k entries per row in topk_idx / topk_w.
+__device__ __forceinline__ void route_row(const float* __restrict__ lrow, int E, int k, const RouteRule rule,
+                                          int* __restrict__ idx_out, float* __restrict__ w_out, int lane) {
   constexpr int PER = 16;  // experts per lane (E <= 512)
   float v[PER];
   float mx = -INFINITY;
@@ -34,9 +43,55 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lrow, int E,
     mx = fmaxf(mx, v[i]);
   }
   mx = warp_max(mx);
+  float total = 0.f;   // softmax normaliser, only needed when the weights are not renormalised
 #pragma unroll
-  for (int i = 0; i < PER; ++i)
-    v[i] = (lane + 32 * i) < E ? __expf(v[i] - mx) : -1.f;  // probabilities (unnormalised); -1 marks "taken / absent"
+  for (int i = 0; i < PER; ++i) {
+    // softmax: unnormalised probabilities; -1 marks "taken / absent"
+    const bool in = (lane + 32 * i) < E;
+    if (rule.sigmoid) v[i] = in ? 1.f / (1.f + expf(-v[i])) : -1.f;
+    else v[i] = in ? __expf(v[i] - mx) : -1.f;
+    total += in ? v[i] : 0.f;
+  }
+  if (rule.groups > 1) {
+    const int size = E / rule.groups;
+    float mine = -INFINITY;      // lane g keeps the score of group g (groups <= 32)
+    for (int g = 0; g < rule.groups; ++g) {
+      float a = -1.f, b = -1.f;  // two best of the group among this lane's experts
+#pragma unroll
+      for (int i = 0; i < PER; ++i) {
+        const int e = lane + 32 * i;
+        if (e >= g * size && e < (g + 1) * size) {
+          if (v[i] > a) { b = a; a = v[i]; }
+          else b = fmaxf(b, v[i]);
+        }
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float oa = __shfl_xor_sync(0xffffffffu, a, o), ob = __shfl_xor_sync(0xffffffffu, b, o);
+        b = fmaxf(fminf(a, oa), fmaxf(b, ob));
+        a = fmaxf(a, oa);
+      }
+      const float score = a + fmaxf(b, 0.f);    // a group of one expert has no second score
+      if (lane == g) mine = score;
+    }
+    unsigned kept = 0;
+    for (int r = 0; r < rule.keep; ++r) {
+      float bv = (kept >> lane) & 1u ? -INFINITY : mine;
+      int bi = lane;
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+        if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
+      }
+      kept |= 1u << bi;
+    }
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const int e = lane + 32 * i;
+      if (e < E && !((kept >> (e / size)) & 1u)) v[i] = -1.f;
+    }
+  }
   float wsum = 0.f;
   float myw = 0.f;
   int myid = 0;
@@ -59,19 +114,22 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lrow, int E,
     wsum += bv;
     if (lane == r) { myw = bv; myid = bi; }
   }
+  float norm = wsum;                                // renormalised: the softmax normaliser cancels
+  if (!rule.renorm) norm = rule.sigmoid ? 1.f : warp_sum(total);
   if (lane < k) {
     idx_out[lane] = myid;
-    w_out[lane] = myw / wsum;  // softmax normaliser cancels: p_i / sum p_topk
+    w_out[lane] = myw / norm;
   }
 }
 
 __global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict__ logits, int ld, int T, int E, int k,
-                                                        int* __restrict__ topk_idx, float* __restrict__ topk_w) {
+                                                        const RouteRule rule, int* __restrict__ topk_idx,
+                                                        float* __restrict__ topk_w) {
   pdl_wait();
   pdl_launch_dependents();
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (warp >= T) return;
-  route_row(logits + (size_t)warp * ld, E, k, topk_idx + (size_t)warp * k, topk_w + (size_t)warp * k, lane);
+  route_row(logits + (size_t)warp * ld, E, k, rule, topk_idx + (size_t)warp * k, topk_w + (size_t)warp * k, lane);
 }
 
 // ---------------------------------------------------------------- decode rows: router logits + routing in one launch
@@ -85,6 +143,7 @@ struct RouterRowsParams {
   float* logits;            // [M][ld]
   int M, R, H, ld, E, k;
   int shared_slot, has_gate;
+  RouteRule rule;
   int* topk_idx;            // [M][k + shared_slot]
   float* topk_w;
   int* ticket;              // one zeroed word; left zero
@@ -150,7 +209,7 @@ __global__ void __launch_bounds__(256) moe_router_rows_kernel(const RouterRowsPa
   const int stride = p.k + p.shared_slot;
   for (int m = warp; m < p.M; m += 8) {
     const float* lrow = p.logits + (size_t)m * p.ld;
-    route_row(lrow, p.E, p.k, p.topk_idx + (size_t)m * stride, p.topk_w + (size_t)m * stride, lane);
+    route_row(lrow, p.E, p.k, p.rule, p.topk_idx + (size_t)m * stride, p.topk_w + (size_t)m * stride, lane);
     if (p.shared_slot && lane == 0) {
       p.topk_idx[(size_t)m * stride + p.k] = p.E;
       p.topk_w[(size_t)m * stride + p.k] = p.has_gate ? 1.f / (1.f + __expf(-__ldcg(lrow + p.E))) : 1.f;
@@ -325,20 +384,28 @@ __global__ void __launch_bounds__(256) moe_combine_rows_kernel(const float* __re
 
 }  // namespace
 
-extern "C" int b2_moe_route(const float* logits, int ld, int T, int E, int k, int* topk_idx, float* topk_w,
-                            void* stream) {
-  if (E > 512 || k > 32 || k < 1) return -1;
+static bool route_ok(int E, int k, const RouteRule& r) {
+  if (E < 1 || E > 512 || k > 32 || k < 1) return false;
+  if (r.groups <= 1) return k <= E;
+  return r.groups <= 32 && E % r.groups == 0 && r.keep >= 1 && r.keep <= r.groups && k <= r.keep * (E / r.groups);
+}
+
+extern "C" int b2_moe_route(const float* logits, int ld, int T, int E, int k, int sigmoid, int groups, int keep, int renorm,
+                            int* topk_idx, float* topk_w, void* stream) {
+  const RouteRule rule{sigmoid, groups, keep, renorm};
+  if (!route_ok(E, k, rule)) return -1;
   const int blocks = (T * 32 + 255) / 256;
   return b2_launch(moe_route_kernel, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, true, logits, ld, T, E, k,
-                   topk_idx, topk_w);
+                   rule, topk_idx, topk_w);
 }
 
 extern "C" int b2_moe_router_rows(const void* w, const void* x, float* logits, int M, int R, int H, int ld, int E, int k,
-                                  int shared_slot, int has_gate, int* topk_idx, float* topk_w, int* ticket,
-                                  void* stream) {
-  if (E > 512 || k > 32 || k < 1 || H % 8 || M < 1 || R < E + (has_gate ? 1 : 0) || ld < R) return -1;
+                                  int shared_slot, int has_gate, int sigmoid, int groups, int keep, int renorm,
+                                  int* topk_idx, float* topk_w, int* ticket, void* stream) {
+  const RouteRule rule{sigmoid, groups, keep, renorm};
+  if (!route_ok(E, k, rule) || H % 8 || M < 1 || R < E + (has_gate ? 1 : 0) || ld < R) return -1;
   RouterRowsParams p{(const __nv_bfloat16*)w, (const __nv_bfloat16*)x, logits, M, R, H, ld, E, k, shared_slot, has_gate,
-                     topk_idx, topk_w, ticket};
+                     rule, topk_idx, topk_w, ticket};
   return b2_launch(moe_router_rows_kernel, dim3((R + 7) / 8), dim3(256), 0, (cudaStream_t)stream, true, p);
 }
 

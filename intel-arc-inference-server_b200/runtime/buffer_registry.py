@@ -35,8 +35,26 @@ def _tensors(obj):
     return {n: v for n, v in vars(obj).items() if isinstance(v, torch.Tensor)}
 
 
+def _audit_listed(buf, kv, cfg: ModelConfig, kv_dtype: str) -> Dict[str, int]:
+    """The same promise for a model that lists its layers: step scratch and latent pages within the planner's figures."""
+    groups = {"step": buf.scratch.nbytes, "kv": sum(t.numel() * t.element_size() for t in kv.latent), "state": 0}
+    for name, t in _tensors(buf).items():
+        if name not in STEP_BUFFERS:
+            raise AssertionError(f"ListedBuffers.{name} has no entry in runtime/buffer_registry.py")
+        groups["step"] += t.numel() * t.element_size()
+    planned = MP.step_scratch_bytes(cfg, buf.max_rows)
+    if groups["step"] > planned:
+        raise AssertionError(f"step buffers hold {groups['step']} bytes, the planner budgets {planned}")
+    if groups["kv"] != kv.num_pages * MP.kv_bytes_per_page(cfg, kv_dtype):
+        raise AssertionError(f"latent pool holds {groups['kv']} bytes, the planner counts "
+                             f"{kv.num_pages * MP.kv_bytes_per_page(cfg, kv_dtype)}")
+    return groups
+
+
 def audit(buf, kv, cfg: ModelConfig, kv_dtype: str = "bf16", max_seqs: int = 1) -> Dict[str, int]:
     """Checks ``buf`` (StepBuffers) and ``kv`` (KVCache) against the tables and the planner; returns bytes per group."""
+    if cfg.layer_specs:
+        return _audit_listed(buf, kv, cfg, kv_dtype)
     groups = {"step": 0, "kv": 0, "state": 0}
     for obj, table, what in ((buf, STEP_BUFFERS, "StepBuffers"), (kv, KV_BUFFERS, "KVCache")):
         for name, t in _tensors(obj).items():

@@ -35,6 +35,15 @@ class Row:
     block: int = 0      # 1: a block drafter's row, which attends to all positions of its request's rows in the step
 
 
+def _starts(entries) -> List[int]:
+    """Index of every entry's first token in the flattened step."""
+    out, n = [], 0
+    for _, toks, _ in entries:
+        out.append(n)
+        n += len(toks)
+    return out
+
+
 class Engine:
     def __init__(self, weights: ModelWeights, max_seqs: int = 1, max_len: int = 4096, kv_dtype: str = "bf16",
                  max_rows: int = 64, use_graphs: bool = True, int8_head: bool = False, num_pages: Optional[int] = None,
@@ -46,6 +55,8 @@ class Engine:
         self.tp = tp if tp is not None and tp.world > 1 else None
         self.device = weights.embed.device
         self.max_seqs, self.max_len, self.max_rows = max_seqs, max_len, max_rows
+        if cfg.layer_specs and weights.embed.dtype == torch.float32:
+            kv_dtype = "f32"        # a model served in 32-bit keeps its cache in 32-bit
         self.max_blocks = (max_len + PAGE - 1) // PAGE
         if num_pages is None:
             num_pages = max_seqs * self.max_blocks + 1
@@ -80,6 +91,7 @@ class Engine:
         if os.environ.get("B200SERVE_AUDIT", "0") == "1":     # every buffer has a planner entry (see buffer_registry.py)
             from .buffer_registry import audit
             audit(self.model.buf, self.kv, cfg, kv_dtype, max_seqs)
+        self._batch = None          # runner of mixed batches (models that list their layers)
         self.launches_per_step: Dict[Tuple[int, bool, bool], int] = {}
 
     def close(self):
@@ -172,9 +184,7 @@ class Engine:
                              "gated delta-net layers is the one after the last position)")
         pages = list(self.pool.table(slot))[begin // PAGE: (end + PAGE - 1) // PAGE]
         idx = torch.as_tensor(pages, device=self.device, dtype=torch.int64)
-        tensors = {"k": self.kv.k, "v": self.kv.v}
-        if self.kv.kv_int8:
-            tensors.update({"k_scale": self.kv.k_scale, "v_scale": self.kv.v_scale})
+        tensors = self.kv.page_tensors()
         out = {"begin": begin, "end": end, "kv_dtype": self.kv_dtype}
         if self.kv.gdn_state is not None:      # the recurrent state and the convolution window after position end - 1
             for name, t in (("gdn_conv", self.kv.gdn_conv), ("gdn_state", self.kv.gdn_state)):
@@ -196,9 +206,7 @@ class Engine:
         self._ensure_pages(slot, end)
         pages = list(self.pool.table(slot))[begin // PAGE: (end + PAGE - 1) // PAGE]
         idx = torch.as_tensor(pages, device=self.device, dtype=torch.int64)
-        tensors = {"k": self.kv.k, "v": self.kv.v}
-        if self.kv.kv_int8:
-            tensors.update({"k_scale": self.kv.k_scale, "v_scale": self.kv.v_scale})
+        tensors = self.kv.page_tensors()
         for name, t in tensors.items():
             t.index_copy_(1, idx, blob[name].to(self.device, non_blocking=True))
         if self.kv.gdn_state is not None:
@@ -300,10 +308,54 @@ class Engine:
         """fp32 logits of the last step's rows (device tensor view)."""
         return self.model.buf.logits[:m]
 
+    @property
+    def mixed_batches(self) -> bool:
+        """Prompt portions and decode rows of several requests run as one batch of any size (``forward_batch``)."""
+        return bool(self.cfg.layer_specs)
+
+    def forward_batch(self, entries: Sequence[Tuple[int, Sequence[int], Sequence[int]]]) -> torch.Tensor:
+        """One step over ``entries`` (slot, next tokens, wanted places among them): prompt portions beside decode rows of
+        other requests, each continuing its slot.  Returns the fp32 logits of the wanted places [n][vocab], in order
+        (a device tensor, valid until the next step)."""
+        self.require_ok()
+        entries = [(s, list(t), list(w)) for s, t, w in entries if len(t)]
+        n = sum(len(t) for _, t, _ in entries)
+        if n == 0:
+            return self.logits(0)
+        if n > self.max_rows and self.mixed_batches:
+            out = self._batch_runner().run(entries)
+            self.check_failed_sync("batch")
+            return out
+        got = []
+        todo = [Row(s, self.seq_len[s] + i, t) for s, toks, _ in entries for i, t in enumerate(toks)]
+        want = [j + w for j, (_, toks, ws) in zip(_starts(entries), entries) for w in ws]
+        for c0 in range(0, n, self.max_rows):      # models without mixed batches: row steps
+            part = todo[c0: c0 + self.max_rows]
+            self.forward_rows(part, advance=False, read=False)
+            sel = [w - c0 for w in want if c0 <= w < c0 + len(part)]
+            if sel:
+                got.append(self.logits(len(part))[sel] if n > self.max_rows or sel != list(range(len(part)))
+                           else self.logits(len(part)))
+        self.check_failed_sync("batch")
+        return torch.cat(got) if len(got) > 1 else (got[0] if got else self.logits(0))
+
+    def check_failed_sync(self, what: str):
+        torch.cuda.current_stream().synchronize()
+        self.check_failed(what)
+
+    def _batch_runner(self):
+        if self._batch is None:
+            from .batch import BatchRunner
+            self._batch = BatchRunner(self)
+        return self._batch
+
     def prefill(self, slot: int, ids: Sequence[int], chunk: Optional[int] = None) -> int:
         """Ingest ``ids`` after the slot's current length; returns the greedy next token."""
         self.require_ok()
         ids = list(ids)
+        if self.mixed_batches and len(ids) > self.max_rows:
+            self.last_prefill_row = 0
+            return self._batch_runner().prefill(slot, ids, chunk)
         if self._use_tc_prefill(len(ids)):
             if self._prefill is None:
                 if self.tp is not None:
@@ -335,7 +387,7 @@ class Engine:
     def _use_tc_prefill(self, n: int) -> bool:
         """Prompt chunks longer than the row kernels take go through the tcgen05 path when the shape
         has one (head size 128, bf16 KV, dense FFN or MoE with a grouped path)."""
-        if self.prefill_backend == "rows" or n <= self.max_rows:
+        if self.prefill_backend == "rows" or n <= self.max_rows or self.mixed_batches:
             return False
         if self.cfg.n_gdn_layers and (self.kv.kv_int8 or self.tp is not None or self.model.nccl is not None):
             return False        # hybrid models: the layer-major int8-KV pass and the parallel runners know no GDN layers

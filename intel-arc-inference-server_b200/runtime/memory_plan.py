@@ -49,6 +49,9 @@ class MemoryPlan:
 
 def weight_bytes(cfg: ModelConfig, int8_head: bool = False, tp: int = 1, ep: int = 1) -> int:
     h = cfg.hidden
+    if cfg.layer_specs:
+        from ..models.latent import padded_weight_elems
+        return int(padded_weight_elems(cfg) * 2)
     int4 = 0.5 + 2.0 / 64
     per = cfg._mixer_params() * int4 / tp      # attention projections, or a gated delta-net layer's (mean over layers)
     if cfg.is_moe:
@@ -62,6 +65,9 @@ def weight_bytes(cfg: ModelConfig, int8_head: bool = False, tp: int = 1, ep: int
 
 
 def kv_bytes_per_page(cfg: ModelConfig, kv_dtype: str, tp: int = 1) -> int:
+    if cfg.layer_specs:
+        from ..models.latent import LatentGeometry
+        return sum(LatentGeometry.of(s.mixer).lc for s in cfg.layer_specs) * cfg.page_size * (4 if kv_dtype == "f32" else 2)
     per_tok_head = cfg.head_dim * (1 if kv_dtype == "int8" else 2) + (4 if kv_dtype == "int8" else 0)
     return (cfg.n_layers - cfg.n_gdn_layers + cfg.mtp_layers) * 2 * (cfg.n_kv_heads // tp) * per_tok_head * cfg.page_size
 
@@ -77,6 +83,9 @@ def gdn_state_bytes_per_slot(cfg: ModelConfig) -> int:
 
 def step_scratch_bytes(cfg: ModelConfig, max_rows: int = 64, nsplit: int = 32) -> int:
     h = cfg.hidden
+    if cfg.layer_specs:
+        from ..models.latent import step_scratch_elems
+        return max_rows * cfg.vocab * 4 + 4 * step_scratch_elems(cfg, max_rows) + (1 << 16)
     b = max_rows * (2 * h * 2 + 2 * cfg.q_dim * 2 + cfg.vocab * 4)
     b += max_rows * cfg.n_q_heads * nsplit * (cfg.head_dim + 2) * 4
     b += 16 * max_rows * (cfg.qkv_dim + 2 * h + 2 * max(cfg.ffn, cfg.expert_ffn * max(cfg.top_k, 1))) * 4
@@ -89,6 +98,9 @@ def step_scratch_bytes(cfg: ModelConfig, max_rows: int = 64, nsplit: int = 32) -
 
 def prefill_scratch_bytes(cfg: ModelConfig, chunk: int, backend: str) -> int:
     h = cfg.hidden
+    if cfg.layer_specs:      # rows of a mixed batch, and expanded keys / values of a window before it
+        from ..models.latent import step_scratch_elems
+        return 4 * step_scratch_elems(cfg, chunk, keys=2 * chunk)
     ffn = cfg.ffn if not cfg.is_moe else max(cfg.expert_ffn, cfg.shared_ffn)
     b = chunk * (2 * h * 2 + cfg.qkv_dim * 4 + 2 * cfg.q_dim * 2 + ffn * 2)
     biggest = max(cfg.qkv_dim * h, h * cfg.q_dim, 2 * ffn * h)
@@ -110,6 +122,8 @@ def plan(cfg: ModelConfig, max_seqs: int, max_len, kv_dtype: str = "bf16", int8_
     budget = budget or device_budget()
     w = weight_bytes(cfg, int8_head, tp, ep)
     resident = 0
+    if cfg.layer_specs:
+        prefill_backend = "listed"      # unquantised weights: the batch path reads them as they are
     if prefill_backend == "auto":    # the prompt pass keeps bf16 copies when they take at most 45 % of the memory
         prefill_backend = "bf16-resident" if 2 * cfg.param_count() / max(tp * ep, 1) <= 0.45 * budget else "bf16"
     if prefill_backend == "bf16-resident":

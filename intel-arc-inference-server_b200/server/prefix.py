@@ -46,7 +46,7 @@ class EngineKV:
         self.e = engine
         self.torch = torch
         kv = engine.kv
-        self.tensors = [kv.k, kv.v] + ([kv.k_scale, kv.v_scale] if kv.kv_int8 else [])
+        self.tensors = list(kv.page_tensors().values())
         self.page_bytes = sum(int(t[:, 0].numel()) * t.element_size() for t in self.tensors)
         self.form = f"{engine.kv_dtype}/{engine.cfg.name}"
 
