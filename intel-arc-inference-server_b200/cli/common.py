@@ -91,6 +91,8 @@ def parallel_auto(cfg, n_gpus: int, mem_bytes: int, max_seqs: int = 1, kv_dtype:
         if n > n_gpus:
             break
         heads_ok = cfg.n_kv_heads % n == 0 and cfg.n_q_heads % n == 0 and not cfg.n_gdn_layers
+        if cfg.layer_specs:
+            break           # one GPU only
         if cfg.is_moe and cfg.n_experts % n == 0 and fits(ep=n):
             return f"ep{n}"
         if not cfg.is_moe and heads_ok and fits(tp=n):
@@ -98,14 +100,23 @@ def parallel_auto(cfg, n_gpus: int, mem_bytes: int, max_seqs: int = 1, kv_dtype:
     raise SystemExit(f"{cfg.name} does not fit on {n_gpus} GPU(s) of {mem_bytes / 2**30:.0f} GiB in any placement")
 
 
-def load_model(spec: str, device, seed: int = 0, int8_head: bool = False, tp=(0, 1)):
-    """A preset name gives random-init weights in that shape; anything else is a snapshot."""
+def load_model(spec: str, device, seed: int = 0, int8_head: bool = False, tp=(0, 1), dtype: str = "bfloat16"):
+    """A preset name gives random-init weights in that shape; anything else is a snapshot.  ``dtype`` float32: served in
+    32-bit (models that list their layers)."""
+    cfg = peek_config(spec)
+    if cfg.layer_specs and (int8_head or tp[1] != 1):
+        raise SystemExit(f"{cfg.name} runs on one GPU with an unquantised head")
+    if dtype != "bfloat16" and not cfg.layer_specs:
+        raise SystemExit(f"{cfg.name}: this family is served in bfloat16 only")
+    if spec in PRESETS and cfg.layer_specs:
+        from ..models.latent import random_listed_weights
+        sys.stderr.write(f"load: preset {spec} with random-init {dtype} weights (seed {seed})\n")
+        return random_listed_weights(cfg, device, seed, dtype=getattr(torch, dtype))
     if spec in PRESETS:
-        cfg = preset(spec)
         sys.stderr.write(f"load: preset {spec} with random-init W4A16 weights (seed {seed})\n")
         return random_weights(cfg, device=device, seed=seed)
     from ..loader.loader import load
-    return load(spec, device=device, int8_head=int8_head, tp=tp)
+    return load(spec, device=device, int8_head=int8_head, tp=tp, dtype=dtype)
 
 
 def find_tokenizer(spec: str):

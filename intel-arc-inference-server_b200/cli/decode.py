@@ -36,7 +36,7 @@ def main(argv=None):
     from . import common
     common.hardware_gate(1)
     torch.cuda.set_device(0)
-    w = common.load_model(f.model, "cuda", f.seed, f.int8_head)
+    w = common.load_model(f.model, "cuda", f.seed, f.int8_head, dtype=f.dtype)
     cfg = w.cfg
     depth = f.depth if (f.bench or f.profile) else 0
     ids = _ids(f.ids) if f.ids else None
@@ -103,6 +103,13 @@ def _profile(eng, f, first):
     raw = {}
     names = [n for n in dir(K) if callable(getattr(K, n)) and n in (
         "gemv_w4", "resid_norm", "rope_append", "attn_decode", "head_gemv", "argmax_finish")]
+    mods = {n: K for n in names}
+    if eng.cfg.layer_specs:
+        from ..ops import latent as L, moe as M
+        mods.update({n: L for n in ("embed_rows", "gemv_bf16", "prep", "absorb", "rows", "simple", "merge", "sublayer_norm",
+                                    "gemv_bf16_experts", "layer_norm_rows", "linear_f32", "linear_f32_experts")})
+        mods["router_rows"] = M
+        names = list(mods)
     pending = []
 
     def wrap(name, fn):
@@ -115,8 +122,8 @@ def _profile(eng, f, first):
             return r
         return inner
     for n in names:
-        raw[n] = getattr(K, n)
-        setattr(K, n, wrap(n, raw[n]))
+        raw[n] = getattr(mods[n], n)
+        setattr(mods[n], n, wrap(n, raw[n]))
     try:
         eng.use_graphs = False
         pos, tok = eng.seq_len[0], first
@@ -131,7 +138,7 @@ def _profile(eng, f, first):
                 times.setdefault(name, []).append(e0.elapsed_time(e1) * 1e3)
     finally:
         for n in names:
-            setattr(K, n, raw[n])
+            setattr(mods[n], n, raw[n])
     print("| kernel family | launches/step | us/step (mean) | share |")
     print("|---|---|---|---|")
     tot = sum(sum(v) for v in times.values()) / f.steps

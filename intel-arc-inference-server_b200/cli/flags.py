@@ -47,7 +47,8 @@ def parse(cls, argv, prog: str, description: str):
 class ServeFlags:
     """Flags of ``b200-serve`` (the reference's b70-serve surface, src/cli/b70_serve.cc:83-147)."""
     model: Optional[str] = flag(None, "snapshot directory, Hugging Face repo id, or a preset name "
-                                      "(tiny-dense, small-dense, dense-27b, moe-35b-a3b) with random weights",
+                                      "(tiny-dense, small-dense, dense-27b, moe-35b-a3b, mumusun-16b) with random "
+                                      "weights",
                                 positional=True)
     spec: str = flag("auto", "speculative decoding", ["auto", "off", "mtp", "dflash", "lookup", "dflash-lookup"])
     spec_max: int = flag(3, "most drafts per step")
@@ -65,6 +66,7 @@ class ServeFlags:
     kv_cache: str = flag("bf16", "KV cache element type", ["bf16", "int8"])
     prefill_backend: str = flag("auto", "prompt-pass GEMM path",
                                 ["auto", "w4", "bf16", "bf16-resident", "int8", "l0", "l0-int8", "rows"])
+    dtype: str = flag("bfloat16", "element type; float32 serves a Mumusun model in 32-bit", ["bfloat16", "float32"])
     int8_head: bool = flag(False, "quantise lm_head to int8 with per-row scales")
     draft_vocab: int = flag(0, "reduced draft vocabulary size (0: full)")
     draft_vocab_ids: Optional[str] = flag(None, "file with the ranked ids of the draft vocabulary")
@@ -91,5 +93,6 @@ class DecodeFlags:
     repeats: int = flag(3, "--profile / --bench: repetitions, the median is reported")
     kv_cache: str = flag("bf16", "KV cache element type", ["bf16", "int8"])
     prefill_backend: str = flag("auto", "prompt-pass GEMM path", ["auto", "w4", "bf16", "bf16-resident", "int8", "rows"])
+    dtype: str = flag("bfloat16", "element type; float32 runs a Mumusun model in 32-bit", ["bfloat16", "float32"])
     int8_head: bool = flag(False, "int8 lm_head")
     seed: int = flag(0, "seed of random-init weights (preset models)")

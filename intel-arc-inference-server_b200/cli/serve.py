@@ -42,13 +42,14 @@ def main(argv=None):
         from ..parallel.launch import serve_parallel
         return serve_parallel(f, par, world)
     torch.cuda.set_device(0)
-    weights = common.load_model(f.model, "cuda", f.seed, f.int8_head)
+    weights = common.load_model(f.model, "cuda", f.seed, f.int8_head, dtype=f.dtype)
     cfg = weights.cfg
     backend = {"l0": "bf16", "l0-int8": "int8"}.get(f.prefill_backend, f.prefill_backend)
-    mp = plan(cfg, f.max_num_seqs, f.max_len if f.max_len == "auto" else int(f.max_len), f.kv_cache, f.int8_head,
+    kv_form = "f32" if f.dtype == "float32" else f.kv_cache
+    mp = plan(cfg, f.max_num_seqs, f.max_len if f.max_len == "auto" else int(f.max_len), kv_form, f.int8_head,
               backend, budget=torch.cuda.get_device_properties(0).total_memory)
     sys.stderr.write(mp.line() + "\n")
-    engine = Engine(weights, max_seqs=f.max_num_seqs, max_len=mp.max_len, kv_dtype=f.kv_cache,
+    engine = Engine(weights, max_seqs=f.max_num_seqs, max_len=mp.max_len, kv_dtype=kv_form,
                     int8_head=f.int8_head, prefill_backend=backend, num_pages=mp.num_pages)
     tok = common.find_tokenizer(f.model)
     template = ChatTemplate.from_snapshot(f.model) if f.model not in PRESETS else ChatTemplate()

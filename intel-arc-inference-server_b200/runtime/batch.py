@@ -22,6 +22,23 @@ SEGMENT = 32        # tokens from which an entry is attended as a prompt segment
 ALIGN = 4           # int32 words: table parts start on 16-byte boundaries
 
 
+def segment_keys(segments: Sequence[Tuple[int, int, int]], window: int, per: int):
+    """Key rows and query tiles of prompt segments (slot, first position, rows): the slots and positions of every key some
+    row of its segment sees, segment after segment, and tiles of at most ``per`` query rows as (first query row, rows,
+    position of that row and key row of position 0, both counted from the segment's first key)."""
+    kreq, kpos, tiles = [], [], []
+    krow = qrow = 0
+    for slot, p, n in segments:
+        lo = max(0, p - window + 1) if window else 0       # first position any of the segment's rows sees
+        kreq.append(np.full(p + n - lo, slot))
+        kpos.append(np.arange(lo, p + n))
+        tiles += [(qrow + r, min(per, n - r), p + r - lo, krow) for r in range(0, n, per)]
+        krow += p + n - lo
+        qrow += n
+    tiles.sort(key=lambda t: -(t[2] + t[1]))               # tiles with many keys first
+    return np.concatenate(kreq), np.concatenate(kpos), tiles
+
+
 class BatchRunner:
     def __init__(self, engine, max_tokens: int = 4096):
         self.eng, self.max_tokens = engine, max_tokens
@@ -49,19 +66,8 @@ class BatchRunner:
                  "token": add(np.concatenate([np.asarray(t) for _, _, t in both])), "want": add(want)}
         keys = {}
         for window, per in self.forms if segments else ():
-            kreq, kpos, tiles = [], [], []
-            krow = qrow = 0
-            for slot, p, toks in segments:
-                n = len(toks)
-                lo = max(0, p - window + 1) if window else 0       # first position any of the segment's rows sees
-                kreq.append(np.full(p + n - lo, slot))
-                kpos.append(np.arange(lo, p + n))
-                for r in range(0, n, per):
-                    tiles.append((qrow + r, min(per, n - r), p + r - lo, krow))
-                krow += p + n - lo
-                qrow += n
-            tiles.sort(key=lambda t: -(t[2] + t[1]))               # tiles with many keys first
-            keys[(window, per)] = (krow, add(np.concatenate(kreq)), add(np.concatenate(kpos)), len(tiles), add(tiles))
+            kreq, kpos, tiles = segment_keys([(s, p, len(t)) for s, p, t in segments], window, per)
+            keys[(window, per)] = (len(kreq), add(kreq), add(kpos), len(tiles), add(tiles))
         return np.concatenate(parts), spans, keys
 
     def _walk(self, entries: Sequence[Tuple[int, List[int]]], want: Sequence[Tuple[int, int]]):

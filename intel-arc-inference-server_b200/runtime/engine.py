@@ -11,6 +11,7 @@ sequence is.
 """
 from __future__ import annotations
 
+import gc
 from dataclasses import dataclass
 from typing import Dict, List, Optional, Sequence, Tuple
 
@@ -243,8 +244,16 @@ class Engine:
                 self.kv.gdn_conv.copy_(saved_gdn[0])
                 self.kv.gdn_state.copy_(saved_gdn[1])
             g = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(g):
-                self._enqueue(m, advance)
+            # no garbage collection while the stream captures: a dead engine's graphs and buffers released in the middle
+            # of it abort the process
+            collects = gc.isenabled()
+            gc.disable()
+            try:
+                with torch.cuda.graph(g):
+                    self._enqueue(m, advance)
+            finally:
+                if collects:
+                    gc.enable()
             self.ctrl.copy_(saved)
             self.graphs[key] = g
         g.replay()
@@ -338,6 +347,15 @@ class Engine:
                            else self.logits(len(part)))
         self.check_failed_sync("batch")
         return torch.cat(got) if len(got) > 1 else (got[0] if got else self.logits(0))
+
+    def argmax(self, logits: torch.Tensor) -> List[int]:
+        """Arg-max of fp32 logit rows (ties to the lower id)."""
+        from ..ops import latent as L
+        m, n = logits.shape
+        val = torch.empty(m, dtype=torch.float32, device=logits.device)
+        idx = torch.empty(m, dtype=torch.int32, device=logits.device)
+        L.row_argmax(logits, m, n, val, idx)
+        return idx.tolist()
 
     def check_failed_sync(self, what: str):
         torch.cuda.current_stream().synchronize()

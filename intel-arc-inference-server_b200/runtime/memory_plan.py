@@ -121,6 +121,8 @@ def plan(cfg: ModelConfig, max_seqs: int, max_len, kv_dtype: str = "bf16", int8_
     numbers when it cannot fit."""
     budget = budget or device_budget()
     w = weight_bytes(cfg, int8_head, tp, ep)
+    if cfg.layer_specs and kv_dtype == "f32":      # served in 32-bit
+        w *= 2
     resident = 0
     if cfg.layer_specs:
         prefill_backend = "listed"      # unquantised weights: the batch path reads them as they are

@@ -316,7 +316,7 @@ class SpecAdapter:
         self.inner = inner
         self.e: Engine = inner.e
         self.spec, self.k_max = spec, spec_max
-        if self.e.cfg.is_moe:
+        if self.e.cfg.is_moe or self.e.cfg.layer_specs:
             # never validated: the one run of a draft head over a mixture-of-experts trunk ended in an illegal memory
             # access, so the combination is refused until its cause is found
             raise NotImplementedError("draft heads (--spec mtp / dflash) are not available for mixture-of-experts models; "

@@ -26,6 +26,7 @@ class EngineAdapter(EngineIface):
         self.eos_ids = tuple(eos_ids)
         self._rows_of: Dict[int, range] = {}
         self._logits_host = None
+        self._logits_dev = None     # logits of the last mixed batch (else the engine's step buffer holds them)
         self._samp = None       # (pinned host words, device words, device out) of the device sampler
 
     def reset(self, slot):
@@ -48,8 +49,29 @@ class EngineAdapter(EngineIface):
         tok = self.e.prefill(slot, list(ids))
         r = self.e.last_prefill_row
         self._rows_of = {slot: range(r, r + 1)}
-        self._logits_host = None
+        self._logits_host = self._logits_dev = None
         return tok
+
+    @property
+    def mixed_batches(self):
+        return self.e.mixed_batches
+
+    def step_mixed(self, slot, ids, rows: Dict[int, List[int]]):
+        entries, spans, n = [], {}, 0
+        for s, toks in rows.items():
+            spans[s] = range(n, n + len(toks))
+            n += len(toks)
+            entries.append((s, [int(t) for t in toks], list(range(len(toks)))))
+        entries.append((slot, list(ids), [len(ids) - 1]))
+        spans[slot] = range(n, n + 1)
+        lg = self.e.forward_batch(entries)
+        out = self.e.argmax(lg)
+        self._rows_of, self._logits_host, self._logits_dev = spans, None, lg
+        return out[n], {s: [out[i] for i in spans[s]] for s in rows}
+
+    def _device_logits(self):
+        n = max(r.stop for r in self._rows_of.values())
+        return self.e.logits(n) if self._logits_dev is None else self._logits_dev[:n]
 
     def step(self, rows: Dict[int, List[int]]):
         flat, spans = [], {}
@@ -59,13 +81,12 @@ class EngineAdapter(EngineIface):
             flat += [Row(slot, base + i, int(t)) for i, t in enumerate(toks)]
         out = self.e.forward_rows(flat, advance=False, read=True)
         self._rows_of = spans
-        self._logits_host = None
+        self._logits_host = self._logits_dev = None
         return {slot: [out[i] for i in span] for slot, span in spans.items()}
 
     def logits(self, slot, row=0):
         if self._logits_host is None:
-            n = max(r.stop for r in self._rows_of.values())
-            self._logits_host = self.e.logits(n).float().cpu().numpy()
+            self._logits_host = self._device_logits().float().cpu().numpy()
         return self._logits_host[self._rows_of[slot][row]]
 
     def logits_shard(self, slot, row=0):
@@ -106,7 +127,7 @@ class EngineAdapter(EngineIface):
             host[self._SAMP_HEAD: self._SAMP_HEAD + len(hist)] = torch.tensor(hist, dtype=torch.int32)
         n = self._SAMP_HEAD + len(hist)
         dev[:n].copy_(host[:n], non_blocking=True)
-        lg = self.e.logits(max(r.stop for r in self._rows_of.values()))[self._rows_of[slot][row]: self._rows_of[slot][row] + 1]
+        lg = self._device_logits()[self._rows_of[slot][row]: self._rows_of[slot][row] + 1]
         df = dev[:4].view(torch.float32)
         K.sample_rows(lg, 1, self.vocab_size, df[0:1], dev[1:2], df[2:3], dev[4:6], out[0:1], out[1:2],
                       penalty=df[3:4] if hist else None, hist=dev[self._SAMP_HEAD:].view(1, -1) if hist else None,

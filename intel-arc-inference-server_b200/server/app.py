@@ -188,11 +188,16 @@ class Server:
                 if s.slot < 0:      # still waiting for a slot: no release action will come for it
                     self.http.close(s.http_id)
                     self.sessions.pop(s.http_id, None)
-        for a in self.sched.tick():
+        acts = list(self.sched.tick())
+        mixed = getattr(self.engine, "mixed_batches", False)
+        while acts:
+            a = acts.pop(0)
+            # a prompt chunk and the decode rows of the same tick run as one batch where the engine can
+            b = acts.pop(0) if mixed and a["kind"] == "prefill" and acts and acts[0]["kind"] == "decode" else None
             try:
-                self._act(a)
+                self._act(a) if b is None else self._mixed(a, b)
             except Exception as e:  # noqa: BLE001   (whatever a request trips over fails that request, not the server)
-                slots = [a["slot"]] if "slot" in a else list(a.get("slots", ()))
+                slots = ([a["slot"]] if "slot" in a else list(a.get("slots", ()))) + (list(b["slots"]) if b else [])
                 for slot in slots:
                     s = self.by_slot.get(slot)
                     if s is not None and not s.finished:
@@ -227,6 +232,24 @@ class Server:
         except Exception as e:  # noqa: BLE001
             self._fail(s, e)
             return self._recover_engine()
+        self._prefill_done(a, s, tok)
+
+    def _mixed(self, a, b):
+        """A prompt chunk and a decode step as one engine call (engines with ``mixed_batches``)."""
+        rows, s_q = self._decode_rows(b)
+        if not rows:
+            return self._prefill(a)
+        s = self.by_slot[a["slot"]]
+        try:
+            tok, res = self.engine.step_mixed(s.slot, s.prompt_ids[a["begin"]: a["end"]], rows)
+        except Exception as e:  # noqa: BLE001   (one step: it fails for everyone in it)
+            for slot in [s.slot] + list(rows):
+                self._fail(self.by_slot[slot], e)
+            return self._recover_engine()
+        self._prefill_done(a, s, tok)
+        self._decode_done(rows, res, s_q)
+
+    def _prefill_done(self, a, s: Session, tok: int):
         self.sched.prefill_done(s.slot, a["end"])
         if a["last"]:
             if self.prefix:
@@ -257,6 +280,20 @@ class Server:
         return int(H.sample(lg, self.engine.vocab_size, r.temperature, r.top_k, r.top_p, seed))
 
     def _decode(self, a):
+        rows, s_q = self._decode_rows(a)
+        if not rows:
+            return
+        try:
+            res = self.engine.step(rows)
+        except Exception as e:  # noqa: BLE001   (a failing step fails its rows, not the server)
+            for slot in rows:
+                self._fail(self.by_slot[slot], e)
+            self._recover_engine()
+            return
+        self._decode_done(rows, res, s_q)
+
+    def _decode_rows(self, a):
+        """The step's rows per slot (pending token, then drafts) and the drafts' distributions where they were drawn."""
         rows = {}
         ask = {}       # slot -> (pending, k, temperature, seed): drafts the engine's head makes, all slots in one call
         for slot, n in zip(a["slots"], a["rows"]):
@@ -278,15 +315,9 @@ class Server:
                 rows[slot] = rows[slot] + [int(t) for t in drafts]
                 if ask[slot][2] > 0 and hasattr(self.engine, "draft_q"):
                     s_q[slot] = self.engine.draft_q(slot)
-        if not rows:
-            return
-        try:
-            res = self.engine.step(rows)
-        except Exception as e:  # noqa: BLE001   (a failing step fails its rows, not the server)
-            for slot in rows:
-                self._fail(self.by_slot[slot], e)
-            self._recover_engine()
-            return
+        return rows, s_q
+
+    def _decode_done(self, rows, res, s_q):
         for slot, toks in rows.items():
             s = self.by_slot[slot]
             out = res[slot]

@@ -17,6 +17,7 @@ class EngineIface:
     max_len: int = 0
     max_seqs: int = 1
     eos_ids: Sequence[int] = ()
+    mixed_batches: bool = False       # the engine has ``step_mixed``
 
     def reset(self, slot: int) -> None: ...
     def length(self, slot: int) -> int: ...
@@ -26,6 +27,8 @@ class EngineIface:
     def step(self, rows: Dict[int, List[int]]) -> Dict[int, List[int]]:
         """For every slot, run its row tokens at consecutive positions (the first is the pending token,
         the rest are drafts); returns the arg-max after each row."""
+    def step_mixed(self, slot: int, ids: Sequence[int], rows: Dict[int, List[int]]):
+        """``prefill(slot, ids)`` and ``step(rows)`` as one batch; returns (token, step result)."""
     def logits(self, slot: int, row: int = 0) -> np.ndarray:
         """fp32 logits of ``row`` of ``slot`` from the last prefill / step (for host sampling)."""
     def kv_form(self) -> str:
@@ -98,6 +101,11 @@ class MockEngine(EngineIface):
             out[slot] = res
             self._logits[slot] = lg
         return out
+
+    def step_mixed(self, slot, ids, rows):
+        self.mixed_steps = getattr(self, "mixed_steps", 0) + 1
+        out = self.step(rows)
+        return self.prefill(slot, ids), out
 
     def logits(self, slot, row=0):
         return self._logits[slot][row]

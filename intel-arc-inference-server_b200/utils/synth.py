@@ -158,3 +158,20 @@ def write_drafter(head, cfg: ModelConfig, path: str, fmt: str = "int4", prefix: 
     with open(os.path.join(path, "config.json"), "w") as f:
         json.dump(hf, f, indent=1)
     return path
+
+
+def write_listed(cfg: ModelConfig, path: str, seed: int = 0, make=None) -> Dict[str, torch.Tensor]:
+    """A snapshot of a model that lists its layers (``config.json`` in the design's keys, one safetensors file) with
+    random weights; ``make(name, tensor)`` may replace a tensor.  Returns the tensors written."""
+    from ..models.latent import tensor_shapes
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in tensor_shapes(cfg).items():
+        t = 1.0 + 0.2 * torch.randn(shape, generator=g) if len(shape) == 1 else torch.randn(shape, generator=g) * (
+            1.0 if name == "embed" else shape[1] ** -0.5)
+        out[name] = (t if make is None else make(name, t)).to(torch.bfloat16)
+    os.makedirs(path, exist_ok=True)
+    save_file(out, os.path.join(path, "model.safetensors"))
+    with open(os.path.join(path, "config.json"), "w") as f:
+        json.dump(cfg.to_listed_config(), f)
+    return out
