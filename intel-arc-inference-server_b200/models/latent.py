@@ -16,6 +16,7 @@ weights are fp32 run everything in 32-bit (no reduced-precision product anywhere
 """
 from __future__ import annotations
 
+import os
 from dataclasses import dataclass
 from typing import Callable, Dict, Optional
 
@@ -30,6 +31,9 @@ from .oracle import rope_tables
 from .weights import ExpertStack, LatentWeights, LayerWeights, ModelWeights, interleave16
 
 SMS = 148
+# Experts of more rows than this go through the expert-sorted grouped GEMMs, which read every chosen expert once; the
+# GEMVs read one expert per (row, slot).
+EXPERT_GEMV_ROWS = int(os.environ.get("B2_EXPERT_GEMV_ROWS", "4"))
 
 
 def pad64(n: int) -> int:
@@ -275,12 +279,12 @@ class ListedLayers:
         return self._rows_form[g]
 
     def nsplit(self, a: LatentAttention, g: LatentGeometry, m: int) -> int:
-        """KV splits of the decode attention: about one CTA per SM, at least two key tiles per split."""
+        """KV splits of the decode attention: about one CTA per SM, at least one key tile per split."""
         if not self.rows_form(g):
             return 1
         keys = min(a.window, self.max_pos) if a.window else self.max_pos
         groups = (a.heads + 31) // 32 if a.heads > 16 else 1
-        return max(1, min(32, SMS // (m * groups), (keys + 127) // 128))
+        return max(1, min(64, SMS // (m * groups), (keys + 63) // 64))
 
     def linear(self, sc: ListedScratch, name: str, w: torch.Tensor, x: torch.Tensor, m: int):
         """fp32 ``x[:m] @ w.T`` as (slices [s][m][n], s)."""
@@ -350,8 +354,8 @@ class ListedLayers:
         h = sc.get("h", m, wp)
         logits = sc.get("router", m, er, f32)
         idx, wt = sc.get("topk_idx", m, k, i32), sc.get("topk_w", m, k, f32)
-        few = m <= L.GEMV_ROWS
-        if not self.f32 and few:
+        few = m <= EXPERT_GEMV_ROWS
+        if not self.f32 and m <= L.GEMV_ROWS:
             M.router_rows(w.router, h, logits, m, f.experts, wp, er, f.experts, k, False, False, idx, wt,
                           sc.get("ticket", 1, 1, i32), rule=f.rule)
         else:

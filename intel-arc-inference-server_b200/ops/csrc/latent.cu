@@ -72,24 +72,42 @@ struct PrepParams {
   void* cache;           // [page][16][kvp + rp]
 };
 
+constexpr int kRopeShared = 128;    // angle pairs kept in shared memory
+
 template <typename T>
 __global__ void __launch_bounds__(512) latent_prep_kernel(const PrepParams p) {
-  extern __shared__ float v[];       // the row's qp + kvp + rp values
+  extern __shared__ __align__(16) float v[];       // the row's qp + kvp + rp values
   __shared__ float red[2][16];
   pdl_launch_dependents();
   pdl_wait();
+  __shared__ float s_cos[kRopeShared], s_sin[kRopeShared];
   const int m = blockIdx.x, n = p.qp + p.kvp + p.rp, tid = threadIdx.x, nw = blockDim.x >> 5;
+  const int pos = p.rows.pos[m], req = p.rows.req[m];
   float sq = 0.f, sc = 0.f;
   for (int i = tid * 4; i < n; i += blockDim.x * 4) {
-    float4 a = *reinterpret_cast<const float4*>(p.part + (size_t)m * n + i);
-    for (int s = 1; s < p.S; ++s) {
-      const float4 b = *reinterpret_cast<const float4*>(p.part + ((size_t)s * p.M + m) * n + i);
-      a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w;
-    }
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b[8];
+#pragma unroll
+    for (int s = 0; s < 8; ++s)          // every slice's value requested before the first is used (S <= 8)
+      b[s] = s < p.S ? __ldcg(reinterpret_cast<const float4*>(p.part + ((size_t)s * p.M + m) * n + i)) : a;
+#pragma unroll
+    for (int s = 0; s < 8; ++s) { a.x += b[s].x; a.y += b[s].y; a.z += b[s].z; a.w += b[s].w; }
     *reinterpret_cast<float4*>(v + i) = a;
     const float q = a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;   // padding columns are zero
     if (i < p.qp) sq += q;
     else if (i < p.qp + p.kvp) sc += q;
+  }
+  // the page and the angles while the slices arrive
+  const int page = p.block_table[(size_t)req * p.max_blocks + (pos >> 4)], half = p.rope.dims >> 1;
+  Rope rope = p.rope;
+  int rope_pos = pos;
+  if (half <= kRopeShared) {
+    for (int i = tid; i < half; i += blockDim.x) {
+      s_cos[i] = p.rope.cos_t[(size_t)pos * half + i];
+      s_sin[i] = p.rope.sin_t[(size_t)pos * half + i];
+    }
+    rope.cos_t = s_cos;
+    rope.sin_t = s_sin;
+    rope_pos = 0;
   }
   sq = warp_sum(sq);
   sc = warp_sum(sc);
@@ -98,15 +116,14 @@ __global__ void __launch_bounds__(512) latent_prep_kernel(const PrepParams p) {
   sq = sc = 0.f;
   for (int i = 0; i < nw; ++i) { sq += red[0][i]; sc += red[1][i]; }
   const float rq = 1.f / sqrtf(sq / (float)p.q_rank + p.eps), rc = 1.f / sqrtf(sc / (float)p.kv_rank + p.eps);
-  const int pos = p.rows.pos[m], lc = p.kvp + p.rp;
+  const int lc = p.kvp + p.rp;
   T* cq = reinterpret_cast<T*>(p.cq) + (size_t)m * p.qp;
   for (int i = tid; i < p.qp; i += blockDim.x) cq[i] = from_f<T>(i < p.q_rank ? v[i] * rq * p.q_norm[i] : 0.f);
-  const int page = p.block_table[(size_t)p.rows.req[m] * p.max_blocks + (pos >> 4)];
   T* dst = reinterpret_cast<T*>(p.cache) + ((size_t)page * 16 + (pos & 15)) * lc;
   for (int i = tid; i < lc; i += blockDim.x) {
     float o = 0.f;
     if (i < p.kv_rank) o = v[p.qp + i] * rc * p.kv_norm[i];
-    else if (i >= p.kvp && i - p.kvp < p.rot) o = rope_at(v + p.qp + p.kvp, i - p.kvp, pos, p.rope);
+    else if (i >= p.kvp && i - p.kvp < p.rot) o = rope_at(v + p.qp + p.kvp, i - p.kvp, rope_pos, rope);
     dst[i] = from_f<T>(o);
   }
 }
@@ -129,6 +146,13 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const AbsorbParams p
   const int dk = p.dn + p.rp, lc = p.kvp + p.rp, tid = threadIdx.x;
   float* qs = sm;
   float* red = sm + 8 * dk;
+  const int sl = tid >> 6, r = r0 + (tid & 63) * 2, per = p.dn / 4;
+  const T* w = reinterpret_cast<const T*>(p.w_uk) + ((size_t)h * p.dn + sl * per) * p.kvp + r;
+  float2 wv[16];           // the first weights do not wait for the queries
+  if (r < p.kvp) {
+#pragma unroll
+    for (int u = 0; u < 16; ++u) wv[u] = load2(w + (size_t)u * p.kvp);
+  }
   pdl_launch_dependents();
   pdl_wait();
   for (int i = tid; i < 8 * dk; i += 256) {
@@ -139,18 +163,12 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const AbsorbParams p
     qs[i] = a;
   }
   __syncthreads();
-  const int sl = tid >> 6, r = r0 + (tid & 63) * 2;
   float acc[8][2];
 #pragma unroll
   for (int m = 0; m < 8; ++m) acc[m][0] = acc[m][1] = 0.f;
   if (r < p.kvp) {
-    const int per = p.dn / 4;
-    const T* w = reinterpret_cast<const T*>(p.w_uk) + ((size_t)h * p.dn + sl * per) * p.kvp + r;
     const float* q = qs + sl * per;
     for (int d = 0; d < per; d += 16) {      // dn is a multiple of 64
-      float2 wv[16];
-#pragma unroll
-      for (int u = 0; u < 16; ++u) wv[u] = load2(w + (size_t)(d + u) * p.kvp);
 #pragma unroll
       for (int m = 0; m < 8; ++m)
         if (m < mt) {
@@ -161,6 +179,10 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const AbsorbParams p
             acc[m][1] = fmaf(qv, wv[u].y, acc[m][1]);
           }
         }
+      if (d + 16 < per) {
+#pragma unroll
+        for (int u = 0; u < 16; ++u) wv[u] = load2(w + (size_t)(d + 16 + u) * p.kvp);
+      }
     }
   }
 #pragma unroll
@@ -220,12 +242,14 @@ __device__ __forceinline__ void split_range(int pos, int window, int nsplit, int
   hi = min(pos + 1, lo + pps * 16);
 }
 
-// MT: tiles of 16 heads per CTA.  Scores: the eight warps are MT head tiles x 8 / MT slices of the tile's keys; product
+// MT: tiles of 16 heads per CTA; KVC: blocks of 64 latent dims; QREG: the queries' fragments stay in registers (one head
+// tile, one block of rotated dims), which saves each warp reading them from shared memory again for every tile.  Scores: the eight warps are MT head tiles x 8 / MT slices of the tile's keys; product
 // with the values: MT head tiles x 8 / MT slices of the latent's dims.  The weights pass between the two through shared
 // memory as bf16 limbs (hi + lo).  Two tiles of keys in flight.
-template <int MT>
+template <int MT, int KVC, bool QREG>
 __global__ void __launch_bounds__(kRowsThreads, 1) latent_rows_kernel(const __grid_constant__ RowsParams p) {
-  constexpr int QR = MT * 16, NSL = 8 / MT, KSL = KT / NSL, NJ = KSL / 8, MAXT = 8 * MT;
+  constexpr int QR = MT * 16, NSL = 8 / MT, KSL = KT / NSL, NJ = KSL / 8;
+  constexpr int NT = KVC * MT, DW = NT * 8;        // this warp's slice of the latent's dims: NT groups of 8
   extern __shared__ uint8_t smem_raw[];
   __shared__ float s_mx[QR][NSL];
   const int nc = p.lc >> 6;
@@ -273,32 +297,56 @@ __global__ void __launch_bounds__(kRowsThreads, 1) latent_rows_kernel(const __gr
   }
   __syncthreads();
 
-  const int dw = p.kvp / NSL, nt = dw >> 3;       // this warp's slice of the latent's dims
-  float o[MAXT][4];
+  float o[NT][4];
 #pragma unroll
-  for (int j = 0; j < MAXT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+  for (int j = 0; j < NT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
   float mx[2] = {-INFINITY, -INFINITY}, lsum[2] = {0.f, 0.f};
+  // ldmatrix lanes: a block of 64 dims keeps a row's 16-byte pieces at (piece XOR row mod 8), so a lane's address in it
+  // is a base plus one of eight swizzled offsets that do not change from block to block
+  const uint32_t qrow = q_s + (mt * 16 + (lane & 15)) * 128, qsw = lane & 7, qhi = lane >> 4;
+  const uint32_t krow = (sl * KSL + (lane & 7)) * 128, kmi = lane >> 3;
+  uint32_t qa[QREG ? KVC + 1 : 1][4][4];
+  if (QREG) {
+#pragma unroll
+    for (int c = 0; c < KVC + 1; ++c)
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+        ldsm_x4(qrow + c * (QR * 128) + (((2 * k + qhi) ^ qsw) << 4), qa[c][k][0], qa[c][k][1], qa[c][k][2], qa[c][k][3]);
+  }
   bool ok = true;
   for (int i = 0; i < ntile; ++i) {
     const uint32_t kt = kv_s + (i & 1) * kvB;
     if (ok) ok = mbar_wait(bar0 + 8 * (i & 1), (i >> 1) & 1, ERR_ATTN_WAIT);
-    // ---- scores of this warp's heads x keys; two chains so that consecutive MMAs do not wait for one another
-    float s[2][NJ][4];
+    // ---- scores of this warp's heads x keys: per block of 64 dims all operands first, then four independent chains
+    float s[4][NJ][4];
 #pragma unroll
-    for (int c = 0; c < 2; ++c)
+    for (int c = 0; c < 4; ++c)
 #pragma unroll
       for (int j = 0; j < NJ; ++j) s[c][j][0] = s[c][j][1] = s[c][j][2] = s[c][j][3] = 0.f;
+    auto block = [&](int c, const uint32_t (&a)[4][4]) {
+      uint32_t b[NJ][2][4];
+#pragma unroll
+      for (int j = 0; j < NJ; ++j)
+#pragma unroll
+        for (int k = 0; k < 2; ++k)
+          ldsm_x4(kt + c * (KT * 128) + krow + j * 1024 + (((4 * k + kmi) ^ qsw) << 4), b[j][k][0], b[j][k][1], b[j][k][2], b[j][k][3]);
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+#pragma unroll
+        for (int j = 0; j < NJ; ++j)
+          mma_bf16_16816(s[k][j], a[k][0], a[k][1], a[k][2], a[k][3], b[j][k >> 1][2 * (k & 1)], b[j][k >> 1][2 * (k & 1) + 1]);
+    };
+    if constexpr (QREG) {
+#pragma unroll
+      for (int c = 0; c < KVC + 1; ++c) block(c, qa[c]);
+    } else {
 #pragma unroll 2
-    for (int kk = 0; kk < nc * 4; kk += 2) {
-      uint32_t a[2][4], b[4];
+      for (int c = 0; c < nc; ++c) {
+        uint32_t a[4][4];
 #pragma unroll
-      for (int c = 0; c < 2; ++c)
-        ldsm_x4(q_s + tile_off<QR>(mt * 16 + (lane & 15), 16 * (kk + c) + 8 * (lane >> 4)), a[c][0], a[c][1], a[c][2], a[c][3]);
-#pragma unroll
-      for (int j = 0; j < NJ; ++j) {
-        ldsm_x4(kt + tile_off<KT>(sl * KSL + 8 * j + (lane & 7), 16 * kk + 8 * (lane >> 3)), b[0], b[1], b[2], b[3]);
-        mma_bf16_16816(s[0][j], a[0][0], a[0][1], a[0][2], a[0][3], b[0], b[1]);
-        mma_bf16_16816(s[1][j], a[1][0], a[1][1], a[1][2], a[1][3], b[2], b[3]);
+        for (int k = 0; k < 4; ++k)
+          ldsm_x4(qrow + c * (QR * 128) + (((2 * k + qhi) ^ qsw) << 4), a[k][0], a[k][1], a[k][2], a[k][3]);
+        block(c, a);
       }
     }
     float mnew[2] = {-INFINITY, -INFINITY};
@@ -307,7 +355,7 @@ __global__ void __launch_bounds__(kRowsThreads, 1) latent_rows_kernel(const __gr
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int key = key0 + i * KT + sl * KSL + 8 * j + 2 * t + (e & 1);
-        const float v = key < key1 && key >= klo ? (s[0][j][e] + s[1][j][e]) * p.scale_log2 : -INFINITY;
+        const float v = key < key1 && key >= klo ? ((s[0][j][e] + s[1][j][e]) + (s[2][j][e] + s[3][j][e])) * p.scale_log2 : -INFINITY;
         s[0][j][e] = v;
         mnew[e >> 1] = fmaxf(mnew[e >> 1], v);
       }
@@ -350,28 +398,25 @@ __global__ void __launch_bounds__(kRowsThreads, 1) latent_rows_kernel(const __gr
     __syncthreads();
     // ---- O += P C over this warp's dims
 #pragma unroll
-    for (int j = 0; j < MAXT; ++j) {
+    for (int j = 0; j < NT; ++j) {
       o[j][0] *= corr[0]; o[j][1] *= corr[0]; o[j][2] *= corr[1]; o[j][3] *= corr[1];
     }
 #pragma unroll
     for (int kk = 0; kk < KT / 16; ++kk) {
       uint32_t ph[4], pl[4];
-      const uint32_t off = tile_off<QR>(mt * 16 + (lane & 15), 16 * kk + 8 * (lane >> 4));
+      const uint32_t off = (mt * 16 + (lane & 15)) * 128 + (((2 * kk + qhi) ^ qsw) << 4);
       ldsm_x4(ph_s + off, ph[0], ph[1], ph[2], ph[3]);
       ldsm_x4(pl_s + off, pl[0], pl[1], pl[2], pl[3]);
 #pragma unroll
-      for (int j = 0; j < MAXT; j += 2) {
-        if (j < nt) {
-          uint32_t b0, b1, b2, b3;
-          const int mi = lane >> 3, jd = min(j + (mi >> 1), nt - 1);
-          ldsm_x4_trans(kt + tile_off<KT>(16 * kk + 8 * (mi & 1) + (lane & 7), sl * dw + 8 * jd), b0, b1, b2, b3);
-          mma_bf16_16816(o[j], ph[0], ph[1], ph[2], ph[3], b0, b1);
-          mma_bf16_16816(o[j], pl[0], pl[1], pl[2], pl[3], b0, b1);
-          if (j + 1 < nt) {
-            mma_bf16_16816(o[j + 1], ph[0], ph[1], ph[2], ph[3], b2, b3);
-            mma_bf16_16816(o[j + 1], pl[0], pl[1], pl[2], pl[3], b2, b3);
-          }
-        }
+      for (int j = 0; j < NT; j += 2) {
+        const int mi = lane >> 3, d = sl * DW + 8 * min(j + (mi >> 1), NT - 1);
+        uint32_t b[4];
+        ldsm_x4_trans(kt + (d >> 6) * (KT * 128) + (16 * kk + 8 * (mi & 1) + (lane & 7)) * 128 + ((((uint32_t)(d & 63) >> 3) ^ qsw) << 4),
+                      b[0], b[1], b[2], b[3]);
+        mma_bf16_16816(o[j], ph[0], ph[1], ph[2], ph[3], b[0], b[1]);
+        if (j + 1 < NT) mma_bf16_16816(o[j + 1], ph[0], ph[1], ph[2], ph[3], b[2], b[3]);
+        mma_bf16_16816(o[j], pl[0], pl[1], pl[2], pl[3], b[0], b[1]);
+        if (j + 1 < NT) mma_bf16_16816(o[j + 1], pl[0], pl[1], pl[2], pl[3], b[2], b[3]);
       }
     }
   }
@@ -399,9 +444,8 @@ __global__ void __launch_bounds__(kRowsThreads, 1) latent_rows_kernel(const __gr
       p.ml_part[2 * row + 1] = l;
     }
 #pragma unroll
-    for (int j = 0; j < MAXT; ++j)
-      if (j < nt)
-        *reinterpret_cast<float2*>(p.o_part + row * p.kvp + sl * dw + 8 * j + 2 * t) = make_float2(o[j][2 * hf], o[j][2 * hf + 1]);
+    for (int j = 0; j < NT; ++j)
+      *reinterpret_cast<float2*>(p.o_part + row * p.kvp + sl * DW + 8 * j + 2 * t) = make_float2(o[j][2 * hf], o[j][2 * hf + 1]);
   }
 }
 
@@ -473,7 +517,9 @@ __global__ void __launch_bounds__(128) latent_simple_kernel(const SimpleParams p
 }
 
 // ------------------------------------------------------------------ merge of the splits + value up projection
-// grid (head, dv / 64, row groups of 8), 256 threads: the rows' merged latents in shared memory, a warp per 8 value dims
+// grid (head, dv / 16, row groups of 8), 256 threads: the rows' merged latents in shared memory (every CTA of a head
+// merges them for itself: the partials come from L2), then a warp per two value dims, whose weights are requested before
+// the kernel waits for its predecessor
 struct MergeParams {
   const float *o_part, *ml_part;
   int M, H, nsplit, kvp, dv;
@@ -482,14 +528,40 @@ struct MergeParams {
   int ld;
 };
 
+// eight consecutive values
+struct Raw8f { float4 a, b; };
+__device__ __forceinline__ void fetch8(const float* p, Raw8f& r) {
+  r.a = __ldg(reinterpret_cast<const float4*>(p));
+  r.b = __ldg(reinterpret_cast<const float4*>(p) + 1);
+}
+__device__ __forceinline__ void fetch8(const __nv_bfloat16* p, uint4& r) { r = __ldg(reinterpret_cast<const uint4*>(p)); }
+__device__ __forceinline__ void expand8(const Raw8f& r, float (&v)[8]) {
+  v[0] = r.a.x; v[1] = r.a.y; v[2] = r.a.z; v[3] = r.a.w; v[4] = r.b.x; v[5] = r.b.y; v[6] = r.b.z; v[7] = r.b.w;
+}
+__device__ __forceinline__ void expand8(const uint4& r, float (&v)[8]) {
+  v[0] = bf16_lo(r.x); v[1] = bf16_hi(r.x); v[2] = bf16_lo(r.y); v[3] = bf16_hi(r.y);
+  v[4] = bf16_lo(r.z); v[5] = bf16_hi(r.z); v[6] = bf16_lo(r.w); v[7] = bf16_hi(r.w);
+}
+template <typename T> struct Raw8 { using type = uint4; };
+template <> struct Raw8<float> { using type = Raw8f; };
+
 template <typename T>
 __global__ void __launch_bounds__(256) latent_merge_kernel(const MergeParams p) {
-  extern __shared__ float lat[];          // [8][kvp]
+  extern __shared__ __align__(16) float lat[];          // [8][kvp], then the partial merges of split groups [G - 1][mt][kvp]
   __shared__ float wt[8][64];
+  const int h = blockIdx.x, m0 = blockIdx.z * 8, mt = min(8, p.M - m0);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, v0 = blockIdx.y * 16 + warp * 2;
+  typename Raw8<T>::type raw[2][2];
+  const T* w = reinterpret_cast<const T*>(p.w_uv) + ((size_t)h * p.dv + v0) * p.kvp;
+#pragma unroll
+  for (int d = 0; d < 2; ++d)
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int r = i * 256 + lane * 8;
+      if (r < p.kvp) fetch8(w + (size_t)d * p.kvp + r, raw[d][i]);
+    }
   pdl_launch_dependents();
   pdl_wait();
-  const int h = blockIdx.x, v0 = blockIdx.y * 64, m0 = blockIdx.z * 8, mt = min(8, p.M - m0);
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   if (warp < mt) {      // nsplit <= 64: two splits per lane
     const float* ml = p.ml_part + ((size_t)(m0 + warp) * p.H + h) * p.nsplit * 2;
     float mx[2], l[2];
@@ -511,51 +583,76 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(const MergeParams p) 
     for (int i = 0; i < 2; ++i) wt[warp][lane + 32 * i] = e[i] * inv;
   }
   __syncthreads();
-  for (int i = tid * 4; i < mt * p.kvp; i += 256 * 4) {
-    const int m = i / p.kvp, r = i - m * p.kvp;
+  const int vecs = mt * p.kvp / 4;
+  int G = 1;                         // groups of threads that share the splits of few rows
+  while (G < 8 && 2 * G * vecs <= 256 && 2 * G <= p.nsplit) G *= 2;
+  const int per = (p.nsplit + G - 1) / G;
+  for (int u = tid; u < G * vecs; u += 256) {
+    const int grp = u / vecs, i = (u - grp * vecs) * 4, m = i / p.kvp, r = i - m * p.kvp;
+    const int s_lo = grp * per, s_hi = min(p.nsplit, s_lo + per);
     const float* o = p.o_part + ((size_t)(m0 + m) * p.H + h) * p.nsplit * p.kvp + r;
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int s0 = 0; s0 < p.nsplit; s0 += 8) {
-      float4 v[8];
+    for (int s0 = s_lo; s0 < s_hi; s0 += 16) {
+      float4 v[16];
 #pragma unroll
-      for (int u = 0; u < 8; ++u)
-        v[u] = s0 + u < p.nsplit ? *reinterpret_cast<const float4*>(o + (size_t)(s0 + u) * p.kvp) : make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int q = 0; q < 16; ++q)
+        v[q] = s0 + q < s_hi ? __ldcg(reinterpret_cast<const float4*>(o + (size_t)(s0 + q) * p.kvp)) : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-      for (int u = 0; u < 8; ++u) {
-        const float w = s0 + u < p.nsplit ? wt[m][s0 + u] : 0.f;
-        a.x = fmaf(w, v[u].x, a.x); a.y = fmaf(w, v[u].y, a.y); a.z = fmaf(w, v[u].z, a.z); a.w = fmaf(w, v[u].w, a.w);
+      for (int q = 0; q < 16; ++q) {
+        const float x = s0 + q < s_hi ? wt[m][s0 + q] : 0.f;
+        a.x = fmaf(x, v[q].x, a.x); a.y = fmaf(x, v[q].y, a.y); a.z = fmaf(x, v[q].z, a.z); a.w = fmaf(x, v[q].w, a.w);
       }
     }
-    *reinterpret_cast<float4*>(lat + i) = a;
+    *reinterpret_cast<float4*>(lat + (grp ? (size_t)8 * p.kvp + (size_t)(grp - 1) * mt * p.kvp : 0) + i) = a;
   }
   __syncthreads();
-  for (int j0 = 0; j0 < 8; j0 += 2) {       // two value dims at a time: 2 x 8 row sums in registers
-    const int v = v0 + warp * 8 + j0;
-    const T* w = reinterpret_cast<const T*>(p.w_uv) + ((size_t)h * p.dv + v) * p.kvp;
-    float acc[2][8];
-#pragma unroll
-    for (int m = 0; m < 8; ++m) acc[0][m] = acc[1][m] = 0.f;
-    for (int r = lane * 2; r < p.kvp; r += 64) {
-      const float2 w0 = load2(w + r), w1 = load2(w + p.kvp + r);
-#pragma unroll
-      for (int m = 0; m < 8; ++m)
-        if (m < mt) {
-          const float2 x = *reinterpret_cast<const float2*>(lat + m * p.kvp + r);
-          acc[0][m] = fmaf(w0.x, x.x, fmaf(w0.y, x.y, acc[0][m]));
-          acc[1][m] = fmaf(w1.x, x.x, fmaf(w1.y, x.y, acc[1][m]));
-        }
+  if (G > 1) {
+    for (int i = tid; i < mt * p.kvp; i += 256) {
+      float a = lat[i];
+      for (int q = 1; q < G; ++q) a += lat[8 * p.kvp + (q - 1) * mt * p.kvp + i];
+      lat[i] = a;
     }
+    __syncthreads();
+  }
+  float acc[2][8];
+#pragma unroll
+  for (int m = 0; m < 8; ++m) acc[0][m] = acc[1][m] = 0.f;
+  auto accumulate = [&](int r, const typename Raw8<T>::type& r0, const typename Raw8<T>::type& r1) {
+    float w0[8], w1[8];
+    expand8(r0, w0);
+    expand8(r1, w1);
 #pragma unroll
     for (int m = 0; m < 8; ++m)
       if (m < mt) {
-        const float a = warp_sum(acc[0][m]), b = warp_sum(acc[1][m]);
-        if (lane == 0) {
-          T* dst = reinterpret_cast<T*>(p.out) + (size_t)(m0 + m) * p.ld + (size_t)h * p.dv + v;
-          dst[0] = from_f<T>(a);
-          dst[1] = from_f<T>(b);
+        float x[8];
+        *reinterpret_cast<float4*>(x) = *reinterpret_cast<const float4*>(lat + m * p.kvp + r);
+        *reinterpret_cast<float4*>(x + 4) = *reinterpret_cast<const float4*>(lat + m * p.kvp + r + 4);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          acc[0][m] = fmaf(w0[j], x[j], acc[0][m]);
+          acc[1][m] = fmaf(w1[j], x[j], acc[1][m]);
         }
       }
+  };
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+    if (i * 256 + lane * 8 < p.kvp) accumulate(i * 256 + lane * 8, raw[0][i], raw[1][i]);
+  for (int r = 512 + lane * 8; r < p.kvp; r += 256) {
+    typename Raw8<T>::type r0, r1;
+    fetch8(w + r, r0);
+    fetch8(w + p.kvp + r, r1);
+    accumulate(r, r0, r1);
   }
+#pragma unroll
+  for (int m = 0; m < 8; ++m)
+    if (m < mt) {
+      const float a = warp_sum(acc[0][m]), b = warp_sum(acc[1][m]);
+      if (lane == 0) {
+        T* dst = reinterpret_cast<T*>(p.out) + (size_t)(m0 + m) * p.ld + (size_t)h * p.dv + v0;
+        dst[0] = from_f<T>(a);
+        dst[1] = from_f<T>(b);
+      }
+    }
 }
 
 // ------------------------------------------------------------------ prompt form: keys of the segments, queries
@@ -610,18 +707,40 @@ EncodeTiledFn encode_fn() {
 
 int rows_smem(int mt, int lc) { return 1024 + (lc / 64) * (mt * 16 + 2 * KT) * 128 + 2 * mt * 16 * 128 + 32; }
 
-template <int MT>
-int launch_rows(const RowsParams& p, int M, cudaStream_t st) {
+template <int MT, int KVC, bool QREG>
+int launch_rows_kernel(const RowsParams& p, int M, cudaStream_t st) {
   static bool configured[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
   if (!configured[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(latent_rows_kernel<MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - 4096);
+    cudaError_t e = cudaFuncSetAttribute(latent_rows_kernel<MT, KVC, QREG>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - 4096);
     if (e != cudaSuccess) return (int)e;
     configured[dev & 63] = true;
   }
-  return b2_launch(latent_rows_kernel<MT>, dim3(M, p.nsplit, (p.H + MT * 16 - 1) / (MT * 16)), dim3(kRowsThreads),
+  return b2_launch(latent_rows_kernel<MT, KVC, QREG>, dim3(M, p.nsplit, (p.H + MT * 16 - 1) / (MT * 16)), dim3(kRowsThreads),
                    rows_smem(MT, p.lc), st, true, p);
+}
+
+template <int MT, int KVC>
+int launch_rows_form(const RowsParams& p, int M, cudaStream_t st) {
+  if constexpr (MT == 1)
+    if (p.lc == p.kvp + 64) return launch_rows_kernel<MT, KVC, true>(p, M, st);
+  return launch_rows_kernel<MT, KVC, false>(p, M, st);
+}
+
+template <int MT>
+int launch_rows(const RowsParams& p, int M, cudaStream_t st) {
+  switch (p.kvp / 64) {
+    case 1: return launch_rows_form<MT, 1>(p, M, st);
+    case 2: return launch_rows_form<MT, 2>(p, M, st);
+    case 3: return launch_rows_form<MT, 3>(p, M, st);
+    case 4: return launch_rows_form<MT, 4>(p, M, st);
+    case 5: return launch_rows_form<MT, 5>(p, M, st);
+    case 6: return launch_rows_form<MT, 6>(p, M, st);
+    case 7: return launch_rows_form<MT, 7>(p, M, st);
+    case 8: return launch_rows_form<MT, 8>(p, M, st);
+  }
+  return -1;
 }
 
 template <typename F>
@@ -637,7 +756,7 @@ extern "C" int b2_latent_prep(const float* part, int S, int M, int q_rank, int q
                               const float* q_norm, const float* kv_norm, float eps, const int* req, const int* pos,
                               const int* block_table, int max_blocks, const float* cos_t, const float* sin_t, int rope_dims,
                               void* cq, void* cache, int f32, void* stream) {
-  if (M < 1 || S < 1 || qp % 64 || kvp % 64 || rp % 64 || rope_dims % 2 || rope_dims > rot || rot > rp) return -1;
+  if (M < 1 || S < 1 || S > 8 || qp % 64 || kvp % 64 || rp % 64 || rope_dims % 2 || rope_dims > rot || rot > rp) return -1;
   PrepParams p{part, S, M, q_rank, qp, kv_rank, kvp, rot, rp, q_norm, kv_norm, eps, {req, pos}, block_table, max_blocks,
                {cos_t, sin_t, rope_dims}, cq, cache};
   const size_t smem = (size_t)(qp + kvp + rp) * 4;
@@ -699,8 +818,8 @@ extern "C" int b2_latent_merge(const float* o_part, const float* ml_part, int M,
                                const void* w_uv, void* out, int ld, int f32, void* stream) {
   if (M < 1 || M > 8 * 65535 || nsplit < 1 || nsplit > 64 || kvp % 64 || dv % 64) return -1;
   MergeParams p{o_part, ml_part, M, H, nsplit, kvp, dv, w_uv, out, ld};
-  const size_t smem = (size_t)8 * kvp * 4;
-  const dim3 grid(H, dv / 64, (M + 7) / 8);
+  const size_t smem = (size_t)8 * kvp * 4 + 4096;     // split groups only form where they share at most 1024 values
+  const dim3 grid(H, dv / 16, (M + 7) / 8);
   int rc = f32 ? set_smem(latent_merge_kernel<float>, smem) : set_smem(latent_merge_kernel<__nv_bfloat16>, smem);
   if (rc) return rc;
   return f32 ? b2_launch(latent_merge_kernel<float>, grid, dim3(256), smem, (cudaStream_t)stream, true, p)

@@ -46,6 +46,7 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lrow, int E,
   float total = 0.f;   // softmax normaliser, only needed when the weights are not renormalised
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
+    if (32 * i >= E) { v[i] = -1.f; continue; }
     // softmax: unnormalised probabilities; -1 marks "taken / absent"
     const bool in = (lane + 32 * i) < E;
     if (rule.sigmoid) v[i] = in ? 1.f / (1.f + expf(-v[i])) : -1.f;
@@ -59,6 +60,7 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lrow, int E,
       float a = -1.f, b = -1.f;  // two best of the group among this lane's experts
 #pragma unroll
       for (int i = 0; i < PER; ++i) {
+        if (32 * i >= E) break;
         const int e = lane + 32 * i;
         if (e >= g * size && e < (g + 1) * size) {
           if (v[i] > a) { b = a; a = v[i]; }
@@ -88,6 +90,7 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lrow, int E,
     }
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
+      if (32 * i >= E) break;
       const int e = lane + 32 * i;
       if (e < E && !((kept >> (e / size)) & 1u)) v[i] = -1.f;
     }
@@ -101,6 +104,7 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lrow, int E,
     int bi = 0x7fffffff;
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
+      if (32 * i >= E) break;
       const int e = lane + 32 * i;
       if (v[i] > bv) { bv = v[i]; bi = e; }  // e ascends with i inside a lane: the first maximum is the lowest id
     }

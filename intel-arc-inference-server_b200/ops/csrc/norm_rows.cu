@@ -20,6 +20,7 @@ namespace cg = cooperative_groups;
 namespace {
 
 constexpr int kThreads = 256;
+constexpr int kTerms = 256;     // slots x slices of a row
 
 struct SubNormParams {
   const void* y;             // fp32 (or bf16 with y_bf16) values
@@ -55,14 +56,22 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 // CS: CTAs per row (cluster size); columns of the row's part live in shared memory between the passes
 template <int CS>
 __global__ void __launch_bounds__(kThreads) sublayer_norm_kernel(const SubNormParams p) {
-  extern __shared__ float vals[];
-  __shared__ float red[kThreads / 32], stat[2];
+  extern __shared__ __align__(16) float vals[];
+  __shared__ float red[kThreads / 32], stat[2], t_w[kTerms];
+  __shared__ long long t_off[kTerms];
   pdl_wait();
   pdl_launch_dependents();
   const int m = blockIdx.x / CS, part = CS > 1 ? blockIdx.x % CS : 0;
   const int per = ((p.ld / 4 + CS - 1) / CS) * 4;            // columns per CTA, in fours
   const int c0 = part * per, c1 = min(p.ld, c0 + per);
   const int terms = p.slots * p.slices;
+  for (int t = threadIdx.x; t < terms; t += kThreads) {       // where the row's values are and what they count
+    const int s = t / p.slices, q = t - s * p.slices;
+    const long long r = p.row_of ? p.row_of[m * p.slots + s] : (long long)m * p.slots + s;
+    t_off[t] = r * p.row + q * p.slice;
+    t_w[t] = p.slot_w ? p.slot_w[m * p.slots + s] : 1.f;
+  }
+  __syncthreads();
   float sum = 0.f;
   for (int c = c0 + threadIdx.x * 4; c < c1; c += kThreads * 4) {
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -75,15 +84,13 @@ __global__ void __launch_bounds__(kThreads) sublayer_norm_kernel(const SubNormPa
         v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
         wt[u] = 0.f;
         if (t < terms) {
-          const int s = t / p.slices, q = t - s * p.slices;
-          const long long r = p.row_of ? p.row_of[m * p.slots + s] : (long long)m * p.slots + s;
-          const long long off = r * p.row + q * p.slice + c;
-          wt[u] = p.slot_w ? p.slot_w[m * p.slots + s] : 1.f;
+          const long long off = t_off[t] + c;
+          wt[u] = t_w[t];
           if (p.y_bf16) {
-            const uint2 raw = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p.y) + off);
+            const uint2 raw = __ldcg(reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p.y) + off));
             v[u] = make_float4(bf16_lo(raw.x), bf16_hi(raw.x), bf16_lo(raw.y), bf16_hi(raw.y));
           } else {
-            v[u] = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.y) + off);
+            v[u] = __ldcg(reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.y) + off));
           }
         }
       }
@@ -98,9 +105,9 @@ __global__ void __launch_bounds__(kThreads) sublayer_norm_kernel(const SubNormPa
     float e[4] = {a.x, a.y, a.z, a.w};
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      vals[c - c0 + j] = e[j];
       if (c + j < p.width) sum += e[j];
     }
+    *reinterpret_cast<float4*>(vals + c - c0) = a;
   }
   float mean = 0.f, rstd = 1.f;
   if (p.w) {
@@ -141,8 +148,9 @@ __global__ void __launch_bounds__(kThreads) sublayer_norm_kernel(const SubNormPa
     for (int j = 0; j < 4; ++j) {
       if (c + j < p.width) e[j] += p.w ? (vals[c - c0 + j] - mean) * rstd * p.w[c + j] : vals[c - c0 + j];
       else e[j] = 0.f;
-      store_h(p.h, p.h_f32, (size_t)m * p.ld + c + j, e[j]);
     }
+    if (p.h_f32) reinterpret_cast<float4*>(p.h)[((size_t)m * p.ld + c) / 4] = make_float4(e[0], e[1], e[2], e[3]);
+    else reinterpret_cast<uint2*>(p.h)[((size_t)m * p.ld + c) / 4] = make_uint2(pack_bf16(e[0], e[1]), pack_bf16(e[2], e[3]));
     *xr = make_float4(e[0], e[1], e[2], e[3]);
   }
   if (CS > 1) cg::this_cluster().sync();    // no CTA leaves while another may still read its statistics
@@ -223,13 +231,14 @@ int launch_subnorm(const SubNormParams& p, cudaStream_t st) {
   cfg.dynamicSmemBytes = smem;
   cfg.stream = st;
   cudaLaunchAttribute attr[2];
-  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  attr[0].val.programmaticStreamSerializationAllowed = 1;
-  attr[1].id = cudaLaunchAttributeClusterDimension;
-  attr[1].val.clusterDim.x = CS;
-  attr[1].val.clusterDim.y = attr[1].val.clusterDim.z = 1;
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = CS;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr;
-  cfg.numAttrs = CS > 1 ? 2 : 1;
+  static const bool no_pdl = getenv("B2_NO_PDL") != nullptr;  // measurement switch, as in b2_launch
+  cfg.numAttrs = no_pdl ? 1 : 2;
   return (int)cudaLaunchKernelEx(&cfg, sublayer_norm_kernel<CS>, p);
 }
 
@@ -238,7 +247,7 @@ int launch_subnorm(const SubNormParams& p, cudaStream_t st) {
 extern "C" int b2_sublayer_norm(const void* y, int y_bf16, const int* row_of, const float* slot_w, long long slice,
                                 long long row, int slots, int slices, int M, int width, int ld, const float* w, float eps,
                                 float* x, void* h, int h_f32, int add, void* stream) {
-  if (M < 1 || slots < 1 || slices < 1 || ld % 4 || width > ld || row % 4 || slice % 4) return -1;
+  if (M < 1 || slots < 1 || slices < 1 || slots * slices > kTerms || ld % 4 || width > ld || row % 4 || slice % 4) return -1;
   SubNormParams p{y, row_of, slot_w, slice, row, slots, slices, y_bf16, M, width, ld, w, eps, x, h, h_f32, add};
   cudaStream_t st = (cudaStream_t)stream;
   // the split over CTAs changes the order of the statistics' sums, so it depends on the width alone up to the row
