@@ -72,6 +72,8 @@ template <int NDK_, int NDV_, int NW_, int KVS_, bool PAGED_>
 struct Form {
   static constexpr int NDK = NDK_, NDV = NDV_, NW = NW_, KVS = KVS_, DV = NDV_ * 64;
   static constexpr bool PAGED = PAGED_;
+  // softmax weights enter P V as one bf16 value, or (contiguous form) as two bf16 limbs, hi + lo, 16 bits of mantissa
+  static constexpr bool P2 = !PAGED_;
   static constexpr int QT_BYTES = BQ * NDK * 128;           // a query tile: [d-blocks][128 rows][64]
   static constexpr int Q_BYTES = NW * QT_BYTES;
   static constexpr int K_BYTES = BK2 * NDK * 128;           // a K tile: [d-blocks][64 keys][64]
@@ -91,6 +93,15 @@ __device__ __forceinline__ uint64_t make_desc_v2(uint32_t smem_addr) {
   d |= (uint64_t)1 << 46;
   d |= (uint64_t)2 << 61;
   return d;
+}
+
+// 16 packed columns of the thread's row into tensor memory
+__device__ __forceinline__ void st_16(uint32_t taddr, const uint32_t (&r)[16]) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%16], {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15};" ::"r"(r[0]),
+      "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]),
+      "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(taddr)
+      : "memory");
 }
 
 // map_r: contiguous form, the key part shared by all heads [rows][64 x blocks]; a head's key is dn columns of map_k
@@ -250,7 +261,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       auto issue_qk = [&](int j) -> bool {
         const int s = j & 1, ks = j % KVS;
         if (!mbar_wait(b_kfull + 8 * ks, (j / KVS) & 1, ERR_ATTN_WAIT)) return false;
-        // the buffer's first 32 columns hold P(j - 2) until that tile's P V product has read them
+        // the buffer holds P(j - 2) until that tile's P V product has read it
         if (j >= 2 && !mbar_wait(b_odone(w, s), ((j >> 1) - 1) & 1, ERR_ATTN_WAIT)) return false;
         tc_fence_after();
         const uint32_t kl = k_lo0 + ks * (F::K_BYTES >> 4), ts = t_s(w, s);
@@ -291,6 +302,11 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
 #pragma unroll
         for (int k = 0; k < 4; ++k)   // 4 x 16 keys: P comes from tensor memory, 8 columns (16 bf16) per step
           umma_f16_ts_w(to, tp + 8 * k, vl + ((k * 16 * 128) >> 4), hi_v, idesc_pv, (i | k) != 0);
+        if (F::P2) {
+#pragma unroll
+          for (int k = 0; k < 4; ++k)   // the low limbs, in the score buffer's other half
+            umma_f16_ts_w(to, tp + 32 + 8 * k, vl + ((k * 16 * 128) >> 4), hi_v, idesc_pv, 1u);
+        }
         tc_commit(b_odone(w, s));
         tc_commit(b_vempty + 8 * ks);
       }
@@ -388,7 +404,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       unsigned long long sc2, nm2, acc0 = 0ull, acc1 = 0ull;
       asm("mov.b64 %0, {%1, %1};" : "=l"(sc2) : "f"(p.scale_log2));
       asm("mov.b64 %0, {%1, %1};" : "=l"(nm2) : "f"(nmref));
-      uint32_t pk[16];
+      uint32_t pk[16], pl[F::P2 ? 16 : 1];
 #pragma unroll
       for (int j = 0; j < 16; ++j) {
         unsigned long long xy;
@@ -405,17 +421,14 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         else
           asm("add.rn.f32x2 %0, %0, %1;" : "+l"(acc0) : "l"(ee));
         pk[j] = pack_bf16(e0, e1);
+        if (F::P2) pl[F::P2 ? j : 0] = pack_bf16(e0 - bf16_lo(pk[j]), e1 - bf16_hi(pk[j]));
       }
       if (ok) {
         // P goes back into tensor memory, over the first 32 columns of the score buffer it came from (both halves
         // of the row have their scores in registers: they met at the barrier above): 16 packed columns per thread,
         // the A operand of P V without a trip through shared memory
-        asm volatile(
-            "tcgen05.st.sync.aligned.32x32b.x16.b32 [%16], {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15};" ::"r"(pk[0]),
-            "r"(pk[1]), "r"(pk[2]), "r"(pk[3]), "r"(pk[4]), "r"(pk[5]), "r"(pk[6]), "r"(pk[7]), "r"(pk[8]), "r"(pk[9]),
-            "r"(pk[10]), "r"(pk[11]), "r"(pk[12]), "r"(pk[13]), "r"(pk[14]), "r"(pk[15]),
-            "r"(t_s(w, sb) + lane_addr + half * 16)
-            : "memory");
+        st_16(t_s(w, sb) + lane_addr + half * 16, pk);
+        if constexpr (F::P2) st_16(t_s(w, sb) + lane_addr + 32 + half * 16, pl);
         tmem_st_wait();
       }
       {

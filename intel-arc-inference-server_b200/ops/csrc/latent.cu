@@ -288,12 +288,26 @@ __global__ void __launch_bounds__(kRowsThreads, 1) latent_rows_kernel(const __gr
     if (ntile > 0) issue(0);
     if (ntile > 1) issue(1);
   }
-  for (int i = tid; i < QR * (p.lc / 8); i += kRowsThreads) {
-    const int r = i / (p.lc / 8), v = i - r * (p.lc / 8);
-    uint4 x = make_uint4(0, 0, 0, 0);
-    if (h0 + r < p.H) x = *reinterpret_cast<const uint4*>(p.q + ((size_t)m * p.H + h0 + r) * p.lc + v * 8);
-    asm volatile("st.shared.v4.u32 [%0], {%1,%2,%3,%4};" ::"r"(q_s + tile_off<QR>(r, v * 8)), "r"(x.x), "r"(x.y), "r"(x.z), "r"(x.w)
-                 : "memory");
+  {
+    // the queries: a batch of vectors per thread requested before the first is stored
+    const int vpr = p.lc / 8, total = min(QR, p.H - h0) * vpr;
+    constexpr int B = 6;
+    for (int i0 = tid; i0 < QR * vpr; i0 += B * kRowsThreads) {
+      uint4 x[B];
+#pragma unroll
+      for (int u = 0; u < B; ++u) {       // rows of one (row, head group) are contiguous
+        const int i = i0 + u * kRowsThreads;
+        x[u] = i < total ? __ldcg(reinterpret_cast<const uint4*>(p.q + ((size_t)m * p.H + h0) * p.lc) + i) : make_uint4(0, 0, 0, 0);
+      }
+#pragma unroll
+      for (int u = 0; u < B; ++u) {
+        const int i = i0 + u * kRowsThreads, r = i / vpr, v = i - r * vpr;
+        if (i < QR * vpr)
+          asm volatile("st.shared.v4.u32 [%0], {%1,%2,%3,%4};" ::"r"(q_s + tile_off<QR>(r, v * 8)), "r"(x[u].x), "r"(x[u].y), "r"(x[u].z),
+                       "r"(x[u].w)
+                       : "memory");
+      }
+    }
   }
   __syncthreads();
 
@@ -801,7 +815,9 @@ extern "C" int b2_latent_rows(const void* q, const void* cache, int num_pages, i
   p.q = (const __nv_bfloat16*)q; p.o_part = o_part; p.ml_part = ml_part; p.rows = {req, pos};
   p.block_table = block_table; p.max_blocks = max_blocks; p.H = H; p.kvp = kvp; p.lc = lc; p.nsplit = nsplit;
   p.window = window > 0 ? window : 0; p.scale_log2 = scale * 1.4426950408889634f;
-  return H > 16 ? launch_rows<2>(p, M, (cudaStream_t)stream) : launch_rows<1>(p, M, (cudaStream_t)stream);
+  // two head tiles per CTA halve the cache reads; a step too small to fill half the GPU that way takes one
+  const bool pair = H > 16 && M * nsplit * ((H + 31) / 32) > 74;
+  return pair ? launch_rows<2>(p, M, (cudaStream_t)stream) : launch_rows<1>(p, M, (cudaStream_t)stream);
 }
 
 extern "C" int b2_latent_simple(const void* q, const void* cache, int M, int H, int kvp, int rp, const int* req, const int* pos,

@@ -30,7 +30,9 @@ struct RouteRule {
 
 // logits fp32 [T][ld], the first E columns are the experts (E <= 512).  topk_idx int32 [T][k], topk_w fp32 [T][k].
 // One row's routing by a whole warp: scores of E logits, top-k by repeated arg-max (ties to the lower id).
-// `stride` >= k entries per row in topk_idx / topk_w.
+// `stride` >= k entries per row in topk_idx / topk_w.  PLAIN: the rule is softmax, no groups, renormalised (the code of the
+// other rules costs the decode step's router 1.5 us a layer when it is compiled in).
+template <bool PLAIN>
 __device__ __forceinline__ void route_row(const float* __restrict__ lrow, int E, int k, const RouteRule rule,
                                           int* __restrict__ idx_out, float* __restrict__ w_out, int lane) {
   constexpr int PER = 16;  // experts per lane (E <= 512)
@@ -46,14 +48,14 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lrow, int E,
   float total = 0.f;   // softmax normaliser, only needed when the weights are not renormalised
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
-    if (32 * i >= E) { v[i] = -1.f; continue; }
+    if (!PLAIN && 32 * i >= E) { v[i] = -1.f; continue; }
     // softmax: unnormalised probabilities; -1 marks "taken / absent"
     const bool in = (lane + 32 * i) < E;
-    if (rule.sigmoid) v[i] = in ? 1.f / (1.f + expf(-v[i])) : -1.f;
+    if (!PLAIN && rule.sigmoid) v[i] = in ? 1.f / (1.f + expf(-v[i])) : -1.f;
     else v[i] = in ? __expf(v[i] - mx) : -1.f;
-    total += in ? v[i] : 0.f;
+    if (!PLAIN) total += in ? v[i] : 0.f;
   }
-  if (rule.groups > 1) {
+  if (!PLAIN && rule.groups > 1) {
     const int size = E / rule.groups;
     float mine = -INFINITY;      // lane g keeps the score of group g (groups <= 32)
     for (int g = 0; g < rule.groups; ++g) {
@@ -104,7 +106,7 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lrow, int E,
     int bi = 0x7fffffff;
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
-      if (32 * i >= E) break;
+      if (!PLAIN && 32 * i >= E) break;
       const int e = lane + 32 * i;
       if (v[i] > bv) { bv = v[i]; bi = e; }  // e ascends with i inside a lane: the first maximum is the lowest id
     }
@@ -119,13 +121,14 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lrow, int E,
     if (lane == r) { myw = bv; myid = bi; }
   }
   float norm = wsum;                                // renormalised: the softmax normaliser cancels
-  if (!rule.renorm) norm = rule.sigmoid ? 1.f : warp_sum(total);
+  if (!PLAIN && !rule.renorm) norm = rule.sigmoid ? 1.f : warp_sum(total);
   if (lane < k) {
     idx_out[lane] = myid;
     w_out[lane] = myw / norm;
   }
 }
 
+template <bool PLAIN>
 __global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict__ logits, int ld, int T, int E, int k,
                                                         const RouteRule rule, int* __restrict__ topk_idx,
                                                         float* __restrict__ topk_w) {
@@ -133,7 +136,7 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict_
   pdl_launch_dependents();
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (warp >= T) return;
-  route_row(logits + (size_t)warp * ld, E, k, rule, topk_idx + (size_t)warp * k, topk_w + (size_t)warp * k, lane);
+  route_row<PLAIN>(logits + (size_t)warp * ld, E, k, rule, topk_idx + (size_t)warp * k, topk_w + (size_t)warp * k, lane);
 }
 
 // ---------------------------------------------------------------- decode rows: router logits + routing in one launch
@@ -153,6 +156,7 @@ struct RouterRowsParams {
   int* ticket;              // one zeroed word; left zero
 };
 
+template <bool PLAIN>
 __global__ void __launch_bounds__(256) moe_router_rows_kernel(const RouterRowsParams p) {
   __shared__ int s_last;
   pdl_wait();
@@ -213,7 +217,7 @@ __global__ void __launch_bounds__(256) moe_router_rows_kernel(const RouterRowsPa
   const int stride = p.k + p.shared_slot;
   for (int m = warp; m < p.M; m += 8) {
     const float* lrow = p.logits + (size_t)m * p.ld;
-    route_row(lrow, p.E, p.k, p.rule, p.topk_idx + (size_t)m * stride, p.topk_w + (size_t)m * stride, lane);
+    route_row<PLAIN>(lrow, p.E, p.k, p.rule, p.topk_idx + (size_t)m * stride, p.topk_w + (size_t)m * stride, lane);
     if (p.shared_slot && lane == 0) {
       p.topk_idx[(size_t)m * stride + p.k] = p.E;
       p.topk_w[(size_t)m * stride + p.k] = p.has_gate ? 1.f / (1.f + __expf(-__ldcg(lrow + p.E))) : 1.f;
@@ -388,6 +392,8 @@ __global__ void __launch_bounds__(256) moe_combine_rows_kernel(const float* __re
 
 }  // namespace
 
+static bool route_plain(const RouteRule& r) { return !r.sigmoid && r.groups <= 1 && r.renorm; }
+
 static bool route_ok(int E, int k, const RouteRule& r) {
   if (E < 1 || E > 512 || k > 32 || k < 1) return false;
   if (r.groups <= 1) return k <= E;
@@ -399,7 +405,7 @@ extern "C" int b2_moe_route(const float* logits, int ld, int T, int E, int k, in
   const RouteRule rule{sigmoid, groups, keep, renorm};
   if (!route_ok(E, k, rule)) return -1;
   const int blocks = (T * 32 + 255) / 256;
-  return b2_launch(moe_route_kernel, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, true, logits, ld, T, E, k,
+  return b2_launch(route_plain(rule) ? moe_route_kernel<true> : moe_route_kernel<false>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, true, logits, ld, T, E, k,
                    rule, topk_idx, topk_w);
 }
 
@@ -410,7 +416,7 @@ extern "C" int b2_moe_router_rows(const void* w, const void* x, float* logits, i
   if (!route_ok(E, k, rule) || H % 8 || M < 1 || R < E + (has_gate ? 1 : 0) || ld < R) return -1;
   RouterRowsParams p{(const __nv_bfloat16*)w, (const __nv_bfloat16*)x, logits, M, R, H, ld, E, k, shared_slot, has_gate,
                      rule, topk_idx, topk_w, ticket};
-  return b2_launch(moe_router_rows_kernel, dim3((R + 7) / 8), dim3(256), 0, (cudaStream_t)stream, true, p);
+  return b2_launch(route_plain(rule) ? moe_router_rows_kernel<true> : moe_router_rows_kernel<false>, dim3((R + 7) / 8), dim3(256), 0, (cudaStream_t)stream, true, p);
 }
 
 // counts must hold E zeros on entry (the caller clears it on the stream).
