@@ -109,7 +109,7 @@ def load_model(spec: str, device, seed: int = 0, int8_head: bool = False, tp=(0,
     if dtype != "bfloat16" and not cfg.layer_specs:
         raise SystemExit(f"{cfg.name}: this family is served in bfloat16 only")
     if spec in PRESETS and cfg.layer_specs:
-        from ..models.latent import random_listed_weights
+        from ..models.listed import random_listed_weights
         sys.stderr.write(f"load: preset {spec} with random-init {dtype} weights (seed {seed})\n")
         return random_listed_weights(cfg, device, seed, dtype=getattr(torch, dtype))
     if spec in PRESETS:

@@ -40,7 +40,7 @@ def main(argv=None):
     cfg = w.cfg
     depth = f.depth if (f.bench or f.profile) else 0
     ids = _ids(f.ids) if f.ids else None
-    need = max(depth, len(ids or []), f.prefill_length) + (f.tg + 4) * max(1, f.repeats if cfg.n_gdn_layers else 1) + f.n + 64
+    need = max(depth, len(ids or []), f.prefill_length) + (f.tg + 4) * max(1, f.repeats if cfg.recurrent else 1) + f.n + 64
     eng = Engine(w, max_seqs=1, max_len=need, kv_dtype=f.kv_cache, int8_head=f.int8_head,
                  prefill_backend=f.prefill_backend if f.prefill or f.bench else "rows")
     if ids is not None and not (f.bench or f.profile):
@@ -56,7 +56,7 @@ def main(argv=None):
     hbm, _, src = peaks()
     rows = []
     for _ in range(f.repeats):
-        if not cfg.n_gdn_layers:    # (a recurrent state is not rewound: a hybrid model's repeats continue the sequence)
+        if not cfg.recurrent:    # (a recurrent state is not rewound: such a model's repeats continue the sequence)
             eng.truncate(0, len(prompt))
         eng.decode_begin([0], [first])
         for _ in range(4):
@@ -109,6 +109,8 @@ def _profile(eng, f, first):
         mods.update({n: L for n in ("embed_rows", "gemv_bf16", "prep", "absorb", "rows", "simple", "merge", "sublayer_norm",
                                     "gemv_bf16_experts", "layer_norm_rows", "linear_f32", "linear_f32_experts")})
         mods["router_rows"] = M
+        from ..ops import mlstm as R, paged as P, streams as S
+        mods.update({"gemv_bf16_glu": L, "embed": S, "boundary": S, "append": P, "step": R})
         names = list(mods)
     pending = []
 

@@ -238,7 +238,7 @@ def _load_ffn(lw: LayerWeights, view: NameView, cfg: ModelConfig, prefix: str, q
 def load_listed(st: SafetensorsSet, cfg: ModelConfig, device, dtype: str = "bfloat16") -> ModelWeights:
     """A model that lists its layers: unquantised tensors under the design's own names, checked against the
     configuration before anything is assembled; ``dtype`` float32 keeps everything in 32-bit."""
-    from ..models.latent import assemble, tensor_shapes
+    from ..models.listed import assemble, tensor_shapes
     bad = []
     for name, shape in tensor_shapes(cfg).items():
         if not st.has(name):

@@ -36,6 +36,76 @@ class LatentAttention:
     rope_base: float
     window: int = 0               # a position sees itself and the window - 1 positions before it (0: all)
 
+    def linear_elems(self, h: int) -> int:
+        return (self.q_rank + self.kv_rank + self.rot_dim) * h + self.heads * (self.dim + self.rot_dim) * self.q_rank \
+            + self.heads * (self.dim + self.vdim) * self.kv_rank + h * self.heads * self.vdim
+
+    @property
+    def kv_elems(self) -> int:
+        return self.kv_rank + self.rot_dim
+
+
+@dataclass(frozen=True)
+class GroupedAttention:
+    """Grouped-query attention without a rotation; the cache holds keys and values per key/value head."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    chunk: int = 0                # a position sees its own chunk of this many positions up to itself (0: all before it)
+    bias: float = 0.0             # distance bias -(i - j) 2^(-bias (h + 1) / heads) on head h's scores (0: none)
+    sink: bool = False            # one learned term per head in the softmax's denominator
+    kv_from: int = -1             # layer whose cached keys and values are read (-1: the layer's own)
+
+    def linear_elems(self, h: int) -> int:
+        return h * (self.heads * (self.dim + self.vdim) + (self.kv_heads * (self.dim + self.vdim) if self.kv_from < 0 else 0))
+
+    @property
+    def kv_elems(self) -> int:
+        return self.kv_heads * (self.dim + self.vdim) if self.kv_from < 0 else 0
+
+
+@dataclass(frozen=True)
+class MatrixLstm:
+    """Recurrent mixer with a matrix memory per head (mLSTM): exponential input gate, sigmoid forget gate, both capped."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+    def linear_elems(self, h: int) -> int:
+        return h * self.heads * (2 * self.dim + 3 * self.vdim + 2)
+
+    @property
+    def kv_elems(self) -> int:
+        return 0
+
+
+@dataclass(frozen=True)
+class DenseFfn:
+    """down (g sigmoid(alpha g) (u + shift)), g = min(gate, limit), u = clamp(up, -limit, limit)."""
+    ff: int
+    limit: float = float("inf")
+    alpha: float = 1.0
+    shift: float = 0.0
+
+    def linear_elems(self, h: int) -> tuple:
+        return (3 * self.ff * h,) * 2
+
+
+@dataclass(frozen=True)
+class StreamBlock:
+    """Residual of several streams around pre-normed sublayers (hyper-connections): a sublayer reads a mix of the streams,
+    its result goes to all of them, times ``mult``.  Norms have one number for all columns; ``shift``: what a mixer reads is
+    mixed with the previous token's; the streams start as the embedding plus a sinusoidal position vector (``sinusoid``:
+    its base, 0: none)."""
+    streams: int
+    mult: float
+    shift: bool = True
+    scale: bool = True            # a learned factor per column on every sublayer's result
+    sinusoid: float = 10000.0
+
 
 @dataclass(frozen=True)
 class ExpertFfn:
@@ -54,13 +124,18 @@ class ExpertFfn:
     def rule(self) -> tuple:
         return (int(self.score == "sigmoid"), self.groups, self.keep, int(self.renorm))
 
+    def linear_elems(self, h: int) -> tuple:
+        """(weights a token's step reads, weights held)."""
+        one = 3 * self.ff * h
+        return self.experts * h + self.top * one, self.experts * (h + one)
+
 
 @dataclass(frozen=True)
 class LayerSpec:
-    """One layer of a model that lists its layers: a mixer and a feed-forward (or none), each followed by a layer norm
-    of its output, added to an fp32 residual stream."""
-    mixer: LatentAttention
-    ffn: Optional[ExpertFfn]
+    """One layer of a model that lists its layers: a mixer and a feed-forward (or none).  How they meet the fp32 residual
+    is ``ModelConfig.block``: None adds layer norms of the sublayers' outputs to one stream."""
+    mixer: object                 # LatentAttention, GroupedAttention or MatrixLstm
+    ffn: object                   # ExpertFfn, DenseFfn or None
 
 
 @dataclass(frozen=True)
@@ -97,9 +172,10 @@ class ModelConfig:
     gdn_k_heads: int = 0
     gdn_v_heads: int = 0
     gdn_head_dim: int = 128
-    # models that list their layers one by one (unquantised weights, fp32 residual stream, norms on sublayer outputs);
-    # the scalar fields above then hold the largest values over the layers
+    # models that list their layers one by one (unquantised weights, fp32 residual); the scalar fields above then hold the
+    # largest values over the layers
     layer_specs: tuple = ()
+    block: Optional[StreamBlock] = None
 
     @property
     def q_dim(self) -> int:
@@ -133,6 +209,12 @@ class ModelConfig:
     @property
     def n_gdn_layers(self) -> int:
         return sum(1 for i in range(self.n_layers) if self.is_gdn_layer(i))
+
+    @property
+    def recurrent(self) -> bool:
+        """Sequences carry a state that cannot be rewound position by position."""
+        return self.n_gdn_layers > 0 or any(isinstance(s.mixer, MatrixLstm) for s in self.layer_specs) \
+            or (self.block is not None and self.block.shift)
 
     @property
     def gdn_key_dim(self) -> int:
@@ -202,14 +284,9 @@ class ModelConfig:
 
     def layer_linears(self, spec: LayerSpec):
         """(weights a token's step reads, weights held) of one listed layer."""
-        a, h = spec.mixer, self.hidden
-        mix = (a.q_rank + a.kv_rank + a.rot_dim) * h + a.heads * (a.dim + a.rot_dim) * a.q_rank \
-            + a.heads * (a.dim + a.vdim) * a.kv_rank + h * a.heads * a.vdim
-        if spec.ffn is None:
-            return mix, mix
-        f = spec.ffn
-        one = 3 * f.ff * h
-        return mix + f.experts * h + f.top * one, mix + f.experts * (h + one)
+        mix = spec.mixer.linear_elems(self.hidden)
+        read, held = spec.ffn.linear_elems(self.hidden) if spec.ffn is not None else (0, 0)
+        return mix + read, mix + held
 
     def param_count(self) -> int:
         h = self.hidden
@@ -243,23 +320,14 @@ class ModelConfig:
 
     def kv_bytes_per_token(self, kv_dtype: str = "bf16") -> int:
         if self.layer_specs:
-            return sum((s.mixer.kv_rank + s.mixer.rot_dim) * (4 if kv_dtype == "f32" else 2) for s in self.layer_specs)
+            return sum(s.mixer.kv_elems for s in self.layer_specs) * (4 if kv_dtype == "f32" else 2)
         per_head = self.head_dim * (2 if kv_dtype == "bf16" else 1) + (4 if kv_dtype == "int8" else 0)
         return (self.n_layers - self.n_gdn_layers) * 2 * self.n_kv_heads * per_head
 
     def to_listed_config(self) -> dict:
         """The inverse of the listed designs' readers."""
-        def layer(s):
-            m, f = s.mixer, s.ffn
-            mixer = {"dim": m.dim, "heads": m.heads, "kv_rank": m.kv_rank, "q_rank": m.q_rank, "rot_dim": m.rot_dim,
-                     "vdim": m.vdim, "scale": m.scale, "rot": {"base": m.rope_base, "dims": m.rope_dims}}
-            if m.window:
-                mixer["mask"] = {"size": m.window}
-            mlp = None if f is None else {"kind": "moe", "expert": {"ff": f.ff}, "router": {
-                "experts": f.experts, "top": f.top, "groups": {"count": f.groups, "keep": f.keep}}}
-            return {"type": "latent_attention", "mixer": mixer, "mlp": mlp}
         return {"architecture": self.architecture, "name": self.name, "width": self.hidden, "vocab": self.vocab,
-                "norm": {"eps": self.rms_eps}, "layers": [layer(s) for s in self.layer_specs]}
+                "norm": {"eps": self.rms_eps}, **LISTED_WRITERS[self.architecture](self)}
 
     def to_hf_config(self) -> dict:
         if self.layer_specs:
@@ -321,14 +389,17 @@ class ModelConfig:
         )
 
 
-def listed_config(name: str, architecture: str, specs, hidden: int, vocab: int, eps: float) -> ModelConfig:
+def listed_config(name: str, architecture: str, specs, hidden: int, vocab: int, eps: float,
+                  block: Optional[StreamBlock] = None) -> ModelConfig:
     """A model given by its layers; the scalar fields other parts of the framework read hold the largest values."""
     specs = tuple(specs)
     ffns = [s.ffn for s in specs if s.ffn is not None]
-    return ModelConfig(name, len(specs), hidden, max(s.mixer.heads for s in specs), 1, max(s.mixer.dim + s.mixer.rot_dim for s in specs),
-                       0, vocab, rms_eps=eps, n_experts=max((f.experts for f in ffns), default=0),
-                       top_k=max((f.top for f in ffns), default=0), expert_ffn=max((f.ff for f in ffns), default=0),
-                       architecture=architecture, layer_specs=specs)
+    most = lambda field: max((getattr(f, field, 0) for f in ffns), default=0)     # noqa: E731
+    return ModelConfig(name, len(specs), hidden, max(s.mixer.heads for s in specs), max(getattr(s.mixer, "kv_heads", 1) for s in specs),
+                       max(s.mixer.dim + getattr(s.mixer, "rot_dim", 0) for s in specs), 0, vocab, rms_eps=eps,
+                       n_experts=most("experts"), top_k=most("top"),
+                       expert_ffn=max((f.ff for f in ffns if isinstance(f, ExpertFfn)), default=0),
+                       architecture=architecture, layer_specs=specs, block=block)
 
 
 def mumusun_config(d: dict) -> ModelConfig:
@@ -356,7 +427,72 @@ def mumusun_config(d: dict) -> ModelConfig:
     return listed_config(d.get("name", "mumusun"), "Mumusun", specs, d["width"], d["vocab"], float(d["norm"]["eps"]))
 
 
-LISTED_ARCHITECTURES = {"Mumusun": mumusun_config}
+def mumusun_keys(c: ModelConfig) -> dict:
+    def layer(s):
+        m, f = s.mixer, s.ffn
+        mixer = {"dim": m.dim, "heads": m.heads, "kv_rank": m.kv_rank, "q_rank": m.q_rank, "rot_dim": m.rot_dim,
+                 "vdim": m.vdim, "scale": m.scale, "rot": {"base": m.rope_base, "dims": m.rope_dims}}
+        if m.window:
+            mixer["mask"] = {"size": m.window}
+        mlp = None if f is None else {"kind": "moe", "expert": {"ff": f.ff}, "router": {
+            "experts": f.experts, "top": f.top, "groups": {"count": f.groups, "keep": f.keep}}}
+        return {"type": "latent_attention", "mixer": mixer, "mlp": mlp}
+    return {"layers": [layer(s) for s in c.layer_specs]}
+
+
+def napadra_config(d: dict) -> ModelConfig:
+    """``config.json`` of a Napadra checkpoint: chunked attention with a distance bias and sinks, layers that read another
+    layer's keys and values, mLSTM layers, clamped feed-forwards, over several residual streams."""
+    specs = []
+    for i, layer in enumerate(d["layers"]):
+        m, f = layer["mixer"], layer["mlp"]
+        if layer["type"] == "attention":
+            mixer = GroupedAttention(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]),
+                                     (m.get("mask") or {}).get("size", 0) or 0, 8.0, True, m.get("kv_from", -1))
+            if mixer.heads % mixer.kv_heads:
+                raise ValueError(f"layer {i}: {mixer.heads} query heads over {mixer.kv_heads} key/value heads")
+            if mixer.kv_from >= 0:
+                src = specs[mixer.kv_from].mixer if mixer.kv_from < i else None
+                if not isinstance(src, GroupedAttention) or src.kv_from >= 0 or \
+                        (src.kv_heads, src.dim, src.vdim) != (mixer.kv_heads, mixer.dim, mixer.vdim):
+                    raise ValueError(f"layer {i}: layer {mixer.kv_from} has no keys and values that fit it")
+        elif layer["type"] == "mlstm":
+            mixer = MatrixLstm(m["heads"], m["dim"], m["vdim"], float(m["gate_cap"]))
+            if mixer.dim > 512 or mixer.vdim > 512:
+                raise ValueError(f"layer {i}: mLSTM heads of {mixer.dim} x {mixer.vdim} (512 at most)")
+        else:
+            raise ValueError(f"layer {i}: mixer {layer['type']!r} is not part of Napadra")
+        ffn = None
+        if f is not None:
+            if f["kind"] != "dense":
+                raise ValueError(f"layer {i}: feed-forward {f['kind']!r} is not part of Napadra")
+            ffn = DenseFfn(f["ff"], float(f["limit"]), 1.702, 1.0)
+        specs.append(LayerSpec(mixer, ffn))
+    if not 1 <= d["streams"] <= 8:
+        raise ValueError(f"{d['streams']} residual streams (1 to 8)")
+    return listed_config(d.get("name", "napadra"), "Napadra", specs, d["width"], d["vocab"], float(d["norm"]["eps"]),
+                         StreamBlock(d["streams"], float(d["residual_mult"])))
+
+
+def napadra_keys(c: ModelConfig) -> dict:
+    def layer(s):
+        m, f = s.mixer, s.ffn
+        mixer = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim}
+        if isinstance(m, MatrixLstm):
+            mixer["gate_cap"] = m.gate_cap
+        else:
+            mixer.update(kv_heads=m.kv_heads, scale=m.scale)
+            if m.chunk:
+                mixer["mask"] = {"size": m.chunk}
+            if m.kv_from >= 0:
+                mixer["kv_from"] = m.kv_from
+        return {"type": "mlstm" if isinstance(m, MatrixLstm) else "attention", "mixer": mixer,
+                "mlp": None if f is None else {"kind": "dense", "ff": f.ff, "limit": f.limit}}
+    return {"streams": c.block.streams, "residual_mult": c.block.mult, "layers": [layer(s) for s in c.layer_specs]}
+
+
+LISTED_ARCHITECTURES = {"Mumusun": mumusun_config, "Napadra": napadra_config}
+LISTED_WRITERS = {"Mumusun": mumusun_keys, "Napadra": napadra_keys}
 
 
 def tiny_dense() -> ModelConfig:
@@ -429,6 +565,30 @@ def mumusun_16b() -> ModelConfig:
                          102400, 1e-6)
 
 
+def napadra_mini() -> ModelConfig:
+    """Small Napadra: attention layers of unequal sizes and chunks, one that reads another's keys, two mLSTM layers."""
+    att = lambda h, g, dim, vdim, chunk, src=-1: GroupedAttention(h, g, dim, vdim, dim ** -0.5, chunk, 8.0, True, src)  # noqa: E731
+    ff = lambda n, limit: DenseFfn(n, limit, 1.702, 1.0)                                                               # noqa: E731
+    return listed_config("napadra-mini", "Napadra", (
+        LayerSpec(att(6, 2, 40, 72, 96), ff(176, 3.0)), LayerSpec(MatrixLstm(3, 80, 112, 10.0), ff(112, 1.5)),
+        LayerSpec(att(4, 4, 128, 64, 150), None), LayerSpec(MatrixLstm(5, 32, 40, 6.0), None),
+        LayerSpec(att(6, 2, 40, 72, 33, 0), ff(80, 2.5)), LayerSpec(att(8, 1, 72, 136, 0), ff(96, 4.0))), 200, 700, 1e-5,
+        StreamBlock(3, 0.8))
+
+
+def napadra_4b() -> ModelConfig:
+    """A Napadra of real layer sizes: width 4096, 32 layers in groups of two mLSTM layers (8 heads of 256 x 512) and two
+    attention layers (32 / 8 heads of 128, chunks of 8192, the second on the first one's keys), 11008 wide feed-forwards on
+    the attention layers, four streams."""
+    specs = []
+    for i in range(0, 32, 4):
+        att = GroupedAttention(32, 8, 128, 128, 128 ** -0.5, 8192, 8.0, True)
+        specs += [LayerSpec(MatrixLstm(8, 256, 512, 15.0), None)] * 2
+        specs += [LayerSpec(att, DenseFfn(11008, 7.0, 1.702, 1.0)),
+                  LayerSpec(replace(att, kv_from=i + 2), DenseFfn(11008, 7.0, 1.702, 1.0))]
+    return listed_config("napadra-4b", "Napadra", specs, 4096, 64000, 1e-5, StreamBlock(4, 0.5))
+
+
 def dflash_drafter(target: ModelConfig) -> ModelConfig:
     """DFlash-style block drafter: a 2-layer W4A16 decoder at the target's width."""
     return replace(target, name=target.name + "-dflash", n_layers=2, n_experts=0, top_k=0, expert_ffn=0,
@@ -438,7 +598,7 @@ def dflash_drafter(target: ModelConfig) -> ModelConfig:
 
 PRESETS = {
     "tiny-dense": tiny_dense, "tiny-moe": tiny_moe, "small-dense": small_dense, "small-windowed": small_windowed, "small-hybrid": small_hybrid, "small-moe": small_moe, "dense-27b": dense_27b, "hybrid-27b": hybrid_27b, "moe-35b-a3b": moe_35b_a3b,
-    "mumusun-mini": mumusun_mini, "mumusun-16b": mumusun_16b,
+    "mumusun-mini": mumusun_mini, "mumusun-16b": mumusun_16b, "napadra-mini": napadra_mini, "napadra-4b": napadra_4b,
 }
 
 

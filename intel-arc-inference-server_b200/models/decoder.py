@@ -17,7 +17,7 @@ import os
 
 import math
 from dataclasses import dataclass
-from typing import List, Optional
+from typing import Dict, List, Optional
 
 import torch
 
@@ -86,7 +86,7 @@ class ListedBuffers:
     """What the engine and the head read of a listed model's step; the layers' activations are in ``scratch``."""
 
     def __init__(self, cfg: ModelConfig, max_rows: int, wp: int, device, dtype):
-        from .latent import ListedScratch
+        from .listed import ListedScratch
         self.max_rows = max_rows
         self.scratch = ListedScratch(device, dtype, fixed=max_rows)
         self.resid = torch.zeros(max_rows, wp, dtype=torch.float32, device=device)
@@ -98,22 +98,34 @@ class ListedBuffers:
 
 
 class KVCache:
-    """Paged KV: per layer ``[page][kv_head][16][D]`` for K and for V (bf16 or int8 + fp32 scales); latent-attention layers
-    hold one latent row per position instead, ``[page][16][lc]`` (``latent[layer]``)."""
+    """Paged KV: per layer ``[page][kv_head][16][D]`` for K and for V (bf16 or int8 + fp32 scales).  Models that list their
+    layers keep what their mixers ask for, by name and layer: planes of the page pool (``pages``: ``[page][kv_head][16][d]``,
+    or ``[page][16][d]`` for rows shared by the heads).  ``states``: recurrent state ``[layers][slot]...`` by name, of every
+    family that has some."""
 
     def __init__(self, cfg: ModelConfig, n_layers: int, num_pages: int, device, kv_dtype: str = "bf16", n_slots: int = 1):
         self.kv_int8 = kv_dtype == "int8"
         dt = torch.int8 if self.kv_int8 else torch.bfloat16
         self.num_pages = num_pages
         self.n_layers = n_layers                # layers addressed by ``layer`` (trunk + draft-head layers)
-        self.latent = []
+        self.pages: Dict[str, torch.Tensor] = {}
+        self.states: Dict[str, torch.Tensor] = {}
+        self.shift_next = None      # last rows of a step on their way into ``states["shift"]``
         if cfg.layer_specs:
-            from .latent import LatentGeometry
+            from .listed import kind, pad64
             if kv_dtype not in ("bf16", "f32"):
-                raise ValueError(f"latent-attention layers keep a bf16 (or, served in 32-bit, fp32) cache, not {kv_dtype}")
+                raise ValueError(f"{cfg.name} keeps a bf16 (or, served in 32-bit, fp32) cache, not {kv_dtype}")
             ldt = torch.float32 if kv_dtype == "f32" else torch.bfloat16
-            self.latent = [torch.zeros(num_pages, cfg.page_size, LatentGeometry.of(sp.mixer).lc, dtype=ldt, device=device)
-                           for sp in cfg.layer_specs]
+            for li, sp in enumerate(cfg.layer_specs):
+                for name, (heads, cols) in kind(sp.mixer).page_planes(sp.mixer).items():
+                    shape = (num_pages, heads, cfg.page_size, cols) if heads else (num_pages, cfg.page_size, cols)
+                    self.pages[f"{name}{li}"] = torch.zeros(shape, dtype=ldt, device=device)
+                shape = kind(sp.mixer).state_shape(sp.mixer)
+                if shape is not None:
+                    self.states[f"mlstm{li}"] = torch.zeros((1, n_slots) + shape, dtype=torch.float32, device=device)
+            if cfg.block is not None and cfg.block.shift:
+                self.states["shift"] = torch.zeros(cfg.n_layers, n_slots, pad64(cfg.hidden), dtype=torch.float32, device=device)
+                self.shift_next = torch.zeros(n_slots, pad64(cfg.hidden), dtype=torch.float32, device=device)
             self.k = self.v = self.k_scale = self.v_scale = self.gdn_conv = self.gdn_state = None
             return
         # gated delta-net layers hold no KV: only the others get a plane of the cache
@@ -136,16 +148,25 @@ class KVCache:
             self.gdn_conv = torch.zeros(g, n_slots, cfg.gdn_conv_channels, 3, dtype=torch.float32, device=device)
             self.gdn_state = torch.zeros(g, n_slots, cfg.gdn_v_heads, cfg.gdn_head_dim, cfg.gdn_head_dim,
                                          dtype=torch.float32, device=device)
+            self.states = {"gdn_conv": self.gdn_conv, "gdn_state": self.gdn_state}
 
     def reset_slot(self, slot: int):
-        if self.gdn_conv is not None:
+        if self.gdn_conv is not None:       # (listed models start a sequence's first position from zeros themselves)
             self.gdn_conv[:, slot].zero_()
             self.gdn_state[:, slot].zero_()
 
+    def save_states(self, slot: int) -> dict:
+        """A copy of the slot's recurrent state."""
+        return {n: t[:, slot].clone() for n, t in self.states.items()}
+
+    def load_states(self, slot: int, saved: dict):
+        for n, t in self.states.items():
+            t[:, slot].copy_(saved[n], non_blocking=True)
+
     def page_tensors(self) -> dict:
         """Everything that belongs to a page, by name, as tensors ``[planes][page]...``."""
-        if self.latent:
-            return {f"latent{i}": t.unsqueeze(0) for i, t in enumerate(self.latent)}
+        if self.k is None:
+            return {n: t.unsqueeze(0) for n, t in self.pages.items()}
         out = {"k": self.k, "v": self.v}
         if self.kv_int8:
             out.update({"k_scale": self.k_scale, "v_scale": self.v_scale})
@@ -170,10 +191,14 @@ class DecoderModel:
         self.nsplit_attn = nsplit_attn
         self.listed = None
         if cfg.layer_specs:
-            from .latent import ListedLayers
+            from .listed import ListedLayers
             if tp is not None and tp.world > 1 or nccl is not None or int8_head:
                 raise ValueError("models that list their layers run on one GPU with an unquantised head")
             self.listed = ListedLayers(weights, max_pos)
+            self.streams = None
+            if cfg.block is not None:
+                from .streams import StreamWalk
+                self.streams = StreamWalk(self.listed)
             self.buf = ListedBuffers(cfg, max_rows, self.listed.wp, self.device, self.listed.dtype)
             self.tp = self.nccl = None
             self.head_rows, self.vocab_offset, self.max_pos, self.int8_head = cfg.vocab, 0, max_pos, False
@@ -570,29 +595,43 @@ class DecoderModel:
 
     # ------------------------------------------------------------------ models that list their layers
     def listed_walk(self, m: int, rows, block_table, kv: KVCache, scratch, resid, plan=None):
-        """All layers of a listed model for ``m`` rows (``rows``: ``models.latent.StepRows``): the fp32 residual rows are
-        left in ``resid[:m]``.  ``plan``: how a mixed batch's rows are attended (None: every row on its own).
+        """All layers of a listed model for ``m`` rows (``rows``: ``models.listed.StepRows``); returns the rows that
+        ``listed_logits`` selects from.  ``plan``: how a mixed batch's rows are attended (None: every row on its own).
 
-        Per layer: the mixer's slices, folded by the kernel that norms them and adds them to the residual; the experts'
-        slots, weighted and folded by the same kernel."""
+        One residual stream (left in ``resid[:m]``), per layer: the mixer's slices, folded by the kernel that norms them and
+        adds them to the residual; the experts' slots, weighted and folded by the same kernel.  Several streams:
+        ``models.streams.StreamWalk``."""
         from ..ops import latent as L
         ll, cfg = self.listed, self.cfg
+        if self.streams is not None:
+            return self.streams.run(m, rows, block_table, kv, scratch, self.buf.flag, plan)
         h = scratch.get("h", m, ll.wp)
         L.embed_rows(self.w.embed, rows.token, m, resid, h, self.buf.flag)
         for li, (spec, lw) in enumerate(zip(cfg.layer_specs, self.w.layers)):
-            part, s = ll.mixer(scratch, li, m, rows, block_table, kv.latent[li], plan)
+            part, s = ll.mixers[li].run(scratch, m, rows, block_table, kv, plan)
             L.sublayer_norm(part, m, cfg.hidden, lw.input_norm, cfg.rms_eps, resid, h, slices=s, slice_elems=m * ll.wp,
                             row_elems=ll.wp)
-            if spec.ffn is not None:
+            if lw.dense is not None:
+                part, s = ll.dense(scratch, spec.ffn, lw.dense, m)
+                L.sublayer_norm(part, m, cfg.hidden, lw.post_norm, cfg.rms_eps, resid, h, slices=s, slice_elems=m * ll.wp,
+                                row_elems=ll.wp)
+            elif spec.ffn is not None:
                 L.sublayer_norm(m=m, width=cfg.hidden, w=lw.post_norm, eps=cfg.rms_eps, x=resid, h=h,
                                 **ll.experts(scratch, spec.ffn, lw.moe, m))
+        return resid
 
-    def listed_logits(self, resid, sel, n: int, scratch, logits):
-        """Output norm and head of residual rows ``sel[:n]`` (None: rows 0..n - 1) into ``logits[:n]``."""
+    def listed_logits(self, final, sel, n: int, scratch, logits):
+        """Head of rows ``sel[:n]`` (None: rows 0..n - 1) of what ``listed_walk`` returned into ``logits[:n]``."""
         from ..ops import latent as L
         ll, cfg, b = self.listed, self.cfg, self.buf
-        x = scratch.get("head_x", n, ll.wp)
-        L.layer_norm_rows(resid, sel, self.w.final_norm, cfg.rms_eps, n, cfg.hidden, x)
+        if self.streams is None:
+            x = scratch.get("head_x", n, ll.wp)
+            L.layer_norm_rows(final, sel, self.w.final_norm, cfg.rms_eps, n, cfg.hidden, x)
+        elif sel is None:
+            x = final
+        else:                   # rows by index, the same kernel as an embedding
+            x = scratch.get("head_x", n, ll.wp)
+            L.embed_rows(final, sel, n, scratch.get("head_x32", n, ll.wp, torch.float32), x, self.buf.flag)
         if ll.f32:
             L.linear_f32(x, self.w.lm_head, logits, n)
             L.row_argmax(logits, n, cfg.vocab, b.cand_val, b.cand_idx)
@@ -600,12 +639,12 @@ class DecoderModel:
             K.head_gemv(self.w.lm_head, x, logits, n, cfg.vocab, ll.wp, b.cand_val, b.cand_idx)
 
     def _listed_step(self, m: int, ctrl, block_table, kv: KVCache, advance: bool):
-        from .latent import StepRows
+        from .listed import StepRows
         b = self.buf
         rows = StepRows(ctrl[K.CTRL_ROW_REQ: K.CTRL_ROW_REQ + m], ctrl[K.CTRL_ROW_POS: K.CTRL_ROW_POS + m],
                         ctrl[K.CTRL_CUR_TOKEN: K.CTRL_CUR_TOKEN + m])
-        self.listed_walk(m, rows, block_table, kv, b.scratch, b.resid)
-        self.listed_logits(b.resid, None, m, b.scratch, b.logits)
+        final = self.listed_walk(m, rows, block_table, kv, b.scratch, b.resid)
+        self.listed_logits(final, None, m, b.scratch, b.logits)
         K.argmax_finish(b.cand_val, b.cand_idx, b.ncand, m, ctrl, advance)
 
     def _nccl_reduce(self, part, splits: int, m: int):

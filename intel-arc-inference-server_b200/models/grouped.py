@@ -1,0 +1,143 @@
+"""Grouped-query attention mixers over paged keys and values of any head size, without a rotation; optional distance bias,
+chunked mask, sinks, and layers that read another layer's keys and values.
+
+Rows of a step are attended one by one (split-KV kernel) or, for long segments of a prompt, in query tiles by the tcgen05
+prompt attention straight over the pages.  The projection of a prompt stays in the GEMM's bf16 rows: the prompt attention
+reads its queries there.
+"""
+from __future__ import annotations
+
+import math
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from ..ops import gemm as G
+from ..ops import latent as L
+from ..ops import paged as P
+from .config import GroupedAttention, ModelConfig
+from .listed import SMS, BatchPlan, ListedLayers, ListedScratch, StepRows, pad64
+from .weights import GroupedWeights
+
+LOG2E = math.log2(math.e)
+
+
+@dataclass(frozen=True)
+class GroupedGeometry:
+    """Kernel sizes: ``dk`` / ``dv`` columns of a key / value head."""
+    heads: int
+    kv_heads: int
+    dk: int
+    dv: int
+
+    @staticmethod
+    def of(a: GroupedAttention) -> "GroupedGeometry":
+        return GroupedGeometry(a.heads, a.kv_heads, pad64(a.dim), pad64(a.vdim))
+
+    @property
+    def nq(self) -> int:
+        return self.heads * self.dk
+
+    @property
+    def groups(self) -> int:
+        """CTAs per row and split of the row attention: 16 query heads of one key/value head each."""
+        return self.kv_heads * ((self.heads // self.kv_heads + 15) // 16)
+
+    @property
+    def nkv(self) -> int:
+        return self.kv_heads * (self.dk + self.dv)
+
+
+def shapes(cfg: ModelConfig, p: str, a: GroupedAttention) -> dict:
+    h = cfg.hidden
+    out = {p + "mix.q": (a.heads * a.dim, h), p + "mix.o": (h, a.heads * a.vdim)}
+    if a.kv_from < 0:
+        out.update({p + "mix.k": (a.kv_heads * a.dim, h), p + "mix.v": (a.kv_heads * a.vdim, h)})
+    if a.sink:
+        out[p + "mix.sink"] = (a.heads,)
+    return out
+
+
+def assemble(t, p: str, a: GroupedAttention) -> GroupedWeights:
+    """``t``: ``listed.Assembler``."""
+    g = GroupedGeometry.of(a)
+    parts = [t.heads(t.t(p + "mix.q"), a.heads, [(a.dim, g.dk)], t.wp)]
+    if a.kv_from < 0:
+        parts += [t.heads(t.t(p + "mix.k"), a.kv_heads, [(a.dim, g.dk)], t.wp), t.heads(t.t(p + "mix.v"), a.kv_heads, [(a.vdim, g.dv)], t.wp)]
+    slope2 = None
+    if a.bias:
+        slope2 = torch.tensor([2.0 ** (-a.bias * (h + 1) / a.heads) * LOG2E for h in range(a.heads)], dtype=torch.float32, device=t.device)
+    sink2 = t.vec(p + "mix.sink") * LOG2E if a.sink else None
+    return GroupedWeights(torch.cat(parts), t.out_proj(p + "mix.o", a.heads, a.vdim, g.dv), slope2, sink2)
+
+
+def weight_elems(cfg: ModelConfig, a: GroupedAttention) -> int:
+    g = GroupedGeometry.of(a)
+    return pad64(cfg.hidden) * (g.nq + (g.nkv if a.kv_from < 0 else 0) + g.heads * g.dv)
+
+
+def scratch_elems(cfg: ModelConfig, a: GroupedAttention, rows: int, keys: int) -> int:
+    g = GroupedGeometry.of(a)
+    return rows * (9 * (g.nq + g.nkv) + g.nq + 2 * g.heads * g.dv)  \
+        + max(rows, Mixer.partials(g)) * (g.dv + 2)
+
+
+def page_planes(a: GroupedAttention) -> dict:
+    """Per position: plane name -> (heads, columns)."""
+    g = GroupedGeometry.of(a)
+    return {} if a.kv_from >= 0 else {"k": (g.kv_heads, g.dk), "v": (g.kv_heads, g.dv)}
+
+
+def state_shape(a: GroupedAttention) -> Optional[tuple]:
+    return None
+
+
+class Mixer:
+    def __init__(self, ll: ListedLayers, li: int, a: GroupedAttention, w: GroupedWeights):
+        self.ll, self.li, self.a, self.w, self.g = ll, li, a, w, GroupedGeometry.of(a)
+        self.src = li if a.kv_from < 0 else a.kv_from
+        on_gpu = ll.device.type == "cuda" and not ll.f32
+        self.tile_rows = P.segments_per_tile(self.g) if on_gpu else 0
+        self.rows_form = on_gpu and P.rows_ok(self.g)
+        self.form = ("tiles", a.chunk, self.tile_rows) if self.tile_rows else None
+
+    def nsplit(self, m: int) -> int:
+        """KV splits of the row attention: about two CTAs per SM, at least two pages per warp of a split."""
+        a = self.a
+        keys = min(a.chunk, self.ll.max_pos) if a.chunk else self.ll.max_pos
+        return max(1, min(64, 2 * SMS // (m * self.g.groups), keys // 128))
+
+    @staticmethod
+    def partials(g: GroupedGeometry) -> int:
+        """Most (row, head, split) partials a call with several splits leaves."""
+        return (2 * SMS // g.groups + 1) * g.heads
+
+    def run(self, sc: ListedScratch, m: int, rows: StepRows, block_table, kv, plan: Optional[BatchPlan]):
+        """Attention of the step's rows: fp32 slices of its output projection."""
+        ll, a, g, w = self.ll, self.a, self.g, self.w
+        own = a.kv_from < 0
+        k, v = kv.pages[f"k{self.src}"], kv.pages[f"v{self.src}"]
+        h = sc.get("h", m, ll.wp)
+        out = sc.get("attn", m, g.heads * g.dv)
+        n1 = m if plan is None or not self.tile_rows else plan.n_single
+        if ll.f32 or m <= L.GEMV_ROWS:
+            part, s = ll.linear(sc, "qkv", w.qkv, h, m)
+            q = sc.get("q_rows", m, g.nq)
+            P.append(part, s, m, g, own, rows.req, rows.pos, block_table, q, k, v)
+        else:
+            q = sc.get("qkv_rows", m, w.qkv.shape[0])
+            G.gemm_bf16(h, w.qkv, q)
+            if own:
+                P.append_rows(q, m, g, rows.req, rows.pos, block_table, k, v)
+        if n1 and self.rows_form:
+            ns, cap = self.nsplit(n1), self.partials(g)
+            op = sc.get("o_part", cap, g.dv, torch.float32) if ns > 1 else None
+            ml = sc.get("ml_part", cap, 2, torch.float32) if ns > 1 else None
+            P.rows(q, k, v, n1, g, rows.req, rows.pos, block_table, ns, a.chunk, a.scale, w.slope2, w.sink2, op, ml, out)
+        elif n1:
+            P.simple(q, k, v, n1, g, rows.req, rows.pos, block_table, a.chunk, a.scale, w.slope2, w.sink2, out)
+        if n1 < m:
+            t = plan.tables[self.form]
+            P.attn_segments(q[n1:], k, v, block_table, out[n1:], t.tiles, t.n_tiles, m - n1, g, a.scale, a.chunk, w.slope2, w.sink2)
+        return ll.linear(sc, "o", w.o, out, m)

@@ -1,0 +1,340 @@
+"""Models that list their layers: what every such model shares.
+
+A layer is a mixer and a feed-forward (``LayerSpec``).  Each kind of mixer has a module of its own (``latent``, ``grouped``,
+``mlstm``) with the same functions: ``shapes`` and ``assemble`` (checkpoint tensors, kernel-layout weights),
+``weight_elems`` and ``scratch_elems`` (the planner's figures), ``page_planes`` (what it keeps per position in the page
+pool), ``state_shape`` (what it keeps per sequence) and ``Mixer``, whose ``run`` enqueues its kernels for the rows of a step.
+The residual around the sublayers is ``streams.StreamWalk``, or the layer-normed single stream of
+``DecoderModel.listed_walk``.  ``Engine`` gives both the rows of a decode step (control block, CUDA graphs) or of a mixed
+batch (``runtime/batch.py``).
+
+Kernel sizes are whole 64s: weights are padded with zeros when they are loaded (rows and columns), and padded activation
+columns are zero; norms, rotations and scales use the true sizes.
+
+Few rows (up to 16) take the weight-streaming GEMVs, more rows the tcgen05 GEMMs.  Models whose weights are fp32 run
+everything in 32-bit (no reduced-precision product anywhere).
+"""
+from __future__ import annotations
+
+import os
+from dataclasses import dataclass
+from typing import Callable, Dict, Optional
+
+import torch
+
+from ..ops import gemm as G
+from ..ops import latent as L
+from ..ops import moe as M
+from .config import DenseFfn, ExpertFfn, GroupedAttention, LatentAttention, MatrixLstm, ModelConfig
+from .weights import DenseWeights, ExpertStack, LayerWeights, ModelWeights, interleave16
+
+SMS = 148
+# Experts of more rows than this go through the expert-sorted grouped GEMMs, which read every chosen expert once; the
+# GEMVs read one expert per (row, slot).
+EXPERT_GEMV_ROWS = int(os.environ.get("B2_EXPERT_GEMV_ROWS", "4"))
+
+
+def pad64(n: int) -> int:
+    return (n + 63) // 64 * 64
+
+
+def kind(mixer):
+    """The module of a mixer's kind."""
+    from . import grouped, latent, mlstm
+    return {LatentAttention: latent, GroupedAttention: grouped, MatrixLstm: mlstm}[type(mixer)]
+
+
+# ------------------------------------------------------------------ weights
+def tensor_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
+    """Checkpoint tensors of a listed model, by name."""
+    from . import streams
+    h = cfg.hidden
+    norm = (h,) if cfg.block is None else ()
+    out = {"embed": (cfg.vocab, h), "final.norm": norm, "head": (cfg.vocab, h)}
+    for i, s in enumerate(cfg.layer_specs):
+        p, f = f"l{i}.", s.ffn
+        out[p + "norm1"] = norm
+        out.update(kind(s.mixer).shapes(cfg, p, s.mixer))
+        if cfg.block is not None:
+            out.update(streams.shapes(cfg, p, s))
+        if f is None:
+            continue
+        out[p + "norm2"] = norm
+        if isinstance(f, DenseFfn):
+            out.update({p + "mlp.gate": (f.ff, h), p + "mlp.up": (f.ff, h), p + "mlp.down": (h, f.ff)})
+        else:
+            out[p + "mlp.router"] = (f.experts, h)
+            for e in range(f.experts):
+                out.update({f"{p}mlp.e{e}.gate": (f.ff, h), f"{p}mlp.e{e}.up": (f.ff, h), f"{p}mlp.e{e}.down": (h, f.ff)})
+    return out
+
+
+class Assembler:
+    """Checkpoint tensors (``get(name)``) in kernel layout on one device."""
+
+    def __init__(self, cfg: ModelConfig, get: Callable[[str], torch.Tensor], device, dtype):
+        self.cfg, self.get, self.device, self.dtype = cfg, get, device, dtype
+        self.wp = pad64(cfg.hidden)
+
+    def t(self, name: str) -> torch.Tensor:
+        return self.get(name).to(device=self.device, dtype=self.dtype)
+
+    def vec(self, name: str, cols: int = 0) -> torch.Tensor:
+        """fp32 vector (or single number), padded with zeros to ``cols``."""
+        v = self.get(name).float().to(self.device).reshape(-1)
+        if cols > len(v):
+            v = torch.cat([v, torch.zeros(cols - len(v), device=self.device)])
+        return v.contiguous()
+
+    def zeros(self, *shape) -> torch.Tensor:
+        return torch.zeros(*shape, dtype=self.dtype, device=self.device)
+
+    def padded(self, w: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
+        out = self.zeros(rows, cols)
+        out[: w.shape[0], : w.shape[1]] = w
+        return out
+
+    def heads(self, w: torch.Tensor, n: int, parts, cols: int) -> torch.Tensor:
+        """Head-major rows: each head's parts (true size, padded size) in turn."""
+        out = self.zeros(n, sum(p for _, p in parts), cols)
+        v = w.reshape(n, sum(s for s, _ in parts), w.shape[1])
+        src = dst = 0
+        for size, pad in parts:
+            out[:, dst: dst + size, : w.shape[1]] = v[:, src: src + size]
+            src, dst = src + size, dst + pad
+        return out.reshape(-1, cols)
+
+    def out_proj(self, name: str, heads: int, size: int, pad: int) -> torch.Tensor:
+        """Output projection over concatenated heads: [wp][heads * pad]."""
+        o = self.zeros(self.wp, heads, pad)
+        o[: self.cfg.hidden, :, :size] = self.t(name).reshape(self.cfg.hidden, heads, size)
+        return o.reshape(self.wp, heads * pad)
+
+    def gate_up(self, gate: str, up: str, ffp: int) -> torch.Tensor:
+        return interleave16(self.padded(self.t(gate), ffp, self.wp), self.padded(self.t(up), ffp, self.wp))
+
+
+def assemble(cfg: ModelConfig, get: Callable[[str], torch.Tensor], device, dtype=torch.bfloat16) -> ModelWeights:
+    """Kernel-layout weights from checkpoint tensors (``get(name)``)."""
+    from . import streams
+    a = Assembler(cfg, get, device, dtype)
+    wp, layers = a.wp, []
+    for i, s in enumerate(cfg.layer_specs):
+        p, f = f"l{i}.", s.ffn
+        lw = LayerWeights(input_norm=a.vec(p + "norm1"), post_norm=a.vec(p + "norm2") if f is not None else None, qkv=None, o=None)
+        lw.mixer = kind(s.mixer).assemble(a, p, s.mixer)
+        if cfg.block is not None:
+            lw.streams = streams.assemble(a, p, s)
+        if isinstance(f, DenseFfn):
+            ffp = pad64(f.ff)
+            lw.dense = DenseWeights(a.gate_up(p + "mlp.gate", p + "mlp.up", ffp), a.padded(a.t(p + "mlp.down"), wp, ffp))
+        elif f is not None:
+            ffp = pad64(f.ff)
+            gu, dn = a.zeros(f.experts, 2 * ffp, wp), a.zeros(f.experts, wp, ffp)
+            for e in range(f.experts):
+                q = f"{p}mlp.e{e}."
+                gu[e] = a.gate_up(q + "gate", q + "up", ffp)
+                dn[e, : cfg.hidden, : f.ff] = a.t(q + "down")
+            lw.moe = ExpertStack(a.padded(a.t(p + "mlp.router"), (f.experts + 7) // 8 * 8, wp), gu, dn)
+        layers.append(lw)
+    return ModelWeights(cfg, a.padded(a.t("embed"), cfg.vocab, wp), a.padded(a.t("head"), cfg.vocab, wp), a.vec("final.norm"), layers)
+
+
+def random_listed_weights(cfg: ModelConfig, device="cpu", seed: int = 0, std: float = 0.02,
+                          dtype=torch.bfloat16) -> ModelWeights:
+    from . import streams
+    shapes = tensor_shapes(cfg)
+    g = torch.Generator(device=device)
+    g.manual_seed(seed)
+
+    def get(name):
+        shape = shapes[name]
+        plain = streams.plain_value(cfg, name, shape)
+        if plain is not None:
+            return plain.to(device)
+        if len(shape) < 2:
+            return torch.ones(shape, device=device)
+        return torch.empty(shape, dtype=torch.bfloat16, device=device).normal_(0, std if name == "head" else shape[1] ** -0.5, generator=g)
+    return assemble(cfg, get, device, dtype)
+
+
+def padded_weight_elems(cfg: ModelConfig) -> int:
+    """Elements of the assembled weights (host arithmetic, the memory planner's figure)."""
+    wp, n = pad64(cfg.hidden), 2 * cfg.vocab * pad64(cfg.hidden)
+    for s in cfg.layer_specs:
+        f = s.ffn
+        n += kind(s.mixer).weight_elems(cfg, s.mixer)
+        if isinstance(f, DenseFfn):
+            n += 3 * pad64(f.ff) * wp
+        elif f is not None:
+            n += (f.experts + 7) // 8 * 8 * wp + 3 * f.experts * pad64(f.ff) * wp
+    return n
+
+
+def step_scratch_elems(cfg: ModelConfig, rows: int, keys: int = 0) -> int:
+    """Upper bound, in 32-bit words, of what a step of ``rows`` rows allocates (``keys``: expanded key rows)."""
+    wp, n = pad64(cfg.hidden), 0
+    for s in cfg.layer_specs:
+        f = s.ffn
+        one = rows * 10 * wp + kind(s.mixer).scratch_elems(cfg, s.mixer, rows, keys)
+        if isinstance(f, DenseFfn):
+            one += rows * 3 * pad64(f.ff)
+        elif f is not None:
+            slots = rows * f.top + (f.experts + 1) * 128
+            one += slots * (4 * wp + pad64(f.ff)) + rows * f.experts
+        n = max(n, one)
+    # layers of unequal sizes keep scratch of their own
+    n = n * len(set(cfg.layer_specs)) + rows * wp * 4
+    return n + (rows * wp * (2 * cfg.block.streams + 2) if cfg.block is not None else 0)
+
+
+# ------------------------------------------------------------------ scratch of a step
+class ListedScratch:
+    """Activations of a step by name.  The decode step's (``fixed`` rows) are allocated once, because captured graphs
+    keep their addresses; a mixed batch's grow with the largest batch."""
+
+    def __init__(self, device, dtype, fixed: int = 0):
+        self.device, self.dtype, self.fixed = device, dtype, fixed
+        self._t: Dict[tuple, torch.Tensor] = {}
+
+    def get(self, name: str, rows: int, cols: int, dtype=None, mult: int = 1) -> torch.Tensor:
+        """``[rows][cols]`` view; ``mult``: value rows per row of the step.  New memory is zeroed: padding that nothing
+        writes is zero and stale rows are finite."""
+        dtype = dtype or self.dtype
+        key = (name, cols, mult, dtype)
+        t = self._t.get(key)
+        need = max(rows, self.fixed * mult) * cols
+        if t is None or t.numel() < need:
+            if self.fixed and t is not None:
+                raise RuntimeError(f"the decode step's scratch {name!r} cannot grow under captured graphs")
+            t = self._t[key] = torch.zeros(need, dtype=dtype, device=self.device)
+        return t[: rows * cols].view(rows, cols)
+
+    @property
+    def nbytes(self) -> int:
+        return sum(t.numel() * t.element_size() for t in self._t.values())
+
+
+@dataclass
+class StepRows:
+    """The rows of a step: device int32 arrays of request slots, positions and tokens.  Rows of a request are consecutive."""
+    req: torch.Tensor
+    pos: torch.Tensor
+    token: torch.Tensor
+
+    def tail(self, n: int) -> "StepRows":
+        return StepRows(self.req[n:], self.pos[n:], self.token[n:])
+
+
+@dataclass
+class BatchPlan:
+    """How a mixed batch's rows are handled: rows before ``n_single`` one by one, the rest as prompt segments, described by
+    one table per form the model's mixers use (``tables[form]``, see ``runtime/batch.py``)."""
+    n_single: int
+    tables: Dict[tuple, object]
+
+
+class ListedLayers:
+    """Mixers and feed-forwards of a listed model over one device's weights."""
+
+    def __init__(self, weights: ModelWeights, max_pos: int):
+        self.w, self.cfg = weights, weights.cfg
+        self.device, self.dtype = weights.embed.device, weights.embed.dtype
+        self.f32 = self.dtype == torch.float32
+        self.wp = weights.embed.shape[1]
+        self.max_pos = max_pos
+        self.shared: Dict[tuple, object] = {}        # what layers of equal sizes share (angle tables and the like)
+        self._splits: Dict[tuple, int] = {}
+        self.mixers = [kind(s.mixer).Mixer(self, i, s.mixer, lw.mixer)
+                       for i, (s, lw) in enumerate(zip(self.cfg.layer_specs, weights.layers))]
+
+    def forms(self):
+        """Tables the mixers want of a mixed batch's prompt segments."""
+        return sorted({m.form for m in self.mixers if m.form is not None})
+
+    def linear(self, sc: ListedScratch, name: str, w: torch.Tensor, x: torch.Tensor, m: int):
+        """fp32 ``x[:m] @ w.T`` as (slices [s][m][n], s)."""
+        n, k = w.shape
+        if self.f32 or m > L.GEMV_ROWS:
+            out = sc.get(name, m, n, torch.float32)
+            if self.f32:
+                L.linear_f32(x, w, out, m)
+            else:
+                G.gemm_bf16(x[:m], w, out, epi=G.EPI_F32)
+            return out, 1
+        s = self.splits(n, k)
+        out = sc.get(name, m * s, n, torch.float32, mult=s)
+        L.gemv_bf16(w, x, out, m, n, k, s)
+        return out, s
+
+    def splits(self, n: int, k: int) -> int:
+        s = self._splits.get((n, k))
+        if s is None:
+            s = self._splits[(n, k)] = L.gemv_splits(n, k)
+        return s
+
+    # ---------------------------------------------------------------- feed-forwards
+    def dense(self, sc: ListedScratch, f: DenseFfn, w: DenseWeights, m: int):
+        """Gated feed-forward of the step's rows: fp32 slices of its down projection."""
+        h = sc.get("h", m, self.wp)
+        n = w.gate_up.shape[0]
+        act = sc.get("ffn_act", m, n // 2)
+        if self.f32:
+            gu = sc.get("gate_up", m, n)
+            L.linear_f32(h, w.gate_up, gu, m)
+            L.glu_rows_f32(gu, act, m, n, f.limit, f.alpha, f.shift)
+        elif m <= L.GEMV_ROWS:
+            L.gemv_bf16_glu(w.gate_up, h, act, m, n, self.wp, f.limit, f.alpha, f.shift)
+        else:
+            G.gemm_glu(h, w.gate_up, act, f.limit, f.alpha, f.shift)
+        return self.linear(sc, "ffn_down", w.down, act, m)
+
+    def experts(self, sc: ListedScratch, f: ExpertFfn, w: ExpertStack, m: int):
+        """Routed experts of the step's rows: arguments of ``sublayer_norm`` that describe the weighted slots."""
+        k, wp, er = f.top, self.wp, w.router.shape[0]
+        ffp = w.down.shape[2]
+        i32, f32 = torch.int32, torch.float32
+        h = sc.get("h", m, wp)
+        logits = sc.get("router", m, er, f32)
+        idx, wt = sc.get("topk_idx", m, k, i32), sc.get("topk_w", m, k, f32)
+        few = m <= EXPERT_GEMV_ROWS
+        if not self.f32 and m <= L.GEMV_ROWS:
+            M.router_rows(w.router, h, logits, m, f.experts, wp, er, f.experts, k, False, False, idx, wt,
+                          sc.get("ticket", 1, 1, i32), rule=f.rule)
+        else:
+            if self.f32:
+                L.linear_f32(h, w.router, logits, m)
+            else:
+                G.gemm_bf16(h, w.router, logits, epi=G.EPI_F32)
+            M.route(logits, er, m, f.experts, k, idx, wt, rule=f.rule)
+        if self.f32:
+            act, y = sc.get("act", m * k, ffp, mult=k), sc.get("y", m * k, wp, mult=k)
+            L.linear_f32_experts(w.gate_up, idx.view(-1), m * k, h, k, act, True)
+            L.linear_f32_experts(w.down, idx.view(-1), m * k, act, 1, y, False)
+            return dict(y=y, slots=k, row_elems=wp, slot_w=wt)
+        if few:
+            act = sc.get("act", m * k, ffp, mult=k)
+            L.gemv_bf16_experts(w.gate_up, idx, m * k, h, k, act, 2 * ffp, wp, epi=L.EPI_SILU)
+            s = self._splits.get((wp, ffp, "experts"))
+            if s is None:
+                s = self._splits[(wp, ffp, "experts")] = min(2, L.gemv_splits(wp, ffp))
+            y = sc.get("y", m * k * s, wp, f32, mult=k * s)
+            L.gemv_bf16_experts(w.down, idx, m * k, act, 1, y, wp, ffp, splits=s)
+            return dict(y=y, slots=k, slices=s, row_elems=s * wp, slice_elems=wp, slot_w=wt)
+        # expert-sorted rows in blocks of 128 for the grouped GEMMs; counts stay on the device
+        e = f.experts
+        blk = (m * k + 127) // 128 + e
+        cap = (max(m, sc.fixed) * k + 127) // 128 + e
+        meta = sc.get(f"moe_tables_{e}_{k}", 2 * e + 3 * cap + 2, 1, i32).view(-1)
+        counts, base, n_blk = meta[:e], meta[e: 2 * e], meta[2 * e: 2 * e + 1]
+        total, tabs = meta[2 * e + 1: 2 * e + 2], meta[2 * e + 2:]
+        be, br, bn = tabs[:blk], tabs[cap: cap + blk], tabs[2 * cap: 2 * cap + blk]
+        rank, row_of = sc.get("moe_rank", m, k, i32), sc.get("moe_row", m, k, i32)
+        xs, act, y = (sc.get(f"{nm}_{e}_{k}" if sc.fixed else nm, cap * 128, c) for nm, c in (("moe_x", wp), ("moe_act", ffp), ("moe_y", wp)))
+        counts.zero_()
+        M.sort(idx, m, k, e, blk, counts, rank, base, be, br, bn, n_blk, total)
+        M.scatter(idx, rank, base, m, k, h, wp, row_of, xs)
+        blocks = (be, br, bn, n_blk, blk)
+        G.gemm_grouped_bf16(xs, w.gate_up, act, blocks, epi=G.EPI_SILU_MUL)
+        G.gemm_grouped_bf16(act, w.down, y, blocks)
+        return dict(y=y, slots=k, row_elems=wp, slot_w=wt, row_of=row_of)

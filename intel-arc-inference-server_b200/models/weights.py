@@ -97,6 +97,41 @@ class LatentWeights:
 
 
 @dataclass
+class GroupedWeights:
+    """A grouped-query attention mixer, unquantised, heads padded to whole 64s."""
+    qkv: torch.Tensor              # [heads * dk + kv_heads * (dk + dv)][Wp], or the queries' rows alone
+    o: torch.Tensor                # [Wp][heads * dv]
+    slope2: Optional[torch.Tensor]     # fp32 [heads] distance bias times log2 e
+    sink2: Optional[torch.Tensor]      # fp32 [heads] sinks times log2 e
+
+
+@dataclass
+class MlstmWeights:
+    """An mLSTM mixer, unquantised, heads padded to whole 64s."""
+    proj: torch.Tensor             # [heads * 2 (dk + dv) + gates][Wp]: q, k, v, output gate, input gates, forget gates
+    gate_bias: torch.Tensor        # fp32 [2 * heads]
+    norm: torch.Tensor             # fp32 [heads * dv]
+    o: torch.Tensor                # [Wp][heads * dv]
+
+
+@dataclass
+class DenseWeights:
+    """Unquantised gated feed-forward, padded to whole 64s."""
+    gate_up: torch.Tensor          # [2 * ffp][Wp], interleave16
+    down: torch.Tensor             # [Wp][ffp]
+
+
+@dataclass
+class StreamWeights:
+    """How a layer's sublayers (mixer, feed-forward) read and write the residual streams; fp32."""
+    w_in: list                     # [streams]
+    w_out: list                    # [streams]
+    w_mix: list                    # [streams (from)][streams (to)]
+    scale: list                    # [Wp] or None: layer scale
+    shift: Optional[torch.Tensor]  # [Wp]: token shift of what the mixer reads
+
+
+@dataclass
 class ExpertStack:
     """Unquantised routed experts of one layer, padded to whole 64s."""
     router: torch.Tensor           # [E rounded up to 8][Wp]
@@ -120,9 +155,12 @@ class LayerWeights:
     experts_gate_up_w4b: Optional[torch.Tensor] = None
     experts_down_w4b: Optional[torch.Tensor] = None
     gdn: Optional[GdnWeights] = None               # set instead of qkv / o on gated delta-net layers
-    # listed layers: input_norm / post_norm then belong to the mixer's and the feed-forward's OUTPUT
-    latent: Optional[LatentWeights] = None
+    # listed layers: the norms then belong to the mixer's and the feed-forward's OUTPUT (one residual stream), or are
+    # single numbers for what they read (``streams`` set)
+    mixer: object = None                           # LatentWeights, GroupedWeights or MlstmWeights
     moe: Optional[ExpertStack] = None
+    dense: Optional[DenseWeights] = None
+    streams: Optional[StreamWeights] = None
 
 
 @dataclass
@@ -158,9 +196,9 @@ class ModelWeights:
                 tot += lw.experts_gate_up_w4b.numel() + lw.experts_down_w4b.numel()
             if lw.shared is not None:
                 tot += lw.shared.gate_up.nbytes + lw.shared.down.nbytes
-            for part in (lw.latent, lw.moe):
+            for part in (lw.mixer, lw.moe, lw.dense):
                 if part is not None:
-                    tot += sum(t.numel() * t.element_size() for t in vars(part).values())
+                    tot += sum(t.numel() * t.element_size() for t in vars(part).values() if t is not None)
         return tot
 
 
@@ -233,7 +271,7 @@ def random_weights(cfg: ModelConfig, device="cpu", seed: int = 0, exact: Optiona
     if exact is None:
         exact = cfg.param_count() < 100_000_000
     if cfg.layer_specs:
-        from .latent import random_listed_weights
+        from .listed import random_listed_weights
         return random_listed_weights(cfg, device, seed, std)
     h = cfg.hidden
     hr = cfg.vocab if head_rows is None else head_rows

@@ -1,5 +1,7 @@
-// Causal flash attention for prompt chunks on tcgen05 / TMEM: over the paged KV cache (head_dim 128), and over contiguous
-// key / value rows with their own head sizes (latent attention, whose keys and values are expanded before).
+// Causal flash attention for prompt chunks on tcgen05 / TMEM: over the paged KV cache (head_dim 128), over contiguous
+// key / value rows with their own head sizes (latent attention, whose keys and values are expanded before), and over
+// paged keys and values of any sizes for the segments of a mixed batch (tiles that name their sequence; optional distance
+// bias, sink and chunked mask, as in paged.cu).
 //
 //   O[r] = softmax( q[r] . K[0 .. pos(r)]^T / sqrt(D) ) V[0 .. pos(r)]      pos(r) = pos0 + r
 //
@@ -34,7 +36,11 @@ struct AttnPfParams {
   __nv_bfloat16* out;  // [C][n_q * D]
   // contiguous form: one entry per CTA column (blockIdx.x) of kTileWords ints: first row in q and out, rows (<= 128 per
   // query tile), position of the first row and key row of position 0, both counted from the segment's first key
+  // paged segments: first row in q and out, rows, absolute position of the first row, sequence (row of block_table)
   const int* tiles;
+  int chunk;           // paged segments, > 0: a row sees the keys of its own chunk of this many positions only
+  const float* slope2; // [n_q] distance bias per head, and sink2 [n_q], both times log2 e, or null
+  const float* sink2;
   int dn;              // columns of a head in the key matrix (a multiple of 64; the shared part fills up the head)
 };
 constexpr int kTileWords = 4;
@@ -67,13 +73,14 @@ constexpr int BK2 = 64;
 constexpr int kThreads2 = 608;    // TMA warp, MMA warp of tile 0, 2 tiles x 2 column halves x 4 softmax warps, MMA warp of tile 1
 constexpr int kMmaWarp1 = 18;
 // A form of the kernel: blocks of 64 dims of a query / key (NDK) and of a value (NDV), query tiles per CTA (NW; one where
-// two do not fit), ring depth (KVS: K / V tiles in flight), K / V from pages or from contiguous rows.
-template <int NDK_, int NDV_, int NW_, int KVS_, bool PAGED_>
+// two do not fit), ring depth (KVS: K / V tiles in flight), K / V from pages or from contiguous rows; SEG: paged segments.
+template <int NDK_, int NDV_, int NW_, int KVS_, bool PAGED_, bool SEG_ = false>
 struct Form {
   static constexpr int NDK = NDK_, NDV = NDV_, NW = NW_, KVS = KVS_, DV = NDV_ * 64;
-  static constexpr bool PAGED = PAGED_;
-  // softmax weights enter P V as one bf16 value, or (contiguous form) as two bf16 limbs, hi + lo, 16 bits of mantissa
-  static constexpr bool P2 = !PAGED_;
+  static constexpr bool PAGED = PAGED_, SEG = SEG_;
+  // softmax weights enter P V as one bf16 value, or (contiguous form, segments) as two bf16 limbs, hi + lo, 16 bits of
+  // mantissa
+  static constexpr bool P2 = !PAGED_ || SEG_;
   static constexpr int QT_BYTES = BQ * NDK * 128;           // a query tile: [d-blocks][128 rows][64]
   static constexpr int Q_BYTES = NW * QT_BYTES;
   static constexpr int K_BYTES = BK2 * NDK * 128;           // a K tile: [d-blocks][64 keys][64]
@@ -131,12 +138,15 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
   // row0: first row inside the chunk (segment); C rows; pos0: position of chunk row 0, counted from the first key;
   // qrow: row of q / out that holds chunk row 0; krow: key row of position 0 (contiguous form)
   int row0 = qt * F::NW * BQ, C = p.C, pos0 = p.pos0, qrow = 0, krow = 0;
-  if (!F::PAGED) {
+  const int* block_table = p.block_table;
+  if (!F::PAGED || F::SEG) {
     const int* tile = p.tiles + blockIdx.x * kTileWords;
     row0 = 0; qrow = tile[0]; C = tile[1]; pos0 = tile[2]; krow = tile[3];
+    if (F::SEG) block_table += (size_t)krow * p.max_blocks;
   }
   // key tiles each query tile needs, counted from the first tile any of the CTA's rows needs
-  const int t0 = p.window > 0 ? max(0, pos0 + row0 - p.window + 1) / BK2 : 0;
+  const int t0 = F::SEG ? (p.chunk > 0 ? (pos0 - pos0 % p.chunk) / BK2 : 0)
+                        : p.window > 0 ? max(0, pos0 + row0 - p.window + 1) / BK2 : 0;
   int n_w[2];
   n_w[0] = (pos0 + min(row0 + BQ, C) - 1) / BK2 + 1 - t0;
   n_w[1] = F::NW > 1 && row0 + BQ < C ? (pos0 + min(row0 + 2 * BQ, C) - 1) / BK2 + 1 - t0 : 0;
@@ -195,7 +205,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
 #pragma unroll
         for (int pg = 0; pg < n_pages && F::PAGED; ++pg) {
           const int pi = (t0 + i) * n_pages + pg;
-          const int page = pi < p.max_blocks ? __ldg(p.block_table + pi) : 0;
+          const int page = pi < p.max_blocks ? __ldg(block_table + pi) : 0;
           rowc[pg] = (page * p.n_kv + kh) * 16;
         }
         // contiguous rows: those past the segment are another's, or rows the workspace keeps finite, and masked out
@@ -206,8 +216,8 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         if (F::PAGED) {
 #pragma unroll
           for (int pg = 0; pg < n_pages; ++pg) {
-            tma_load_2d(k_s + pg * 2048, &map_k, 0, rowc[pg], b_kfull + 8 * s);
-            tma_load_2d(k_s + BK2 * 128 + pg * 2048, &map_k, 64, rowc[pg], b_kfull + 8 * s);
+#pragma unroll
+            for (int c = 0; c < NDK; ++c) tma_load_2d(k_s + c * (BK2 * 128) + pg * 2048, &map_k, c * 64, rowc[pg], b_kfull + 8 * s);
           }
         } else {
           const int cn = p.dn >> 6;
@@ -226,8 +236,8 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         if (F::PAGED) {
 #pragma unroll
           for (int pg = 0; pg < n_pages; ++pg) {
-            tma_load_2d(v_s + pg * 2048, &map_v, 0, rowc[pg], b_vfull + 8 * s);
-            tma_load_2d(v_s + BK2 * 128 + pg * 2048, &map_v, 64, rowc[pg], b_vfull + 8 * s);
+#pragma unroll
+            for (int c = 0; c < NDV; ++c) tma_load_2d(v_s + c * (BK2 * 128) + pg * 2048, &map_v, c * 64, rowc[pg], b_vfull + 8 * s);
           }
         } else {
 #pragma unroll
@@ -323,10 +333,13 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const int r = quarter * 32 + lane;    // row inside the tile
     const int rowg = row0 + w * BQ + r;   // row inside the chunk
     const int qpos = pos0 + rowg;
-    const int qlo = p.window > 0 ? qpos - p.window + 1 : 0;   // the row's keys: qlo <= key <= qpos
+    // the row's keys: qlo <= key <= qpos
+    const int qlo = F::SEG ? (p.chunk > 0 ? qpos - qpos % p.chunk : 0) : p.window > 0 ? qpos - p.window + 1 : 0;
     const bool row_ok = rowg < C;
     const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
     const int first_pos = pos0 + row0 + w * BQ;             // position of the tile's first row
+    const int last_lo = !F::SEG || p.chunk <= 0 ? 0 : first_pos + BQ - 1 - (first_pos + BQ - 1) % p.chunk;   // first key of its last row
+    const float slope = F::SEG && p.slope2 ? p.slope2[head] : 0.f;
     const int nt = n_w[w];
     // float [tile w][tile parity][half][128 rows]: the halves of a row exchange their maxima (and, at the end, sums)
     const uint32_t xch = bars + 256 + (uint32_t)w * (2 * 2 * 128 * 4);
@@ -350,7 +363,22 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       }
       // only tiles that reach past the tile's first row, or below the window of its last row, need the mask; a
       // masked score becomes -inf and drops out of the maximum and (2^-inf = 0) of the sums below
-      if (key0 + 31 > first_pos || (p.window > 0 && key0 < first_pos + BQ - p.window)) {
+      if constexpr (F::SEG) {      // scores in powers of two with the distance bias, as packed pairs
+        unsigned long long sc2, sl2, d2;
+        const float d0 = (float)(key0 - qpos);
+        asm("mov.b64 %0, {%1, %1};" : "=l"(sc2) : "f"(p.scale_log2));
+        asm("mov.b64 %0, {%1, %1};" : "=l"(sl2) : "f"(slope));
+#pragma unroll
+        for (int j = 0; j < 16; ++j) {
+          unsigned long long xy;
+          asm("mov.b64 %0, {%1, %2};" : "=l"(d2) : "f"(d0 + (float)(2 * j)), "f"(d0 + (float)(2 * j + 1)));
+          asm("mov.b64 %0, {%1, %2};" : "=l"(xy) : "r"(v[2 * j]), "r"(v[2 * j + 1]));
+          asm("mul.rn.f32x2 %0, %0, %1;" : "+l"(d2) : "l"(sl2));
+          asm("fma.rn.f32x2 %0, %0, %1, %2;" : "+l"(xy) : "l"(sc2), "l"(d2));
+          asm("mov.b64 {%0, %1}, %2;" : "=r"(v[2 * j]), "=r"(v[2 * j + 1]) : "l"(xy));
+        }
+      }
+      if (key0 + 31 > first_pos || (F::SEG ? key0 < last_lo : p.window > 0 && key0 < first_pos + BQ - p.window)) {
 #pragma unroll
         for (int j = 0; j < 32; ++j) {
           const int kj = key0 + j;
@@ -371,7 +399,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       asm volatile("bar.sync %0, 256;" ::"r"(2 + w) : "memory");
       float other;
       asm volatile("ld.shared.f32 %0, [%1];" : "=f"(other) : "r"(xch + (uint32_t)((sb * 2 + (half ^ 1)) * 128 + r) * 4));
-      tmax = fmaxf(tmax, other) * p.scale_log2;
+      tmax = fmaxf(tmax, other) * (F::SEG ? 1.f : p.scale_log2);
       APROF_T(t3_);
       float alpha = 1.f;
       if (tmax > mref + kLazy || (mref == -INFINITY && tmax > -INFINITY)) {
@@ -409,7 +437,8 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       for (int j = 0; j < 16; ++j) {
         unsigned long long xy;
         asm("mov.b64 %0, {%1, %2};" : "=l"(xy) : "r"(v[2 * j]), "r"(v[2 * j + 1]));
-        asm("fma.rn.f32x2 %0, %0, %1, %2;" : "+l"(xy) : "l"(sc2), "l"(nm2));
+        if (F::SEG) asm("add.rn.f32x2 %0, %0, %1;" : "+l"(xy) : "l"(nm2));
+        else asm("fma.rn.f32x2 %0, %0, %1, %2;" : "+l"(xy) : "l"(sc2), "l"(nm2));
         float x0, x1, e0, e1;
         asm("mov.b64 {%0, %1}, %2;" : "=f"(x0), "=f"(x1) : "l"(xy));
         asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e0) : "f"(x0));
@@ -458,6 +487,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       float lo;
       asm volatile("ld.shared.f32 %0, [%1];" : "=f"(lo) : "r"(xch + (uint32_t)((sb * 2 + (half ^ 1)) * 128 + r) * 4));
       l += lo;
+      if (F::SEG && p.sink2) l += exp2f(p.sink2[head] - mref);     // one more term without a key
     }
     // the last product (and, accumulating in issue order, every product before it)
     if (ok && nt > 0) ok = mbar_wait(b_odone(w, (nt - 1) & 1), ((nt - 1) >> 1) & 1, ERR_ATTN_WAIT);
@@ -505,11 +535,11 @@ EncodeTiledFn encode_fn() {
   }
   return fn;
 }
-int make_map_bf16(CUtensorMap* map, const void* ptr, uint64_t rows, uint64_t cols, uint32_t box_rows) {
+int make_map_bf16(CUtensorMap* map, const void* ptr, uint64_t rows, uint64_t cols, uint32_t box_rows, uint64_t ld = 0) {
   EncodeTiledFn fn = encode_fn();
   if (!fn) return -100;
   cuuint64_t dims[2] = {cols, rows};
-  cuuint64_t strides[1] = {cols * 2};
+  cuuint64_t strides[1] = {(ld ? ld : cols) * 2};
   cuuint32_t box[2] = {64, box_rows};
   cuuint32_t estr[2] = {1, 1};
   CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), dims, strides, box, estr,
@@ -603,6 +633,51 @@ extern "C" int b2_attn_prefill_rows(const void* q, const void* k, const void* kr
     case 24: return launch_form<Form<2, 4, 1, 3, false>>(mq, mk, mv, mr, p, n_tiles, H, st);
     case 34: return launch_form<Form<3, 4, 1, 3, false>>(mq, mk, mv, mr, p, n_tiles, H, st);
     case 44: return launch_form<Form<4, 4, 1, 2, false>>(mq, mk, mv, mr, p, n_tiles, H, st);
+  }
+  return -1;
+}
+
+// Query rows per CTA of the paged segments' form: 256, 128, or 0 when no form covers the sizes.
+extern "C" int b2_attn_segments_per_tile(int dk, int dv) {
+  if (dk % 64 || dv % 64 || dk < 64 || dk > 256 || dv < 64 || dv > 256) return 0;
+  return dk <= 192 && dv <= 128 ? 256 : 128;
+}
+
+template <int NDK>
+static int launch_segments(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const AttnPfParams& p, int ndv,
+                           int n_tiles, cudaStream_t st) {
+  constexpr int NW = NDK <= 3 ? 2 : 1;
+  switch (ndv) {
+    case 1: return launch_form<Form<NDK, 1, NW, NDK <= 2 ? 4 : 3, true, true>>(mq, mk, mv, mv, p, n_tiles, p.n_q, st);
+    case 2: return launch_form<Form<NDK, 2, NW, NDK <= 2 ? 4 : 3, true, true>>(mq, mk, mv, mv, p, n_tiles, p.n_q, st);
+    case 3: return launch_form<Form<NDK, 3, 1, NDK == 4 ? 2 : 3, true, true>>(mq, mk, mv, mv, p, n_tiles, p.n_q, st);
+    case 4: return launch_form<Form<NDK, 4, 1, NDK == 4 ? 2 : 3, true, true>>(mq, mk, mv, mv, p, n_tiles, p.n_q, st);
+  }
+  return -1;
+}
+
+// q: bf16 rows of ldq elements (the first H * dk of each are the queries); k / v caches [num_pages][G][16][dk | dv];
+// block_table [slots][max_blocks]; out [q_rows][H * dv].  tiles: n_tiles x 4 ints: first row of q, rows, position of that
+// row, slot.
+extern "C" int b2_attn_prefill_segments(const void* q, int ldq, const void* k_cache, const void* v_cache,
+                                        const int* block_table, int max_blocks, void* out, const int* tiles, int n_tiles,
+                                        int q_rows, int H, int G, int dk, int dv, int num_pages, float scale, int chunk,
+                                        const float* slope2, const float* sink2, void* stream) {
+  if (!b2_attn_segments_per_tile(dk, dv) || n_tiles < 1 || H < 1 || H % G || ldq % 8 || ldq < H * dk || chunk < 0) return -1;
+  CUtensorMap mq, mk, mv;
+  int rc = make_map_bf16(&mq, q, (uint64_t)q_rows, (uint64_t)H * dk, BQ, (uint64_t)ldq);
+  if (!rc) rc = make_map_bf16(&mk, k_cache, (uint64_t)num_pages * G * 16, (uint64_t)dk, 16);
+  if (!rc) rc = make_map_bf16(&mv, v_cache, (uint64_t)num_pages * G * 16, (uint64_t)dv, 16);
+  if (rc) return rc;
+  AttnPfParams p = {};
+  p.block_table = block_table; p.max_blocks = max_blocks; p.n_q = H; p.n_kv = G; p.scale_log2 = scale * 1.4426950408889634f;
+  p.out = (__nv_bfloat16*)out; p.tiles = tiles; p.chunk = chunk; p.slope2 = slope2; p.sink2 = sink2;
+  cudaStream_t st = (cudaStream_t)stream;
+  switch (dk / 64) {
+    case 1: return launch_segments<1>(mq, mk, mv, p, dv / 64, n_tiles, st);
+    case 2: return launch_segments<2>(mq, mk, mv, p, dv / 64, n_tiles, st);
+    case 3: return launch_segments<3>(mq, mk, mv, p, dv / 64, n_tiles, st);
+    case 4: return launch_segments<4>(mq, mk, mv, p, dv / 64, n_tiles, st);
   }
   return -1;
 }

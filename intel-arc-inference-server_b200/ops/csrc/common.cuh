@@ -273,6 +273,15 @@ __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + __expf(-x)); }
+// Gated product of two projections: g' sigmoid(alpha g') (u' + shift) with g' = min(g, limit), u' = clamp(u, -limit, limit)
+struct Glu {
+  float limit, alpha, shift;
+};
+__device__ __forceinline__ float glu(const Glu& p, float g, float u) {
+  g = fminf(g, p.limit);
+  u = fminf(fmaxf(u, -p.limit), p.limit);
+  return g / (1.0f + __expf(-p.alpha * g)) * (u + p.shift);
+}
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

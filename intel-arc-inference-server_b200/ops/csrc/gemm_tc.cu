@@ -41,7 +41,7 @@ constexpr int BM = 128;
 constexpr int BKB = 128;  // bytes of K per stage row (64 bf16 or 128 int8)
 constexpr int kThreads = 192;
 
-enum Epi : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SILU_MUL = 2, EPI_RESID_ADD = 3, EPI_RS_PUSH = 4, EPI_EP_RETURN = 5 };
+enum Epi : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SILU_MUL = 2, EPI_RESID_ADD = 3, EPI_RS_PUSH = 4, EPI_EP_RETURN = 5, EPI_GLU = 6 };
 
 struct GemmParams {
   int M, N, K;       // K in elements
@@ -81,6 +81,7 @@ struct GemmParams {
   // ---- W4 form: B as W4B blocks [expert][ceil(N / 128)][K / 64][4352 bytes]
   const uint8_t* w4;
   long long w4_expert_bytes;
+  Glu glu;           // EPI_GLU: SiLU(gate) * up with other constants
 };
 
 constexpr int kW4Block = 4352;     // one W4B block: 128 rows x 64 k of nibbles (4096 B) + 128 fp16 scales
@@ -380,13 +381,14 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
           float f[32];
 #pragma unroll
           for (int j = 0; j < 32; ++j) f[j] = __uint_as_float(v[j]);
-          if (p.epi == EPI_SILU_MUL) {
+          if (p.epi == EPI_SILU_MUL || p.epi == EPI_GLU) {
             // columns alternate 16 gate, 16 up: 16 outputs per 32 accumulator columns
             __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.C) + (size_t)grow * p.ldc + (n0 >> 1);
             uint32_t o[8];
 #pragma unroll
             for (int j = 0; j < 8; ++j)
-              o[j] = pack_bf16(silu(f[2 * j]) * f[16 + 2 * j], silu(f[2 * j + 1]) * f[17 + 2 * j]);
+              o[j] = p.epi == EPI_GLU ? pack_bf16(glu(p.glu, f[2 * j], f[16 + 2 * j]), glu(p.glu, f[2 * j + 1], f[17 + 2 * j]))
+                                      : pack_bf16(silu(f[2 * j]) * f[16 + 2 * j], silu(f[2 * j + 1]) * f[17 + 2 * j]);
             *reinterpret_cast<uint4*>(dst) = make_uint4(o[0], o[1], o[2], o[3]);
             *reinterpret_cast<uint4*>(dst + 8) = make_uint4(o[4], o[5], o[6], o[7]);
           } else if (p.epi == EPI_F32) {
@@ -624,9 +626,10 @@ static int gemm_tc_impl(const void* a, const void* b, void* c, int M, int N, int
                         const void* resid, const float* a_scale, const float* b_scale, const int* blk_expert,
                         const int* blk_row0, const int* blk_rows, const int* n_blk, int max_blk, int n_experts,
                         int bn, const void* rs_table, int rs_rank, int rs_world, int rs_tpr, const int* ag_cnt,
-                        int ag_expect, const int* blk_wait, const int* row_src, const void* ret_table, void* stream) {
+                        int ag_expect, const int* blk_wait, const int* row_src, const void* ret_table, void* stream,
+                        const Glu& glu = Glu{}) {
   if (K % (i8 ? 128 : 64) != 0 || M < 1 || N % 8 != 0) return -1;
-  if (epi == EPI_SILU_MUL && N % 32 != 0) return -2;
+  if ((epi == EPI_SILU_MUL || epi == EPI_GLU) && N % 32 != 0) return -2;
   if (epi == EPI_RS_PUSH && (!rs_table || rs_world < 1 || rs_world > kMaxRanks || rs_rank < 0 || rs_rank >= rs_world ||
                              rs_tpr < 1 || N % 64 != 0 || blk_expert || (M + BM - 1) / BM > rs_tpr * rs_world))
     return -3;
@@ -637,7 +640,7 @@ static int gemm_tc_impl(const void* a, const void* b, void* c, int M, int N, int
   if (epi == EPI_EP_RETURN && (!row_src || !ret_table || !blk_expert || N % 64 != 0)) return -4;
   p.mt_rot = (epi == EPI_RS_PUSH) ? (rs_rank * rs_tpr) % ((M + BM - 1) / BM) : 0;
   p.M = M; p.N = N; p.K = K; p.ldc = ldc; p.C = c; p.resid = (const __nv_bfloat16*)resid;
-  p.a_scale = a_scale; p.b_scale = b_scale; p.epi = epi;
+  p.a_scale = a_scale; p.b_scale = b_scale; p.epi = epi; p.glu = glu;
   p.blk_expert = blk_expert; p.blk_row0 = blk_row0; p.blk_rows = blk_rows; p.n_blk = n_blk; p.max_blk = max_blk;
   if (bn != 128 && bn != 256) bn = (N >= 256 && (N % 256 == 0 || N > 2048)) ? 256 : 128;
   CUtensorMap ma, mb;
@@ -658,6 +661,13 @@ extern "C" int b2_gemm_tc(const void* a, const void* b, void* c, int M, int N, i
                           int bn, void* stream) {
   return gemm_tc_impl(a, b, c, M, N, K, ldc, i8, epi, resid, a_scale, b_scale, blk_expert, blk_row0, blk_rows, n_blk,
                       max_blk, n_experts, bn, nullptr, 0, 1, 1, nullptr, 0, nullptr, nullptr, nullptr, stream);
+}
+
+// bf16 C [M][N / 2] = gated product of the interleave16 columns of A * B^T (common.cuh, Glu)
+extern "C" int b2_gemm_tc_glu(const void* a, const void* b, void* c, int M, int N, int K, int ldc, float limit, float alpha,
+                              float shift, void* stream) {
+  return gemm_tc_impl(a, b, c, M, N, K, ldc, 0, EPI_GLU, nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, 0, 1, 0,
+                      nullptr, 0, 1, 1, nullptr, 0, nullptr, nullptr, nullptr, stream, Glu{limit, alpha, shift});
 }
 
 // Tensor-parallel forms of the same kernel.  epi = 4 (row-parallel GEMM -> reduce-scatter): c is unused, the

@@ -6,11 +6,12 @@
 //                      activations as A and the weight rows as B, in a k order chosen so that a lane's 16-byte vector is
 //                      its fragment (as in the lm_head kernel).  The first weight vectors are requested before the
 //                      kernel waits for its predecessor.
-//                      Epilogues: fp32 slices [split][m][N] (the consumer folds them), bf16, or SiLU(gate) * up over
-//                      interleave16 rows.  Batched form: batch b multiplies activation row b / x_div with the weight of
+//                      Epilogues: fp32 slices [split][m][N] (the consumer folds them), bf16, or SiLU(gate) * up (or another
+//                      gated product) over interleave16 rows.  Batched form: batch b multiplies activation row b / x_div with the weight of
 //                      expert ids[b] (mixture-of-experts decode rows).
 //   linear_f32_kernel  C[M][N] = A[M][K] B[N][K]^T in fp32 FMA arithmetic (models served in 32-bit)
 //   linear_f32_rows    the batched expert form of it: one warp per output
+//   glu_rows_f32       gated product of interleave16 columns
 //
 // The role of the reference's bf16 GEMV (src/kernels/gemv_bf16.cl).
 #include "common.cuh"
@@ -19,7 +20,7 @@ using namespace b2;
 
 namespace {
 
-enum Epi : int { EPI_PART = 0, EPI_BF16 = 1, EPI_SILU = 2 };
+enum Epi : int { EPI_PART = 0, EPI_BF16 = 1, EPI_SILU = 2, EPI_GLU = 3 };
 
 struct GemvBfParams {
   const __nv_bfloat16* w;    // [N][K], or [E][N][K] in the batched form
@@ -27,6 +28,7 @@ struct GemvBfParams {
   const __nv_bfloat16* x;    // [rows][ldx]
   void* out;
   int M, N, K, ldx, splits, epi, x_div;
+  Glu glu;                   // EPI_GLU
 };
 
 constexpr int kStages = 4, kWarps = 4, NG = 4, KU = 2;
@@ -119,7 +121,7 @@ __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const GemvBfPara
 #pragma unroll
     for (int e = 0; e < 4; ++e) red[(warp * 16 + g + 8 * (e >> 1)) * 33 + 8 * j + 2 * t + (e & 1)] = acc[j][e];
   __syncthreads();
-  if (p.epi == EPI_SILU) {
+  if (p.epi >= EPI_SILU) {
     for (int i = threadIdx.x; i < M * 16; i += kWarps * 32) {
       const int m = i >> 4, c = i & 15;
       float gt = 0.f, up = 0.f;
@@ -129,7 +131,7 @@ __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const GemvBfPara
         up += red[(q * 16 + m) * 33 + 16 + c];
       }
       if (n0 + 16 + c < p.N)
-        reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)(batched ? batch : m) * (p.N / 2) + n0 / 2 + c] = __float2bfloat16(silu(gt) * up);
+        reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)(batched ? batch : m) * (p.N / 2) + n0 / 2 + c] = __float2bfloat16(p.epi == EPI_GLU ? glu(p.glu, gt, up) : silu(gt) * up);
     }
     return;
   }
@@ -207,6 +209,16 @@ __global__ void __launch_bounds__(256) linear_f32_rows_kernel(const float* __res
   if (lane == 0) out[(size_t)b * outs + o] = do_silu ? u / (1.f + expf(-u)) * v : u;
 }
 
+__global__ void __launch_bounds__(256) glu_rows_f32_kernel(const float* __restrict__ in, float* __restrict__ out, int N, const Glu p) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int o = blockIdx.x * 256 + threadIdx.x;
+  if (o >= N / 2) return;
+  const float* r = in + (size_t)blockIdx.y * N + (o >> 4) * 32 + (o & 15);
+  const float g = fminf(r[0], p.limit), u = fminf(fmaxf(r[16], -p.limit), p.limit);
+  out[(size_t)blockIdx.y * (N / 2) + o] = g / (1.f + expf(-p.alpha * g)) * (u + p.shift);
+}
+
 int sm_count() {
   static int n[64] = {};
   int dev = 0;
@@ -250,9 +262,24 @@ extern "C" int b2_gemv_bf16(const void* w, const int* ids, int batches, const vo
   if (K % 64 || N < 1 || M < 1 || M > 16 || splits < 1 || ldx % 8 || (epi != EPI_PART && splits != 1)) return -1;
   if (epi == EPI_SILU && N % 32) return -2;
   if (ids && (M != 1 || x_div < 1)) return -3;
-  GemvBfParams p{(const __nv_bfloat16*)w, ids, (const __nv_bfloat16*)x, out, M, N, K, ldx, splits, epi, x_div};
+  GemvBfParams p{(const __nv_bfloat16*)w, ids, (const __nv_bfloat16*)x, out, M, N, K, ldx, splits, epi, x_div, {}};
   return M <= 8 ? launch_gemv<1>(p, ids ? batches : 1, (cudaStream_t)stream)
                 : launch_gemv<2>(p, ids ? batches : 1, (cudaStream_t)stream);
+}
+
+// bf16 out [M][N / 2] = gated product of the interleave16 columns of x W^T
+extern "C" int b2_gemv_bf16_glu(const void* w, const void* x, int ldx, void* out, int M, int N, int K, float limit, float alpha,
+                                float shift, void* stream) {
+  if (K % 64 || N % 32 || M < 1 || M > 16 || ldx % 8) return -1;
+  GemvBfParams p{(const __nv_bfloat16*)w, nullptr, (const __nv_bfloat16*)x, out, M, N, K, ldx, 1, EPI_GLU, 1, {limit, alpha, shift}};
+  return M <= 8 ? launch_gemv<1>(p, 1, (cudaStream_t)stream) : launch_gemv<2>(p, 1, (cudaStream_t)stream);
+}
+
+// in fp32 [M][N] interleave16 -> out [M][N / 2]
+extern "C" int b2_glu_rows_f32(const float* in, float* out, int M, int N, float limit, float alpha, float shift, void* stream) {
+  if (M < 1 || M > 65535 || N % 32) return -1;
+  return b2_launch(glu_rows_f32_kernel, dim3((N / 2 + 255) / 256, M), dim3(256), 0, (cudaStream_t)stream, true, in, out, N,
+                   Glu{limit, alpha, shift});
 }
 
 extern "C" int b2_linear_f32(const float* a, const float* w, float* c, int M, int N, int K, void* stream) {

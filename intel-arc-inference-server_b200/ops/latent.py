@@ -31,6 +31,17 @@ def gemv_bf16(w, x, out, m: int, n: int, k: int, splits: int = 1, epi: int = EPI
              "gemv_bf16")
 
 
+def gemv_bf16_glu(w, x, out, m: int, n: int, k: int, limit: float, alpha: float, shift: float):
+    """The gated product of ``gemm.gemm_glu`` for ``m`` <= 16 rows."""
+    K._check(K.lib().b2_gemv_bf16_glu(K._p(w), K._p(x), x.stride(0), K._p(out), m, n, k, ctypes.c_float(limit), ctypes.c_float(alpha),
+                                      ctypes.c_float(shift), K._stream()), "gemv_bf16_glu")
+
+
+def glu_rows_f32(x, out, m: int, n: int, limit: float, alpha: float, shift: float):
+    K._check(K.lib().b2_glu_rows_f32(K._p(x), K._p(out), m, n, ctypes.c_float(limit), ctypes.c_float(alpha), ctypes.c_float(shift),
+                                     K._stream()), "glu_rows_f32")
+
+
 def gemv_bf16_experts(w, ids, batches: int, x, x_div: int, out, n: int, k: int, splits: int = 1, epi: int = EPI_PART):
     """Batch ``b``: row ``b // x_div`` of ``x`` against expert ``ids[b]`` of ``w`` ``[E][n][k]``."""
     K._check(K.lib().b2_gemv_bf16(K._p(w), K._p(ids), batches, K._p(x), x.stride(0), x_div, K._p(out), 1, n, k, splits, epi,

@@ -1,25 +1,84 @@
 """Mixed batches: prompt portions of some requests beside decode rows of others, as one walk over the layers.
 
 The decode step's control block holds 64 rows.  A batch here has a row table of its own (slot, position, token per row),
-uploaded with one copy together with everything else the kernels need: the wanted rows, and for every window of the
-model the cache rows the prompt segments see and their query tiles.  Entries of fewer than ``SEGMENT`` tokens are attended
-row by row over the latent, longer ones as prompt segments over expanded keys and values; both kinds share every linear
-and every expert of the step.  The walk itself is ``DecoderModel.listed_walk``, as in decode steps.
+uploaded with one copy together with everything else the kernels need: the wanted rows, and for every form of prompt
+segments the model's mixers use (``Mixer.form``) a table of its own.  Entries of fewer than ``SEGMENT`` tokens are handled
+row by row, longer ones as prompt segments; both kinds share every linear and every expert of the step.  The walk itself is
+``DecoderModel.listed_walk``, as in decode steps.
+
+Forms: ``("keys", window, rows per tile)`` lists the cache rows the segments see, to be expanded, and query tiles over them;
+``("tiles", chunk, rows per tile)`` query tiles over the pages; ``("chunks",)`` the segments of a recurrence.
 
 Takes the place of the reference's chunk walk (src/runtime/prefill/step.cc:102-319) for models that list their layers.
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import List, Optional, Sequence, Tuple
 
 import numpy as np
 import torch
 
-from ..models.latent import BatchPlan, KeyPlan, ListedScratch, StepRows
+from ..models.listed import BatchPlan, ListedScratch, StepRows
 from ..ops import lib as K
 
-SEGMENT = 32        # tokens from which an entry is attended as a prompt segment
+SEGMENT = 32        # tokens from which an entry is handled as a prompt segment
+CHUNK = 64          # rows of a recurrence's chunk
 ALIGN = 4           # int32 words: table parts start on 16-byte boundaries
+
+
+@dataclass
+class KeyPlan:
+    """Cache rows whose keys and values the segments see, and the query tiles over them."""
+    n_keys: int
+    kreq: torch.Tensor
+    kpos: torch.Tensor
+    n_tiles: int
+    tiles: torch.Tensor
+
+
+@dataclass
+class TilePlan:
+    """Query tiles over the pages."""
+    n_tiles: int
+    tiles: torch.Tensor
+
+
+@dataclass
+class ChunkPlan:
+    """Segments of a recurrence: [n][4] (first row, rows, slot, first chunk); chunks in total and in the longest one."""
+    n_segs: int
+    segs: torch.Tensor
+    chunks: int
+    most: int
+
+
+def segment_tiles(segments: Sequence[Tuple[int, int, int]], chunk: int, per: int):
+    """Query tiles of prompt segments (slot, first position, rows) as (first query row, rows, position of that row, slot):
+    at most ``per`` rows, and none across a border of chunks that hold more rows than a tile."""
+    tiles, qrow = [], 0
+    for slot, p, n in segments:
+        r = 0
+        while r < n:
+            c = min(per, n - r)
+            if chunk > per:
+                c = min(c, chunk - (p + r) % chunk)
+            tiles.append((qrow + r, c, p + r, slot))
+            r += c
+        qrow += n
+    keys = lambda t: t[2] % chunk + t[1] if chunk else t[2] + t[1]     # noqa: E731
+    tiles.sort(key=lambda t: -keys(t))                     # tiles with many keys first
+    return tiles
+
+
+def segment_chunks(segments: Sequence[Tuple[int, int, int]]):
+    """Prompt segments of a recurrence as (first row, rows, slot, first chunk), and the number of chunks."""
+    out, row, chunks = [], 0, 0
+    for slot, _, n in segments:
+        out.append((row, n, slot, chunks))
+        row += n
+        chunks += (n + CHUNK - 1) // CHUNK
+    return out, chunks
 
 
 def segment_keys(segments: Sequence[Tuple[int, int, int]], window: int, per: int):
@@ -44,8 +103,7 @@ class BatchRunner:
         self.eng, self.max_tokens = engine, max_tokens
         ll = engine.model.listed
         self.scratch = ListedScratch(engine.device, ll.dtype)
-        # forms of the expanded attention the model's layers use: (window, query rows per tile)
-        self.forms = sorted({(s.mixer.window, ll.tile_rows(g)) for s, g in zip(engine.cfg.layer_specs, ll.geo) if ll.tile_rows(g)})
+        self.forms = ll.forms()
 
     # ------------------------------------------------------------------ tables
     def _tables(self, singles, segments, want: np.ndarray):
@@ -64,15 +122,24 @@ class BatchRunner:
         spans = {"req": add(np.concatenate([np.full(len(t), s) for s, _, t in both])),
                  "pos": add(np.concatenate([np.arange(p, p + len(t)) for _, p, t in both])),
                  "token": add(np.concatenate([np.asarray(t) for _, _, t in both])), "want": add(want)}
-        keys = {}
-        for window, per in self.forms if segments else ():
-            kreq, kpos, tiles = segment_keys([(s, p, len(t)) for s, p, t in segments], window, per)
-            keys[(window, per)] = (len(kreq), add(kreq), add(kpos), len(tiles), add(tiles))
-        return np.concatenate(parts), spans, keys
+        segs, tables = [(s, p, len(t)) for s, p, t in segments], {}
+        for form in self.forms if segments else ():
+            if form[0] == "keys":
+                kreq, kpos, tiles = segment_keys(segs, form[1], form[2])
+                k, t = (add(kreq), add(kpos)), add(tiles)
+                tables[form] = lambda cut, n=len(kreq), k=k, nt=len(tiles), t=t: KeyPlan(n, cut(k[0]), cut(k[1]), nt, cut(t))
+            elif form[0] == "tiles":
+                tiles = segment_tiles(segs, form[1], form[2])
+                tables[form] = lambda cut, nt=len(tiles), t=add(tiles): TilePlan(nt, cut(t))
+            else:
+                rows, chunks = segment_chunks(segs)
+                most = max((n + CHUNK - 1) // CHUNK for _, _, n in segs)
+                tables[form] = lambda cut, n=len(rows), t=add(rows), c=chunks, most=most: ChunkPlan(n, cut(t), c, most)
+        return np.concatenate(parts), spans, tables
 
     def _walk(self, entries: Sequence[Tuple[int, List[int]]], want: Sequence[Tuple[int, int]]):
         """One batch: ``entries`` (slot, tokens) through all layers, K / V appended.  ``want``: (entry, place) pairs.
-        Returns (residual rows, device indices of the wanted ones)."""
+        Returns (the walk's rows, device indices of the wanted ones)."""
         eng, m = self.eng, self.eng.model
         slots = [s for s, _ in entries]
         if len(set(slots)) != len(slots):
@@ -87,17 +154,16 @@ class BatchRunner:
             n += len(entries[i][1])
         item = lambda i: (entries[i][0], eng.seq_len[entries[i][0]], entries[i][1])   # noqa: E731
         singles, segments = [item(i) for i in order if not seg[i]], [item(i) for i in order if seg[i]]
-        host, spans, keys = self._tables(singles, segments, np.asarray([start[i] + j for i, j in want], dtype=np.int32))
+        host, spans, tables = self._tables(singles, segments, np.asarray([start[i] + j for i, j in want], dtype=np.int32))
         dev = torch.from_numpy(host).pin_memory().to(eng.device, non_blocking=True)
         cut = lambda span: dev[span[0]: span[0] + span[1]]                              # noqa: E731
         rows = StepRows(cut(spans["req"]), cut(spans["pos"]), cut(spans["token"]))
-        plan = BatchPlan(sum(len(t) for _, _, t in singles),
-                         {f: KeyPlan(nk, cut(a), cut(b), nt, cut(c)) for f, (nk, a, b, nt, c) in keys.items()})
-        resid = self.scratch.get("resid", n, m.listed.wp, torch.float32)
-        m.listed_walk(n, rows, eng.block_table, eng.kv, self.scratch, resid, plan)
+        plan = BatchPlan(sum(len(t) for _, _, t in singles), {f: make(cut) for f, make in tables.items()})
+        resid = self.scratch.get("resid", n, m.listed.wp, torch.float32) if m.streams is None else None
+        final = m.listed_walk(n, rows, eng.block_table, eng.kv, self.scratch, resid, plan)
         for s, t in entries:
             eng.seq_len[s] += len(t)
-        return resid, cut(spans["want"])
+        return final, cut(spans["want"])
 
     # ------------------------------------------------------------------ whole steps
     def run(self, entries: Sequence[Tuple[int, List[int], List[int]]]) -> torch.Tensor:
@@ -120,13 +186,13 @@ class BatchRunner:
                     room -= k
             want = [(j, w - lo) for j, (i, lo, k) in enumerate(now) for w in sorted(set(entries[i][2])) if lo <= w < lo + k]
             dst = [where[(now[j][0], w + now[j][1])] for j, w in want]
-            resid, sel = self._walk([(entries[i][0], entries[i][1][lo: lo + k]) for i, lo, k in now], want)
-            self._logits(resid, sel, dst, out)
+            final, sel = self._walk([(entries[i][0], entries[i][1][lo: lo + k]) for i, lo, k in now], want)
+            self._logits(final, sel, dst, out)
             for i, lo, k in now:
                 cut[i] = lo + k
         return out[:total]
 
-    def _logits(self, resid, sel, dst, out):
+    def _logits(self, final, sel, dst, out):
         m = self.eng.model
         step = m.buf.max_rows
         for c0 in range(0, len(dst), step):
@@ -134,7 +200,7 @@ class BatchRunner:
             n = len(d)
             straight = d == [[d[0][0] + i] for i in range(n)]
             lg = out[d[0][0]: d[0][0] + n] if straight else self.scratch.get("logits_part", n, self.eng.cfg.vocab, torch.float32)
-            m.listed_logits(resid, sel[c0: c0 + n], n, self.scratch, lg)
+            m.listed_logits(final, sel[c0: c0 + n], n, self.scratch, lg)
             if not straight:
                 for i, rows in enumerate(d):
                     for r in rows:
@@ -147,7 +213,7 @@ class BatchRunner:
         for c0 in range(0, len(ids), chunk):
             part = ids[c0: c0 + chunk]
             last = c0 + chunk >= len(ids)
-            resid, sel = self._walk([(slot, part)], [(0, len(part) - 1)] if last else [])
-        m.listed_logits(resid, sel, 1, self.scratch, m.buf.logits)
+            final, sel = self._walk([(slot, part)], [(0, len(part) - 1)] if last else [])
+        m.listed_logits(final, sel, 1, self.scratch, m.buf.logits)
         K.argmax_finish(m.buf.cand_val, m.buf.cand_idx, m.buf.ncand, 1, eng.ctrl, False)
         return eng._read_out(1)[0]

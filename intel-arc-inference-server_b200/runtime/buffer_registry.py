@@ -35,9 +35,10 @@ def _tensors(obj):
     return {n: v for n, v in vars(obj).items() if isinstance(v, torch.Tensor)}
 
 
-def _audit_listed(buf, kv, cfg: ModelConfig, kv_dtype: str) -> Dict[str, int]:
-    """The same promise for a model that lists its layers: step scratch and latent pages within the planner's figures."""
-    groups = {"step": buf.scratch.nbytes, "kv": sum(t.numel() * t.element_size() for t in kv.latent), "state": 0}
+def _audit_listed(buf, kv, cfg: ModelConfig, kv_dtype: str, max_seqs: int) -> Dict[str, int]:
+    """The same promise for a model that lists its layers: step scratch, pages and states within the planner's figures."""
+    size = lambda ts: sum(t.numel() * t.element_size() for t in ts)       # noqa: E731
+    groups = {"step": buf.scratch.nbytes, "kv": size(kv.pages.values()), "state": size(kv.states.values())}
     for name, t in _tensors(buf).items():
         if name not in STEP_BUFFERS:
             raise AssertionError(f"ListedBuffers.{name} has no entry in runtime/buffer_registry.py")
@@ -46,15 +47,17 @@ def _audit_listed(buf, kv, cfg: ModelConfig, kv_dtype: str) -> Dict[str, int]:
     if groups["step"] > planned:
         raise AssertionError(f"step buffers hold {groups['step']} bytes, the planner budgets {planned}")
     if groups["kv"] != kv.num_pages * MP.kv_bytes_per_page(cfg, kv_dtype):
-        raise AssertionError(f"latent pool holds {groups['kv']} bytes, the planner counts "
+        raise AssertionError(f"page pool holds {groups['kv']} bytes, the planner counts "
                              f"{kv.num_pages * MP.kv_bytes_per_page(cfg, kv_dtype)}")
+    if groups["state"] > max_seqs * MP.state_bytes_per_slot(cfg):
+        raise AssertionError(f"recurrent state holds {groups['state']} bytes, the planner budgets {max_seqs * MP.state_bytes_per_slot(cfg)}")
     return groups
 
 
 def audit(buf, kv, cfg: ModelConfig, kv_dtype: str = "bf16", max_seqs: int = 1) -> Dict[str, int]:
     """Checks ``buf`` (StepBuffers) and ``kv`` (KVCache) against the tables and the planner; returns bytes per group."""
     if cfg.layer_specs:
-        return _audit_listed(buf, kv, cfg, kv_dtype)
+        return _audit_listed(buf, kv, cfg, kv_dtype, max_seqs)
     groups = {"step": 0, "kv": 0, "state": 0}
     for obj, table, what in ((buf, STEP_BUFFERS, "StepBuffers"), (kv, KV_BUFFERS, "KVCache")):
         for name, t in _tensors(obj).items():
@@ -73,7 +76,7 @@ def audit(buf, kv, cfg: ModelConfig, kv_dtype: str = "bf16", max_seqs: int = 1) 
     planned_kv = kv.num_pages * per_page
     if groups["kv"] != planned_kv:
         raise AssertionError(f"KV pool holds {groups['kv']} bytes, the planner counts {planned_kv} for {kv.num_pages} pages")
-    planned_state = max_seqs * MP.gdn_state_bytes_per_slot(cfg)
+    planned_state = max_seqs * MP.state_bytes_per_slot(cfg)
     if groups["state"] > planned_state:
         raise AssertionError(f"recurrent state holds {groups['state']} bytes, the planner budgets {planned_state}")
     return groups

@@ -76,7 +76,7 @@ class Engine:
         self.out_host = torch.zeros(K.CTRL_WORDS, dtype=torch.int32).pin_memory()
         self.block_table = torch.zeros(max_seqs, self.max_blocks, dtype=torch.int32, device=self.device)
         self.seq_len = [0] * max_seqs
-        self._gdn_snap = None       # (rows, {slot: state before them}) of the last forward_rows step of a hybrid model
+        self._snap = None           # (rows, {slot: recurrent state before them}) of the last step of a recurrent model
         self.use_graphs = use_graphs
         self.graphs: Dict[Tuple[int, bool, bool], torch.cuda.CUDAGraph] = {}
         self._one_request = False   # the rows last written are consecutive positions of one request
@@ -112,33 +112,32 @@ class Engine:
         for s in slots:
             self.pool.release(s)
             self.seq_len[s] = 0
-            self.kv.reset_slot(s)       # recurrent state of gated delta-net layers
+            self.kv.reset_slot(s)       # recurrent state
 
     def truncate(self, slot: int, length: int):
         """Drop everything after ``length`` positions (rejected draft rows)."""
         assert length <= self.seq_len[slot]
         replay = None
-        if length < self.seq_len[slot] and self.cfg.n_gdn_layers:
+        if length == 0 < self.seq_len[slot]:
+            self.kv.reset_slot(slot)
+        elif length < self.seq_len[slot] and self.kv.states:
             # A recurrent state cannot be rewound.  The last multi-row step left a copy of the slot's state from
             # before its rows (the reference snapshots its GDN state the same way around verify rows): put it
             # back and run the rows that stay once more.
-            snap = self._gdn_snap
+            snap = self._snap
             rows = [] if snap is None else [r for r in snap[0] if r.slot == slot]
             if not rows or slot not in snap[1] or length < rows[0].pos or self.seq_len[slot] != rows[-1].pos + 1:
-                raise NotImplementedError("a gated delta-net layer's recurrent state can only be rewound to a position "
-                                          "inside the last multi-row step (prefix reuse is not available for the "
-                                          "hybrid family)")
-            conv, state = snap[1][slot]
-            self.kv.gdn_conv[:, slot].copy_(conv)
-            self.kv.gdn_state[:, slot].copy_(state)
+                raise NotImplementedError("a recurrent state can only be rewound to a position inside the last multi-row "
+                                          "step (prefix reuse is not available for recurrent families)")
+            self.kv.load_states(slot, snap[1][slot])
             replay = [r for r in rows if r.pos < length]
             self.seq_len[slot] = rows[0].pos
-            self._gdn_snap = None
+            self._snap = None
         self.seq_len[slot] = min(self.seq_len[slot], length)
         self.pool.truncate(slot, (length + PAGE - 1) // PAGE)
         if replay:
             self.forward_rows(replay, advance=False, read=False)
-            self._gdn_snap = None       # one rewind per step
+            self._snap = None           # one rewind per step
 
     def _ensure_pages(self, slot: int, upto_len: int):
         if upto_len > self.max_len:
@@ -180,18 +179,17 @@ class Engine:
         the layout is ``[layer][page][kv head][16][head dim]`` per tensor and does not depend on the parallel mode."""
         if begin % PAGE or (end % PAGE and end != self.seq_len[slot]) or not 0 <= begin <= end <= self.seq_len[slot]:
             raise ValueError("save_kv takes whole pages inside the sequence")
-        if self.kv.gdn_state is not None and end != self.seq_len[slot]:
-            raise ValueError("save_kv: a hybrid model's snapshot ends at the sequence end (the recurrent state of its "
-                             "gated delta-net layers is the one after the last position)")
+        if self.kv.states and end != self.seq_len[slot]:
+            raise ValueError("save_kv: a recurrent model's snapshot ends at the sequence end (its state is the one after the "
+                             "last position)")
         pages = list(self.pool.table(slot))[begin // PAGE: (end + PAGE - 1) // PAGE]
         idx = torch.as_tensor(pages, device=self.device, dtype=torch.int64)
         tensors = self.kv.page_tensors()
         out = {"begin": begin, "end": end, "kv_dtype": self.kv_dtype}
-        if self.kv.gdn_state is not None:      # the recurrent state and the convolution window after position end - 1
-            for name, t in (("gdn_conv", self.kv.gdn_conv), ("gdn_state", self.kv.gdn_state)):
-                host = torch.empty((t.shape[0],) + tuple(t.shape[2:]), dtype=t.dtype).pin_memory()
-                host.copy_(t[:, slot], non_blocking=True)
-                out[name] = host
+        for name, t in self.kv.states.items():      # the recurrent state after position end - 1
+            host = torch.empty((t.shape[0],) + tuple(t.shape[2:]), dtype=t.dtype).pin_memory()
+            host.copy_(t[:, slot], non_blocking=True)
+            out[name] = host
         for name, t in tensors.items():
             host = torch.empty((t.shape[0], len(pages)) + tuple(t.shape[2:]), dtype=t.dtype).pin_memory()
             host.copy_(t.index_select(1, idx), non_blocking=True)
@@ -210,12 +208,11 @@ class Engine:
         tensors = self.kv.page_tensors()
         for name, t in tensors.items():
             t.index_copy_(1, idx, blob[name].to(self.device, non_blocking=True))
-        if self.kv.gdn_state is not None:
-            if "gdn_state" not in blob:
-                raise ValueError("load_kv: the blob holds no recurrent state for this hybrid model")
-            self.kv.gdn_conv[:, slot].copy_(blob["gdn_conv"].to(self.device, non_blocking=True))
-            self.kv.gdn_state[:, slot].copy_(blob["gdn_state"].to(self.device, non_blocking=True))
-            self._gdn_snap = None
+        if self.kv.states:
+            if any(name not in blob for name in self.kv.states):
+                raise ValueError("load_kv: the blob holds no recurrent state for this model")
+            self.kv.load_states(slot, blob)
+            self._snap = None
         self.seq_len[slot] = end
 
     # ------------------------------------------------------------------ running a step
@@ -233,16 +230,15 @@ class Engine:
             # warm-up outside capture (sets function attributes, allocates split-K scratch), then
             # restore the control block the warm-up advanced
             saved = self.ctrl.clone()
-            # KV appends repeat harmlessly; a gated delta-net layer's recurrent update does not: its state is put back
-            saved_gdn = None if self.kv.gdn_state is None else (self.kv.gdn_conv.clone(), self.kv.gdn_state.clone())
+            # KV appends repeat harmlessly; a recurrent update does not: the state is put back
+            saved_states = {n: t.clone() for n, t in self.kv.states.items()}
             n0 = K.launch_count
             self._enqueue(m, advance)
             self.launches_per_step[key] = K.launch_count - n0
             torch.cuda.current_stream().synchronize()
             self.ctrl.copy_(saved)
-            if saved_gdn is not None:
-                self.kv.gdn_conv.copy_(saved_gdn[0])
-                self.kv.gdn_state.copy_(saved_gdn[1])
+            for n, t in saved_states.items():
+                self.kv.states[n].copy_(t)
             g = torch.cuda.CUDAGraph()
             # no garbage collection while the stream captures: a dead engine's graphs and buffers released in the middle
             # of it abort the process
@@ -302,16 +298,18 @@ class Engine:
         self.require_ok()
         for r in rows:
             self._ensure_pages(r.slot, r.pos + 1)
-        self._gdn_snap = None
-        if self.kv.gdn_state is not None:
-            slots = sorted({r.slot for r in rows})
-            self._gdn_snap = (list(rows), {s: (self.kv.gdn_conv[:, s].clone(), self.kv.gdn_state[:, s].clone())
-                                           for s in slots})
+        self._snapshot(rows)
         self._write_rows(rows)
         self._run(len(rows), advance)
         for r in rows:
             self.seq_len[r.slot] = max(self.seq_len[r.slot], r.pos + 1)
         return self._read_out(len(rows)) if read else None
+
+    def _snapshot(self, rows: Sequence[Row]):
+        """Keeps the recurrent state from before a step's rows, so that its last rows can be taken back (``truncate``)."""
+        self._snap = None
+        if self.kv.states and rows:
+            self._snap = (list(rows), {s: self.kv.save_states(s) for s in sorted({r.slot for r in rows})})
 
     def logits(self, m: int) -> torch.Tensor:
         """fp32 logits of the last step's rows (device tensor view)."""
@@ -332,6 +330,9 @@ class Engine:
         if n == 0:
             return self.logits(0)
         if n > self.max_rows and self.mixed_batches:
+            # rows of entries short enough to be a decode step's can be taken back afterwards, as in ``forward_rows``
+            self._snapshot([Row(s, self.seq_len[s] + i, t) for s, toks, _ in entries if 1 < len(toks) <= 16
+                            for i, t in enumerate(toks)])
             out = self._batch_runner().run(entries)
             self.check_failed_sync("batch")
             return out
@@ -373,6 +374,7 @@ class Engine:
         ids = list(ids)
         if self.mixed_batches and len(ids) > self.max_rows:
             self.last_prefill_row = 0
+            self._snap = None
             return self._batch_runner().prefill(slot, ids, chunk)
         if self._use_tc_prefill(len(ids)):
             if self._prefill is None:

@@ -50,7 +50,7 @@ class MemoryPlan:
 def weight_bytes(cfg: ModelConfig, int8_head: bool = False, tp: int = 1, ep: int = 1) -> int:
     h = cfg.hidden
     if cfg.layer_specs:
-        from ..models.latent import padded_weight_elems
+        from ..models.listed import padded_weight_elems
         return int(padded_weight_elems(cfg) * 2)
     int4 = 0.5 + 2.0 / 64
     per = cfg._mixer_params() * int4 / tp      # attention projections, or a gated delta-net layer's (mean over layers)
@@ -66,15 +66,23 @@ def weight_bytes(cfg: ModelConfig, int8_head: bool = False, tp: int = 1, ep: int
 
 def kv_bytes_per_page(cfg: ModelConfig, kv_dtype: str, tp: int = 1) -> int:
     if cfg.layer_specs:
-        from ..models.latent import LatentGeometry
-        return sum(LatentGeometry.of(s.mixer).lc for s in cfg.layer_specs) * cfg.page_size * (4 if kv_dtype == "f32" else 2)
+        from ..models.listed import kind
+        planes = [pl for s in cfg.layer_specs for pl in kind(s.mixer).page_planes(s.mixer).values()]
+        return sum(max(1, heads) * cols for heads, cols in planes) * cfg.page_size * (4 if kv_dtype == "f32" else 2)
     per_tok_head = cfg.head_dim * (1 if kv_dtype == "int8" else 2) + (4 if kv_dtype == "int8" else 0)
     return (cfg.n_layers - cfg.n_gdn_layers + cfg.mtp_layers) * 2 * (cfg.n_kv_heads // tp) * per_tok_head * cfg.page_size
 
 
-def gdn_state_bytes_per_slot(cfg: ModelConfig) -> int:
-    """Recurrent state (fp32, one head_dim x head_dim matrix per value head) and convolution window of the gated
-    delta-net layers of one sequence slot; twice, for the copy that rewinds rejected rows."""
+def state_bytes_per_slot(cfg: ModelConfig) -> int:
+    """Recurrent state of one sequence slot; twice, for the copy that rewinds rejected rows.  Gated delta-net layers: fp32,
+    one head_dim x head_dim matrix per value head, and the convolution window.  Listed models: their mixers' states, and the
+    token shift's row per layer."""
+    if cfg.layer_specs:
+        from ..models.listed import kind, pad64
+        n = sum(sum(kind(s.mixer).state_shape(s.mixer) or (0,)) for s in cfg.layer_specs)
+        if cfg.block is not None and cfg.block.shift:
+            n += (cfg.n_layers + 1) * pad64(cfg.hidden)
+        return 2 * 4 * n
     if not cfg.n_gdn_layers:
         return 0
     per = cfg.gdn_v_heads * cfg.gdn_head_dim * cfg.gdn_head_dim * 4 + cfg.gdn_conv_channels * 3 * 4
@@ -84,7 +92,7 @@ def gdn_state_bytes_per_slot(cfg: ModelConfig) -> int:
 def step_scratch_bytes(cfg: ModelConfig, max_rows: int = 64, nsplit: int = 32) -> int:
     h = cfg.hidden
     if cfg.layer_specs:
-        from ..models.latent import step_scratch_elems
+        from ..models.listed import step_scratch_elems
         return max_rows * cfg.vocab * 4 + 4 * step_scratch_elems(cfg, max_rows) + (1 << 16)
     b = max_rows * (2 * h * 2 + 2 * cfg.q_dim * 2 + cfg.vocab * 4)
     b += max_rows * cfg.n_q_heads * nsplit * (cfg.head_dim + 2) * 4
@@ -99,7 +107,7 @@ def step_scratch_bytes(cfg: ModelConfig, max_rows: int = 64, nsplit: int = 32) -
 def prefill_scratch_bytes(cfg: ModelConfig, chunk: int, backend: str) -> int:
     h = cfg.hidden
     if cfg.layer_specs:      # rows of a mixed batch, and expanded keys / values of a window before it
-        from ..models.latent import step_scratch_elems
+        from ..models.listed import step_scratch_elems
         return 4 * step_scratch_elems(cfg, chunk, keys=2 * chunk)
     ffn = cfg.ffn if not cfg.is_moe else max(cfg.expert_ffn, cfg.shared_ffn)
     b = chunk * (2 * h * 2 + cfg.qkv_dim * 4 + 2 * cfg.q_dim * 2 + ffn * 2)
@@ -135,7 +143,7 @@ def plan(cfg: ModelConfig, max_seqs: int, max_len, kv_dtype: str = "bf16", int8_
     st = step_scratch_bytes(cfg)
     pf = prefill_scratch_bytes(cfg, prefill_chunk, prefill_backend)
     page = kv_bytes_per_page(cfg, kv_dtype, tp)
-    fixed = w + resident + st + pf + RESERVE_BYTES + max_seqs * gdn_state_bytes_per_slot(cfg)
+    fixed = w + resident + st + pf + RESERVE_BYTES + max_seqs * state_bytes_per_slot(cfg)
     if fixed >= budget:
         raise ValueError(f"{cfg.name}: weights and scratch need {fixed / 2**30:.1f} GiB of {budget / 2**30:.1f} GiB "
                          "before any KV cache")

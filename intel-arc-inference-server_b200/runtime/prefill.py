@@ -209,7 +209,7 @@ class PrefillRunner:
         eng, cfg, m = self.eng, self.cfg, self.eng.model
         c, h = len(ids), cfg.hidden
         eng._ensure_pages(slot, pos0 + c)
-        eng._gdn_snap = None      # (a hybrid model's recurrent state moves on: nothing to rewind to)
+        eng._snap = None      # (a hybrid model's recurrent state moves on: nothing to rewind to)
         ids_host = self.ids_stage.begin()
         ids_host[:c] = torch.as_tensor(ids, dtype=torch.int64)
         self.ids_stage.push(self.ids_dev[:c], ids_host[:c])

@@ -163,11 +163,11 @@ def write_drafter(head, cfg: ModelConfig, path: str, fmt: str = "int4", prefix: 
 def write_listed(cfg: ModelConfig, path: str, seed: int = 0, make=None) -> Dict[str, torch.Tensor]:
     """A snapshot of a model that lists its layers (``config.json`` in the design's keys, one safetensors file) with
     random weights; ``make(name, tensor)`` may replace a tensor.  Returns the tensors written."""
-    from ..models.latent import tensor_shapes
+    from ..models.listed import tensor_shapes
     g = torch.Generator().manual_seed(seed)
     out = {}
     for name, shape in tensor_shapes(cfg).items():
-        t = 1.0 + 0.2 * torch.randn(shape, generator=g) if len(shape) == 1 else torch.randn(shape, generator=g) * (
+        t = 1.0 + 0.2 * torch.randn(shape, generator=g) if len(shape) < 2 else torch.randn(shape, generator=g) * (
             1.0 if name == "embed" else shape[1] ** -0.5)
         out[name] = (t if make is None else make(name, t)).to(torch.bfloat16)
     os.makedirs(path, exist_ok=True)

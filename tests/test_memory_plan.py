@@ -84,8 +84,8 @@ def test_plan_counts_the_recurrent_state_of_hybrid_models():
     from b200serve.models.config import preset
     from b200serve.runtime import memory_plan as MP
     dense, hyb = preset("dense-27b"), preset("hybrid-27b")
-    per_slot = MP.gdn_state_bytes_per_slot(hyb)
-    assert MP.gdn_state_bytes_per_slot(dense) == 0
+    per_slot = MP.state_bytes_per_slot(hyb)
+    assert MP.state_bytes_per_slot(dense) == 0
     assert per_slot == 2 * 48 * (48 * 128 * 128 * 4 + (2 * 16 * 128 + 48 * 128) * 3 * 4)
     # only the 16 attention layers hold KV pages
     assert MP.kv_bytes_per_page(hyb, "bf16") * 4 == MP.kv_bytes_per_page(dense, "bf16")

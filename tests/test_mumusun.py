@@ -204,7 +204,8 @@ class Attn:
     """One mixer with random weights, a scattered page table, and ``n`` positions of two requests in its cache."""
 
     def __init__(self, shape, window, n, dtype, seed=0):
-        from b200serve.models.latent import LatentGeometry, assemble, tensor_shapes
+        from b200serve.models.latent import LatentGeometry
+        from b200serve.models.listed import assemble, tensor_shapes
         from b200serve.models.oracle import rope_tables
         g = gen(seed)
         self.a = a = mixer_of(shape, window)
@@ -214,7 +215,7 @@ class Attn:
         raw = {k: (1 + 0.3 * torch.randn(s, generator=g) if len(s) == 1 else torch.randn(s, generator=g) * s[1] ** -0.5).bfloat16()
                for k, s in tensor_shapes(self.cfg).items()}
         self.raw = {k: v.double() for k, v in raw.items()}
-        self.w = assemble(self.cfg, lambda k: raw[k], DEV, dtype).layers[0].latent
+        self.w = assemble(self.cfg, lambda k: raw[k], DEV, dtype).layers[0].mixer
         self.dtype, self.n = dtype, n
         blocks = (n + 15) // 16
         perm = torch.randperm(2 * blocks, generator=g) + 1
@@ -609,8 +610,8 @@ def test_saved_pages_and_prefix_store(model):
 
 def test_weights_in_both_element_types_run_what_they_say(model):
     e32, e16 = model.engine("float32"), model.engine("bfloat16")
-    assert e32.kv_dtype == "f32" and all(t.dtype == torch.float32 for t in e32.kv.latent)
-    assert e16.kv_dtype == "bf16" and all(t.dtype == torch.bfloat16 for t in e16.kv.latent)
+    assert e32.kv_dtype == "f32" and all(t.dtype == torch.float32 for t in e32.kv.pages.values())
+    assert e16.kv_dtype == "bf16" and all(t.dtype == torch.bfloat16 for t in e16.kv.pages.values())
 
 
 def test_served_over_http(model):

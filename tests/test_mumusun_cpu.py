@@ -66,7 +66,7 @@ def test_loaded_weights_compute_the_layer(snapshot):
     hp[:, : cfg.hidden] = h
     pos = torch.arange(n)
     for i, (spec, lw, js) in enumerate(zip(cfg.layer_specs, w.layers, cfg.to_listed_config()["layers"])):
-        a, g, m = spec.mixer, LatentGeometry.of(spec.mixer), lw.latent
+        a, g, m = spec.mixer, LatentGeometry.of(spec.mixer), lw.mixer
         d = hp @ m.down.double().T
         assert torch.all(d[:, a.q_rank: g.qp] == 0) and torch.all(d[:, g.qp + a.kv_rank: g.qp + g.kvp] == 0)
         cq = torch.zeros(n, g.qp, dtype=torch.float64)
@@ -137,14 +137,16 @@ def test_segment_keys_cover_what_rows_see():
 def test_batch_tables_number_single_rows_first():
     from b200serve.runtime.batch import BatchRunner
     b = BatchRunner.__new__(BatchRunner)
-    b.forms = [(64, 256)]
-    host, spans, keys = b._tables([(1, 9, [5]), (3, 0, [7, 8])], [(0, 100, list(range(40)))], np.asarray([2, 42]))
+    form = ("keys", 64, 256)
+    b.forms = [form]
+    host, spans, tables = b._tables([(1, 9, [5]), (3, 0, [7, 8])], [(0, 100, list(range(40)))], np.asarray([2, 42]))
     cut = lambda s: host[s[0]: s[0] + s[1]].tolist()     # noqa: E731
     assert cut(spans["req"])[:4] == [1, 3, 3, 0] and cut(spans["pos"])[:4] == [9, 0, 1, 100]
     assert cut(spans["token"])[:4] == [5, 7, 8, 0] and cut(spans["want"]) == [2, 42]
-    n, kr, kp, nt, tiles = keys[(64, 256)]
-    assert n == 40 + 63 and cut(kp)[0] == 37 and nt == 1 and cut(tiles) == [0, 40, 63, 0]
-    assert all(s[0] % 4 == 0 for s in (*spans.values(), kr, kp, tiles))
+    used = []
+    t = tables[form](lambda span: used.append(span) or cut(span))
+    assert t.n_keys == 40 + 63 and t.kpos[0] == 37 and t.n_tiles == 1 and t.tiles == [0, 40, 63, 0]
+    assert all(s[0] % 4 == 0 for s in (*spans.values(), *used))
 
 
 def test_planner_counts_pages_and_refuses():
@@ -167,7 +169,7 @@ def test_planner_counts_pages_and_refuses():
 
 
 def test_step_scratch_stays_within_the_planner_figure():
-    from b200serve.models.latent import ListedScratch
+    from b200serve.models.listed import ListedScratch
     sc = ListedScratch("cpu", torch.float32, fixed=8)
     a = sc.get("x", 3, 16)
     assert a.shape == (3, 16) and sc.get("x", 8, 16).data_ptr() == a.data_ptr()
