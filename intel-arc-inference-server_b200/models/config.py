@@ -576,17 +576,15 @@ def napadra_mini() -> ModelConfig:
         StreamBlock(3, 0.8))
 
 
-def napadra_4b() -> ModelConfig:
+def napadra_7b() -> ModelConfig:
     """A Napadra of real layer sizes: width 4096, 32 layers in groups of two mLSTM layers (8 heads of 256 x 512) and two
-    attention layers (32 / 8 heads of 128, chunks of 8192, the second on the first one's keys), 11008 wide feed-forwards on
-    the attention layers, four streams."""
-    specs = []
+    attention layers (32 / 8 heads of 128, chunks of 8192, the second on the first one's keys), 11008 wide feed-forwards, four
+    streams."""
+    ffn, specs = DenseFfn(11008, 7.0, 1.702, 1.0), []
     for i in range(0, 32, 4):
         att = GroupedAttention(32, 8, 128, 128, 128 ** -0.5, 8192, 8.0, True)
-        specs += [LayerSpec(MatrixLstm(8, 256, 512, 15.0), None)] * 2
-        specs += [LayerSpec(att, DenseFfn(11008, 7.0, 1.702, 1.0)),
-                  LayerSpec(replace(att, kv_from=i + 2), DenseFfn(11008, 7.0, 1.702, 1.0))]
-    return listed_config("napadra-4b", "Napadra", specs, 4096, 64000, 1e-5, StreamBlock(4, 0.5))
+        specs += [LayerSpec(MatrixLstm(8, 256, 512, 15.0), ffn)] * 2 + [LayerSpec(att, ffn), LayerSpec(replace(att, kv_from=i + 2), ffn)]
+    return listed_config("napadra-7b", "Napadra", specs, 4096, 64000, 1e-5, StreamBlock(4, 0.5))
 
 
 def dflash_drafter(target: ModelConfig) -> ModelConfig:
@@ -598,7 +596,7 @@ def dflash_drafter(target: ModelConfig) -> ModelConfig:
 
 PRESETS = {
     "tiny-dense": tiny_dense, "tiny-moe": tiny_moe, "small-dense": small_dense, "small-windowed": small_windowed, "small-hybrid": small_hybrid, "small-moe": small_moe, "dense-27b": dense_27b, "hybrid-27b": hybrid_27b, "moe-35b-a3b": moe_35b_a3b,
-    "mumusun-mini": mumusun_mini, "mumusun-16b": mumusun_16b, "napadra-mini": napadra_mini, "napadra-4b": napadra_4b,
+    "mumusun-mini": mumusun_mini, "mumusun-16b": mumusun_16b, "napadra-mini": napadra_mini, "napadra-7b": napadra_7b,
 }
 
 

@@ -39,8 +39,8 @@ class MlstmGeometry:
 
     @property
     def state_elems(self) -> int:
-        """Per value block of 64: S [dk][64], n [dk], the running maximum and padding."""
-        return self.heads * (self.dv // 64) * (self.dk * 65 + 4)
+        """Per value block of 32: S [dk][32], n [dk], the running maximum and padding."""
+        return self.heads * (self.dv // 32) * (self.dk * 33 + 4)
 
 
 def shapes(cfg: ModelConfig, p: str, a: MatrixLstm) -> dict:

@@ -1,5 +1,5 @@
 // Matrix-memory recurrence with exponential gates (mLSTM): per head a state S [dk][dv], a normaliser n [dk] and a running
-// maximum m, all fp32, one block per (slot, head, 64 value dims).
+// maximum m, all fp32, one block per (slot, head, 32 value dims); every block has its own copy of n and m.
 //
 //   m' = max(f + m, i);  S' = e^(f + m - m') S + e^(i - m') k v^T;  n' likewise with k alone
 //   o  = S'^T q / (max(|n' . q|, e^(-m')) + 1e-6)          q scaled by dim^-1/2
@@ -9,7 +9,7 @@
 //   mlstm_step_kernel   rows in order, one token at a time: a cluster of dv / 64 CTAs per (sequence, head) folds the
 //                       projection's slices, updates the state and writes the gated output; either element type
 //   mlstm_gates_kernel  prompt segments: gates of all rows, and the running maximum at every chunk of 64 rows
-//   mlstm_scan_kernel   prompt segments: a CTA walks the chunks of one (segment, head, 64 value dims) on the tensor cores
+//   mlstm_scan_kernel   prompt segments: a CTA walks the chunks of one (segment, head, 32 value dims) on the tensor cores
 //   mlstm_out_kernel    prompt segments: head norm and output gate
 //
 // Chunk form.  With F_t the sum of f over the chunk's rows up to t, a_s = i_s - F_s and M_t = max(m0, max_{s <= t} a_s):
@@ -38,7 +38,8 @@ __device__ __forceinline__ float log_forget_gate(float z, float cap) {
   const float x = cap * tanhf(z / cap);
   return fminf(x, 0.f) - log1pf(expf(-fabsf(x)));
 }
-__host__ __device__ constexpr int state_block(int dk) { return dk * 65 + 4; }     // S [dk][64], n [dk], m
+constexpr int VB = 32;                                                                // value dims of a state block
+__host__ __device__ constexpr int state_block(int dk) { return dk * (VB + 1) + 4; }   // S [dk][32], n [dk], m, padding
 
 // ------------------------------------------------------------------ one token at a time
 struct StepParams {
@@ -48,7 +49,7 @@ struct StepParams {
   const float* gate_bias; // [2 H]
   float cap, q_scale, eps;
   const float* norm;      // [H dv], padding 0
-  float* state;           // [slots][H][dv / 64][state_block]
+  float* state;           // [slots][H][dv / 32][state_block]
   void* out;              // [M][H dv]
 };
 
@@ -64,19 +65,21 @@ __global__ void __launch_bounds__(256) mlstm_step_kernel(const StepParams p) {
   pdl_wait();
   const int slot = p.req[row0];
   if (row0 > 0 && p.req[row0 - 1] == slot) return;        // the whole cluster leaves: another CTA walks this sequence
-  float* st = p.state + (((size_t)slot * p.H + h) * nvb + vb) * state_block(dk);
+  constexpr int SB = state_block(dk);
+  float* blk = p.state + (((size_t)slot * p.H + h) * nvb + vb) * 2 * SB;      // two blocks per CTA
+  float* st = blk + (c >> 5) * SB + (c & 31);
   float4 S[NS];
   float n[NN], m = 0.f;
   const bool fresh = p.pos[row0] == 0;
 #pragma unroll
   for (int i = 0; i < NS; ++i)
-    S[i] = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : __ldcg(reinterpret_cast<const float4*>(st + (16 * i + grp) * 64 + c));
+    S[i] = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : __ldcg(reinterpret_cast<const float4*>(st + (16 * i + grp) * VB));
 #pragma unroll
   for (int i = 0; i < NN; ++i) {
     const int d = tid + 256 * i;
-    n[i] = fresh || d >= dk ? 0.f : __ldcg(st + dk * 64 + d);
+    n[i] = fresh || d >= dk ? 0.f : __ldcg(blk + dk * VB + d);
   }
-  if (!fresh) m = __ldcg(st + dk * 65);
+  if (!fresh) m = __ldcg(blk + SB - 4);
   const int Hk = p.H * dk, Hv = p.H * p.dv;
   cg::cluster_group cl = cg::this_cluster();
   for (int row = row0; row < p.M && p.req[row] == slot; ++row) {
@@ -163,11 +166,11 @@ __global__ void __launch_bounds__(256) mlstm_step_kernel(const StepParams p) {
     }
   }
 #pragma unroll
-  for (int i = 0; i < NS; ++i) *reinterpret_cast<float4*>(st + (16 * i + grp) * 64 + c) = S[i];
+  for (int i = 0; i < NS; ++i) *reinterpret_cast<float4*>(st + (16 * i + grp) * VB) = S[i];
 #pragma unroll
   for (int i = 0; i < NN; ++i)
-    if (tid + 256 * i < dk) st[dk * 64 + tid + 256 * i] = n[i];
-  if (tid == 0) st[dk * 65] = m;
+    if (tid + 256 * i < dk) blk[dk * VB + tid + 256 * i] = blk[SB + dk * VB + tid + 256 * i] = n[i];
+  if (tid < 2) blk[tid * SB + SB - 4] = m;
 }
 
 // ------------------------------------------------------------------ prompt segments
@@ -236,7 +239,7 @@ __global__ void __launch_bounds__(256) mlstm_gates_kernel(const GatesParams p) {
   }
   __syncthreads();
   if (threadIdx.x == 0) {
-    float m = p.pos[row0] == 0 ? 0.f : p.state[((size_t)slot * p.H + h) * p.nvb * state_block(p.dk) + p.dk * 65];
+    float m = p.pos[row0] == 0 ? 0.f : p.state[((size_t)slot * p.H + h) * p.nvb * state_block(p.dk) + state_block(p.dk) - 4];
     for (int c = 0; c < nch; ++c) {
       const float next = sm[2 * c] + fmaxf(m, sm[2 * c + 1]);
       sm[2 * c] = m;
@@ -281,34 +284,44 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
 // byte offset of a 16-byte piece (8 bf16) of a row of 128 bytes, 128-byte swizzle
 __device__ __forceinline__ uint32_t piece(int row, int pc) { return (uint32_t)(row * 128 + ((pc ^ (row & 7)) << 4)); }
 
+constexpr int kScanWork = 256, kScanThreads = kScanWork + 32;     // eight working warps and one that fetches
+
 template <int KB>
 struct Scan {
   static constexpr int BLK = CH * 128;                       // 64 rows x 64 dims
   static constexpr int OFF_K = KB * BLK, OFF_V = 2 * KB * BLK, OFF_G = OFF_V + BLK;
   static constexpr int STAGE = OFF_G + kGateBlock * 4;
-  static constexpr int OFF_PH = 2 * STAGE, OFF_PL = OFF_PH + BLK, OFF_NT = OFF_PL + BLK;
-  static constexpr int OFF_F = OFF_NT + KB * 1024;           // n [dk], inter [64], inv [64], b [64]
-  static constexpr int OFF_BAR = OFF_F + (KB * 64 + 3 * CH) * 4;
-  static constexpr int SMEM = OFF_BAR + 16 + 1024;
+  static constexpr int NST = KB <= 2 ? 3 : 2;                // chunks in flight
+  static constexpr int OFF_P = NST * STAGE;                  // P as two limbs, of two chunks
+  static constexpr int OFF_NT = OFF_P + 4 * BLK;             // n's limbs, of two chunks
+  static constexpr int OFF_X = OFF_NT + 2 * KB * 1024;       // partial read-outs [8 warps][4 row groups][2][32 lanes][4]
+  static constexpr int OFF_F = OFF_X + 8 * 4 * 1024;         // row sums of P [2 chunks][2][64], n . q [2][64], b [2 chunks][64]
+  static constexpr int OFF_BAR = OFF_F + 8 * CH * 4;
+  static constexpr int SMEM = OFF_BAR + 32 + 1024;
+  static_assert(SMEM <= 227 * 1024, "shared memory of one CTA");
 };
 
-// Four warps; a warp owns 16 value columns of the state, S^T [16][dk] in MMA accumulators for the whole walk.  Products
-// are written with the value dimension as M, so accumulators become A operands in registers.  n rides through the products
-// with the queries as two more key rows (its bf16 limbs).  Two chunks in flight.
+// Eight warps.  The state is S^T [32 value columns][dk] in MMA accumulators for the whole walk: warp = (tile of 16 value
+// columns, quarter of the key dims).  Products are written with the value dimension as M, so accumulators become A operands
+// in registers; the quarters' read-outs meet in shared memory, each warp finishing 16 of the chunk's 64 rows.  For the
+// products with the keys a warp owns 16 rows and every second group of 16 keys up to them; n . q are products with two more
+// key rows, n's bf16 limbs.  Between two barriers the warps read out and update the state for one chunk and make the next
+// chunk's P, which does not depend on the state.  A ninth warp fetches.
 template <int KB>
-__global__ void __launch_bounds__(128, 1) mlstm_scan_kernel(const __grid_constant__ ScanParams p) {
+__global__ void __launch_bounds__(kScanThreads) mlstm_scan_kernel(const __grid_constant__ ScanParams p) {
   using L = Scan<KB>;
-  constexpr int dk = KB * 64;
+  constexpr int dk = KB * 64, RG = KB == 1 ? 8 : KB == 2 ? 4 : 2;      // RG: lanes that share two dims of n
   extern __shared__ uint8_t smem_raw[];
   uint8_t* sp = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const uint32_t base = smem_u32(sp), bar0 = base + L::OFF_BAR;
-  float* s_n = reinterpret_cast<float*>(sp + L::OFF_F);
-  float *s_inter = s_n + dk, *s_inv = s_inter + CH, *s_b = s_inv + CH;
+  float* s_sum = reinterpret_cast<float*>(sp + L::OFF_F);
+  float *s_nq = s_sum + 4 * CH, *s_b = s_nq + 2 * CH;
   const int vb = blockIdx.x, nvb = gridDim.x, h = blockIdx.y, *seg = p.segs + blockIdx.z * kSegWords;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  const int vt = warp & 1, dq = warp >> 1;              // state: value tile, quarter of the key dims
+  const int rt = warp >> 1, ke = warp & 1;              // scores: row tile, parity of the key groups
   if (tid == 0) {
-    mbar_init(bar0, 1);
-    mbar_init(bar0 + 8, 1);
+    for (int i = 0; i < L::NST; ++i) mbar_init(bar0 + 8 * i, 1);
     mbar_fence_init();
     prefetch_tmap(&p.map);
   }
@@ -319,214 +332,330 @@ __global__ void __launch_bounds__(128, 1) mlstm_scan_kernel(const __grid_constan
   float* st_g = p.state + (((size_t)slot * p.H + h) * nvb + vb) * state_block(dk);
   const bool fresh = p.pos[row0] == 0;
   __syncthreads();
-  auto fetch = [&](int c) {
-    const uint32_t dst = base + (c & 1) * L::STAGE, bar = bar0 + 8 * (c & 1);
-    const int y = row0 + c * CH;
-    mbar_expect_tx(bar, L::STAGE);
+  auto stage = [](int c) { return c % L::NST; };
+  auto arrived = [&](int c) { return mbar_wait(bar0 + 8 * stage(c), (c / L::NST) & 1, ERR_GDN_WAIT); };
+  bool ok = true;
+  if (warp == 8) {
+    auto fetch = [&](int c) {
+      const uint32_t dst = base + stage(c) * L::STAGE, bar = bar0 + 8 * stage(c);
+      const int y = row0 + c * CH;
+      mbar_expect_tx(bar, L::STAGE);
 #pragma unroll
-    for (int b = 0; b < KB; ++b) {
-      tma_load_2d(dst + b * L::BLK, &p.map, h * dk + b * 64, y, bar);
-      tma_load_2d(dst + L::OFF_K + b * L::BLK, &p.map, (p.H + h) * dk + b * 64, y, bar);
+      for (int b = 0; b < KB; ++b) {
+        tma_load_2d(dst + b * L::BLK, &p.map, h * dk + b * 64, y, bar);
+        tma_load_2d(dst + L::OFF_K + b * L::BLK, &p.map, (p.H + h) * dk + b * 64, y, bar);
+      }
+      tma_load_2d(dst + L::OFF_V, &p.map, 2 * p.H * dk + h * p.dv + (vb >> 1) * 64, y, bar);
+      bulk_g2s(dst + L::OFF_G, gates + (size_t)c * kGateBlock, kGateBlock * 4, bar);
+    };
+    int issued = min(L::NST, nch);
+    if (lane == 0)
+      for (int c = 0; c < issued; ++c) fetch(c);
+    __syncthreads();
+    for (int c = 0; c < nch; ++c) {
+      if (!__syncthreads_and(1)) {      // a copy gave up: wait (bounded) for those in flight
+        if (lane == 0)
+          for (int i = c; i < issued; ++i) arrived(i);
+        break;
+      }
+      __syncthreads();                  // chunk c's stage is free
+      if (c + L::NST < nch) {
+        if (lane == 0) fetch(c + L::NST);
+        issued = c + L::NST + 1;
+      }
     }
-    tma_load_2d(dst + L::OFF_V, &p.map, 2 * p.H * dk + h * p.dv + vb * 64, y, bar);
-    bulk_g2s(dst + L::OFF_G, gates + (size_t)c * kGateBlock, kGateBlock * 4, bar);
-  };
-  if (tid == 0)
-    for (int c = 0; c < min(2, nch); ++c) fetch(c);
-  // S^T: st[j] covers key dims 8 j ..; [0], [1]: value column 16 warp + g, dims 8 j + 2 t, + 1; [2], [3]: column + 8
-  float st[KB * 8][4];
-  const int vc = 16 * warp + g;
+    return;
+  }
+  // st[j] covers key dims dq dk / 4 + 8 j ..; [0], [1]: value column vc, dims 2 t, + 1 of them; [2], [3]: column vc + 8
+  float st[KB * 2][4];
+  const int vc = 16 * vt + g, d0 = dq * (KB * 16);
 #pragma unroll
-  for (int j = 0; j < KB * 8; ++j)
+  for (int j = 0; j < KB * 2; ++j)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) st[j][e] = fresh ? 0.f : st_g[(8 * j + 2 * t + (e & 1)) * 64 + vc + 8 * (e >> 1)];
-  auto put_n = [&](int d, float v) {       // n as fp32 and as its two limbs' rows
-    s_n[d] = v;
-    const __nv_bfloat16 hi = __float2bfloat16(v), lo = __float2bfloat16(v - __bfloat162float(hi));
-    uint8_t* tile = sp + L::OFF_NT + (d >> 6) * 1024;
-    *reinterpret_cast<__nv_bfloat16*>(tile + piece(0, (d & 63) >> 3) + (d & 7) * 2) = hi;
-    *reinterpret_cast<__nv_bfloat16*>(tile + piece(1, (d & 63) >> 3) + (d & 7) * 2) = lo;
+    for (int e = 0; e < 4; ++e) st[j][e] = fresh ? 0.f : st_g[(d0 + 8 * j + 2 * t + (e & 1)) * VB + vc + 8 * (e >> 1)];
+  // n: RG lanes share dims nd, nd + 1 (all hold them, each sums over its own rows)
+  const int nd = (warp * (32 / RG) + lane / RG) * 2, nr = lane % RG;
+  float n0 = 0.f, n1 = 0.f;
+  if (!fresh && nd < dk) {
+    n0 = st_g[dk * VB + nd];
+    n1 = st_g[dk * VB + nd + 1];
+  }
+  auto put_n = [&](int buf) {              // the limbs' rows
+    if (nd < dk && nr == 0) {
+      uint8_t* tile = sp + L::OFF_NT + buf * KB * 1024 + (nd >> 6) * 1024 + (nd & 7) * 2;
+      uint32_t hi, lo;
+      split2(n0, n1, hi, lo);
+      *reinterpret_cast<uint32_t*>(tile + piece(0, (nd & 63) >> 3)) = hi;
+      *reinterpret_cast<uint32_t*>(tile + piece(1, (nd & 63) >> 3)) = lo;
+    }
   };
-  for (int i = tid; i < KB * 256; i += 128) reinterpret_cast<uint32_t*>(sp + L::OFF_NT)[i] = 0u;
+  for (int i = tid; i < 2 * KB * 256; i += kScanWork) reinterpret_cast<uint32_t*>(sp + L::OFF_NT)[i] = 0u;
   __syncthreads();
-  for (int d = tid; d < dk; d += 128) put_n(d, fresh ? 0.f : st_g[dk * 64 + d]);
-  const uint32_t ph = base + L::OFF_PH, pl = base + L::OFF_PL, nt = base + L::OFF_NT;
+  put_n(0);
+  float4* xch = reinterpret_cast<float4*>(sp + L::OFF_X) + lane;          // [warp][row group][2][32]
   // ldmatrix lanes: A rows (row lane & 15, piece half lane >> 4); B rows of two n-tiles (row .., piece half (lane >> 3) & 1)
   const int ar = lane & 15, ah = lane >> 4, br = (lane & 7) + ((lane >> 4) << 3), bh = (lane >> 3) & 1;
-  float m_last = 0.f;
-  bool ok = true;
-  for (int c = 0; c < nch; ++c) {
-    const uint32_t sb = base + (c & 1) * L::STAGE, ks = sb + L::OFF_K, vs = sb + L::OFF_V;
-    const float* gt = reinterpret_cast<const float*>(sp + (c & 1) * L::STAGE + L::OFF_G);
-    ok = mbar_wait(bar0 + 8 * (c & 1), (c >> 1) & 1, ERR_GDN_WAIT);
-    if (!__syncthreads_and(ok)) {
-      // a copy gave up: wait (bounded) for the other stage's, which may still be in flight, and leave the state alone
-      if (tid == 0 && c + 1 < nch) mbar_wait(bar0 + 8 * ((c + 1) & 1), ((c + 1) >> 1) & 1, ERR_GDN_WAIT);
-      ok = false;
-      break;
-    }
-    const float m0 = gt[3 * CH], M_end = gt[CH + CH - 1], keep = __expf(m0 - M_end);
-    m_last = gt[2 * CH + CH - 1];
-    if (tid < CH) s_b[tid] = __expf(gt[tid] - M_end);
-    // ---- P of this warp's 16 rows: products with the keys of rows up to them, and with n
-    {
-      float x[8][4], xn[4] = {0.f, 0.f, 0.f, 0.f};
+
+  // P of chunk c: 16 rows with this warp's key groups 2 u + ke up to them, and the rows' weights in the state after it
+  auto scores = [&](int c) {
+    const uint32_t sb = base + stage(c) * L::STAGE, ks = sb + L::OFF_K;
+    const float* gt = reinterpret_cast<const float*>(sp + stage(c) * L::STAGE + L::OFF_G);
+    const uint32_t ph = base + L::OFF_P + (c & 1) * 2 * L::BLK, pl = ph + L::BLK;
+    if (tid < CH) s_b[(c & 1) * CH + tid] = __expf(gt[tid] - gt[2 * CH - 1]);
+    float sum[2] = {0.f, 0.f};
+    const int tr[2] = {16 * rt + g, 16 * rt + g + 8};
+    if (ke <= rt) {
+      float x[4][4];
 #pragma unroll
-      for (int j = 0; j < 8; ++j) x[j][0] = x[j][1] = x[j][2] = x[j][3] = 0.f;
+      for (int j = 0; j < 4; ++j) x[j][0] = x[j][1] = x[j][2] = x[j][3] = 0.f;
 #pragma unroll
       for (int kk = 0; kk < KB * 4; kk += 2) {
-        uint32_t a[2][4], bn[4];
+        uint32_t a[2][4];
         const uint32_t blk = (kk >> 2) * L::BLK;
 #pragma unroll
-        for (int u = 0; u < 2; ++u) ldsm_x4(sb + blk + piece(16 * warp + ar, 2 * ((kk + u) & 3) + ah), a[u]);
-        ldsm_x4(nt + (kk >> 2) * 1024 + piece(lane & 7, 2 * (kk & 3) + (lane >> 3)), bn);
-        mma_bf16_16816(xn, a[0][0], a[0][1], a[0][2], a[0][3], bn[0], bn[1]);
-        mma_bf16_16816(xn, a[1][0], a[1][1], a[1][2], a[1][3], bn[2], bn[3]);
+        for (int u = 0; u < 2; ++u) ldsm_x4(sb + blk + piece(16 * rt + ar, 2 * ((kk + u) & 3) + ah), a[u]);
 #pragma unroll
-        for (int jp = 0; jp < 4; ++jp)
-          if (jp <= warp) {
+        for (int u = 0; u < 2; ++u)
+          if (2 * u + ke <= rt) {
+            uint32_t b[2][4];
 #pragma unroll
-            for (int u = 0; u < 2; ++u) {
-              uint32_t b[4];
-              ldsm_x4(ks + blk + piece(16 * jp + br, 2 * ((kk + u) & 3) + bh), b);
-              mma_bf16_16816(x[2 * jp], a[u][0], a[u][1], a[u][2], a[u][3], b[0], b[1]);
-              mma_bf16_16816(x[2 * jp + 1], a[u][0], a[u][1], a[u][2], a[u][3], b[2], b[3]);
+            for (int w = 0; w < 2; ++w) ldsm_x4(ks + blk + piece(16 * (2 * u + ke) + br, 2 * ((kk + w) & 3) + bh), b[w]);
+#pragma unroll
+            for (int w = 0; w < 2; ++w) {
+              mma_bf16_16816(x[2 * u], a[w][0], a[w][1], a[w][2], a[w][3], b[w][0], b[w][1]);
+              mma_bf16_16816(x[2 * u + 1], a[w][0], a[w][1], a[w][2], a[w][3], b[w][2], b[w][3]);
             }
           }
       }
-      float sum[2] = {0.f, 0.f};
-      const int tr[2] = {16 * warp + g, 16 * warp + g + 8};
       const float Mt[2] = {gt[CH + tr[0]], gt[CH + tr[1]]};
+      // all weights before the first store: the stores are barriers for the compiler
 #pragma unroll
-      for (int j = 0; j < 8; ++j)
-        if (j < 2 * warp + 2) {
-          const int s0 = 8 * j + 2 * t;
-          const float a0 = gt[s0], a1 = gt[s0 + 1];
+      for (int u = 0; u < 2; ++u)
+        if (2 * u + ke <= rt)
 #pragma unroll
-          for (int hf = 0; hf < 2; ++hf) {
-            const float p0 = s0 <= tr[hf] ? __expf(a0 - Mt[hf]) * (x[j][2 * hf] * p.q_scale) : 0.f;
-            const float p1 = s0 + 1 <= tr[hf] ? __expf(a1 - Mt[hf]) * (x[j][2 * hf + 1] * p.q_scale) : 0.f;
-            sum[hf] += p0 + p1;
-            uint32_t hi, lo;
-            split2(p0, p1, hi, lo);
-            const uint32_t off = piece(tr[hf], j) + 4 * t;
-            asm volatile("st.shared.u32 [%0], %1;" ::"r"(ph + off), "r"(hi) : "memory");
-            asm volatile("st.shared.u32 [%0], %1;" ::"r"(pl + off), "r"(lo) : "memory");
+          for (int v = 0; v < 2; ++v) {
+            const int s0 = 8 * (2 * (2 * u + ke) + v) + 2 * t;
+            const float2 as = *reinterpret_cast<const float2*>(gt + s0);
+#pragma unroll
+            for (int hf = 0; hf < 2; ++hf) {
+              float* e = x[2 * u + v] + 2 * hf;
+              e[0] = s0 <= tr[hf] ? __expf(as.x - Mt[hf]) * (e[0] * p.q_scale) : 0.f;
+              e[1] = s0 + 1 <= tr[hf] ? __expf(as.y - Mt[hf]) * (e[1] * p.q_scale) : 0.f;
+              sum[hf] += e[0] + e[1];
+            }
           }
-        }
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+        if (2 * u + ke <= rt)
+#pragma unroll
+          for (int v = 0; v < 2; ++v)
+#pragma unroll
+            for (int hf = 0; hf < 2; ++hf) {
+              uint32_t hi, lo;
+              split2(x[2 * u + v][2 * hf], x[2 * u + v][2 * hf + 1], hi, lo);
+              const uint32_t off = piece(tr[hf], 2 * (2 * u + ke) + v) + 4 * t;
+              asm volatile("st.shared.u32 [%0], %1;" ::"r"(ph + off), "r"(hi) : "memory");
+              asm volatile("st.shared.u32 [%0], %1;" ::"r"(pl + off), "r"(lo) : "memory");
+            }
 #pragma unroll
       for (int hf = 0; hf < 2; ++hf) {
         sum[hf] += __shfl_xor_sync(0xffffffffu, sum[hf], 1);
         sum[hf] += __shfl_xor_sync(0xffffffffu, sum[hf], 2);
-        if (t == 0) {
-          const float inter = __expf(m0 - Mt[hf]) * p.q_scale;
-          const float nq = fmaf(inter, xn[2 * hf] + xn[2 * hf + 1], sum[hf]);
-          s_inter[tr[hf]] = inter;
-          s_inv[tr[hf]] = 1.f / (fmaxf(fabsf(nq), expf(-gt[2 * CH + tr[hf]])) + 1e-6f);
-        }
       }
     }
-    __syncthreads();
-    // ---- O^T [16 value columns][64 rows]: the state's part, then this chunk's
-    uint32_t va[4][4];
+    if (t == 0) {
+      s_sum[((c & 1) * 2 + ke) * CH + tr[0]] = sum[0];
+      s_sum[((c & 1) * 2 + ke) * CH + tr[1]] = sum[1];
+    }
+  };
+
+  if (nch > 0) {
+    ok = arrived(0);
+    if (ok) scores(0);
+  }
+  float m_last = 0.f;
+  for (int c = 0; c < nch; ++c) {
+    const uint32_t sb = base + stage(c) * L::STAGE, ks = sb + L::OFF_K, vs = sb + L::OFF_V;
+    const float* gt = reinterpret_cast<const float*>(sp + stage(c) * L::STAGE + L::OFF_G);
+    const float* bw = s_b + (c & 1) * CH;
+    if (!__syncthreads_and(ok)) {      // a copy gave up: leave the state alone
+      ok = false;
+      break;
+    }
+    const float m0 = gt[3 * CH], keep = __expf(m0 - gt[2 * CH - 1]);
+    m_last = gt[3 * CH - 1];
+    // of the rows this warp finishes: the old state's factor, their sum of P and the denominator's floor
+    float2 fac[2], psum[2], flr[2];
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int i = 16 * dq + 8 * u + 2 * t;
+      const float2 M = *reinterpret_cast<const float2*>(gt + CH + i), mr = *reinterpret_cast<const float2*>(gt + 2 * CH + i);
+      const float2 p0 = *reinterpret_cast<const float2*>(s_sum + (c & 1) * 2 * CH + i);
+      const float2 p1 = *reinterpret_cast<const float2*>(s_sum + ((c & 1) * 2 + 1) * CH + i);
+      fac[u] = make_float2(__expf(m0 - M.x) * p.q_scale, __expf(m0 - M.y) * p.q_scale);
+      flr[u] = make_float2(__expf(-mr.x), __expf(-mr.y));
+      psum[u] = make_float2(p0.x + p1.x, p0.y + p1.y);
+    }
+    // ---- n . q of 16 rows, half of the dims per warp
     {
-      float o[8][4];
+      float xn[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-      for (int j = 0; j < 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+      for (int kk = 0; kk < KB * 4; kk += 2)
+        if (((kk >> 1) & 1) == ke) {
+          uint32_t a[2][4], bn[4];
 #pragma unroll
-      for (int kk = 0; kk < KB * 4; ++kk) {
-        uint32_t hi[4], lo[4];
-        split2(st[2 * kk][0], st[2 * kk][1], hi[0], lo[0]);
-        split2(st[2 * kk][2], st[2 * kk][3], hi[1], lo[1]);
-        split2(st[2 * kk + 1][0], st[2 * kk + 1][1], hi[2], lo[2]);
-        split2(st[2 * kk + 1][2], st[2 * kk + 1][3], hi[3], lo[3]);
-#pragma unroll
-        for (int jj = 0; jj < 4; ++jj) {
-          uint32_t b[4];
-          ldsm_x4(sb + (kk >> 2) * L::BLK + piece(16 * jj + br, 2 * (kk & 3) + bh), b);
-#pragma unroll
-          for (int u = 0; u < 2; ++u) {
-            mma_bf16_16816(o[2 * jj + u], hi[0], hi[1], hi[2], hi[3], b[2 * u], b[2 * u + 1]);
-            mma_bf16_16816(o[2 * jj + u], lo[0], lo[1], lo[2], lo[3], b[2 * u], b[2 * u + 1]);
-          }
+          for (int u = 0; u < 2; ++u) ldsm_x4(sb + (kk >> 2) * L::BLK + piece(16 * rt + ar, 2 * ((kk + u) & 3) + ah), a[u]);
+          ldsm_x4(base + L::OFF_NT + (c & 1) * KB * 1024 + (kk >> 2) * 1024 + piece(lane & 7, 2 * (kk & 3) + (lane >> 3)), bn);
+          mma_bf16_16816(xn, a[0][0], a[0][1], a[0][2], a[0][3], bn[0], bn[1]);
+          mma_bf16_16816(xn, a[1][0], a[1][1], a[1][2], a[1][3], bn[2], bn[3]);
         }
+      if (t == 0) {
+        s_nq[ke * CH + 16 * rt + g] = xn[0] + xn[1];
+        s_nq[ke * CH + 16 * rt + g + 8] = xn[2] + xn[3];
       }
+    }
+    // ---- O^T [16 value columns][64 rows] from this quarter of the state; rows of the other quarters' warps are handed over
+    float o[8][4];
 #pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        const float2 f = *reinterpret_cast<const float2*>(s_inter + 8 * j + 2 * t);
-        o[j][0] *= f.x; o[j][1] *= f.y; o[j][2] *= f.x; o[j][3] *= f.y;
-      }
+    for (int j = 0; j < 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
 #pragma unroll
-      for (int kk = 0; kk < 4; ++kk) ldsm_x4_trans(vs + piece(16 * kk + br, 2 * warp + bh), va[kk]);
+    for (int kk = 0; kk < KB; ++kk) {
+      uint32_t hi[4], lo[4];
+      split2(st[2 * kk][0], st[2 * kk][1], hi[0], lo[0]);
+      split2(st[2 * kk][2], st[2 * kk][3], hi[1], lo[1]);
+      split2(st[2 * kk + 1][0], st[2 * kk + 1][1], hi[2], lo[2]);
+      split2(st[2 * kk + 1][2], st[2 * kk + 1][3], hi[3], lo[3]);
+      const int d = d0 + 16 * kk;
+      uint32_t b[4][4];
+#pragma unroll
+      for (int jj = 0; jj < 4; ++jj) ldsm_x4(sb + (d >> 6) * L::BLK + piece(16 * jj + br, ((d & 63) >> 3) + bh), b[jj]);
 #pragma unroll
       for (int jj = 0; jj < 4; ++jj)
 #pragma unroll
-        for (int kk = 0; kk <= jj; ++kk) {
+        for (int u = 0; u < 2; ++u) mma_bf16_16816(o[2 * jj + u], hi[0], hi[1], hi[2], hi[3], b[jj][2 * u], b[jj][2 * u + 1]);
+#pragma unroll
+      for (int jj = 0; jj < 4; ++jj)
+#pragma unroll
+        for (int u = 0; u < 2; ++u) mma_bf16_16816(o[2 * jj + u], lo[0], lo[1], lo[2], lo[3], b[jj][2 * u], b[jj][2 * u + 1]);
+    }
+    float4 own[2];
+#pragma unroll
+    for (int jj = 0; jj < 4; ++jj)
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const float4 v = make_float4(o[2 * jj + u][0], o[2 * jj + u][1], o[2 * jj + u][2], o[2 * jj + u][3]);
+        if (jj != dq) xch[((warp * 4 + jj) * 2 + u) * 32] = v;
+        else own[u] = v;
+      }
+    uint32_t va[4][4];
+#pragma unroll
+    for (int kk = 0; kk < 4; ++kk) ldsm_x4_trans(vs + piece(16 * kk + br, 4 * (vb & 1) + 2 * vt + bh), va[kk]);
+    // ---- the chunk's own values for this warp's 16 rows
+    float r[2][4] = {};
+    {
+      const uint32_t ph = base + L::OFF_P + (c & 1) * 2 * L::BLK, pl = ph + L::BLK;
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk)
+        if (kk <= dq) {
           uint32_t b[4], bl[4];
-          ldsm_x4(ph + piece(16 * jj + br, 2 * kk + bh), b);
-          ldsm_x4(pl + piece(16 * jj + br, 2 * kk + bh), bl);
+          ldsm_x4(ph + piece(16 * dq + br, 2 * kk + bh), b);
+          ldsm_x4(pl + piece(16 * dq + br, 2 * kk + bh), bl);
 #pragma unroll
-          for (int u = 0; u < 2; ++u) {
-            mma_bf16_16816(o[2 * jj + u], va[kk][0], va[kk][1], va[kk][2], va[kk][3], b[2 * u], b[2 * u + 1]);
-            mma_bf16_16816(o[2 * jj + u], va[kk][0], va[kk][1], va[kk][2], va[kk][3], bl[2 * u], bl[2 * u + 1]);
-          }
-        }
-      float* dst = p.o + (size_t)(row0 + c * CH) * (p.H * p.dv) + h * p.dv + vb * 64 + vc;
-      const int valid = rows - c * CH;
+          for (int u = 0; u < 2; ++u) mma_bf16_16816(r[u], va[kk][0], va[kk][1], va[kk][2], va[kk][3], b[2 * u], b[2 * u + 1]);
 #pragma unroll
-      for (int j = 0; j < 8; ++j)
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int r = 8 * j + 2 * t + e;
-          if (r < valid) {
-            const float inv = s_inv[r];
-            dst[(size_t)r * (p.H * p.dv)] = o[j][e] * inv;
-            dst[(size_t)r * (p.H * p.dv) + 8] = o[j][2 + e] * inv;
-          }
+          for (int u = 0; u < 2; ++u) mma_bf16_16816(r[u], va[kk][0], va[kk][1], va[kk][2], va[kk][3], bl[2 * u], bl[2 * u + 1]);
         }
     }
     // ---- state after the chunk
 #pragma unroll
-    for (int j = 0; j < KB * 8; ++j) { st[j][0] *= keep; st[j][1] *= keep; st[j][2] *= keep; st[j][3] *= keep; }
+    for (int j = 0; j < KB * 2; ++j) { st[j][0] *= keep; st[j][1] *= keep; st[j][2] *= keep; st[j][3] *= keep; }
 #pragma unroll
     for (int kk = 0; kk < 4; ++kk) {
       uint32_t hi[4], lo[4];
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const float2 w = *reinterpret_cast<const float2*>(s_b + 16 * kk + 8 * (e >> 1) + 2 * t);
+        const float2 w = *reinterpret_cast<const float2*>(bw + 16 * kk + 8 * (e >> 1) + 2 * t);
         split2(bf16_lo(va[kk][e]) * w.x, bf16_hi(va[kk][e]) * w.y, hi[e], lo[e]);
       }
+      uint32_t b[KB][4];
 #pragma unroll
-      for (int q = 0; q < KB * 4; ++q) {
-        uint32_t b[4];
-        ldsm_x4_trans(ks + (q >> 2) * L::BLK + piece(16 * kk + (lane & 7) + (bh << 3), 2 * (q & 3) + ah), b);
-#pragma unroll
-        for (int u = 0; u < 2; ++u) {
-          mma_bf16_16816(st[2 * q + u], hi[0], hi[1], hi[2], hi[3], b[2 * u], b[2 * u + 1]);
-          mma_bf16_16816(st[2 * q + u], lo[0], lo[1], lo[2], lo[3], b[2 * u], b[2 * u + 1]);
-        }
+      for (int q = 0; q < KB; ++q) {
+        const int d = d0 + 16 * q;
+        ldsm_x4_trans(ks + (d >> 6) * L::BLK + piece(16 * kk + (lane & 7) + (bh << 3), ((d & 63) >> 3) + ah), b[q]);
       }
+#pragma unroll
+      for (int q = 0; q < KB; ++q)
+#pragma unroll
+        for (int u = 0; u < 2; ++u) mma_bf16_16816(st[2 * q + u], hi[0], hi[1], hi[2], hi[3], b[q][2 * u], b[q][2 * u + 1]);
+#pragma unroll
+      for (int q = 0; q < KB; ++q)
+#pragma unroll
+        for (int u = 0; u < 2; ++u) mma_bf16_16816(st[2 * q + u], lo[0], lo[1], lo[2], lo[3], b[q][2 * u], b[q][2 * u + 1]);
     }
-    for (int d = tid; d < dk; d += 128) {
-      const uint8_t* kp = sp + (c & 1) * L::STAGE + L::OFF_K + (d >> 6) * L::BLK + (d & 7) * 2;
+    // ---- n after the chunk
+    {
+      const int ndc = nd < dk ? nd : 0;
+      const uint8_t* kp = sp + stage(c) * L::STAGE + L::OFF_K + (ndc >> 6) * L::BLK + (ndc & 7) * 2;
+      const int pc = (ndc & 63) >> 3;
       float a0 = 0.f, a1 = 0.f;
-#pragma unroll 8
-      for (int s = 0; s < CH; s += 2) {
-        a0 = fmaf(s_b[s], __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(kp + piece(s, (d & 63) >> 3))), a0);
-        a1 = fmaf(s_b[s + 1], __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(kp + piece(s + 1, (d & 63) >> 3))), a1);
+#pragma unroll
+      for (int i = 0; i < CH / RG; ++i) {
+        const int s = i * RG + nr;
+        const uint32_t k2 = *reinterpret_cast<const uint32_t*>(kp + piece(s, pc));
+        const float w = bw[s];
+        a0 = fmaf(w, bf16_lo(k2), a0);
+        a1 = fmaf(w, bf16_hi(k2), a1);
       }
-      put_n(d, fmaf(keep, s_n[d], a0 + a1));
+#pragma unroll
+      for (int o2 = 1; o2 < RG; o2 <<= 1) {
+        a0 += __shfl_xor_sync(0xffffffffu, a0, o2);
+        a1 += __shfl_xor_sync(0xffffffffu, a1, o2);
+      }
+      n0 = fmaf(keep, n0, a0);
+      n1 = fmaf(keep, n1, a1);
+      put_n((c + 1) & 1);
+    }
+    if (c + 1 < nch) {
+      ok = arrived(c + 1);
+      if (ok) scores(c + 1);
     }
     __syncthreads();
-    if (tid == 0 && c + 2 < nch) fetch(c + 2);
+    // ---- this warp's 16 rows: the four quarters of the state's part, the denominators
+    {
+      float* dst = p.o + (size_t)(row0 + c * CH + 16 * dq + 2 * t) * (p.H * p.dv) + h * p.dv + vb * VB + vc;
+      const int valid = rows - c * CH - 16 * dq - 2 * t;
+      float4 part[2][3];
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+#pragma unroll
+        for (int q = 1; q < 4; ++q) part[u][q - 1] = xch[((((dq + q) & 3) * 2 + vt) * 4 + dq) * 64 + u * 32];
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const int i = 16 * dq + 8 * u + 2 * t;
+        const float2 q0 = *reinterpret_cast<const float2*>(s_nq + i), q1 = *reinterpret_cast<const float2*>(s_nq + CH + i);
+        const float i0 = __fdividef(1.f, fmaxf(fabsf(fmaf(fac[u].x, q0.x + q1.x, psum[u].x)), flr[u].x) + 1e-6f);
+        const float i1 = __fdividef(1.f, fmaxf(fabsf(fmaf(fac[u].y, q0.y + q1.y, psum[u].y)), flr[u].y) + 1e-6f);
+        float4 a = own[u];
+#pragma unroll
+        for (int q = 0; q < 3; ++q) { a.x += part[u][q].x; a.y += part[u][q].y; a.z += part[u][q].z; a.w += part[u][q].w; }
+        const float v0 = fmaf(a.x, fac[u].x, r[u][0]) * i0, v1 = fmaf(a.y, fac[u].y, r[u][1]) * i1;
+        const float v2 = fmaf(a.z, fac[u].x, r[u][2]) * i0, v3 = fmaf(a.w, fac[u].y, r[u][3]) * i1;
+        float* row = dst + (size_t)(8 * u) * (p.H * p.dv);
+        if (8 * u < valid) { row[0] = v0; row[8] = v2; }
+        if (8 * u + 1 < valid) { row[p.H * p.dv] = v1; row[p.H * p.dv + 8] = v3; }
+      }
+    }
   }
   if (ok) {
 #pragma unroll
-    for (int j = 0; j < KB * 8; ++j)
+    for (int j = 0; j < KB * 2; ++j)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) st_g[(8 * j + 2 * t + (e & 1)) * 64 + vc + 8 * (e >> 1)] = st[j][e];
-    for (int d = tid; d < dk; d += 128) st_g[dk * 64 + d] = s_n[d];
-    if (tid == 0) st_g[dk * 65] = m_last;
+      for (int e = 0; e < 4; ++e) st_g[(d0 + 8 * j + 2 * t + (e & 1)) * VB + vc + 8 * (e >> 1)] = st[j][e];
+    if (nd < dk && nr == 0) {
+      st_g[dk * VB + nd] = n0;
+      st_g[dk * VB + nd + 1] = n1;
+    }
+    if (tid == 0) st_g[state_block(dk) - 4] = m_last;
   }
 }
 
@@ -615,13 +744,13 @@ int launch_scan(const ScanParams& p, int n_segs, cudaStream_t st) {
     if (e != cudaSuccess) return (int)e;
     configured[dev & 63] = true;
   }
-  return b2_launch(mlstm_scan_kernel<KB>, dim3(p.dv / 64, p.H, n_segs), dim3(128), Scan<KB>::SMEM, st, true, p);
+  return b2_launch(mlstm_scan_kernel<KB>, dim3(p.dv / VB, p.H, n_segs), dim3(kScanThreads), Scan<KB>::SMEM, st, true, p);
 }
 
 }  // namespace
 
 // fp32 elements of one slot's state
-extern "C" int b2_mlstm_state_elems(int H, int dk, int dv) { return H * (dv / 64) * state_block(dk); }
+extern "C" int b2_mlstm_state_elems(int H, int dk, int dv) { return H * (dv / VB) * state_block(dk); }
 
 // rows of a sequence are consecutive; part as in StepParams
 extern "C" int b2_mlstm_step(const float* part, int slices, int M, int N, int H, int dk, int dv, int dim, int vdim, const int* req,
@@ -649,7 +778,7 @@ extern "C" int b2_mlstm_segments(const void* proj, int N, const float* z, int ld
   const size_t gsm = (size_t)most_chunks * 2 * sizeof(float);
   if (gsm > 48 * 1024) return -5;
   cudaStream_t st = (cudaStream_t)stream;
-  GatesParams gp{z, ldz, H, dk, dv / 64, chunks, segs, pos, gate_bias, cap, state, gates};
+  GatesParams gp{z, ldz, H, dk, dv / VB, chunks, segs, pos, gate_bias, cap, state, gates};
   int rc = b2_launch(mlstm_gates_kernel, dim3(H, n_segs), dim3(256), gsm, st, true, gp);
   if (rc) return rc;
   ScanParams p;

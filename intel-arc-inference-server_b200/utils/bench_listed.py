@@ -2,8 +2,7 @@
 
 Decode: captured steps of 1, 8, 16 and 64 requests at one depth (one row each, positions advance on the device).  Prompt:
 whole prompt passes through ``Engine.prefill``.  Both are timed with CUDA events after warm-up; the weights a step reads
-are far more than the L2 holds.  The comparison model has the same width, layers, experts, experts per token, query heads
-and window, grouped-query attention instead of latents, and the framework's W4A16 weights.
+are far more than the L2 holds.  The comparison models have the framework's W4A16 weights.
 """
 from __future__ import annotations
 
@@ -11,14 +10,15 @@ import dataclasses
 
 import torch
 
-from ..models.config import ModelConfig, listed_config, preset
+from ..models.config import DenseFfn, GroupedAttention, LayerSpec, MatrixLstm, ModelConfig, listed_config, preset
 from ..models.weights import random_weights
 from ..ops import lib as K
 from ..runtime.engine import Engine
 
 
-def sizes():
-    """(listed model, closest model) pairs."""
+def mumusun_sizes():
+    """(latent-attention mixture of experts, grouped-query mixture of experts) pairs: the same width, layers, experts, experts
+    per token, query heads and window."""
     out = []
     big = preset("mumusun-16b")
     spec = big.layer_specs[0]
@@ -32,6 +32,31 @@ def sizes():
                                      cfg.vocab, n_experts=f.experts, top_k=f.top, expert_ffn=f.ff, shared_ffn=0,
                                      sliding_window=a.window, architecture="B200MoeForCausalLM")))
     return out
+
+
+def napadra_sizes():
+    """(mLSTM and chunked attention over residual streams, gated delta-net and softmax attention) pairs: the same width,
+    layers, feed-forwards, attention heads, and key and value dimensions of the recurrent layers; every second layer is
+    recurrent.  Contexts stay inside one chunk, so the attention layers of both see every earlier position."""
+    out = []
+    big = preset("napadra-7b")
+
+    def like(name, width, layers, heads, kv, rec, ff, vocab):
+        f, specs = DenseFfn(ff, 7.0, 1.702, 1.0), []
+        att = GroupedAttention(heads, kv, 128, 128, 128 ** -0.5, 8192, 8.0, True)
+        for i in range(0, layers, 4):
+            specs += [LayerSpec(rec, f)] * 2 + [LayerSpec(att, f), LayerSpec(dataclasses.replace(att, kv_from=i + 2), f)]
+        return listed_config(name, "Napadra", specs, width, vocab, 1e-5, big.block)
+    for cfg in (big, like("napadra-1b", 2048, 24, 16, 4, MatrixLstm(16, 128, 128, 15.0), 5632, 64000),
+                like("napadra-wide-8l", 8192, 8, 64, 8, MatrixLstm(16, 256, 512, 15.0), 22016, 64000)):
+        r, a, f = cfg.layer_specs[0].mixer, cfg.layer_specs[2].mixer, cfg.layer_specs[0].ffn
+        out.append((cfg, ModelConfig(f"hybrid-like-{cfg.name}", cfg.n_layers, cfg.hidden, a.heads, a.kv_heads, 128, f.ff, cfg.vocab,
+                                     full_attn_every=2, gdn_k_heads=r.heads * r.dim // 128, gdn_v_heads=r.heads * r.vdim // 128,
+                                     architecture="B200HybridForCausalLM")))
+    return out
+
+
+SIZES = {"mumusun": mumusun_sizes, "napadra": napadra_sizes}
 
 
 def _timed(fn, warm: int, reps: int) -> float:
@@ -61,9 +86,14 @@ def bench_model(cfg: ModelConfig, depth: int = 4096, prompt: int = 4096, rows=(1
         for t in eng.kv.page_tensors().values():
             t.index_copy_(1, dst, t.index_select(1, src))
         eng.seq_len[s] = depth
+    states = eng.kv.save_states(0)
     for m in rows:
         for s in range(m):
-            eng.truncate(s, depth)
+            if eng.kv.states:           # positions after ``depth`` are written again; the state goes back to what it was
+                eng.kv.load_states(s, states)
+                eng.seq_len[s] = depth
+            else:
+                eng.truncate(s, depth)
         # unlike tokens, so that the rows' experts differ
         eng.decode_begin(list(range(m)), [(first + 997 * i) % cfg.vocab for i in range(m)])
         ms = _timed(lambda: eng.decode_step(read=False), warm, steps)
@@ -81,9 +111,9 @@ def bench_model(cfg: ModelConfig, depth: int = 4096, prompt: int = 4096, rows=(1
     return out
 
 
-def run(release=lambda: None, which=None) -> dict:
+def run(release=lambda: None, family: str = "mumusun", which=None) -> dict:
     out = {}
-    for cfg, other in sizes():
+    for cfg, other in SIZES[family]():
         if which and cfg.name != which:
             continue
         for c in (cfg, other):
