@@ -117,7 +117,7 @@ class Engine:
     def truncate(self, slot: int, length: int):
         """Drop everything after ``length`` positions (rejected draft rows)."""
         assert length <= self.seq_len[slot]
-        replay = None
+        replay = rest = None
         if length == 0 < self.seq_len[slot]:
             self.kv.reset_slot(slot)
         elif length < self.seq_len[slot] and self.kv.states:
@@ -132,12 +132,14 @@ class Engine:
             self.kv.load_states(slot, snap[1][slot])
             replay = [r for r in rows if r.pos < length]
             self.seq_len[slot] = rows[0].pos
-            self._snap = None
+            # one rewind per step and slot; the step's other slots can still be rewound
+            rest = ([r for r in snap[0] if r.slot != slot], {s: v for s, v in snap[1].items() if s != slot})
         self.seq_len[slot] = min(self.seq_len[slot], length)
         self.pool.truncate(slot, (length + PAGE - 1) // PAGE)
         if replay:
             self.forward_rows(replay, advance=False, read=False)
-            self._snap = None           # one rewind per step
+        if rest is not None:
+            self._snap = rest
 
     def _ensure_pages(self, slot: int, upto_len: int):
         if upto_len > self.max_len:
@@ -309,7 +311,10 @@ class Engine:
         """Keeps the recurrent state from before a step's rows, so that its last rows can be taken back (``truncate``)."""
         self._snap = None
         if self.kv.states and rows:
-            self._snap = (list(rows), {s: self.kv.save_states(s) for s in sorted({r.slot for r in rows})})
+            slots = {r.slot for r in rows}
+            if sum(i == 0 or r.slot != rows[i - 1].slot for i, r in enumerate(rows)) != len(slots):
+                raise ValueError("a recurrent model's step holds a sequence's rows one after another")
+            self._snap = (list(rows), {s: self.kv.save_states(s) for s in sorted(slots)})
 
     def logits(self, m: int) -> torch.Tensor:
         """fp32 logits of the last step's rows (device tensor view)."""
