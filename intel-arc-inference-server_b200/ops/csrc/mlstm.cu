@@ -176,7 +176,13 @@ __global__ void __launch_bounds__(256) mlstm_step_kernel(const StepParams p) {
 // ------------------------------------------------------------------ prompt segments
 constexpr int CH = 64;               // rows of a chunk
 constexpr int kSegWords = 4;         // first row, rows, slot, first chunk (counted over all segments)
-constexpr int kGateBlock = 4 * CH;   // per (head, chunk): a_s, M_t, m_t of the rows; m0
+constexpr int kGateBlock = 4 * CH;   // per (head, chunk): a_s, M_t (both times log2 e), m_t of the rows; m0 (times log2 e)
+constexpr float kLog2e = 1.4426950408889634f;
+__device__ __forceinline__ float exp2_fast(float x) {      // subnormal results are zero
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 
 struct GatesParams {
   const float* z;         // [rows][ldz]: z_i [H] | z_f [H]
@@ -229,7 +235,7 @@ __global__ void __launch_bounds__(256) mlstm_gates_kernel(const GatesParams p) {
     float before = __shfl_up_sync(0xffffffffu, top, 1);
     if (lane == 0) before = -INFINITY;
     float* g = out + (size_t)c * kGateBlock;
-    *reinterpret_cast<float2*>(g + 2 * lane) = make_float2(a[0], a[1]);
+    *reinterpret_cast<float2*>(g + 2 * lane) = make_float2(a[0] * kLog2e, a[1] * kLog2e);
     *reinterpret_cast<float2*>(g + CH + 2 * lane) = make_float2(fmaxf(before, a[0]), top);     // without m0 yet
     *reinterpret_cast<float2*>(g + 2 * CH + 2 * lane) = make_float2(F0, F1);
     if (lane == 31) {
@@ -253,9 +259,9 @@ __global__ void __launch_bounds__(256) mlstm_gates_kernel(const GatesParams p) {
     float2 M = *reinterpret_cast<float2*>(g + CH + 2 * lane), F = *reinterpret_cast<float2*>(g + 2 * CH + 2 * lane);
     M.x = fmaxf(M.x, m0);
     M.y = fmaxf(M.y, m0);
-    *reinterpret_cast<float2*>(g + CH + 2 * lane) = M;
+    *reinterpret_cast<float2*>(g + CH + 2 * lane) = make_float2(M.x * kLog2e, M.y * kLog2e);
     *reinterpret_cast<float2*>(g + 2 * CH + 2 * lane) = make_float2(F.x + M.x, F.y + M.y);
-    if (lane == 0) g[3 * CH] = m0;
+    if (lane == 0) g[3 * CH] = m0 * kLog2e;
   }
 }
 
@@ -263,7 +269,7 @@ struct ScanParams {
   CUtensorMap map;        // the projection [rows][N]: q | k | v | g; boxes of 64 rows x 64 columns
   const int *segs, *pos;
   int H, dv, chunks;
-  float q_scale;
+  float q_scale_log2;
   const float* gates;
   float* state;
   float* o;               // [rows][H dv], before the head norm
@@ -296,7 +302,8 @@ struct Scan {
   static constexpr int OFF_NT = OFF_P + 4 * BLK;             // n's limbs, of two chunks
   static constexpr int OFF_X = OFF_NT + 2 * KB * 1024;       // partial read-outs [8 warps][4 row groups][2][32 lanes][4]
   static constexpr int OFF_F = OFF_X + 8 * 4 * 1024;         // row sums of P [2 chunks][2][64], n . q [2][64], b [2 chunks][64]
-  static constexpr int OFF_BAR = OFF_F + 8 * CH * 4;
+                                                             // (fp32), b's limbs [2 chunks][2][64] (bf16)
+  static constexpr int OFF_BAR = OFF_F + 10 * CH * 4;
   static constexpr int SMEM = OFF_BAR + 32 + 1024;
   static_assert(SMEM <= 227 * 1024, "shared memory of one CTA");
 };
@@ -310,12 +317,13 @@ struct Scan {
 template <int KB>
 __global__ void __launch_bounds__(kScanThreads) mlstm_scan_kernel(const __grid_constant__ ScanParams p) {
   using L = Scan<KB>;
-  constexpr int dk = KB * 64, RG = KB == 1 ? 8 : KB == 2 ? 4 : 2;      // RG: lanes that share two dims of n
+  constexpr int dk = KB * 64;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* sp = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const uint32_t base = smem_u32(sp), bar0 = base + L::OFF_BAR;
   float* s_sum = reinterpret_cast<float*>(sp + L::OFF_F);
   float *s_nq = s_sum + 4 * CH, *s_b = s_nq + 2 * CH;
+  __nv_bfloat16* s_bl = reinterpret_cast<__nv_bfloat16*>(s_b + 2 * CH);
   const int vb = blockIdx.x, nvb = gridDim.x, h = blockIdx.y, *seg = p.segs + blockIdx.z * kSegWords;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
   const int vt = warp & 1, dq = warp >> 1;              // state: value tile, quarter of the key dims
@@ -373,20 +381,23 @@ __global__ void __launch_bounds__(kScanThreads) mlstm_scan_kernel(const __grid_c
   for (int j = 0; j < KB * 2; ++j)
 #pragma unroll
     for (int e = 0; e < 4; ++e) st[j][e] = fresh ? 0.f : st_g[(d0 + 8 * j + 2 * t + (e & 1)) * VB + vc + 8 * (e >> 1)];
-  // n: RG lanes share dims nd, nd + 1 (all hold them, each sums over its own rows)
-  const int nd = (warp * (32 / RG) + lane / RG) * 2, nr = lane % RG;
-  float n0 = 0.f, n1 = 0.f;
-  if (!fresh && nd < dk) {
-    n0 = st_g[dk * VB + nd];
-    n1 = st_g[dk * VB + nd + 1];
-  }
+  // n: lanes 0 .. 3 hold dims d0 + 16 q + 8 vt + 2 t, + 1
+  float n[KB][2];
+#pragma unroll
+  for (int q = 0; q < KB; ++q)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) n[q][e] = fresh || lane > 3 ? 0.f : st_g[dk * VB + d0 + 16 * q + 8 * vt + 2 * t + e];
   auto put_n = [&](int buf) {              // the limbs' rows
-    if (nd < dk && nr == 0) {
-      uint8_t* tile = sp + L::OFF_NT + buf * KB * 1024 + (nd >> 6) * 1024 + (nd & 7) * 2;
-      uint32_t hi, lo;
-      split2(n0, n1, hi, lo);
-      *reinterpret_cast<uint32_t*>(tile + piece(0, (nd & 63) >> 3)) = hi;
-      *reinterpret_cast<uint32_t*>(tile + piece(1, (nd & 63) >> 3)) = lo;
+    if (lane < 4) {
+#pragma unroll
+      for (int q = 0; q < KB; ++q) {
+        const int d = d0 + 16 * q + 8 * vt;
+        uint8_t* tile = sp + L::OFF_NT + buf * KB * 1024 + (d >> 6) * 1024 + 4 * t;
+        uint32_t hi, lo;
+        split2(n[q][0], n[q][1], hi, lo);
+        *reinterpret_cast<uint32_t*>(tile + piece(0, (d & 63) >> 3)) = hi;
+        *reinterpret_cast<uint32_t*>(tile + piece(1, (d & 63) >> 3)) = lo;
+      }
     }
   };
   for (int i = tid; i < 2 * KB * 256; i += kScanWork) reinterpret_cast<uint32_t*>(sp + L::OFF_NT)[i] = 0u;
@@ -401,7 +412,13 @@ __global__ void __launch_bounds__(kScanThreads) mlstm_scan_kernel(const __grid_c
     const uint32_t sb = base + stage(c) * L::STAGE, ks = sb + L::OFF_K;
     const float* gt = reinterpret_cast<const float*>(sp + stage(c) * L::STAGE + L::OFF_G);
     const uint32_t ph = base + L::OFF_P + (c & 1) * 2 * L::BLK, pl = ph + L::BLK;
-    if (tid < CH) s_b[(c & 1) * CH + tid] = __expf(gt[tid] - gt[2 * CH - 1]);
+    if (tid < CH) {
+      const float b = exp2_fast(gt[tid] - gt[2 * CH - 1]);
+      const __nv_bfloat16 hi = __float2bfloat16(b);
+      s_b[(c & 1) * CH + tid] = b;
+      s_bl[(c & 1) * 2 * CH + tid] = hi;
+      s_bl[((c & 1) * 2 + 1) * CH + tid] = __float2bfloat16(b - __bfloat162float(hi));
+    }
     float sum[2] = {0.f, 0.f};
     const int tr[2] = {16 * rt + g, 16 * rt + g + 8};
     if (ke <= rt) {
@@ -427,7 +444,7 @@ __global__ void __launch_bounds__(kScanThreads) mlstm_scan_kernel(const __grid_c
             }
           }
       }
-      const float Mt[2] = {gt[CH + tr[0]], gt[CH + tr[1]]};
+      const float Mt[2] = {gt[CH + tr[0]] - p.q_scale_log2, gt[CH + tr[1]] - p.q_scale_log2};     // the queries' scale rides along
       // all weights before the first store: the stores are barriers for the compiler
 #pragma unroll
       for (int u = 0; u < 2; ++u)
@@ -439,8 +456,12 @@ __global__ void __launch_bounds__(kScanThreads) mlstm_scan_kernel(const __grid_c
 #pragma unroll
             for (int hf = 0; hf < 2; ++hf) {
               float* e = x[2 * u + v] + 2 * hf;
-              e[0] = s0 <= tr[hf] ? __expf(as.x - Mt[hf]) * (e[0] * p.q_scale) : 0.f;
-              e[1] = s0 + 1 <= tr[hf] ? __expf(as.y - Mt[hf]) * (e[1] * p.q_scale) : 0.f;
+              e[0] *= exp2_fast(as.x - Mt[hf]);
+              e[1] *= exp2_fast(as.y - Mt[hf]);
+              if (2 * u + ke == rt) {       // the diagonal: later keys (whose exponent may be above 0) are not seen
+                e[0] = s0 <= tr[hf] ? e[0] : 0.f;
+                e[1] = s0 + 1 <= tr[hf] ? e[1] : 0.f;
+              }
               sum[hf] += e[0] + e[1];
             }
           }
@@ -482,7 +503,7 @@ __global__ void __launch_bounds__(kScanThreads) mlstm_scan_kernel(const __grid_c
       ok = false;
       break;
     }
-    const float m0 = gt[3 * CH], keep = __expf(m0 - gt[2 * CH - 1]);
+    const float m0 = gt[3 * CH], keep = exp2_fast(m0 - gt[2 * CH - 1]);
     m_last = gt[3 * CH - 1];
     // of the rows this warp finishes: the old state's factor, their sum of P and the denominator's floor
     float2 fac[2], psum[2], flr[2];
@@ -492,8 +513,8 @@ __global__ void __launch_bounds__(kScanThreads) mlstm_scan_kernel(const __grid_c
       const float2 M = *reinterpret_cast<const float2*>(gt + CH + i), mr = *reinterpret_cast<const float2*>(gt + 2 * CH + i);
       const float2 p0 = *reinterpret_cast<const float2*>(s_sum + (c & 1) * 2 * CH + i);
       const float2 p1 = *reinterpret_cast<const float2*>(s_sum + ((c & 1) * 2 + 1) * CH + i);
-      fac[u] = make_float2(__expf(m0 - M.x) * p.q_scale, __expf(m0 - M.y) * p.q_scale);
-      flr[u] = make_float2(__expf(-mr.x), __expf(-mr.y));
+      fac[u] = make_float2(exp2_fast(m0 - M.x + p.q_scale_log2), exp2_fast(m0 - M.y + p.q_scale_log2));
+      flr[u] = make_float2(exp2_fast(-kLog2e * mr.x), exp2_fast(-kLog2e * mr.y));
       psum[u] = make_float2(p0.x + p1.x, p0.y + p1.y);
     }
     // ---- n . q of 16 rows, half of the dims per warp
@@ -569,8 +590,12 @@ __global__ void __launch_bounds__(kScanThreads) mlstm_scan_kernel(const __grid_c
     // ---- state after the chunk
 #pragma unroll
     for (int j = 0; j < KB * 2; ++j) { st[j][0] *= keep; st[j][1] *= keep; st[j][2] *= keep; st[j][3] *= keep; }
+    // n's sums ride along: rows 0 and 1 of one more A tile are the limbs of b
+    float ns[KB][4] = {};
+    const uint32_t* bl = reinterpret_cast<const uint32_t*>(s_bl + ((c & 1) * 2 + (g & 1)) * CH);
 #pragma unroll
     for (int kk = 0; kk < 4; ++kk) {
+      const uint32_t b0 = g < 2 ? bl[8 * kk + t] : 0u, b2 = g < 2 ? bl[8 * kk + 4 + t] : 0u;
       uint32_t hi[4], lo[4];
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
@@ -591,30 +616,15 @@ __global__ void __launch_bounds__(kScanThreads) mlstm_scan_kernel(const __grid_c
       for (int q = 0; q < KB; ++q)
 #pragma unroll
         for (int u = 0; u < 2; ++u) mma_bf16_16816(st[2 * q + u], lo[0], lo[1], lo[2], lo[3], b[q][2 * u], b[q][2 * u + 1]);
-    }
-    // ---- n after the chunk
-    {
-      const int ndc = nd < dk ? nd : 0;
-      const uint8_t* kp = sp + stage(c) * L::STAGE + L::OFF_K + (ndc >> 6) * L::BLK + (ndc & 7) * 2;
-      const int pc = (ndc & 63) >> 3;
-      float a0 = 0.f, a1 = 0.f;
 #pragma unroll
-      for (int i = 0; i < CH / RG; ++i) {
-        const int s = i * RG + nr;
-        const uint32_t k2 = *reinterpret_cast<const uint32_t*>(kp + piece(s, pc));
-        const float w = bw[s];
-        a0 = fmaf(w, bf16_lo(k2), a0);
-        a1 = fmaf(w, bf16_hi(k2), a1);
-      }
-#pragma unroll
-      for (int o2 = 1; o2 < RG; o2 <<= 1) {
-        a0 += __shfl_xor_sync(0xffffffffu, a0, o2);
-        a1 += __shfl_xor_sync(0xffffffffu, a1, o2);
-      }
-      n0 = fmaf(keep, n0, a0);
-      n1 = fmaf(keep, n1, a1);
-      put_n((c + 1) & 1);
+      for (int q = 0; q < KB; ++q) mma_bf16_16816(ns[q], b0, 0u, b2, 0u, vt ? b[q][2] : b[q][0], vt ? b[q][3] : b[q][1]);
     }
+#pragma unroll
+    for (int q = 0; q < KB; ++q) {
+      n[q][0] = fmaf(keep, n[q][0], ns[q][0] + __shfl_down_sync(0xffffffffu, ns[q][0], 4));
+      n[q][1] = fmaf(keep, n[q][1], ns[q][1] + __shfl_down_sync(0xffffffffu, ns[q][1], 4));
+    }
+    put_n((c + 1) & 1);
     if (c + 1 < nch) {
       ok = arrived(c + 1);
       if (ok) scores(c + 1);
@@ -651,9 +661,11 @@ __global__ void __launch_bounds__(kScanThreads) mlstm_scan_kernel(const __grid_c
     for (int j = 0; j < KB * 2; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) st_g[(d0 + 8 * j + 2 * t + (e & 1)) * VB + vc + 8 * (e >> 1)] = st[j][e];
-    if (nd < dk && nr == 0) {
-      st_g[dk * VB + nd] = n0;
-      st_g[dk * VB + nd + 1] = n1;
+    if (lane < 4) {
+#pragma unroll
+      for (int q = 0; q < KB; ++q)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) st_g[dk * VB + d0 + 16 * q + 8 * vt + 2 * t + e] = n[q][e];
     }
     if (tid == 0) st_g[state_block(dk) - 4] = m_last;
   }
@@ -791,7 +803,7 @@ extern "C" int b2_mlstm_segments(const void* proj, int N, const float* z, int ld
                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
   if (r != CUDA_SUCCESS) return -101 - (int)r;
-  p.segs = segs; p.pos = pos; p.H = H; p.dv = dv; p.chunks = chunks; p.q_scale = 1.f / sqrtf((float)dim);
+  p.segs = segs; p.pos = pos; p.H = H; p.dv = dv; p.chunks = chunks; p.q_scale_log2 = -0.5f * log2f((float)dim);
   p.gates = gates; p.state = state; p.o = o;
   switch (dk / 64) {
     case 1: rc = launch_scan<1>(p, n_segs, st); break;
