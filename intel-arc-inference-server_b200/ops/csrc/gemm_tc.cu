@@ -642,7 +642,11 @@ static int gemm_tc_impl(const void* a, const void* b, void* c, int M, int N, int
   p.M = M; p.N = N; p.K = K; p.ldc = ldc; p.C = c; p.resid = (const __nv_bfloat16*)resid;
   p.a_scale = a_scale; p.b_scale = b_scale; p.epi = epi; p.glu = glu;
   p.blk_expert = blk_expert; p.blk_row0 = blk_row0; p.blk_rows = blk_rows; p.n_blk = n_blk; p.max_blk = max_blk;
-  if (bn != 128 && bn != 256) bn = (N >= 256 && (N % 256 == 0 || N > 2048)) ? 256 : 128;
+  if (bn != 128 && bn != 256) {
+    bn = (N >= 256 && (N % 256 == 0 || N > 2048)) ? 256 : 128;
+    // few rows: narrower tiles while they still fit in one wave
+    if (!blk_expert && ((M + BM - 1) / BM) * ((N + 127) / 128) <= sm_count()) bn = 128;
+  }
   CUtensorMap ma, mb;
   int rc = make_map(&ma, a, i8 != 0, (uint64_t)M, (uint64_t)K, 0, BM);
   if (rc) return rc;
