@@ -103,15 +103,15 @@ def _profile(eng, f, first):
     raw = {}
     names = [n for n in dir(K) if callable(getattr(K, n)) and n in (
         "gemv_w4", "resid_norm", "rope_append", "attn_decode", "head_gemv", "argmax_finish")]
-    mods = {n: K for n in names}
+    targets = [(n, K, n) for n in names]        # label, module, function
     if eng.cfg.layer_specs:
         from ..ops import latent as L, moe as M
-        mods.update({n: L for n in ("embed_rows", "gemv_bf16", "prep", "absorb", "rows", "simple", "merge", "sublayer_norm",
-                                    "gemv_bf16_experts", "layer_norm_rows", "linear_f32", "linear_f32_experts")})
-        mods["router_rows"] = M
         from ..ops import mlstm as R, paged as P, streams as S
-        mods.update({"gemv_bf16_glu": L, "embed": S, "boundary": S, "append": P, "step": R})
-        names = list(mods)
+        targets += [(n, L, n) for n in ("embed_rows", "gemv_bf16", "prep", "absorb", "rows", "simple", "merge", "sublayer_norm",
+                                        "gemv_bf16_experts", "layer_norm_rows", "linear_f32", "linear_f32_experts", "gemv_bf16_glu",
+                                        "glu_rows_f32")]
+        targets += [("router_rows", M, "router_rows"), ("streams_embed", S, "embed"), ("streams_boundary", S, "boundary"),
+                    ("kv_append", P, "append"), ("paged_rows", P, "rows"), ("paged_simple", P, "simple"), ("mlstm_step", R, "step")]
     pending = []
 
     def wrap(name, fn):
@@ -123,9 +123,9 @@ def _profile(eng, f, first):
             pending.append((name, e0, e1))
             return r
         return inner
-    for n in names:
-        raw[n] = getattr(mods[n], n)
-        setattr(mods[n], n, wrap(n, raw[n]))
+    for label, mod, n in targets:
+        raw[label] = getattr(mod, n)
+        setattr(mod, n, wrap(label, raw[label]))
     try:
         eng.use_graphs = False
         pos, tok = eng.seq_len[0], first
@@ -139,8 +139,8 @@ def _profile(eng, f, first):
             for name, e0, e1 in pending:
                 times.setdefault(name, []).append(e0.elapsed_time(e1) * 1e3)
     finally:
-        for n in names:
-            setattr(mods[n], n, raw[n])
+        for label, mod, n in targets:
+            setattr(mod, n, raw[label])
     print("| kernel family | launches/step | us/step (mean) | share |")
     print("|---|---|---|---|")
     tot = sum(sum(v) for v in times.values()) / f.steps

@@ -311,10 +311,12 @@ class Engine:
         """Keeps the recurrent state from before a step's rows, so that its last rows can be taken back (``truncate``)."""
         self._snap = None
         if self.kv.states and rows:
-            slots = {r.slot for r in rows}
-            if sum(i == 0 or r.slot != rows[i - 1].slot for i, r in enumerate(rows)) != len(slots):
+            runs = [r.slot for i, r in enumerate(rows) if i == 0 or r.slot != rows[i - 1].slot]
+            if len(set(runs)) != len(runs):
                 raise ValueError("a recurrent model's step holds a sequence's rows one after another")
-            self._snap = (list(rows), {s: self.kv.save_states(s) for s in sorted(slots)})
+            several = {r.slot for i, r in enumerate(rows) if i and r.slot == rows[i - 1].slot}
+            if several:       # a lone row of a sequence is its next token, never a draft
+                self._snap = ([r for r in rows if r.slot in several], {s: self.kv.save_states(s) for s in sorted(several)})
 
     def logits(self, m: int) -> torch.Tensor:
         """fp32 logits of the last step's rows (device tensor view)."""
