@@ -50,7 +50,13 @@ def peek_config(spec: str):
         hf = json.load(f)
     if "text_config" in hf:
         hf = hf["text_config"]
-    return ModelConfig.from_hf_config(hf)
+    cfg = ModelConfig.from_hf_config(hf)
+    from ..models.listed import sizes_in_tensors
+    if sizes_in_tensors(cfg):
+        from ..loader.loader import tensor_sizes
+        from ..utils.safetensors_io import SafetensorsSet
+        cfg = tensor_sizes(cfg, SafetensorsSet(resolve_snapshot(spec)))
+    return cfg
 
 
 def chat_format_for(spec: str):

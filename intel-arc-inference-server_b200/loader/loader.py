@@ -235,10 +235,17 @@ def _load_ffn(lw: LayerWeights, view: NameView, cfg: ModelConfig, prefix: str, q
         lw.gate_up, lw.down = mlp(prefix + ".mlp", cfg.ffn)
 
 
+def tensor_sizes(cfg: ModelConfig, st: SafetensorsSet) -> ModelConfig:
+    """The configuration of a listed model with the sizes that its tensors give (0 where a tensor is missing)."""
+    from ..models.listed import with_tensor_sizes
+    return with_tensor_sizes(cfg, lambda name: tuple(st.shape(name)) if st.has(name) else (0, 0))
+
+
 def load_listed(st: SafetensorsSet, cfg: ModelConfig, device, dtype: str = "bfloat16") -> ModelWeights:
     """A model that lists its layers: unquantised tensors under the design's own names, checked against the
     configuration before anything is assembled; ``dtype`` float32 keeps everything in 32-bit."""
     from ..models.listed import assemble, tensor_shapes
+    cfg = tensor_sizes(cfg, st)
     bad = []
     for name, shape in tensor_shapes(cfg).items():
         if not st.has(name):

@@ -57,6 +57,12 @@ class GroupedAttention:
     bias: float = 0.0             # distance bias -(i - j) 2^(-bias (h + 1) / heads) on head h's scores (0: none)
     sink: bool = False            # one learned term per head in the softmax's denominator
     kv_from: int = -1             # layer whose cached keys and values are read (-1: the layer's own)
+    log_bias: bool = False        # distance bias -r1 ln(1 + r2 (i - j)) with two learned numbers per head
+    qkv_bias: bool = False
+    qk_norm: bool = False         # queries and keys: RMS norm per head with a weight shared by the heads
+    v_norm: bool = False          # values are divided by their root mean square per head
+    temp: float = 0.0             # queries at position p times 1 + temp ln(floor((p + 1) / temp_every) + 1)
+    temp_every: int = 1
 
     def linear_elems(self, h: int) -> int:
         return h * (self.heads * (self.dim + self.vdim) + (self.kv_heads * (self.dim + self.vdim) if self.kv_from < 0 else 0))
@@ -73,6 +79,7 @@ class MatrixLstm:
     dim: int
     vdim: int
     gate_cap: float
+    recurrent = True
 
     def linear_elems(self, h: int) -> int:
         return h * self.heads * (2 * self.dim + 3 * self.vdim + 2)
@@ -83,12 +90,108 @@ class MatrixLstm:
 
 
 @dataclass(frozen=True)
+class MinGru:
+    """Recurrent mixer, element by element: S <- (1 - z) S + z c, gates from the current token only; the result is S times
+    SiLU of a third projection."""
+    width: int
+    recurrent = True
+    heads = 1
+
+    @property
+    def dim(self) -> int:
+        return self.width
+
+    def linear_elems(self, h: int) -> int:
+        return 4 * h * self.width
+
+    @property
+    def kv_elems(self) -> int:
+        return 0
+
+
+@dataclass(frozen=True)
+class ParallelMixer:
+    """Two mixers side by side on the same input; the result is the sum of theirs, each times its scale."""
+    left: object
+    right: object
+    left_scale: float
+    right_scale: float
+
+    @property
+    def heads(self) -> int:
+        return max(self.left.heads, self.right.heads)
+
+    @property
+    def kv_heads(self) -> int:
+        return max(getattr(m, "kv_heads", 1) for m in (self.left, self.right))
+
+    @property
+    def dim(self) -> int:
+        return max(self.left.dim, self.right.dim)
+
+    @property
+    def recurrent(self) -> bool:
+        return any(getattr(m, "recurrent", False) for m in (self.left, self.right))
+
+    def linear_elems(self, h: int) -> int:
+        return self.left.linear_elems(h) + self.right.linear_elems(h)
+
+    @property
+    def kv_elems(self) -> int:
+        return self.left.kv_elems + self.right.kv_elems
+
+
+@dataclass(frozen=True)
+class ChannelDelta:
+    """Recurrent mixer: gated delta rule with one decay per head and key channel; short causal convolutions on q, k and v.
+    The ranks of the decay's and the output gate's projections are given by their tensors (0: not known yet)."""
+    heads: int                    # value heads; query / key head of head h: h / (heads / kv_heads)
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int                     # taps
+    a_rank: int = 0
+    g_rank: int = 0
+    recurrent = True
+
+    def linear_elems(self, h: int) -> int:
+        qk, v = self.kv_heads * self.dim, self.heads * self.vdim
+        return h * (2 * qk + 2 * v + self.heads + self.a_rank + self.g_rank) + self.heads * self.dim * self.a_rank + v * self.g_rank
+
+    @property
+    def kv_elems(self) -> int:
+        return 0
+
+
+@dataclass(frozen=True)
+class Wkv:
+    """Recurrent mixer (RWKV-style time mixing): five inputs, each its own mix of the token and the one before; a decay per
+    head and key channel, a bonus for the current token.  The rank of the decay's projection is given by its tensor."""
+    heads: int
+    dim: int
+    w_rank: int = 0
+    recurrent = True
+    shifts = 5                    # shifted inputs
+
+    def linear_elems(self, h: int) -> int:
+        n = self.heads * self.dim
+        return 5 * h * n + self.w_rank * (h + n)
+
+    @property
+    def kv_elems(self) -> int:
+        return 0
+
+
+@dataclass(frozen=True)
 class DenseFfn:
-    """down (g sigmoid(alpha g) (u + shift)), g = min(gate, limit), u = clamp(up, -limit, limit)."""
+    """down (f(g) (u + shift)), g = min(gate, limit), u = clamp(up, -limit, limit), f(g) = g sigmoid(alpha g), or the tanh form
+    of GELU; ``bias``: all three projections have one."""
     ff: int
     limit: float = float("inf")
     alpha: float = 1.0
     shift: float = 0.0
+    gelu: bool = False
+    bias: bool = False
 
     def linear_elems(self, h: int) -> tuple:
         return (3 * self.ff * h,) * 2
@@ -99,12 +202,24 @@ class StreamBlock:
     """Residual of several streams around pre-normed sublayers (hyper-connections): a sublayer reads a mix of the streams,
     its result goes to all of them, times ``mult``.  Norms have one number for all columns; ``shift``: what a mixer reads is
     mixed with the previous token's; the streams start as the embedding plus a sinusoidal position vector (``sinusoid``:
-    its base, 0: none)."""
+    its base, 0: none).  One stream without ``mixing`` is the plain residual x + y; ``columns``: norms have a weight per
+    column, stored around zero."""
     streams: int
     mult: float
     shift: bool = True
     scale: bool = True            # a learned factor per column on every sublayer's result
     sinusoid: float = 10000.0
+    mixing: bool = True
+    columns: bool = False
+
+
+@dataclass(frozen=True)
+class LayerLoop:
+    """Layers ``start`` .. ``stop - 1`` run ``times`` times in a row with the same weights, each pass with its own cache and
+    state.  Ahead of a pass a learned vector is added to the residual, and ahead of all but the first the embedding row too."""
+    start: int
+    stop: int
+    times: int
 
 
 @dataclass(frozen=True)
@@ -134,7 +249,7 @@ class ExpertFfn:
 class LayerSpec:
     """One layer of a model that lists its layers: a mixer and a feed-forward (or none).  How they meet the fp32 residual
     is ``ModelConfig.block``: None adds layer norms of the sublayers' outputs to one stream."""
-    mixer: object                 # LatentAttention, GroupedAttention or MatrixLstm
+    mixer: object                 # LatentAttention, GroupedAttention, MatrixLstm, ParallelMixer, ChannelDelta or Wkv
     ffn: object                   # ExpertFfn, DenseFfn or None
 
 
@@ -176,6 +291,27 @@ class ModelConfig:
     # largest values over the layers
     layer_specs: tuple = ()
     block: Optional[StreamBlock] = None
+    loop: Optional[LayerLoop] = None
+
+    @property
+    def layer_runs(self) -> tuple:
+        """(layer, pass that starts ahead of it or -1) of a listed model, in the order in which the layers run.  Caches and
+        states belong to runs."""
+        n, lp = len(self.layer_specs), self.loop
+        if lp is None:
+            return tuple((i, -1) for i in range(n))
+        body = tuple((i, t if i == lp.start else -1) for t in range(lp.times) for i in range(lp.start, lp.stop))
+        return tuple((i, -1) for i in range(lp.start)) + body + tuple((i, -1) for i in range(lp.stop, n))
+
+    @property
+    def run_specs(self) -> tuple:
+        return tuple(self.layer_specs[i] for i, _ in self.layer_runs)
+
+    @property
+    def shift_runs(self) -> tuple:
+        """Runs whose mixer reads the previous token's input too."""
+        every = self.block is not None and self.block.shift
+        return tuple(j for j, s in enumerate(self.run_specs) if every or getattr(s.mixer, "shifts", 0))
 
     @property
     def q_dim(self) -> int:
@@ -213,8 +349,7 @@ class ModelConfig:
     @property
     def recurrent(self) -> bool:
         """Sequences carry a state that cannot be rewound position by position."""
-        return self.n_gdn_layers > 0 or any(isinstance(s.mixer, MatrixLstm) for s in self.layer_specs) \
-            or (self.block is not None and self.block.shift)
+        return self.n_gdn_layers > 0 or any(getattr(s.mixer, "recurrent", False) for s in self.layer_specs) or bool(self.shift_runs)
 
     @property
     def gdn_key_dim(self) -> int:
@@ -307,7 +442,7 @@ class ModelConfig:
         for every linear that is touched, plus the head."""
         h = self.hidden
         if self.layer_specs:
-            return 2.0 * sum(self.layer_linears(s)[0] for s in self.layer_specs) + self.vocab * h * lm_head_bytes_per_weight
+            return 2.0 * sum(self.layer_linears(s)[0] for s in self.run_specs) + self.vocab * h * lm_head_bytes_per_weight
         int4 = 0.5 + 2.0 / self.group_size
         per = self._mixer_params() * int4
         if self.is_moe:
@@ -320,7 +455,7 @@ class ModelConfig:
 
     def kv_bytes_per_token(self, kv_dtype: str = "bf16") -> int:
         if self.layer_specs:
-            return sum(s.mixer.kv_elems for s in self.layer_specs) * (4 if kv_dtype == "f32" else 2)
+            return sum(s.mixer.kv_elems for s in self.run_specs) * (4 if kv_dtype == "f32" else 2)
         per_head = self.head_dim * (2 if kv_dtype == "bf16" else 1) + (4 if kv_dtype == "int8" else 0)
         return (self.n_layers - self.n_gdn_layers) * 2 * self.n_kv_heads * per_head
 
@@ -390,7 +525,7 @@ class ModelConfig:
 
 
 def listed_config(name: str, architecture: str, specs, hidden: int, vocab: int, eps: float,
-                  block: Optional[StreamBlock] = None) -> ModelConfig:
+                  block: Optional[StreamBlock] = None, loop: Optional[LayerLoop] = None) -> ModelConfig:
     """A model given by its layers; the scalar fields other parts of the framework read hold the largest values."""
     specs = tuple(specs)
     ffns = [s.ffn for s in specs if s.ffn is not None]
@@ -399,7 +534,7 @@ def listed_config(name: str, architecture: str, specs, hidden: int, vocab: int, 
                        max(s.mixer.dim + getattr(s.mixer, "rot_dim", 0) for s in specs), 0, vocab, rms_eps=eps,
                        n_experts=most("experts"), top_k=most("top"),
                        expert_ffn=max((f.ff for f in ffns if isinstance(f, ExpertFfn)), default=0),
-                       architecture=architecture, layer_specs=specs, block=block)
+                       architecture=architecture, layer_specs=specs, block=block, loop=loop)
 
 
 def mumusun_config(d: dict) -> ModelConfig:
@@ -491,8 +626,71 @@ def napadra_keys(c: ModelConfig) -> dict:
     return {"streams": c.block.streams, "residual_mult": c.block.mult, "layers": [layer(s) for s in c.layer_specs]}
 
 
-LISTED_ARCHITECTURES = {"Mumusun": mumusun_config, "Napadra": napadra_config}
-LISTED_WRITERS = {"Mumusun": mumusun_keys, "Napadra": napadra_keys}
+def pefulorn_config(d: dict) -> ModelConfig:
+    """``config.json`` of a Pefulorn checkpoint: delta-rule layers with a decay per key channel, layers of attention with a
+    logarithmic distance bias beside a minGRU, time-mixing layers, dense feed-forwards, over one pre-normed residual; a range
+    of layers may run several times."""
+    specs = []
+    for i, layer in enumerate(d["layers"]):
+        m, f = layer["mixer"], layer["mlp"]
+        if layer["type"] == "channel_delta":
+            mixer = ChannelDelta(m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"])
+            if not 1 <= mixer.conv <= 16:
+                raise ValueError(f"layer {i}: convolution of {mixer.conv} taps (1 to 16)")
+        elif layer["type"] == "parallel":
+            a, t = m["left"], m["left"].get("q_temp") or {"coef": 0.0, "every": 1}
+            left = GroupedAttention(a["heads"], a["kv_heads"], a["dim"], a["vdim"], float(a["scale"]), log_bias=True, qkv_bias=True,
+                                    qk_norm=True, v_norm=True, temp=float(t["coef"]), temp_every=t["every"])
+            if max(left.dim, left.vdim) > 1024 or left.temp_every < 1:
+                raise ValueError(f"layer {i}: attention heads of {left.dim} x {left.vdim} (1024 at most), temperature {t}")
+            mixer = ParallelMixer(left, MinGru(m["right"]["width"]), float(m["left_scale"]), float(m["right_scale"]))
+        elif layer["type"] == "wkv":
+            mixer = Wkv(m["heads"], m["dim"])
+        else:
+            raise ValueError(f"layer {i}: mixer {layer['type']!r} is not part of Pefulorn")
+        if not isinstance(mixer, ParallelMixer) and max(mixer.dim, getattr(mixer, "vdim", 0)) > 512:
+            raise ValueError(f"layer {i}: recurrent heads of {mixer.dim} x {getattr(mixer, 'vdim', mixer.dim)} (512 at most)")
+        heads = mixer.left if isinstance(mixer, ParallelMixer) else mixer
+        if heads.heads % getattr(heads, "kv_heads", 1):
+            raise ValueError(f"layer {i}: {heads.heads} heads over {heads.kv_heads} key heads")
+        ffn = None
+        if f is not None:
+            if f["kind"] != "dense":
+                raise ValueError(f"layer {i}: feed-forward {f['kind']!r} is not part of Pefulorn")
+            ffn = DenseFfn(f["ff"], gelu=True, bias=True)
+        specs.append(LayerSpec(mixer, ffn))
+    loop = d.get("loop")
+    if loop is not None:
+        loop = LayerLoop(loop["start"], loop["stop"], loop["times"])
+        if not 0 <= loop.start < loop.stop <= len(specs) or loop.times < 1:
+            raise ValueError(f"{loop} does not fit {len(specs)} layers")
+    return listed_config(d.get("name", "pefulorn"), "Pefulorn", specs, d["width"], d["vocab"], float(d["norm"]["eps"]),
+                         StreamBlock(1, 1.0, shift=False, scale=False, sinusoid=0.0, mixing=False, columns=True), loop)
+
+
+def pefulorn_keys(c: ModelConfig) -> dict:
+    def layer(s):
+        m, f = s.mixer, s.ffn
+        if isinstance(m, ChannelDelta):
+            kind, mixer = "channel_delta", {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "conv": m.conv}
+        elif isinstance(m, Wkv):
+            kind, mixer = "wkv", {"heads": m.heads, "dim": m.dim}
+        else:
+            a = m.left
+            left = {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim, "scale": a.scale}
+            if a.temp:
+                left["q_temp"] = {"coef": a.temp, "every": a.temp_every}
+            kind, mixer = "parallel", {"left": left, "left_scale": m.left_scale, "right": {"width": m.right.width},
+                                       "right_scale": m.right_scale}
+        return {"type": kind, "mixer": mixer, "mlp": None if f is None else {"kind": "dense", "ff": f.ff}}
+    out = {"layers": [layer(s) for s in c.layer_specs]}
+    if c.loop is not None:
+        out["loop"] = {"start": c.loop.start, "stop": c.loop.stop, "times": c.loop.times}
+    return out
+
+
+LISTED_ARCHITECTURES = {"Mumusun": mumusun_config, "Napadra": napadra_config, "Pefulorn": pefulorn_config}
+LISTED_WRITERS = {"Mumusun": mumusun_keys, "Napadra": napadra_keys, "Pefulorn": pefulorn_keys}
 
 
 def tiny_dense() -> ModelConfig:
@@ -587,6 +785,37 @@ def napadra_7b() -> ModelConfig:
     return listed_config("napadra-7b", "Napadra", specs, 4096, 64000, 1e-5, StreamBlock(4, 0.5))
 
 
+def _parallel(heads, kv, dim, vdim, width, every, coef=0.4, scales=(1.0, 1.0)) -> ParallelMixer:
+    return ParallelMixer(GroupedAttention(heads, kv, dim, vdim, dim ** -0.5, log_bias=True, qkv_bias=True, qk_norm=True, v_norm=True,
+                                          temp=coef, temp_every=every), MinGru(width), *scales)
+
+
+def pefulorn_mini() -> ModelConfig:
+    """Small Pefulorn: every kind of layer with unequal sizes, the middle ones run three times."""
+    ff = lambda n: DenseFfn(n, gelu=True, bias=True)                               # noqa: E731
+    return listed_config("pefulorn-mini", "Pefulorn", (
+        LayerSpec(_parallel(6, 2, 40, 72, 136, 50, 0.7, (0.8, 1.3)), ff(176)), LayerSpec(ChannelDelta(6, 2, 48, 40, 3, 20, 36), ff(112)),
+        LayerSpec(Wkv(3, 72, 28), None), LayerSpec(_parallel(4, 4, 96, 64, 80, 7), None), LayerSpec(Wkv(2, 40, 70), ff(80)),
+        LayerSpec(ChannelDelta(3, 3, 80, 130, 4, 72, 12), ff(96))), 200, 700, 1e-5,
+        StreamBlock(1, 1.0, shift=False, scale=False, sinusoid=0.0, mixing=False, columns=True), LayerLoop(1, 4, 3))
+
+
+def pefulorn_like(name: str, width: int, layers: int, heads: int, kv: int, ff: int, vocab: int, rank: int = 128) -> ModelConfig:
+    """A Pefulorn of real layer sizes: groups of two delta-rule layers, a time-mixing layer and a layer of attention beside a
+    minGRU of the model's width, all heads of 128."""
+    f, specs = DenseFfn(ff, gelu=True, bias=True), []
+    for _ in range(0, layers, 4):
+        specs += [LayerSpec(ChannelDelta(heads, heads, 128, 128, 4, rank, rank), f)] * 2 + [
+            LayerSpec(Wkv(heads, 128, rank), f), LayerSpec(_parallel(heads, kv, 128, 128, width, 8192, 0.1), f)]
+    return listed_config(name, "Pefulorn", specs, width, vocab, 1e-6,
+                         StreamBlock(1, 1.0, shift=False, scale=False, sinusoid=0.0, mixing=False, columns=True))
+
+
+def pefulorn_7b() -> ModelConfig:
+    """32 layers, hidden 4096, 32 heads of 128 (8 key heads in the attention layers), 11008 wide feed-forwards."""
+    return pefulorn_like("pefulorn-7b", 4096, 32, 32, 8, 11008, 64000)
+
+
 def dflash_drafter(target: ModelConfig) -> ModelConfig:
     """DFlash-style block drafter: a 2-layer W4A16 decoder at the target's width."""
     return replace(target, name=target.name + "-dflash", n_layers=2, n_experts=0, top_k=0, expert_ffn=0,
@@ -597,6 +826,7 @@ def dflash_drafter(target: ModelConfig) -> ModelConfig:
 PRESETS = {
     "tiny-dense": tiny_dense, "tiny-moe": tiny_moe, "small-dense": small_dense, "small-windowed": small_windowed, "small-hybrid": small_hybrid, "small-moe": small_moe, "dense-27b": dense_27b, "hybrid-27b": hybrid_27b, "moe-35b-a3b": moe_35b_a3b,
     "mumusun-mini": mumusun_mini, "mumusun-16b": mumusun_16b, "napadra-mini": napadra_mini, "napadra-7b": napadra_7b,
+    "pefulorn-mini": pefulorn_mini, "pefulorn-7b": pefulorn_7b,
 }
 
 

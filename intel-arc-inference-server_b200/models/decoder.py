@@ -99,7 +99,7 @@ class ListedBuffers:
 
 class KVCache:
     """Paged KV: per layer ``[page][kv_head][16][D]`` for K and for V (bf16 or int8 + fp32 scales).  Models that list their
-    layers keep what their mixers ask for, by name and layer: planes of the page pool (``pages``: ``[page][kv_head][16][d]``,
+    layers keep what their mixers ask for, by name and layer run: planes of the page pool (``pages``: ``[page][kv_head][16][d]``,
     or ``[page][16][d]`` for rows shared by the heads).  ``states``: recurrent state ``[layers][slot]...`` by name, of every
     family that has some."""
 
@@ -116,15 +116,14 @@ class KVCache:
             if kv_dtype not in ("bf16", "f32"):
                 raise ValueError(f"{cfg.name} keeps a bf16 (or, served in 32-bit, fp32) cache, not {kv_dtype}")
             ldt = torch.float32 if kv_dtype == "f32" else torch.bfloat16
-            for li, sp in enumerate(cfg.layer_specs):
+            for li, sp in enumerate(cfg.run_specs):
                 for name, (heads, cols) in kind(sp.mixer).page_planes(sp.mixer).items():
                     shape = (num_pages, heads, cfg.page_size, cols) if heads else (num_pages, cfg.page_size, cols)
                     self.pages[f"{name}{li}"] = torch.zeros(shape, dtype=ldt, device=device)
-                shape = kind(sp.mixer).state_shape(sp.mixer)
-                if shape is not None:
-                    self.states[f"mlstm{li}"] = torch.zeros((1, n_slots) + shape, dtype=torch.float32, device=device)
-            if cfg.block is not None and cfg.block.shift:
-                self.states["shift"] = torch.zeros(cfg.n_layers, n_slots, pad64(cfg.hidden), dtype=torch.float32, device=device)
+                for name, shape in kind(sp.mixer).state_shapes(sp.mixer).items():
+                    self.states[f"{name}{li}"] = torch.zeros((1, n_slots) + shape, dtype=torch.float32, device=device)
+            if cfg.shift_runs:
+                self.states["shift"] = torch.zeros(len(cfg.shift_runs), n_slots, pad64(cfg.hidden), dtype=torch.float32, device=device)
                 self.shift_next = torch.zeros(n_slots, pad64(cfg.hidden), dtype=torch.float32, device=device)
             self.k = self.v = self.k_scale = self.v_scale = self.gdn_conv = self.gdn_state = None
             return

@@ -1,9 +1,11 @@
-"""Grouped-query attention mixers over paged keys and values of any head size, without a rotation; optional distance bias,
-chunked mask, sinks, and layers that read another layer's keys and values.
+"""Grouped-query attention mixers over paged keys and values of any head size, without a rotation; optional distance bias
+(linear or logarithmic), chunked mask, sinks, biases and norms of queries, keys and values, query temperature, and layers that
+read another layer's keys and values.
 
 Rows of a step are attended one by one (split-KV kernel) or, for long segments of a prompt, in query tiles by the tcgen05
 prompt attention straight over the pages.  The projection of a prompt stays in the GEMM's bf16 rows: the prompt attention
-reads its queries there.
+reads its queries there.  With biases or norms the projection is fp32 instead, and a kernel of its own makes query rows and
+fills the pages (``core``, which also serves a mixer beside another one).
 """
 from __future__ import annotations
 
@@ -51,25 +53,39 @@ class GroupedGeometry:
 
 def shapes(cfg: ModelConfig, p: str, a: GroupedAttention) -> dict:
     h = cfg.hidden
-    out = {p + "mix.q": (a.heads * a.dim, h), p + "mix.o": (h, a.heads * a.vdim)}
+    out = {p + "q": (a.heads * a.dim, h), p + "o": (h, a.heads * a.vdim)}
     if a.kv_from < 0:
-        out.update({p + "mix.k": (a.kv_heads * a.dim, h), p + "mix.v": (a.kv_heads * a.vdim, h)})
+        out.update({p + "k": (a.kv_heads * a.dim, h), p + "v": (a.kv_heads * a.vdim, h)})
     if a.sink:
-        out[p + "mix.sink"] = (a.heads,)
+        out[p + "sink"] = (a.heads,)
+    if a.qkv_bias:
+        out.update({p + n + ".b": (h * d,) for n, h, d in (("q", a.heads, a.dim), ("k", a.kv_heads, a.dim), ("v", a.kv_heads, a.vdim))})
+    if a.qk_norm:
+        out.update({p + "q.norm": (a.dim,), p + "k.norm": (a.dim,)})
+    if a.log_bias:
+        out.update({p + "r1": (a.heads,), p + "r2": (a.heads,)})
     return out
 
 
 def assemble(t, p: str, a: GroupedAttention) -> GroupedWeights:
     """``t``: ``listed.Assembler``."""
     g = GroupedGeometry.of(a)
-    parts = [t.heads(t.t(p + "mix.q"), a.heads, [(a.dim, g.dk)], t.wp)]
+    parts = [t.heads(t.t(p + "q"), a.heads, [(a.dim, g.dk)], t.wp)]
     if a.kv_from < 0:
-        parts += [t.heads(t.t(p + "mix.k"), a.kv_heads, [(a.dim, g.dk)], t.wp), t.heads(t.t(p + "mix.v"), a.kv_heads, [(a.vdim, g.dv)], t.wp)]
+        parts += [t.heads(t.t(p + "k"), a.kv_heads, [(a.dim, g.dk)], t.wp), t.heads(t.t(p + "v"), a.kv_heads, [(a.vdim, g.dv)], t.wp)]
     slope2 = None
     if a.bias:
         slope2 = torch.tensor([2.0 ** (-a.bias * (h + 1) / a.heads) * LOG2E for h in range(a.heads)], dtype=torch.float32, device=t.device)
-    sink2 = t.vec(p + "mix.sink") * LOG2E if a.sink else None
-    return GroupedWeights(torch.cat(parts), t.out_proj(p + "mix.o", a.heads, a.vdim, g.dv), slope2, sink2)
+    sink2 = t.vec(p + "sink") * LOG2E if a.sink else None
+    w = GroupedWeights(torch.cat(parts), t.out_proj(p + "o", a.heads, a.vdim, g.dv), slope2, sink2)
+    if a.qkv_bias:
+        w.bias = torch.cat([t.fp32_heads(p + n + ".b", h, d, pad, 1).reshape(-1) for n, h, d, pad in (
+            ("q", a.heads, a.dim, g.dk), ("k", a.kv_heads, a.dim, g.dk), ("v", a.kv_heads, a.vdim, g.dv))])
+    if a.qk_norm:
+        w.q_norm, w.k_norm = t.vec(p + "q.norm", g.dk), t.vec(p + "k.norm", g.dk)
+    if a.log_bias:
+        w.r1, w.r2 = t.vec(p + "r1"), t.vec(p + "r2")
+    return w
 
 
 def weight_elems(cfg: ModelConfig, a: GroupedAttention) -> int:
@@ -89,8 +105,8 @@ def page_planes(a: GroupedAttention) -> dict:
     return {} if a.kv_from >= 0 else {"k": (g.kv_heads, g.dk), "v": (g.kv_heads, g.dv)}
 
 
-def state_shape(a: GroupedAttention) -> Optional[tuple]:
-    return None
+def state_shapes(a: GroupedAttention) -> dict:
+    return {}
 
 
 class Mixer:
@@ -100,7 +116,13 @@ class Mixer:
         on_gpu = ll.device.type == "cuda" and not ll.f32
         self.tile_rows = P.segments_per_tile(self.g) if on_gpu else 0
         self.rows_form = on_gpu and P.rows_ok(self.g)
-        self.form = ("tiles", a.chunk, self.tile_rows) if self.tile_rows else None
+        self.forms = [("tiles", a.chunk, self.tile_rows)] if self.tile_rows else []
+        self.normed = a.qkv_bias or a.qk_norm or a.v_norm or a.temp != 0.0
+        if self.normed and a.kv_from >= 0:
+            raise ValueError("layers on another layer's keys have neither biases nor norms of their own")
+        self.cols = self.g.nq + (self.g.nkv if a.kv_from < 0 else 0)      # columns of its projection, and of its rows
+        self.out_cols = self.g.heads * self.g.dv
+        self.logb = (w.r1, w.r2) if a.log_bias else None
 
     def nsplit(self, m: int) -> int:
         """KV splits of the row attention: about two CTAs per SM, at least two pages per warp of a split."""
@@ -115,12 +137,15 @@ class Mixer:
 
     def run(self, sc: ListedScratch, m: int, rows: StepRows, block_table, kv, plan: Optional[BatchPlan]):
         """Attention of the step's rows: fp32 slices of its output projection."""
-        ll, a, g, w = self.ll, self.a, self.g, self.w
-        own = a.kv_from < 0
+        ll, g, w = self.ll, self.g, self.w
+        own = self.a.kv_from < 0
         k, v = kv.pages[f"k{self.src}"], kv.pages[f"v{self.src}"]
         h = sc.get("h", m, ll.wp)
         out = sc.get("attn", m, g.heads * g.dv)
-        n1 = m if plan is None or not self.tile_rows else plan.n_single
+        if self.normed:
+            part, s = ll.linear(sc, "qkv", w.qkv, h, m)
+            self.core(sc, m, rows, block_table, kv, plan, part, s, 0, out)
+            return ll.linear(sc, "o", w.o, out, m)
         if ll.f32 or m <= L.GEMV_ROWS:
             part, s = ll.linear(sc, "qkv", w.qkv, h, m)
             q = sc.get("q_rows", m, g.nq)
@@ -130,14 +155,31 @@ class Mixer:
             G.gemm_bf16(h, w.qkv, q)
             if own:
                 P.append_rows(q, m, g, rows.req, rows.pos, block_table, k, v)
+        self.attend(sc, m, rows, block_table, plan, q, k, v, out)
+        return ll.linear(sc, "o", w.o, out, m)
+
+    def core(self, sc: ListedScratch, m: int, rows: StepRows, block_table, kv, plan: Optional[BatchPlan], part, s: int, col: int, out,
+             mult: float = 1.0):
+        """From its columns of the projection's fp32 slices, which come first, to its rows ``out``, times ``mult``."""
+        if col:
+            raise ValueError("the columns of an attention mixer come first")
+        g, k, v = self.g, kv.pages[f"k{self.li}"], kv.pages[f"v{self.li}"]
+        q = sc.get("q_rows", m, g.nq)
+        P.norm(part, s, m, g, self.a, self.w, self.ll.cfg.rms_eps, rows.req, rows.pos, block_table, q, k, v)
+        self.attend(sc, m, rows, block_table, plan, q, k, v, out, mult)
+
+    def attend(self, sc: ListedScratch, m: int, rows: StepRows, block_table, plan: Optional[BatchPlan], q, k, v, out, mult: float = 1.0):
+        """Attention of query rows ``q`` over the pages, which hold the step's keys and values already."""
+        a, g, w = self.a, self.g, self.w
+        more = dict(logb=self.logb, mult=mult)
+        n1 = m if plan is None or not self.tile_rows else plan.n_single
         if n1 and self.rows_form:
             ns, cap = self.nsplit(n1), self.partials(g)
             op = sc.get("o_part", cap, g.dv, torch.float32) if ns > 1 else None
             ml = sc.get("ml_part", cap, 2, torch.float32) if ns > 1 else None
-            P.rows(q, k, v, n1, g, rows.req, rows.pos, block_table, ns, a.chunk, a.scale, w.slope2, w.sink2, op, ml, out)
+            P.rows(q, k, v, n1, g, rows.req, rows.pos, block_table, ns, a.chunk, a.scale, w.slope2, w.sink2, op, ml, out, **more)
         elif n1:
-            P.simple(q, k, v, n1, g, rows.req, rows.pos, block_table, a.chunk, a.scale, w.slope2, w.sink2, out)
+            P.simple(q, k, v, n1, g, rows.req, rows.pos, block_table, a.chunk, a.scale, w.slope2, w.sink2, out, **more)
         if n1 < m:
-            t = plan.tables[self.form]
-            P.attn_segments(q[n1:], k, v, block_table, out[n1:], t.tiles, t.n_tiles, m - n1, g, a.scale, a.chunk, w.slope2, w.sink2)
-        return ll.linear(sc, "o", w.o, out, m)
+            t = plan.tables[self.forms[0]]
+            P.attn_segments(q[n1:], k, v, block_table, out[n1:], t.tiles, t.n_tiles, m - n1, g, a.scale, a.chunk, w.slope2, w.sink2, **more)

@@ -57,22 +57,22 @@ class LatentGeometry:
 # ------------------------------------------------------------------ weights and sizes
 def shapes(cfg: ModelConfig, p: str, a: LatentAttention) -> dict:
     h = cfg.hidden
-    return {p + "mix.dq": (a.q_rank, h), p + "mix.dq.norm": (a.q_rank,), p + "mix.uq": (a.heads * (a.dim + a.rot_dim), a.q_rank),
-            p + "mix.dkv": (a.kv_rank + a.rot_dim, h), p + "mix.dkv.norm": (a.kv_rank,), p + "mix.uk": (a.heads * a.dim, a.kv_rank),
-            p + "mix.uv": (a.heads * a.vdim, a.kv_rank), p + "mix.o": (h, a.heads * a.vdim)}
+    return {p + "dq": (a.q_rank, h), p + "dq.norm": (a.q_rank,), p + "uq": (a.heads * (a.dim + a.rot_dim), a.q_rank),
+            p + "dkv": (a.kv_rank + a.rot_dim, h), p + "dkv.norm": (a.kv_rank,), p + "uk": (a.heads * a.dim, a.kv_rank),
+            p + "uv": (a.heads * a.vdim, a.kv_rank), p + "o": (h, a.heads * a.vdim)}
 
 
 def assemble(t, p: str, a: LatentAttention) -> LatentWeights:
     """``t``: ``listed.Assembler``."""
     g, h = LatentGeometry.of(a), t.cfg.hidden
-    down, dkv = t.zeros(g.n_down, t.wp), t.t(p + "mix.dkv")
-    down[: a.q_rank, :h] = t.t(p + "mix.dq")
+    down, dkv = t.zeros(g.n_down, t.wp), t.t(p + "dkv")
+    down[: a.q_rank, :h] = t.t(p + "dq")
     down[g.qp: g.qp + a.kv_rank, :h] = dkv[: a.kv_rank]
     down[g.qp + g.kvp: g.qp + g.kvp + a.rot_dim, :h] = dkv[a.kv_rank:]
-    return LatentWeights(down, t.vec(p + "mix.dq.norm"), t.vec(p + "mix.dkv.norm"),
-                         t.heads(t.t(p + "mix.uq"), a.heads, [(a.dim, g.dn), (a.rot_dim, g.rp)], g.qp),
-                         t.heads(t.t(p + "mix.uk"), a.heads, [(a.dim, g.dn)], g.kvp),
-                         t.heads(t.t(p + "mix.uv"), a.heads, [(a.vdim, g.dv)], g.kvp), t.out_proj(p + "mix.o", a.heads, a.vdim, g.dv))
+    return LatentWeights(down, t.vec(p + "dq.norm"), t.vec(p + "dkv.norm"),
+                         t.heads(t.t(p + "uq"), a.heads, [(a.dim, g.dn), (a.rot_dim, g.rp)], g.qp),
+                         t.heads(t.t(p + "uk"), a.heads, [(a.dim, g.dn)], g.kvp),
+                         t.heads(t.t(p + "uv"), a.heads, [(a.vdim, g.dv)], g.kvp), t.out_proj(p + "o", a.heads, a.vdim, g.dv))
 
 
 def weight_elems(cfg: ModelConfig, a: LatentAttention) -> int:
@@ -91,8 +91,8 @@ def page_planes(a: LatentAttention) -> dict:
     return {"latent": (0, LatentGeometry.of(a).lc)}
 
 
-def state_shape(a: LatentAttention) -> Optional[tuple]:
-    return None
+def state_shapes(a: LatentAttention) -> dict:
+    return {}
 
 
 class Mixer:
@@ -106,7 +106,7 @@ class Mixer:
         on_gpu = ll.device.type == "cuda" and not ll.f32
         self.tile_rows = L.prefill_rows_per_tile(self.g) if on_gpu else 0     # query rows per tile of the prompt attention
         self.rows_form = on_gpu and L.rows_ok(self.g)
-        self.form = ("keys", a.window, self.tile_rows) if self.tile_rows else None
+        self.forms = [("keys", a.window, self.tile_rows)] if self.tile_rows else []
 
     def nsplit(self, m: int) -> int:
         """KV splits of the decode attention: about one CTA per SM, at least one key tile per split."""
@@ -142,7 +142,7 @@ class Mixer:
             L.merge(op, ml, n1, g, ns, w.uv, out)
         if n1 < m:
             self._prompt_attention(sc, a, g, w, cq[n1:], m - n1, rows.pos[n1:], block_table, cache,
-                                   plan.tables[self.form], rope, out[n1:])
+                                   plan.tables[self.forms[0]], rope, out[n1:])
         return ll.linear(sc, "o", w.o, out, m)
 
     def _prompt_attention(self, sc, a, g, w, cq, m, pos, block_table, cache, kp, rope, out):

@@ -1,9 +1,12 @@
 """Models that list their layers: what every such model shares.
 
 A layer is a mixer and a feed-forward (``LayerSpec``).  Each kind of mixer has a module of its own (``latent``, ``grouped``,
-``mlstm``) with the same functions: ``shapes`` and ``assemble`` (checkpoint tensors, kernel-layout weights),
-``weight_elems`` and ``scratch_elems`` (the planner's figures), ``page_planes`` (what it keeps per position in the page
-pool), ``state_shape`` (what it keeps per sequence) and ``Mixer``, whose ``run`` enqueues its kernels for the rows of a step.
+``mlstm``, ``mingru``, ``channel_delta``, ``wkv``; ``parallel``: two of them side by side) with the same functions: ``shapes`` and
+``assemble`` (checkpoint tensors, kernel-layout weights), ``tensor_sizes`` (sizes that only the tensors give; not every kind has
+some), ``weight_elems`` and ``scratch_elems`` (the planner's figures), ``page_planes`` (what it keeps per position in the page
+pool), ``state_shapes`` (what it keeps per sequence) and ``Mixer``, whose ``run`` enqueues its kernels for the rows of a step and
+whose ``forms`` are the tables it wants of a mixed batch's prompt segments.  Pages and states belong to layer runs
+(``ModelConfig.layer_runs``): a layer that runs several times in a step has several.
 The residual around the sublayers is ``streams.StreamWalk``, or the layer-normed single stream of
 ``DecoderModel.listed_walk``.  ``Engine`` gives both the rows of a decode step (control block, CUDA graphs) or of a mixed
 batch (``runtime/batch.py``).
@@ -16,6 +19,7 @@ everything in 32-bit (no reduced-precision product anywhere).
 """
 from __future__ import annotations
 
+import dataclasses
 import os
 from dataclasses import dataclass
 from typing import Callable, Dict, Optional
@@ -25,7 +29,8 @@ import torch
 from ..ops import gemm as G
 from ..ops import latent as L
 from ..ops import moe as M
-from .config import DenseFfn, ExpertFfn, GroupedAttention, LatentAttention, MatrixLstm, ModelConfig
+from .config import (ChannelDelta, DenseFfn, ExpertFfn, GroupedAttention, LatentAttention, MatrixLstm, MinGru, ModelConfig,
+                     ParallelMixer, Wkv)
 from .weights import DenseWeights, ExpertStack, LayerWeights, ModelWeights, interleave16
 
 SMS = 148
@@ -40,8 +45,23 @@ def pad64(n: int) -> int:
 
 def kind(mixer):
     """The module of a mixer's kind."""
-    from . import grouped, latent, mlstm
-    return {LatentAttention: latent, GroupedAttention: grouped, MatrixLstm: mlstm}[type(mixer)]
+    from . import channel_delta, grouped, latent, mingru, mlstm, parallel, wkv
+    return {LatentAttention: latent, GroupedAttention: grouped, MatrixLstm: mlstm, MinGru: mingru, ParallelMixer: parallel,
+            ChannelDelta: channel_delta, Wkv: wkv}[type(mixer)]
+
+
+def sizes_in_tensors(cfg: ModelConfig) -> bool:
+    """Some of the model's sizes are given by its tensors only."""
+    return any(hasattr(kind(s.mixer), "tensor_sizes") for s in cfg.layer_specs)
+
+
+def with_tensor_sizes(cfg: ModelConfig, shape: Callable[[str], tuple]) -> ModelConfig:
+    """The configuration with the sizes that only the checkpoint's tensors give (``shape(name)``)."""
+    specs = []
+    for i, s in enumerate(cfg.layer_specs):
+        sizes = getattr(kind(s.mixer), "tensor_sizes", None)
+        specs.append(s if sizes is None else dataclasses.replace(s, mixer=sizes(f"l{i}.mix.", s.mixer, shape)))
+    return dataclasses.replace(cfg, layer_specs=tuple(specs))
 
 
 # ------------------------------------------------------------------ weights
@@ -49,12 +69,12 @@ def tensor_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
     """Checkpoint tensors of a listed model, by name."""
     from . import streams
     h = cfg.hidden
-    norm = (h,) if cfg.block is None else ()
+    norm = (h,) if cfg.block is None or cfg.block.columns else ()
     out = {"embed": (cfg.vocab, h), "final.norm": norm, "head": (cfg.vocab, h)}
     for i, s in enumerate(cfg.layer_specs):
         p, f = f"l{i}.", s.ffn
         out[p + "norm1"] = norm
-        out.update(kind(s.mixer).shapes(cfg, p, s.mixer))
+        out.update(kind(s.mixer).shapes(cfg, p + "mix.", s.mixer))
         if cfg.block is not None:
             out.update(streams.shapes(cfg, p, s))
         if f is None:
@@ -62,10 +82,14 @@ def tensor_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
         out[p + "norm2"] = norm
         if isinstance(f, DenseFfn):
             out.update({p + "mlp.gate": (f.ff, h), p + "mlp.up": (f.ff, h), p + "mlp.down": (h, f.ff)})
+            if f.bias:
+                out.update({p + "mlp.gate.b": (f.ff,), p + "mlp.up.b": (f.ff,), p + "mlp.down.b": (h,)})
         else:
             out[p + "mlp.router"] = (f.experts, h)
             for e in range(f.experts):
                 out.update({f"{p}mlp.e{e}.gate": (f.ff, h), f"{p}mlp.e{e}.up": (f.ff, h), f"{p}mlp.e{e}.down": (h, f.ff)})
+    if cfg.loop is not None:
+        out["loop.step"] = (cfg.loop.times, h)
     return out
 
 
@@ -85,6 +109,21 @@ class Assembler:
         if cols > len(v):
             v = torch.cat([v, torch.zeros(cols - len(v), device=self.device)])
         return v.contiguous()
+
+    def norm(self, name: str) -> torch.Tensor:
+        """Norm weights as factors."""
+        if self.cfg.block is None or not self.cfg.block.columns:
+            return self.vec(name)
+        return self.vec(name, self.wp) + (torch.arange(self.wp, device=self.device) < self.cfg.hidden)
+
+    def stack(self, parts) -> torch.Tensor:
+        return torch.cat(parts).contiguous()
+
+    def fp32_heads(self, name: str, n: int, size: int, pad: int, cols: int) -> torch.Tensor:
+        """fp32 ``[n * pad][cols]`` from head-major rows."""
+        out = torch.zeros(n, pad, cols, dtype=torch.float32, device=self.device)
+        out[:, :size] = self.get(name).float().to(self.device).reshape(n, size, cols)
+        return out.reshape(n * pad, cols)
 
     def zeros(self, *shape) -> torch.Tensor:
         return torch.zeros(*shape, dtype=self.dtype, device=self.device)
@@ -121,13 +160,16 @@ def assemble(cfg: ModelConfig, get: Callable[[str], torch.Tensor], device, dtype
     wp, layers = a.wp, []
     for i, s in enumerate(cfg.layer_specs):
         p, f = f"l{i}.", s.ffn
-        lw = LayerWeights(input_norm=a.vec(p + "norm1"), post_norm=a.vec(p + "norm2") if f is not None else None, qkv=None, o=None)
-        lw.mixer = kind(s.mixer).assemble(a, p, s.mixer)
-        if cfg.block is not None:
+        lw = LayerWeights(input_norm=a.norm(p + "norm1"), post_norm=a.norm(p + "norm2") if f is not None else None, qkv=None, o=None)
+        lw.mixer = kind(s.mixer).assemble(a, p + "mix.", s.mixer)
+        if cfg.block is not None and cfg.block.mixing:
             lw.streams = streams.assemble(a, p, s)
         if isinstance(f, DenseFfn):
             ffp = pad64(f.ff)
             lw.dense = DenseWeights(a.gate_up(p + "mlp.gate", p + "mlp.up", ffp), a.padded(a.t(p + "mlp.down"), wp, ffp))
+            if f.bias:
+                lw.dense.bias = interleave16(a.vec(p + "mlp.gate.b", ffp)[:, None], a.vec(p + "mlp.up.b", ffp)[:, None]).view(-1).contiguous()
+                lw.dense.down_bias = a.vec(p + "mlp.down.b", wp)
         elif f is not None:
             ffp = pad64(f.ff)
             gu, dn = a.zeros(f.experts, 2 * ffp, wp), a.zeros(f.experts, wp, ffp)
@@ -137,7 +179,11 @@ def assemble(cfg: ModelConfig, get: Callable[[str], torch.Tensor], device, dtype
                 dn[e, : cfg.hidden, : f.ff] = a.t(q + "down")
             lw.moe = ExpertStack(a.padded(a.t(p + "mlp.router"), (f.experts + 7) // 8 * 8, wp), gu, dn)
         layers.append(lw)
-    return ModelWeights(cfg, a.padded(a.t("embed"), cfg.vocab, wp), a.padded(a.t("head"), cfg.vocab, wp), a.vec("final.norm"), layers)
+    w = ModelWeights(cfg, a.padded(a.t("embed"), cfg.vocab, wp), a.padded(a.t("head"), cfg.vocab, wp), a.norm("final.norm"), layers)
+    if cfg.loop is not None:
+        w.loop_step = torch.zeros(cfg.loop.times, wp, dtype=torch.float32, device=device)
+        w.loop_step[:, : cfg.hidden] = get("loop.step").float().to(device)
+    return w
 
 
 def random_listed_weights(cfg: ModelConfig, device="cpu", seed: int = 0, std: float = 0.02,
@@ -168,6 +214,18 @@ def padded_weight_elems(cfg: ModelConfig) -> int:
             n += 3 * pad64(f.ff) * wp
         elif f is not None:
             n += (f.experts + 7) // 8 * 8 * wp + 3 * f.experts * pad64(f.ff) * wp
+    return n
+
+
+def state_elems(cfg: ModelConfig) -> int:
+    """fp32 elements of one sequence's recurrent states."""
+    n = 0
+    for s in cfg.run_specs:
+        for shape in kind(s.mixer).state_shapes(s.mixer).values():
+            size = 1
+            for d in shape:
+                size *= d
+            n += size
     return n
 
 
@@ -245,12 +303,18 @@ class ListedLayers:
         self.max_pos = max_pos
         self.shared: Dict[tuple, object] = {}        # what layers of equal sizes share (angle tables and the like)
         self._splits: Dict[tuple, int] = {}
-        self.mixers = [kind(s.mixer).Mixer(self, i, s.mixer, lw.mixer)
-                       for i, (s, lw) in enumerate(zip(self.cfg.layer_specs, weights.layers))]
+        if self.cfg.loop is not None and (self.cfg.block is None or any(getattr(s.mixer, "kv_from", -1) >= 0 for s in self.cfg.layer_specs)):
+            raise ValueError(f"{self.cfg.name}: layers that run several times need the pre-normed residual and keys of their own")
+        self.mixers = [kind(self.cfg.layer_specs[i].mixer).Mixer(self, j, self.cfg.layer_specs[i].mixer, weights.layers[i].mixer)
+                       for j, (i, _) in enumerate(self.cfg.layer_runs)]
 
     def forms(self):
         """Tables the mixers want of a mixed batch's prompt segments."""
-        return sorted({m.form for m in self.mixers if m.form is not None})
+        return sorted({f for m in self.mixers for f in m.forms})
+
+    def shifted(self, sc: ListedScratch, planes: int, m: int) -> torch.Tensor:
+        """``[planes * m][wp]``: what a mixer with several shifted inputs reads."""
+        return sc.get(f"h_shift{planes}", planes * m, self.wp, mult=planes)
 
     def linear(self, sc: ListedScratch, name: str, w: torch.Tensor, x: torch.Tensor, m: int):
         """fp32 ``x[:m] @ w.T`` as (slices [s][m][n], s)."""
@@ -267,6 +331,23 @@ class ListedLayers:
         L.gemv_bf16(w, x, out, m, n, k, s)
         return out, s
 
+    def linear_planes(self, sc: ListedScratch, name: str, w: torch.Tensor, x: torch.Tensor, plane_rows: int, m: int):
+        """``linear`` with activations ``x`` ``[planes][m][k]``: weight rows ``n`` read plane ``min(n // plane_rows, planes - 1)``."""
+        n, k = w.shape
+        if self.f32 or m > L.GEMV_ROWS:
+            out, last = sc.get(name, m, n, torch.float32), x.shape[0] - 1
+            for i in range(x.shape[0]):
+                lo, hi = i * plane_rows, n if i == last else (i + 1) * plane_rows
+                if self.f32:
+                    L.linear_f32(x[i], w[lo:hi], out[:, lo:hi], m)
+                else:
+                    G.gemm_bf16(x[i], w[lo:hi], out[:, lo:hi], epi=G.EPI_F32)
+            return out, 1
+        s = self.splits(n, k)
+        out = sc.get(name, m * s, n, torch.float32, mult=s)
+        L.gemv_bf16_planes(w, x, plane_rows, out, m, n, k, s)
+        return out, s
+
     def splits(self, n: int, k: int) -> int:
         s = self._splits.get((n, k))
         if s is None:
@@ -275,18 +356,18 @@ class ListedLayers:
 
     # ---------------------------------------------------------------- feed-forwards
     def dense(self, sc: ListedScratch, f: DenseFfn, w: DenseWeights, m: int):
-        """Gated feed-forward of the step's rows: fp32 slices of its down projection."""
+        """Gated feed-forward of the step's rows: fp32 slices of its down projection (without its bias)."""
         h = sc.get("h", m, self.wp)
         n = w.gate_up.shape[0]
         act = sc.get("ffn_act", m, n // 2)
         if self.f32:
             gu = sc.get("gate_up", m, n)
             L.linear_f32(h, w.gate_up, gu, m)
-            L.glu_rows_f32(gu, act, m, n, f.limit, f.alpha, f.shift)
+            L.glu_rows_f32(gu, act, m, n, f.limit, f.alpha, f.shift, f.gelu, w.bias)
         elif m <= L.GEMV_ROWS:
-            L.gemv_bf16_glu(w.gate_up, h, act, m, n, self.wp, f.limit, f.alpha, f.shift)
+            L.gemv_bf16_glu(w.gate_up, h, act, m, n, self.wp, f.limit, f.alpha, f.shift, f.gelu, w.bias)
         else:
-            G.gemm_glu(h, w.gate_up, act, f.limit, f.alpha, f.shift)
+            G.gemm_glu(h, w.gate_up, act, f.limit, f.alpha, f.shift, f.gelu, w.bias)
         return self.linear(sc, "ffn_down", w.down, act, m)
 
     def experts(self, sc: ListedScratch, f: ExpertFfn, w: ExpertStack, m: int):

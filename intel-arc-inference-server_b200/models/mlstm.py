@@ -45,21 +45,21 @@ class MlstmGeometry:
 
 def shapes(cfg: ModelConfig, p: str, a: MatrixLstm) -> dict:
     h, n = cfg.hidden, a.heads
-    return {p + "mix.q": (n * a.dim, h), p + "mix.k": (n * a.dim, h), p + "mix.v": (n * a.vdim, h), p + "mix.g": (n * a.vdim, h),
-            p + "mix.o": (h, n * a.vdim), p + "mix.norm": (n * a.vdim,), p + "mix.i": (n, h), p + "mix.i.b": (n,),
-            p + "mix.f": (n, h), p + "mix.f.b": (n,)}
+    return {p + "q": (n * a.dim, h), p + "k": (n * a.dim, h), p + "v": (n * a.vdim, h), p + "g": (n * a.vdim, h),
+            p + "o": (h, n * a.vdim), p + "norm": (n * a.vdim,), p + "i": (n, h), p + "i.b": (n,),
+            p + "f": (n, h), p + "f.b": (n,)}
 
 
 def assemble(t, p: str, a: MatrixLstm) -> MlstmWeights:
     """``t``: ``listed.Assembler``."""
     g, n = MlstmGeometry.of(a), a.heads
-    parts = [t.heads(t.t(p + "mix." + x), n, [(size, pad)], t.wp)
+    parts = [t.heads(t.t(p + "" + x), n, [(size, pad)], t.wp)
              for x, size, pad in (("q", a.dim, g.dk), ("k", a.dim, g.dk), ("v", a.vdim, g.dv), ("g", a.vdim, g.dv))]
-    gates = torch.cat([t.t(p + "mix.i"), t.t(p + "mix.f")])
+    gates = torch.cat([t.t(p + "i"), t.t(p + "f")])
     norm = torch.zeros(n, g.dv, dtype=torch.float32, device=t.device)
-    norm[:, : a.vdim] = t.vec(p + "mix.norm").view(n, a.vdim)
-    return MlstmWeights(torch.cat(parts + [t.padded(gates, pad64(2 * n), t.wp)]), torch.cat([t.vec(p + "mix.i.b"), t.vec(p + "mix.f.b")]),
-                        norm.view(-1), t.out_proj(p + "mix.o", n, a.vdim, g.dv))
+    norm[:, : a.vdim] = t.vec(p + "norm").view(n, a.vdim)
+    return MlstmWeights(torch.cat(parts + [t.padded(gates, pad64(2 * n), t.wp)]), torch.cat([t.vec(p + "i.b"), t.vec(p + "f.b")]),
+                        norm.view(-1), t.out_proj(p + "o", n, a.vdim, g.dv))
 
 
 def weight_elems(cfg: ModelConfig, a: MatrixLstm) -> int:
@@ -76,15 +76,15 @@ def page_planes(a: MatrixLstm) -> dict:
     return {}
 
 
-def state_shape(a: MatrixLstm) -> Optional[tuple]:
-    return (MlstmGeometry.of(a).state_elems,)
+def state_shapes(a: MatrixLstm) -> dict:
+    return {"mlstm": (MlstmGeometry.of(a).state_elems,)}
 
 
 class Mixer:
     def __init__(self, ll: ListedLayers, li: int, a: MatrixLstm, w: MlstmWeights):
         self.ll, self.li, self.a, self.w, self.g = ll, li, a, w, MlstmGeometry.of(a)
         chunks = ll.device.type == "cuda" and not ll.f32 and R.chunks_ok(self.g)
-        self.form = ("chunks",) if chunks else None
+        self.forms = [("chunks",)] if chunks else []
 
     def run(self, sc: ListedScratch, m: int, rows: StepRows, block_table, kv, plan: Optional[BatchPlan]):
         """The recurrence over the step's rows: fp32 slices of its output projection."""
@@ -92,12 +92,12 @@ class Mixer:
         state = kv.states[f"mlstm{self.li}"][0]
         h = sc.get("h", m, ll.wp)
         out = sc.get("mlstm_out", m, g.heads * g.dv)
-        n1 = m if plan is None or self.form is None else plan.n_single
+        n1 = m if plan is None or not self.forms else plan.n_single
         if n1:
             part, s = ll.linear(sc, "mlstm_in", w.proj, h, n1)
             R.step(part, s, n1, w.proj.shape[0], g, a, rows.req, rows.pos, w.gate_bias, eps, w.norm, state, out)
         if n1 < m:
-            t, n = plan.tables[self.form], m - n1
+            t, n = plan.tables[self.forms[0]], m - n1
             proj, z = sc.get("mlstm_rows", n, g.n), sc.get("mlstm_gates", n, g.gates, torch.float32)
             G.gemm_bf16(h[n1:], w.proj[: g.n], proj)
             G.gemm_bf16(h[n1:], w.proj[g.n: g.n + g.gates], z, epi=G.EPI_F32)

@@ -99,10 +99,15 @@ class LatentWeights:
 @dataclass
 class GroupedWeights:
     """A grouped-query attention mixer, unquantised, heads padded to whole 64s."""
-    qkv: torch.Tensor              # [heads * dk + kv_heads * (dk + dv)][Wp], or the queries' rows alone
-    o: torch.Tensor                # [Wp][heads * dv]
+    qkv: Optional[torch.Tensor]    # [heads * dk + kv_heads * (dk + dv)][Wp], or the queries' rows alone
+    o: Optional[torch.Tensor]      # [Wp][heads * dv]
     slope2: Optional[torch.Tensor]     # fp32 [heads] distance bias times log2 e
     sink2: Optional[torch.Tensor]      # fp32 [heads] sinks times log2 e
+    bias: Optional[torch.Tensor] = None      # fp32 [heads * dk + kv_heads * (dk + dv)]
+    q_norm: Optional[torch.Tensor] = None    # fp32 [dk]
+    k_norm: Optional[torch.Tensor] = None    # fp32 [dk]
+    r1: Optional[torch.Tensor] = None        # fp32 [heads] logarithmic distance bias
+    r2: Optional[torch.Tensor] = None
 
 
 @dataclass
@@ -115,10 +120,54 @@ class MlstmWeights:
 
 
 @dataclass
+class MinGruWeights:
+    """A minGRU mixer, unquantised, padded to whole 64s."""
+    proj: Optional[torch.Tensor]   # [3 * wp][Wp]: gate, candidate, output gate
+    o: Optional[torch.Tensor]      # [Wp][wp]
+    bias_z: torch.Tensor           # fp32 [wp]
+    bias_x: torch.Tensor           # fp32 [wp]
+
+
+@dataclass
+class ParallelWeights:
+    """Two mixers side by side: their input projections one below the other, their output projections side by side."""
+    proj: torch.Tensor
+    o: torch.Tensor
+    left: object                   # the two mixers' other weights
+    right: object
+
+
+@dataclass
+class DeltaWeights:
+    """A delta-rule mixer with a decay per key channel, unquantised, heads padded."""
+    proj: torch.Tensor             # [2 * kv_heads * dk + heads * dv + ...][Wp]: q, k, v, step sizes, first halves of decay and gate
+    conv: torch.Tensor             # fp32 [taps][2 * kv_heads * dk + heads * dv]
+    neg_a: torch.Tensor            # fp32 [heads]: exp(A_log)
+    dt_bias: torch.Tensor          # fp32 [heads * dk]
+    second: torch.Tensor           # [heads * (dk + dv)][kp] second halves of decay and gate; bf16: twice side by side, for two limbs
+    norm: torch.Tensor             # fp32 [heads * dv]
+    o: torch.Tensor                # [Wp][heads * dv]
+
+
+@dataclass
+class WkvWeights:
+    """A time-mixing (wkv) mixer, unquantised, heads padded."""
+    proj: torch.Tensor             # [4 * heads * d + ...][Wp]: r, k, v, gate, first half of the decay
+    shift: torch.Tensor            # fp32 [5][Wp]: how much of the previous token r, k, v, gate and decay read
+    u: torch.Tensor                # fp32 [heads * d]
+    w0: torch.Tensor               # fp32 [heads * d]
+    second: torch.Tensor           # [heads * d][kp], as in DeltaWeights
+    norm: torch.Tensor             # fp32 [heads * d]
+    o: torch.Tensor                # [Wp][heads * d]
+
+
+@dataclass
 class DenseWeights:
     """Unquantised gated feed-forward, padded to whole 64s."""
     gate_up: torch.Tensor          # [2 * ffp][Wp], interleave16
     down: torch.Tensor             # [Wp][ffp]
+    bias: Optional[torch.Tensor] = None          # fp32 [2 * ffp], interleave16
+    down_bias: Optional[torch.Tensor] = None     # fp32 [Wp]
 
 
 @dataclass
@@ -155,9 +204,9 @@ class LayerWeights:
     experts_gate_up_w4b: Optional[torch.Tensor] = None
     experts_down_w4b: Optional[torch.Tensor] = None
     gdn: Optional[GdnWeights] = None               # set instead of qkv / o on gated delta-net layers
-    # listed layers: the norms then belong to the mixer's and the feed-forward's OUTPUT (one residual stream), or are
-    # single numbers for what they read (``streams`` set)
-    mixer: object = None                           # LatentWeights, GroupedWeights or MlstmWeights
+    # listed layers: the norms then belong to the mixer's and the feed-forward's OUTPUT, or (``ModelConfig.block``) to what
+    # they read: single numbers or a factor per column
+    mixer: object = None                           # the weights of the mixer's kind
     moe: Optional[ExpertStack] = None
     dense: Optional[DenseWeights] = None
     streams: Optional[StreamWeights] = None
@@ -183,6 +232,7 @@ class ModelWeights:
     layers: List[LayerWeights]
     mtp: Optional[MtpWeights] = None
     lm_head_i8: Optional[tuple] = None    # (int8 [vocab][hidden], fp32 [vocab]) when the int8 head is on
+    loop_step: Optional[torch.Tensor] = None    # fp32 [passes][Wp]: added before every pass of a looped range of layers
 
     def nbytes(self) -> int:
         tot = self.embed.numel() * 2 + self.lm_head.numel() * 2
@@ -198,8 +248,13 @@ class ModelWeights:
                 tot += lw.shared.gate_up.nbytes + lw.shared.down.nbytes
             for part in (lw.mixer, lw.moe, lw.dense):
                 if part is not None:
-                    tot += sum(t.numel() * t.element_size() for t in vars(part).values() if t is not None)
+                    tot += part_nbytes(part)
         return tot
+
+
+def part_nbytes(part) -> int:
+    """Bytes of a container of tensors and containers."""
+    return sum(t.numel() * t.element_size() if isinstance(t, torch.Tensor) else part_nbytes(t) for t in vars(part).values() if t is not None)
 
 
 def _norm_weight(h, device, gen=None):

@@ -1,7 +1,7 @@
 // Causal flash attention for prompt chunks on tcgen05 / TMEM: over the paged KV cache (head_dim 128), over contiguous
 // key / value rows with their own head sizes (latent attention, whose keys and values are expanded before), and over
 // paged keys and values of any sizes for the segments of a mixed batch (tiles that name their sequence; optional distance
-// bias, sink and chunked mask, as in paged.cu).
+// bias (linear or logarithmic), sink and chunked mask, as in paged.cu).
 //
 //   O[r] = softmax( q[r] . K[0 .. pos(r)]^T / sqrt(D) ) V[0 .. pos(r)]      pos(r) = pos0 + r
 //
@@ -41,6 +41,9 @@ struct AttnPfParams {
   int chunk;           // paged segments, > 0: a row sees the keys of its own chunk of this many positions only
   const float* slope2; // [n_q] distance bias per head, and sink2 [n_q], both times log2 e, or null
   const float* sink2;
+  const float *r1, *r2;  // [n_q] logarithmic distance bias (powers of two: r1 log2(1 + r2 distance)), or null
+  int ldo;             // paged segments: elements of an output row
+  float mult;          // paged segments: factor of the result
   int dn;              // columns of a head in the key matrix (a multiple of 64; the shared part fills up the head)
 };
 constexpr int kTileWords = 4;
@@ -339,7 +342,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
     const int first_pos = pos0 + row0 + w * BQ;             // position of the tile's first row
     const int last_lo = !F::SEG || p.chunk <= 0 ? 0 : first_pos + BQ - 1 - (first_pos + BQ - 1) % p.chunk;   // first key of its last row
-    const float slope = F::SEG && p.slope2 ? p.slope2[head] : 0.f;
+    const float slope = !F::SEG ? 0.f : p.r1 ? p.r1[head] : p.slope2 ? p.slope2[head] : 0.f, r2 = F::SEG && p.r1 ? p.r2[head] : 0.f;
     const int nt = n_w[w];
     // float [tile w][tile parity][half][128 rows]: the halves of a row exchange their maxima (and, at the end, sums)
     const uint32_t xch = bars + 256 + (uint32_t)w * (2 * 2 * 128 * 4);
@@ -367,6 +370,12 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         unsigned long long sc2, sl2, d2;
         const float d0 = (float)(key0 - qpos);
         asm("mov.b64 %0, {%1, %1};" : "=l"(sc2) : "f"(p.scale_log2));
+        if (p.r1) {                // keys past the row give NaN here and are masked below
+          const float far = fmaf(-r2, d0, 1.f);
+#pragma unroll
+          for (int j = 0; j < 32; ++j)
+            v[j] = __float_as_uint(fmaf(__uint_as_float(v[j]), p.scale_log2, -slope * __log2f(fmaf(-r2, (float)j, far))));
+        } else {
         asm("mov.b64 %0, {%1, %1};" : "=l"(sl2) : "f"(slope));
 #pragma unroll
         for (int j = 0; j < 16; ++j) {
@@ -376,6 +385,7 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
           asm("mul.rn.f32x2 %0, %0, %1;" : "+l"(d2) : "l"(sl2));
           asm("fma.rn.f32x2 %0, %0, %1, %2;" : "+l"(xy) : "l"(sc2), "l"(d2));
           asm("mov.b64 {%0, %1}, %2;" : "=r"(v[2 * j]), "=r"(v[2 * j + 1]) : "l"(xy));
+        }
         }
       }
       if (key0 + 31 > first_pos || (F::SEG ? key0 < last_lo : p.window > 0 && key0 < first_pos + BQ - p.window)) {
@@ -493,8 +503,8 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     if (ok && nt > 0) ok = mbar_wait(b_odone(w, (nt - 1) & 1), ((nt - 1) >> 1) & 1, ERR_ATTN_WAIT);
     if (ok && nt > 0) {
       tc_fence_after();
-      const float inv = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* dst = p.out + (size_t)(qrow + rowg) * (p.n_q * F::DV) + head * F::DV;
+      const float inv = l > 0.f ? (F::SEG ? p.mult : 1.f) / l : 0.f;
+      __nv_bfloat16* dst = p.out + (size_t)(qrow + rowg) * (F::SEG ? p.ldo : p.n_q * F::DV) + head * F::DV;
 #pragma unroll 1
       for (int c = NDV * half; c < NDV * half + NDV; ++c) {
         uint32_t o[32];
@@ -657,13 +667,16 @@ static int launch_segments(const CUtensorMap& mq, const CUtensorMap& mk, const C
 }
 
 // q: bf16 rows of ldq elements (the first H * dk of each are the queries); k / v caches [num_pages][G][16][dk | dv];
-// block_table [slots][max_blocks]; out [q_rows][H * dv].  tiles: n_tiles x 4 ints: first row of q, rows, position of that
+// block_table [slots][max_blocks]; out: rows of ldo elements, H * dv of them written.  tiles: n_tiles x 4 ints: first row of q, rows, position of that
 // row, slot.
 extern "C" int b2_attn_prefill_segments(const void* q, int ldq, const void* k_cache, const void* v_cache,
                                         const int* block_table, int max_blocks, void* out, const int* tiles, int n_tiles,
                                         int q_rows, int H, int G, int dk, int dv, int num_pages, float scale, int chunk,
-                                        const float* slope2, const float* sink2, void* stream) {
-  if (!b2_attn_segments_per_tile(dk, dv) || n_tiles < 1 || H < 1 || H % G || ldq % 8 || ldq < H * dk || chunk < 0) return -1;
+                                        const float* slope2, const float* sink2, const float* r1, const float* r2, int ldo,
+                                        float mult, void* stream) {
+  if (!b2_attn_segments_per_tile(dk, dv) || n_tiles < 1 || H < 1 || H % G || ldq % 8 || ldq < H * dk || chunk < 0 || ldo % 8 || ldo < H * dv ||
+      (r1 && !r2))
+    return -1;
   CUtensorMap mq, mk, mv;
   int rc = make_map_bf16(&mq, q, (uint64_t)q_rows, (uint64_t)H * dk, BQ, (uint64_t)ldq);
   if (!rc) rc = make_map_bf16(&mk, k_cache, (uint64_t)num_pages * G * 16, (uint64_t)dk, 16);
@@ -672,6 +685,7 @@ extern "C" int b2_attn_prefill_segments(const void* q, int ldq, const void* k_ca
   AttnPfParams p = {};
   p.block_table = block_table; p.max_blocks = max_blocks; p.n_q = H; p.n_kv = G; p.scale_log2 = scale * 1.4426950408889634f;
   p.out = (__nv_bfloat16*)out; p.tiles = tiles; p.chunk = chunk; p.slope2 = slope2; p.sink2 = sink2;
+  p.r1 = r1; p.r2 = r2; p.ldo = ldo; p.mult = mult;
   cudaStream_t st = (cudaStream_t)stream;
   switch (dk / 64) {
     case 1: return launch_segments<1>(mq, mk, mv, p, dv / 64, n_tiles, st);

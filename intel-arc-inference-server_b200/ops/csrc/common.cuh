@@ -273,14 +273,19 @@ __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + __expf(-x)); }
-// Gated product of two projections: g' sigmoid(alpha g') (u' + shift) with g' = min(g, limit), u' = clamp(u, -limit, limit)
+// Gated product of two projections: f(g') (u' + shift) with g' = min(g, limit), u' = clamp(u, -limit, limit);
+// f(x) = x sigmoid(alpha x), or with gelu 1 the tanh form of GELU: x (1 + tanh(y)) / 2 = x / (1 + e^(-2 y)) with
+// y = sqrt(2 / pi) (x + 0.044715 x^3).  bias: fp32, added to the projections' (interleave16) columns first, or null.
 struct Glu {
   float limit, alpha, shift;
+  int gelu;
+  const float* bias;
 };
+__device__ __forceinline__ float gelu_arg(float g) { return 1.5957691216057308f * fmaf(0.044715f * g * g, g, g); }
 __device__ __forceinline__ float glu(const Glu& p, float g, float u) {
   g = fminf(g, p.limit);
   u = fminf(fmaxf(u, -p.limit), p.limit);
-  return g / (1.0f + __expf(-p.alpha * g)) * (u + p.shift);
+  return g / (1.0f + __expf(p.gelu ? -gelu_arg(g) : -p.alpha * g)) * (u + p.shift);
 }
 
 __device__ __forceinline__ float warp_sum(float v) {

@@ -385,6 +385,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
             // columns alternate 16 gate, 16 up: 16 outputs per 32 accumulator columns
             __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.C) + (size_t)grow * p.ldc + (n0 >> 1);
             uint32_t o[8];
+            if (p.epi == EPI_GLU && p.glu.bias) {
+#pragma unroll
+              for (int j = 0; j < 8; ++j) {
+                const float4 b = __ldg(reinterpret_cast<const float4*>(p.glu.bias + n0) + j);
+                f[4 * j] += b.x; f[4 * j + 1] += b.y; f[4 * j + 2] += b.z; f[4 * j + 3] += b.w;
+              }
+            }
 #pragma unroll
             for (int j = 0; j < 8; ++j)
               o[j] = p.epi == EPI_GLU ? pack_bf16(glu(p.glu, f[2 * j], f[16 + 2 * j]), glu(p.glu, f[2 * j + 1], f[17 + 2 * j]))
@@ -669,9 +676,9 @@ extern "C" int b2_gemm_tc(const void* a, const void* b, void* c, int M, int N, i
 
 // bf16 C [M][N / 2] = gated product of the interleave16 columns of A * B^T (common.cuh, Glu)
 extern "C" int b2_gemm_tc_glu(const void* a, const void* b, void* c, int M, int N, int K, int ldc, float limit, float alpha,
-                              float shift, void* stream) {
+                              float shift, int gelu, const float* bias, void* stream) {
   return gemm_tc_impl(a, b, c, M, N, K, ldc, 0, EPI_GLU, nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, 0, 1, 0,
-                      nullptr, 0, 1, 1, nullptr, 0, nullptr, nullptr, nullptr, stream, Glu{limit, alpha, shift});
+                      nullptr, 0, 1, 1, nullptr, 0, nullptr, nullptr, nullptr, stream, Glu{limit, alpha, shift, gelu, bias});
 }
 
 // Tensor-parallel forms of the same kernel.  epi = 4 (row-parallel GEMM -> reduce-scatter): c is unused, the

@@ -28,6 +28,8 @@ struct GemvBfParams {
   const __nv_bfloat16* x;    // [rows][ldx]
   void* out;
   int M, N, K, ldx, splits, epi, x_div;
+  int plane_rows, planes;    // planes > 1: weight rows n read activations of plane min(n / plane_rows, planes - 1),
+  long long plane;           // planes this many elements apart
   Glu glu;                   // EPI_GLU
 };
 
@@ -57,9 +59,10 @@ __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const GemvBfPara
   const __nv_bfloat16* wp[NG];
 #pragma unroll
   for (int i = 0; i < NG; ++i) wp[i] = w + (size_t)min(n0 + 8 * i + g, p.N - 1) * p.K + t * 8;
+  const __nv_bfloat16* x = p.x + (p.planes > 1 ? min(n0 / p.plane_rows, p.planes - 1) * p.plane : 0);
   const __nv_bfloat16* xr[MH];
 #pragma unroll
-  for (int h = 0; h < MH; ++h) xr[h] = p.x + (size_t)(row_x + min(8 * h + g, M - 1)) * p.ldx + t * 8;
+  for (int h = 0; h < MH; ++h) xr[h] = x + (size_t)(row_x + min(8 * h + g, M - 1)) * p.ldx + t * 8;
   constexpr int SB = stage_bytes<MH>();
   unsigned char* ring = ring_smem + warp * kStages * SB + lane * 16;
   const uint32_t ring_s = smem_u32(ring);
@@ -130,6 +133,10 @@ __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const GemvBfPara
         gt += red[(q * 16 + m) * 33 + c];
         up += red[(q * 16 + m) * 33 + 16 + c];
       }
+      if (p.epi == EPI_GLU && p.glu.bias) {
+        gt += p.glu.bias[n0 + c];
+        up += p.glu.bias[n0 + 16 + c];
+      }
       if (n0 + 16 + c < p.N)
         reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)(batched ? batch : m) * (p.N / 2) + n0 / 2 + c] = __float2bfloat16(p.epi == EPI_GLU ? glu(p.glu, gt, up) : silu(gt) * up);
     }
@@ -153,7 +160,7 @@ __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const GemvBfPara
 // ------------------------------------------------------------------ 32-bit linears
 // 64 x 64 tile, 256 threads, 4 x 4 outputs per thread, K in steps of 16
 __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict__ a, const float* __restrict__ b,
-                                                         float* __restrict__ c, int M, int N, int K) {
+                                                         float* __restrict__ c, int M, int N, int K, int ldc) {
   __shared__ float as[16][68], bs[16][68];
   pdl_wait();
   pdl_launch_dependents();
@@ -184,7 +191,7 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict
   for (int i = 0; i < 4; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j)
-      if (m0 + ty * 4 + i < M && n0 + tx * 4 + j < N) c[(size_t)(m0 + ty * 4 + i) * N + n0 + tx * 4 + j] = acc[i][j];
+      if (m0 + ty * 4 + i < M && n0 + tx * 4 + j < N) c[(size_t)(m0 + ty * 4 + i) * ldc + n0 + tx * 4 + j] = acc[i][j];
 }
 
 // batch b: out[b][n] = x[b / x_div] . w[ids[b]][n]; one warp per output.  silu: w rows interleave16, out [b][N / 2]
@@ -215,8 +222,14 @@ __global__ void __launch_bounds__(256) glu_rows_f32_kernel(const float* __restri
   const int o = blockIdx.x * 256 + threadIdx.x;
   if (o >= N / 2) return;
   const float* r = in + (size_t)blockIdx.y * N + (o >> 4) * 32 + (o & 15);
-  const float g = fminf(r[0], p.limit), u = fminf(fmaxf(r[16], -p.limit), p.limit);
-  out[(size_t)blockIdx.y * (N / 2) + o] = g / (1.f + expf(-p.alpha * g)) * (u + p.shift);
+  float g = r[0], u = r[16];
+  if (p.bias) {
+    g += p.bias[(o >> 4) * 32 + (o & 15)];
+    u += p.bias[(o >> 4) * 32 + (o & 15) + 16];
+  }
+  g = fminf(g, p.limit);
+  u = fminf(fmaxf(u, -p.limit), p.limit);
+  out[(size_t)blockIdx.y * (N / 2) + o] = g / (1.f + expf(p.gelu ? -gelu_arg(g) : -p.alpha * g)) * (u + p.shift);
 }
 
 int sm_count() {
@@ -262,30 +275,41 @@ extern "C" int b2_gemv_bf16(const void* w, const int* ids, int batches, const vo
   if (K % 64 || N < 1 || M < 1 || M > 16 || splits < 1 || ldx % 8 || (epi != EPI_PART && splits != 1)) return -1;
   if (epi == EPI_SILU && N % 32) return -2;
   if (ids && (M != 1 || x_div < 1)) return -3;
-  GemvBfParams p{(const __nv_bfloat16*)w, ids, (const __nv_bfloat16*)x, out, M, N, K, ldx, splits, epi, x_div, {}};
+  GemvBfParams p{(const __nv_bfloat16*)w, ids, (const __nv_bfloat16*)x, out, M, N, K, ldx, splits, epi, x_div, 0, 1, 0, {}};
   return M <= 8 ? launch_gemv<1>(p, ids ? batches : 1, (cudaStream_t)stream)
                 : launch_gemv<2>(p, ids ? batches : 1, (cudaStream_t)stream);
 }
 
-// bf16 out [M][N / 2] = gated product of the interleave16 columns of x W^T
+// epi 0 with activations in `planes` planes (`plane` elements apart) of M rows each: weight rows n read plane
+// min(n / plane_rows, planes - 1)
+extern "C" int b2_gemv_bf16_planes(const void* w, const void* x, int ldx, int plane_rows, int planes, long long plane, void* out, int M,
+                                   int N, int K, int splits, void* stream) {
+  if (K % 64 || N < 1 || M < 1 || M > 16 || splits < 1 || ldx % 8 || plane_rows % 32 || plane_rows < 32 || planes < 1 || plane % 8) return -1;
+  GemvBfParams p{(const __nv_bfloat16*)w, nullptr, (const __nv_bfloat16*)x, out, M, N, K, ldx, splits, EPI_PART, 1, plane_rows, planes, plane, {}};
+  return M <= 8 ? launch_gemv<1>(p, 1, (cudaStream_t)stream) : launch_gemv<2>(p, 1, (cudaStream_t)stream);
+}
+
+// bf16 out [M][N / 2] = gated product of the interleave16 columns of x W^T (common.cuh, Glu)
 extern "C" int b2_gemv_bf16_glu(const void* w, const void* x, int ldx, void* out, int M, int N, int K, float limit, float alpha,
-                                float shift, void* stream) {
+                                float shift, int gelu, const float* bias, void* stream) {
   if (K % 64 || N % 32 || M < 1 || M > 16 || ldx % 8) return -1;
-  GemvBfParams p{(const __nv_bfloat16*)w, nullptr, (const __nv_bfloat16*)x, out, M, N, K, ldx, 1, EPI_GLU, 1, {limit, alpha, shift}};
+  GemvBfParams p{(const __nv_bfloat16*)w, nullptr, (const __nv_bfloat16*)x, out, M, N, K, ldx, 1, EPI_GLU, 1, 0, 1, 0,
+                 {limit, alpha, shift, gelu, bias}};
   return M <= 8 ? launch_gemv<1>(p, 1, (cudaStream_t)stream) : launch_gemv<2>(p, 1, (cudaStream_t)stream);
 }
 
 // in fp32 [M][N] interleave16 -> out [M][N / 2]
-extern "C" int b2_glu_rows_f32(const float* in, float* out, int M, int N, float limit, float alpha, float shift, void* stream) {
+extern "C" int b2_glu_rows_f32(const float* in, float* out, int M, int N, float limit, float alpha, float shift, int gelu,
+                               const float* bias, void* stream) {
   if (M < 1 || M > 65535 || N % 32) return -1;
   return b2_launch(glu_rows_f32_kernel, dim3((N / 2 + 255) / 256, M), dim3(256), 0, (cudaStream_t)stream, true, in, out, N,
-                   Glu{limit, alpha, shift});
+                   Glu{limit, alpha, shift, gelu, bias});
 }
 
-extern "C" int b2_linear_f32(const float* a, const float* w, float* c, int M, int N, int K, void* stream) {
-  if (K % 16 || M < 1 || N < 1) return -1;
+extern "C" int b2_linear_f32(const float* a, const float* w, float* c, int M, int N, int K, int ldc, void* stream) {
+  if (K % 16 || M < 1 || N < 1 || ldc < N) return -1;
   return b2_launch(linear_f32_kernel, dim3((N + 63) / 64, (M + 63) / 64), dim3(256), 0, (cudaStream_t)stream, true, a, w, c,
-                   M, N, K);
+                   M, N, K, ldc);
 }
 
 extern "C" int b2_linear_f32_rows(const float* w, const int* ids, int batches, const float* x, int ldx, int x_div, float* out,

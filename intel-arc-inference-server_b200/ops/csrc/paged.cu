@@ -3,13 +3,15 @@
 //
 //   kv_append_kernel    folds the projection's slices (or reads bf16 GEMM rows), stores keys and values at their positions
 //                       and the queries as rows
+//   kv_norm_kernel      the same for heads with biases, norms and a query temperature, a warp per (row, head)
 //   paged_rows_kernel   split-KV attention of single rows (mma.m16n8k16): a CTA serves up to 16 query heads of one KV head
 //                       and one row; its four warps take the pages in turn, each with a cp.async ring and an online
 //                       softmax of its own, and meet in shared memory
 //   paged_merge_kernel  merge of the splits
 //   paged_simple_kernel the same in plain fp32 arithmetic for either element type
 //
-// What a score may carry besides (q . k) scale, each optional: a distance bias -slope_h (i - j); a chunk size, with which a
+// What a score may carry besides (q . k) scale, each optional: a distance bias -slope_h (i - j), or a logarithmic one
+// -r1_h ln(1 + r2_h (i - j)); a chunk size, with which a
 // position sees the keys of its own chunk only (chunks counted from position 0); a sink per head, one more term of the
 // softmax's denominator that has no key.  Scores, weights and sums are fp32; the weights enter their product as two bf16
 // limbs.
@@ -87,6 +89,87 @@ __global__ void __launch_bounds__(128) kv_append_rows_kernel(const AppendParams 
   }
 }
 
+// ------------------------------------------------------------------ heads with biases, norms and a query temperature
+struct NormParams {
+  const float* part;       // [slices][M][N]; columns: queries [H dk] | keys [G dk] | values [G dv] | others
+  int slices, M, N, H, G, dk, dv, dim, vdim;
+  const float* bias;       // [H dk + G dk + G dv], or null
+  const float *q_norm, *k_norm;    // [dk] factors after the division by the root mean square, or null: no such norm
+  int v_norm;              // values are divided by their root mean square
+  float eps, temp;         // queries times 1 + temp ln(floor((p + 1) / every) + 1)
+  int every;
+  const int *req, *pos, *block_table;
+  int max_blocks;
+  void *q, *k, *v;         // q [M][H dk]
+};
+
+// NQ: quads of columns per lane
+template <int NQ, typename T>
+__global__ void __launch_bounds__(128) kv_norm_kernel(const NormParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int m = blockIdx.x, head = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (head >= p.H + 2 * p.G) return;
+  const bool is_q = head < p.H, is_v = head >= p.H + p.G;
+  const int d = is_v ? p.dv : p.dk;
+  const int col = is_v ? (p.H + p.G) * p.dk + (head - p.H - p.G) * p.dv : head * p.dk;
+  const long long slice = (long long)p.M * p.N;
+  const float* src = p.part + (size_t)m * p.N + col;
+  float4 x[NQ];
+  float ssq = 0.f;
+#pragma unroll
+  for (int u = 0; u < NQ; ++u) {
+    const int c = (u * 32 + lane) * 4;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b[8];
+    if (c < d) {
+#pragma unroll
+      for (int s = 0; s < 8; ++s) b[s] = s < p.slices ? __ldcg(reinterpret_cast<const float4*>(src + s * slice + c)) : a;
+#pragma unroll
+      for (int s = 0; s < 8; ++s) { a.x += b[s].x; a.y += b[s].y; a.z += b[s].z; a.w += b[s].w; }
+      if (p.bias) {
+        const float4 w = *reinterpret_cast<const float4*>(p.bias + col + c);
+        a.x += w.x; a.y += w.y; a.z += w.z; a.w += w.w;
+      }
+    }
+    x[u] = a;
+    ssq += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;      // padding columns are zero
+  }
+  const float* w = is_v ? nullptr : is_q ? p.q_norm : p.k_norm;
+  float r = 1.f;
+  if (w || (is_v && p.v_norm)) r = 1.f / sqrtf(warp_sum(ssq) / (float)(is_v ? p.vdim : p.dim) + p.eps);
+  const int pos = p.pos[m];
+  if (is_q && p.temp != 0.f) r *= 1.f + p.temp * logf((float)((pos + 1) / p.every) + 1.f);
+  T* dst;
+  if (is_q) {
+    dst = reinterpret_cast<T*>(p.q) + (size_t)m * p.H * p.dk + col;
+  } else {
+    const int page = p.block_table[(size_t)p.req[m] * p.max_blocks + (pos >> 4)];
+    const int h = head - p.H - (is_v ? p.G : 0);
+    dst = reinterpret_cast<T*>(is_v ? p.v : p.k) + (((size_t)page * p.G + h) * 16 + (pos & 15)) * d;
+  }
+#pragma unroll
+  for (int u = 0; u < NQ; ++u) {
+    const int c = (u * 32 + lane) * 4;
+    if (c >= d) continue;
+    float4 f = make_float4(r, r, r, r);
+    if (w) {
+      const float4 g = *reinterpret_cast<const float4*>(w + c);
+      f = make_float4(r * g.x, r * g.y, r * g.z, r * g.w);
+    }
+    store4(dst + c, make_float4(x[u].x * f.x, x[u].y * f.y, x[u].z * f.z, x[u].w * f.w));
+  }
+}
+
+template <typename T>
+int launch_norm(const NormParams& p, cudaStream_t st) {
+  const dim3 grid(p.M, (p.H + 2 * p.G + 3) / 4);
+  const int quads = ((p.dk > p.dv ? p.dk : p.dv) + 127) / 128;
+  if (quads <= 1) return b2_launch(kv_norm_kernel<1, T>, grid, dim3(128), 0, st, true, p);
+  if (quads <= 2) return b2_launch(kv_norm_kernel<2, T>, grid, dim3(128), 0, st, true, p);
+  if (quads <= 4) return b2_launch(kv_norm_kernel<4, T>, grid, dim3(128), 0, st, true, p);
+  return b2_launch(kv_norm_kernel<8, T>, grid, dim3(128), 0, st, true, p);
+}
+
 // ------------------------------------------------------------------ attention of single rows (tensor cores)
 struct RowsParams {
   const __nv_bfloat16 *q, *k, *v;    // q: rows of ldq elements, the first H dk of each
@@ -94,8 +177,11 @@ struct RowsParams {
   int ldq, max_blocks, H, G, nsplit, chunk;
   float scale_log2;
   const float *slope2, *sink2;       // [H] times log2 e, or null
+  const float *r1, *r2;              // [H] logarithmic distance bias (in powers of two: r1 log2(1 + r2 distance)), or null
   float *o_part, *ml_part;           // [M][H][nsplit][dv], [M][H][nsplit][2]
-  __nv_bfloat16* out;                // [M][H][dv], written when nsplit is 1
+  __nv_bfloat16* out;                // rows of ldo elements [H][dv], written when nsplit is 1
+  int ldo;
+  float mult;                        // factor of the result
 };
 
 constexpr int kWarps = 4;
@@ -170,10 +256,14 @@ __global__ void __launch_bounds__(kWarps * 32) paged_rows_kernel(const RowsParam
       const int r = g + 8 * (e & 1), c = k * 16 + 2 * t + 8 * (e >> 1);
       qa[k][e] = r < nr ? *reinterpret_cast<const uint32_t*>(p.q + (size_t)m * p.ldq + (h0 + r) * dk + c) : 0u;
     }
-  float slope[2] = {0.f, 0.f};
-  if (p.slope2) {
+  float slope[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};      // slope: r1 of a logarithmic bias
+  if (p.slope2 || p.r1) {
 #pragma unroll
-    for (int hf = 0; hf < 2; ++hf) slope[hf] = p.slope2[h0 + min(g + 8 * hf, nr - 1)];
+    for (int hf = 0; hf < 2; ++hf) {
+      const int hd = h0 + min(g + 8 * hf, nr - 1);
+      slope[hf] = p.r1 ? p.r1[hd] : p.slope2[hd];
+      if (p.r1) r2[hf] = p.r2[hd];
+    }
   }
   float o[NDV * 8][4];
 #pragma unroll
@@ -205,7 +295,9 @@ __global__ void __launch_bounds__(kWarps * 32) paged_rows_kernel(const RowsParam
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int key = key0 + 8 * j + 2 * t + (e & 1);
-        const float v = fmaf(slope[e >> 1], (float)(key - pos), (s[0][j][e] + s[1][j][e]) * p.scale_log2);
+        float away = (float)(key - pos);
+        if (p.r1) away = -__log2f(fmaf(-r2[e >> 1], fminf(away, 0.f), 1.f));
+        const float v = fmaf(slope[e >> 1], away, (s[0][j][e] + s[1][j][e]) * p.scale_log2);
         x[j][e] = key >= lo && key <= pos ? v : -INFINITY;
         top[e >> 1] = fmaxf(top[e >> 1], x[j][e]);
       }
@@ -279,8 +371,8 @@ __global__ void __launch_bounds__(kWarps * 32) paged_rows_kernel(const RowsParam
       a.x = fmaf(e, v.x, a.x); a.y = fmaf(e, v.y, a.y); a.z = fmaf(e, v.z, a.z); a.w = fmaf(e, v.w, a.w);
     }
     if (p.nsplit == 1) {
-      const float inv = 1.f / (sum + (p.sink2 ? exp2f(p.sink2[h0 + r] - top) : 0.f));
-      store4(p.out + ((size_t)m * p.H + h0 + r) * dv + c, make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv));
+      const float inv = p.mult / (sum + (p.sink2 ? exp2f(p.sink2[h0 + r] - top) : 0.f));
+      store4(p.out + (size_t)m * p.ldo + (h0 + r) * dv + c, make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv));
     } else {
       const size_t row = ((size_t)m * p.H + h0 + r) * p.nsplit + split;
       *reinterpret_cast<float4*>(p.o_part + row * dv + c) = a;
@@ -298,6 +390,8 @@ struct MergeParams {
   int H, nsplit, dv;
   const float* sink2;
   __nv_bfloat16* out;
+  int ldo;
+  float mult;
 };
 
 __global__ void __launch_bounds__(128) paged_merge_kernel(const MergeParams p) {
@@ -323,7 +417,7 @@ __global__ void __launch_bounds__(128) paged_merge_kernel(const MergeParams p) {
       e[i] = mx[i] == -INFINITY ? 0.f : exp2f(mx[i] - top);
       sum += e[i] * l[i];
     }
-    const float inv = 1.f / (warp_sum(sum) + (p.sink2 ? exp2f(p.sink2[h] - top) : 0.f));
+    const float inv = p.mult / (warp_sum(sum) + (p.sink2 ? exp2f(p.sink2[h] - top) : 0.f));
     wt[tid] = e[0] * inv;
     wt[tid + 32] = e[1] * inv;
   }
@@ -355,7 +449,7 @@ __global__ void __launch_bounds__(128) paged_merge_kernel(const MergeParams p) {
       const float4 b = red[tid + i * quads];
       a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w;
     }
-    store4(p.out + row * p.dv + c, a);
+    store4(p.out + (row / p.H) * p.ldo + h * p.dv + c, a);
   }
 }
 
@@ -365,8 +459,10 @@ struct SimpleParams {
   const int *req, *pos, *block_table;
   int ldq, max_blocks, H, G, dk, dv, chunk;
   float scale;
-  const float *slope2, *sink2;
-  void* out;                   // [M][H][dv]
+  const float *slope2, *sink2, *r1, *r2;
+  void* out;                   // rows of ldo elements [H][dv]
+  int ldo;
+  float mult;
 };
 constexpr int kSimpleDims = 16;    // value dims per thread: dv <= 2048
 constexpr float kLn2 = 0.6931471805599453f;
@@ -381,7 +477,7 @@ __global__ void __launch_bounds__(128) paged_simple_kernel(const SimpleParams p)
   const int m = blockIdx.x, h = blockIdx.y, kh = h / (p.H / p.G), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int pos = p.pos[m];
   const int* bt = p.block_table + (size_t)p.req[m] * p.max_blocks;
-  const float slope = p.slope2 ? p.slope2[h] * kLn2 : 0.f;
+  const float slope = p.slope2 ? p.slope2[h] * kLn2 : 0.f, r1 = p.r1 ? p.r1[h] : 0.f, r2 = p.r1 ? p.r2[h] : 0.f;
   for (int i = tid; i < p.dk; i += 128) qs[i] = to_f(reinterpret_cast<const T*>(p.q)[(size_t)m * p.ldq + h * p.dk + i]);
   float o[kSimpleDims];
 #pragma unroll
@@ -397,7 +493,8 @@ __global__ void __launch_bounds__(128) paged_simple_kernel(const SimpleParams p)
       float s = 0.f;
       for (int d = lane; d < p.dk; d += 32) s = fmaf(qs[d], to_f(c[d]), s);
       s = warp_sum(s);
-      if (lane == 0) sc[j] = s * p.scale - slope * (float)(pos - k0 - j);
+      const float away = (float)(pos - k0 - j);
+      if (lane == 0) sc[j] = s * p.scale - (p.r1 ? r1 * log1pf(r2 * away) : slope * away);
     }
     __syncthreads();
     float mn = mx;
@@ -419,7 +516,7 @@ __global__ void __launch_bounds__(128) paged_simple_kernel(const SimpleParams p)
   if (p.sink2) l += expf(p.sink2[h] * kLn2 - mx);
 #pragma unroll
   for (int i = 0; i < kSimpleDims; ++i)
-    if (tid + 128 * i < p.dv) reinterpret_cast<T*>(p.out)[((size_t)m * p.H + h) * p.dv + tid + 128 * i] = from_f<T>(o[i] / l);
+    if (tid + 128 * i < p.dv) reinterpret_cast<T*>(p.out)[(size_t)m * p.ldo + h * p.dv + tid + 128 * i] = from_f<T>(o[i] / l * p.mult);
 }
 
 template <int NDK, int NDV>
@@ -463,15 +560,31 @@ extern "C" int b2_kv_append(const void* part, int rows_form, int S, int M, int n
              : b2_launch(kv_append_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, true, p);
 }
 
+// Heads with biases, norms and a query temperature (see NormParams): fp32 slices [slices][M][N], whose first columns are
+// q | k | v, to query rows and pages.
+extern "C" int b2_kv_norm(const float* part, int slices, int M, int N, int H, int G, int dk, int dv, int dim, int vdim, const float* bias,
+                          const float* q_norm, const float* k_norm, int v_norm, float eps, float temp, int every, const int* req,
+                          const int* pos, const int* block_table, int max_blocks, void* q, void* k, void* v, int f32, void* stream) {
+  if (M < 1 || slices < 1 || slices > 8 || H < 1 || G < 1 || dk % 64 || dv % 64 || dk > 1024 || dv > 1024 || N % 4 ||
+      N < H * dk + G * (dk + dv) || every < 1 || dim < 1 || vdim < 1)
+    return -1;
+  NormParams p{part, slices, M, N, H, G, dk, dv, dim, vdim, bias, q_norm, k_norm, v_norm, eps, temp, every, req, pos, block_table,
+               max_blocks, q, k, v};
+  return f32 ? launch_norm<float>(p, (cudaStream_t)stream) : launch_norm<__nv_bfloat16>(p, (cudaStream_t)stream);
+}
+
 // 1 when the tensor-core row kernel covers the head sizes
 extern "C" int b2_paged_rows_ok(int dk, int dv) { return dk % 64 == 0 && dv % 64 == 0 && dk >= 64 && dv >= 64 && dk <= 256 && dv <= 256; }
 
 extern "C" int b2_paged_rows(const void* q, int ldq, const void* k, const void* v, int M, int H, int G, int dk, int dv, const int* req,
                              const int* pos, const int* block_table, int max_blocks, int nsplit, int chunk, float scale,
-                             const float* slope2, const float* sink2, float* o_part, float* ml_part, void* out, void* stream) {
-  if (M < 1 || H % G || nsplit < 1 || nsplit > 64 || !b2_paged_rows_ok(dk, dv) || chunk < 0 || ldq < H * dk || ldq % 2) return -1;
+                             const float* slope2, const float* sink2, const float* r1, const float* r2, float* o_part, float* ml_part,
+                             void* out, int ldo, float mult, void* stream) {
+  if (M < 1 || H % G || nsplit < 1 || nsplit > 64 || !b2_paged_rows_ok(dk, dv) || chunk < 0 || ldq < H * dk || ldq % 2 || ldo < H * dv ||
+      ldo % 4 || (r1 && !r2))
+    return -1;
   RowsParams p{(const __nv_bfloat16*)q, (const __nv_bfloat16*)k, (const __nv_bfloat16*)v, req, pos, block_table, ldq, max_blocks, H, G,
-               nsplit, chunk, scale * 1.4426950408889634f, slope2, sink2, o_part, ml_part, (__nv_bfloat16*)out};
+               nsplit, chunk, scale * 1.4426950408889634f, slope2, sink2, r1, r2, o_part, ml_part, (__nv_bfloat16*)out, ldo, mult};
   cudaStream_t st = (cudaStream_t)stream;
   int rc = -1;
   switch (dk / 64) {
@@ -481,15 +594,16 @@ extern "C" int b2_paged_rows(const void* q, int ldq, const void* k, const void* 
     case 4: rc = launch_rows_dv<4>(p, M, dv / 64, st); break;
   }
   if (rc || nsplit == 1) return rc;
-  MergeParams mp{o_part, ml_part, H, nsplit, dv, sink2, (__nv_bfloat16*)out};
+  MergeParams mp{o_part, ml_part, H, nsplit, dv, sink2, (__nv_bfloat16*)out, ldo, mult};
   return b2_launch(paged_merge_kernel, dim3(M * H), dim3(128), 0, st, true, mp);
 }
 
 extern "C" int b2_paged_simple(const void* q, int ldq, const void* k, const void* v, int M, int H, int G, int dk, int dv, const int* req,
                                const int* pos, const int* block_table, int max_blocks, int chunk, float scale,
-                               const float* slope2, const float* sink2, void* out, int f32, void* stream) {
-  if (M < 1 || H % G || H > 65535 || dv > 128 * kSimpleDims || dk > 8192 || chunk < 0) return -1;
-  SimpleParams p{q, k, v, req, pos, block_table, ldq, max_blocks, H, G, dk, dv, chunk, scale, slope2, sink2, out};
+                               const float* slope2, const float* sink2, const float* r1, const float* r2, void* out, int ldo, float mult,
+                               int f32, void* stream) {
+  if (M < 1 || H % G || H > 65535 || dv > 128 * kSimpleDims || dk > 8192 || chunk < 0 || ldo < H * dv || (r1 && !r2)) return -1;
+  SimpleParams p{q, k, v, req, pos, block_table, ldq, max_blocks, H, G, dk, dv, chunk, scale, slope2, sink2, r1, r2, out, ldo, mult};
   const size_t smem = (size_t)dk * 4;
   return f32 ? b2_launch(paged_simple_kernel<float>, dim3(M, H), dim3(128), smem, (cudaStream_t)stream, true, p)
              : b2_launch(paged_simple_kernel<__nv_bfloat16>, dim3(M, H), dim3(128), smem, (cudaStream_t)stream, true, p);

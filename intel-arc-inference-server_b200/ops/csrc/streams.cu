@@ -4,8 +4,12 @@
 //   u    = sum_t in[t] x'_t,  h = u / sqrt(mean(u^2) + eps) g     what the next sublayer reads (g: one number)
 //   h   <- h + (h_before - h) o mu                                optional token shift; h_before: the row before, unshifted
 //
-// y is what a linear left (split-K slices, folded here); everything is fp32, h is rounded at the end.  The first call of a
-// step has no y: all streams start as the embedding row plus a sinusoidal position vector.
+// y is what a linear left (split-K slices, folded here, plus its bias); everything is fp32, h is rounded at the end.  The
+// first call of a step has no y: all streams start as the embedding row plus a sinusoidal position vector.
+//
+// Options: a plain residual (no mix, in, out: one stream, x' = x + y); a norm with a factor per column; what comes before a
+// pass over a range of layers (the embedding row once more, a vector); several shifted results of one row at a time, each
+// with its own mu (a plane of h each).
 //
 // The streams are read from one buffer and written to another, because a row whose predecessor is in the same step
 // computes the predecessor's h again when it belongs to another CTA (a CTA walks `rows_per` rows and keeps the last h).
@@ -43,11 +47,16 @@ struct StreamParams {
   const float* scale;        // [ld] layer scale, or null
   float mult;
   const float* in;           // [S], null: the plain sum
-  const float* g;            // [1]
+  const float* g;            // [1], or [ld] with g_cols
+  int g_cols;
+  const float* bias;         // [ld] of the linear that left y, or null
+  const float* add;          // [ld] added to the streams, or null
+  int again;                 // the embedding row is added to the streams
   float eps;
   void* h;                   // [M][ld]
   int h_f32;
-  const float* mu;           // [ld], null: no shift
+  const float* mu;           // [planes][ld], null: no shift
+  int planes;                // h is [planes][M][ld]
   const float* prev;         // [slots][ld] state of the layer that reads h
   float* next;               // [slots][ld]
   float* commit;             // [slots][ld] state of the layer whose mixer made y, or null
@@ -98,11 +107,11 @@ __global__ void __launch_bounds__(kThreads) streams_kernel(const StreamParams p)
   __shared__ float red[kThreads / 32], stat, s_mix[S * S], s_out[S], s_in[S];
   const int tid = threadIdx.x;
   if (tid < S) {
-    s_out[tid] = p.y ? p.out[tid] * p.mult : 0.f;
+    s_out[tid] = p.y ? (p.out ? p.out[tid] : 1.f) * p.mult : 0.f;
     s_in[tid] = p.in ? p.in[tid] : 1.f;
   }
-  if (tid < S * S) s_mix[tid] = p.y ? p.mix[tid] : 0.f;
-  const float g = p.g[0];
+  if (tid < S * S) s_mix[tid] = !p.y ? 0.f : p.mix ? p.mix[tid] : tid % (S + 1) == 0 ? 1.f : 0.f;
+  const float g = p.g_cols ? 1.f : p.g[0];
   pdl_launch_dependents();
   pdl_wait();
   __syncthreads();
@@ -117,7 +126,7 @@ __global__ void __launch_bounds__(kThreads) streams_kernel(const StreamParams p)
   auto pass = [&](int m, bool store) -> float {
     float ssq = 0.f;
     int tok = 0, pos = 0;
-    if (!p.y) {
+    if (!p.y || p.again) {
       tok = p.tokens[m];
       pos = p.pos[m];
       if (tok < 0 || tok >= p.vocab) {
@@ -137,20 +146,26 @@ __global__ void __launch_bounds__(kThreads) streams_kernel(const StreamParams p)
         float4 y = b[0];
 #pragma unroll
         for (int s = 1; s < 8; ++s) y = fma4(1.f, b[s], y);
+        if (p.bias) y = fma4(1.f, *reinterpret_cast<const float4*>(p.bias + c), y);
         if (p.scale) {
           const float4 w = *reinterpret_cast<const float4*>(p.scale + c);
           y.x *= w.x; y.y *= w.y; y.z *= w.z; y.w *= w.w;
         }
+        float4 ahead = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (p.again) ahead = embedded(p, tok, pos, c);
+        if (p.add) ahead = fma4(1.f, *reinterpret_cast<const float4*>(p.add + c), ahead);
 #pragma unroll
         for (int t = 0; t < S; ++t) {
           float4 v = make_float4(s_out[t] * y.x, s_out[t] * y.y, s_out[t] * y.z, s_out[t] * y.w);
 #pragma unroll
           for (int s = 0; s < S; ++s) v = fma4(s_mix[s * S + t], x[s], v);
+          v = fma4(1.f, ahead, v);
           if (store && p.x_out) *reinterpret_cast<float4*>(p.x_out + ((size_t)m * S + t) * p.ld + c) = v;
           a = fma4(s_in[t], v, a);
         }
       } else {
-        const float4 v = embedded(p, tok, pos, c);
+        float4 v = embedded(p, tok, pos, c);
+        if (p.add) v = fma4(1.f, *reinterpret_cast<const float4*>(p.add + c), v);
 #pragma unroll
         for (int t = 0; t < S; ++t) {
           if (store && p.x_out) *reinterpret_cast<float4*>(p.x_out + ((size_t)m * S + t) * p.ld + c) = v;
@@ -183,7 +198,7 @@ __global__ void __launch_bounds__(kThreads) streams_kernel(const StreamParams p)
         const float r = pass(m - 1, false);
         for (int c = c0 + tid * 4; c < c1; c += kThreads * 4)
 #pragma unroll
-          for (int j = 0; j < 4; ++j) before[c + j] = u[c + j] * r;
+          for (int j = 0; j < 4; ++j) before[c + j] = u[c + j] * r * (p.g_cols ? p.g[c + j] : 1.f);
       }
     }
     const bool last = m + 1 == p.M || p.req[m + 1] != req;
@@ -194,18 +209,28 @@ __global__ void __launch_bounds__(kThreads) streams_kernel(const StreamParams p)
       if (p.commit && last) *reinterpret_cast<float4*>(p.commit + st) = __ldcg(reinterpret_cast<const float4*>(p.next + st));
       float4 h = *reinterpret_cast<const float4*>(u + c);
       h.x *= r; h.y *= r; h.z *= r; h.w *= r;
-      float4 o = h;
+      if (p.g_cols) {
+        const float4 w = *reinterpret_cast<const float4*>(p.g + c);
+        h.x *= w.x; h.y *= w.y; h.z *= w.z; h.w *= w.w;
+      }
+      auto store = [&](int plane, const float4& o) {
+        const size_t at = (((size_t)plane * p.M + m) * p.ld + c) / 4;
+        if (p.h_f32) reinterpret_cast<float4*>(p.h)[at] = o;
+        else reinterpret_cast<uint2*>(p.h)[at] = make_uint2(pack_bf16(o.x, o.y), pack_bf16(o.z, o.w));
+      };
       if (p.mu) {
         float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
         if (follows) b = *reinterpret_cast<const float4*>(before + c);
         else if (!first) b = __ldcg(reinterpret_cast<const float4*>(p.prev + st));
-        const float4 w = *reinterpret_cast<const float4*>(p.mu + c);
-        o = make_float4(fmaf(b.x - h.x, w.x, h.x), fmaf(b.y - h.y, w.y, h.y), fmaf(b.z - h.z, w.z, h.z), fmaf(b.w - h.w, w.w, h.w));
+        for (int i = 0; i < p.planes; ++i) {
+          const float4 w = *reinterpret_cast<const float4*>(p.mu + (size_t)i * p.ld + c);
+          store(i, make_float4(fmaf(b.x - h.x, w.x, h.x), fmaf(b.y - h.y, w.y, h.y), fmaf(b.z - h.z, w.z, h.z), fmaf(b.w - h.w, w.w, h.w)));
+        }
         *reinterpret_cast<float4*>(before + c) = h;
         if (last) *reinterpret_cast<float4*>(p.next + st) = h;
+      } else {
+        store(0, h);
       }
-      if (p.h_f32) reinterpret_cast<float4*>(p.h)[((size_t)m * p.ld + c) / 4] = o;
-      else reinterpret_cast<uint2*>(p.h)[((size_t)m * p.ld + c) / 4] = make_uint2(pack_bf16(o.x, o.y), pack_bf16(o.z, o.w));
     }
     have = m;
   }
@@ -254,12 +279,14 @@ int launch_streams(StreamParams& p, cudaStream_t st) {
 extern "C" int b2_streams(const float* y, long long slice, int slices, const void* embed, const int* tokens, const double* freq,
                           int vocab, int embed_f32, int* flag, const int* req, const int* pos, int M, int streams, int width,
                           int ld, const float* x_in, float* x_out, const float* mix, const float* out, const float* scale,
-                          float mult, const float* in, const float* g, float eps, void* h, int h_f32, const float* mu,
-                          const float* prev, float* next, float* commit, void* stream) {
+                          float mult, const float* in, const float* g, int g_cols, float eps, void* h, int h_f32, const float* mu,
+                          int planes, const float* prev, float* next, float* commit, const float* bias, const float* add, int again,
+                          void* stream) {
   if (M < 1 || ld % 4 || width > ld || slice % 4 || (y && (slices < 1 || slices > 8 || !x_in)) || (!y && !embed)) return -1;
-  if ((mu && (!prev || !next)) || (commit && !next)) return -2;
+  if ((mu && (!prev || !next || planes < 1)) || (commit && !next) || (again && (!embed || !tokens))) return -2;
+  if (y && streams > 1 && (!mix || !out)) return -4;
   StreamParams p{y, slice, slices, embed, tokens, freq, vocab, embed_f32, flag, req, pos, M, width, ld, 1, x_in, x_out, mix,
-                 out, scale, mult, in, g, eps, h, h_f32, mu, prev, next, commit};
+                 out, scale, mult, in, g, g_cols, bias, add, again, eps, h, h_f32, mu, planes, prev, next, commit};
   cudaStream_t st = (cudaStream_t)stream;
   switch (streams) {
     case 1: return launch_streams<1>(p, st);

@@ -31,12 +31,13 @@ def gemm_bf16(a: torch.Tensor, b: torch.Tensor, c: torch.Tensor, epi: int = EPI_
     _launch(a, b, c, m, n, k, c.stride(0), False, epi, resid=resid, bn=bn)
 
 
-def gemm_glu(a: torch.Tensor, b: torch.Tensor, c: torch.Tensor, limit: float, alpha: float, shift: float):
-    """``c`` ``[M][N/2]`` = g sigmoid(alpha g) (u + shift) over the interleave16 columns of ``a @ b.T``, with
-    g = min(gate, limit) and u = clamp(up, -limit, limit)."""
+def gemm_glu(a: torch.Tensor, b: torch.Tensor, c: torch.Tensor, limit: float, alpha: float, shift: float,
+             gelu: bool = False, bias=None):
+    """``c`` ``[M][N/2]`` = g sigmoid(alpha g) (u + shift) over the interleave16 columns of ``a @ b.T + bias``, with
+    g = min(gate, limit) and u = clamp(up, -limit, limit); ``gelu``: the tanh form of GELU in place of g sigmoid(alpha g)."""
     m, k = a.shape
     K._check(K.lib().b2_gemm_tc_glu(K._p(a), K._p(b), K._p(c), m, b.shape[0], k, c.stride(0), ctypes.c_float(limit),
-                                    ctypes.c_float(alpha), ctypes.c_float(shift), K._stream()), "gemm_tc_glu")
+                                    ctypes.c_float(alpha), ctypes.c_float(shift), int(gelu), K._p(bias), K._stream()), "gemm_tc_glu")
 
 
 def gemm_i8(a8, b8, a_scale, b_scale, c, epi: int = EPI_BF16, resid=None, bn: int = 0):

@@ -31,15 +31,22 @@ def gemv_bf16(w, x, out, m: int, n: int, k: int, splits: int = 1, epi: int = EPI
              "gemv_bf16")
 
 
-def gemv_bf16_glu(w, x, out, m: int, n: int, k: int, limit: float, alpha: float, shift: float):
+def gemv_bf16_planes(w, x, plane_rows: int, out, m: int, n: int, k: int, splits: int = 1):
+    """fp32 slices ``[splits][m][n]`` where rows ``n`` of the weight read plane ``min(n // plane_rows, planes - 1)`` of the
+    activations ``x`` ``[planes][m][k]``."""
+    K._check(K.lib().b2_gemv_bf16_planes(K._p(w), K._p(x), x.stride(1), plane_rows, x.shape[0], ctypes.c_longlong(x.stride(0)), K._p(out),
+                                         m, n, k, splits, K._stream()), "gemv_bf16_planes")
+
+
+def gemv_bf16_glu(w, x, out, m: int, n: int, k: int, limit: float, alpha: float, shift: float, gelu: bool = False, bias=None):
     """The gated product of ``gemm.gemm_glu`` for ``m`` <= 16 rows."""
     K._check(K.lib().b2_gemv_bf16_glu(K._p(w), K._p(x), x.stride(0), K._p(out), m, n, k, ctypes.c_float(limit), ctypes.c_float(alpha),
-                                      ctypes.c_float(shift), K._stream()), "gemv_bf16_glu")
+                                      ctypes.c_float(shift), int(gelu), K._p(bias), K._stream()), "gemv_bf16_glu")
 
 
-def glu_rows_f32(x, out, m: int, n: int, limit: float, alpha: float, shift: float):
+def glu_rows_f32(x, out, m: int, n: int, limit: float, alpha: float, shift: float, gelu: bool = False, bias=None):
     K._check(K.lib().b2_glu_rows_f32(K._p(x), K._p(out), m, n, ctypes.c_float(limit), ctypes.c_float(alpha), ctypes.c_float(shift),
-                                     K._stream()), "glu_rows_f32")
+                                     int(gelu), K._p(bias), K._stream()), "glu_rows_f32")
 
 
 def gemv_bf16_experts(w, ids, batches: int, x, x_div: int, out, n: int, k: int, splits: int = 1, epi: int = EPI_PART):
@@ -49,9 +56,9 @@ def gemv_bf16_experts(w, ids, batches: int, x, x_div: int, out, n: int, k: int, 
 
 
 def linear_f32(a, w, c, m: int):
-    """``c[:m] = a[:m] @ w.T`` in fp32."""
+    """``c[:m] = a[:m] @ w.T`` in fp32 (``c``: rows of any stride)."""
     n, k = w.shape
-    K._check(K.lib().b2_linear_f32(K._p(a), K._p(w), K._p(c), m, n, k, K._stream()), "linear_f32")
+    K._check(K.lib().b2_linear_f32(K._p(a), K._p(w), K._p(c), m, n, k, c.stride(0), K._stream()), "linear_f32")
 
 
 def linear_f32_experts(w, ids, batches: int, x, x_div: int, out, silu: bool):

@@ -2,7 +2,7 @@
 
 The decode step's control block holds 64 rows.  A batch here has a row table of its own (slot, position, token per row),
 uploaded with one copy together with everything else the kernels need: the wanted rows, and for every form of prompt
-segments the model's mixers use (``Mixer.form``) a table of its own.  Entries of fewer than ``SEGMENT`` tokens are handled
+segments the model's mixers use (``Mixer.forms``) a table of its own.  Entries of fewer than ``SEGMENT`` tokens are handled
 row by row, longer ones as prompt segments; both kinds share every linear and every expert of the step.  The walk itself is
 ``DecoderModel.listed_walk``, as in decode steps.
 

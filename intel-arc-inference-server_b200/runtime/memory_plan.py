@@ -67,7 +67,7 @@ def weight_bytes(cfg: ModelConfig, int8_head: bool = False, tp: int = 1, ep: int
 def kv_bytes_per_page(cfg: ModelConfig, kv_dtype: str, tp: int = 1) -> int:
     if cfg.layer_specs:
         from ..models.listed import kind
-        planes = [pl for s in cfg.layer_specs for pl in kind(s.mixer).page_planes(s.mixer).values()]
+        planes = [pl for s in cfg.run_specs for pl in kind(s.mixer).page_planes(s.mixer).values()]
         return sum(max(1, heads) * cols for heads, cols in planes) * cfg.page_size * (4 if kv_dtype == "f32" else 2)
     per_tok_head = cfg.head_dim * (1 if kv_dtype == "int8" else 2) + (4 if kv_dtype == "int8" else 0)
     return (cfg.n_layers - cfg.n_gdn_layers + cfg.mtp_layers) * 2 * (cfg.n_kv_heads // tp) * per_tok_head * cfg.page_size
@@ -78,10 +78,10 @@ def state_bytes_per_slot(cfg: ModelConfig) -> int:
     one head_dim x head_dim matrix per value head, and the convolution window.  Listed models: their mixers' states, and the
     token shift's row per layer."""
     if cfg.layer_specs:
-        from ..models.listed import kind, pad64
-        n = sum(sum(kind(s.mixer).state_shape(s.mixer) or (0,)) for s in cfg.layer_specs)
-        if cfg.block is not None and cfg.block.shift:
-            n += (cfg.n_layers + 1) * pad64(cfg.hidden)
+        from ..models.listed import pad64, state_elems
+        n = state_elems(cfg)
+        if cfg.shift_runs:
+            n += (len(cfg.shift_runs) + 1) * pad64(cfg.hidden)
         return 2 * 4 * n
     if not cfg.n_gdn_layers:
         return 0
