@@ -31,14 +31,20 @@ struct GruParams {
   int ldo;
 };
 
-// 1 - z, and z c
+// 1 - z, and z c; FAST: the intrinsics of models served in bf16
+template <bool FAST>
+__device__ __forceinline__ float exp_f(float x) { return FAST ? __expf(x) : expf(x); }
+template <bool FAST>
+__device__ __forceinline__ float div_f(float x, float y) { return FAST ? __fdividef(x, y) : x / y; }
+template <bool FAST>
 __device__ __forceinline__ float2 gates(float a, float u) {
-  const float e = expf(-fabsf(a)), big = 1.f / (1.f + e), small = e / (1.f + e);      // sigmoid(|a|), sigmoid(-|a|)
+  const float e = exp_f<FAST>(-fabsf(a)), big = div_f<FAST>(1.f, 1.f + e), small = e * big;      // sigmoid(|a|), sigmoid(-|a|)
   const float z = a >= 0.f ? big : small, keep = a >= 0.f ? small : big;
-  const float c = u >= 0.f ? u + 0.5f : 1.f / (1.f + expf(-u));
+  const float c = u >= 0.f ? u + 0.5f : div_f<FAST>(1.f, 1.f + exp_f<FAST>(fminf(-u, 80.f)));
   return make_float2(keep, z * c);
 }
-__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+template <bool FAST>
+__device__ __forceinline__ float silu_f(float x) { return div_f<FAST>(x, 1.f + exp_f<FAST>(fminf(-x, 80.f))); }
 
 template <typename T>
 __global__ void __launch_bounds__(128) mingru_rows_kernel(const GruParams p) {
@@ -61,9 +67,9 @@ __global__ void __launch_bounds__(128) mingru_rows_kernel(const GruParams p) {
     float a = 0.f, u = 0.f, g = 0.f;
 #pragma unroll
     for (int q = 0; q < 8; ++q) { a += v[0][q]; u += v[1][q]; g += v[2][q]; }
-    const float2 k = gates(a + ba, u + bu);
+    const float2 k = gates<sizeof(T) == 2>(a + ba, u + bu);
     s = fmaf(k.x, s, k.y);
-    put(reinterpret_cast<T*>(p.out) + (size_t)m * p.ldo + c, p.mult * s * silu_f(g));
+    put(reinterpret_cast<T*>(p.out) + (size_t)m * p.ldo + c, p.mult * s * silu_f<sizeof(T) == 2>(g));
   }
   *st = s;
 }
@@ -103,8 +109,8 @@ __global__ void __launch_bounds__(kParts * 32) mingru_segments_kernel(const GruP
     float gate[kRows];
 #pragma unroll
     for (int i = 0; i < kRows; ++i) {
-      k[i] = r0 + i < rows ? gates(a[i] + ba, u[i] + bu) : make_float2(1.f, 0.f);      // rows past the end keep the state
-      gate[i] = p.mult * silu_f(g[i]);
+      k[i] = r0 + i < rows ? gates<sizeof(T) == 2>(a[i] + ba, u[i] + bu) : make_float2(1.f, 0.f);      // rows past the end keep the state
+      gate[i] = p.mult * silu_f<sizeof(T) == 2>(g[i]);
       ab = make_float2(ab.x * k[i].x, fmaf(k[i].x, ab.y, k[i].y));
     }
     if (b + 1 < blocks) load(b + 1);

@@ -10,7 +10,8 @@ import dataclasses
 
 import torch
 
-from ..models.config import DenseFfn, GroupedAttention, LayerSpec, MatrixLstm, ModelConfig, listed_config, preset
+from ..models.config import (DenseFfn, GroupedAttention, LayerSpec, MatrixLstm, ModelConfig, listed_config, pefulorn_like,
+                             preset)
 from ..models.weights import random_weights
 from ..ops import lib as K
 from ..runtime.engine import Engine
@@ -56,7 +57,20 @@ def napadra_sizes():
     return out
 
 
-SIZES = {"mumusun": mumusun_sizes, "napadra": napadra_sizes}
+def pefulorn_sizes():
+    """(delta rule with channel decays, time mixing and attention beside a minGRU; gated delta-net and softmax attention) pairs:
+    the same width, layers, feed-forwards, attention heads and recurrent heads; three layers of four are recurrent."""
+    out = []
+    for cfg in (preset("pefulorn-7b"), pefulorn_like("pefulorn-1b", 2048, 24, 16, 4, 5632, 64000, 64),
+                pefulorn_like("pefulorn-wide-8l", 8192, 8, 64, 8, 22016, 64000)):
+        a, f = cfg.layer_specs[3].mixer.left, cfg.layer_specs[0].ffn
+        out.append((cfg, ModelConfig(f"hybrid-like-{cfg.name}", cfg.n_layers, cfg.hidden, a.heads, a.kv_heads, 128, f.ff, cfg.vocab,
+                                     full_attn_every=4, gdn_k_heads=a.heads, gdn_v_heads=a.heads,
+                                     architecture="B200HybridForCausalLM")))
+    return out
+
+
+SIZES = {"mumusun": mumusun_sizes, "napadra": napadra_sizes, "pefulorn": pefulorn_sizes}
 
 
 def _timed(fn, warm: int, reps: int) -> float:
