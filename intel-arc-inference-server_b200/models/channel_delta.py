@@ -114,7 +114,13 @@ def weight_elems(cfg: ModelConfig, a: ChannelDelta) -> int:
 
 def scratch_elems(cfg: ModelConfig, a: ChannelDelta, rows: int, keys: int) -> int:
     g = DeltaGeometry.of(a)
-    return rows * (9 * g.n + 2 * g.kp + g.second + g.act + 2 * g.heads * g.dv) + max(rows, 64) * (g.taps - 1) * g.channels
+    return rows * (9 * g.n + 2 * g.kp + g.second + g.act + 2 * g.heads * g.dv) + max(rows, 64) * (g.taps - 1) * g.channels \
+        + block_elems(rows, a.heads, g.dk, g.dv)
+
+
+def block_elems(rows: int, heads: int, dk: int, dv: int) -> int:
+    """32-bit words of the tensor-core form's workspace (at least 32 rows per segment: twice the rows' chunks at most)."""
+    return 0 if dk > 256 else (2 * rows // 16 + 4) * heads * (6 * 16 * (dk + 8) // 2 + dk + 384 + 20 * dv)
 
 
 def page_planes(a: ChannelDelta) -> dict:
@@ -158,9 +164,10 @@ def scan_rows(ll, sc, plan, m: int, rows: StepRows, act, delta: bool, hq: int, h
     raw = sc.get(name + "_raw", m, h * dv, torch.float32) if n1 < m or not R.fused(dk, dv) else None
     sizes = (hq, h, dk, dv, vdim)
     if n1:
-        R.scan(act, delta, n1, *sizes, rows.req, rows.pos, None, 0, state, w.norm, ll.cfg.rms_eps, raw, out, conv_next, conv_state)
+        R.scan(act, delta, n1, *sizes, rows.req, rows.pos, None, state, w.norm, ll.cfg.rms_eps, raw, out, conv_next, conv_state)
     if n1 < m:
-        t = plan.tables[("chunks",)]
-        R.scan(act[n1:], delta, m - n1, *sizes, rows.req[n1:], rows.pos[n1:], t.segs, t.n_segs, state, w.norm, ll.cfg.rms_eps, raw[n1:],
-               out[n1:], conv_next, conv_state)
+        t, block = plan.tables[("chunks",)], 0 if ll.f32 else R.block_bytes(delta, dk, dv)
+        ws = sc.get("channel_blocks", 4 * t.chunks * h, block, torch.uint8).view(-1) if block else None
+        R.scan(act[n1:], delta, m - n1, *sizes, rows.req[n1:], rows.pos[n1:], t, state, w.norm, ll.cfg.rms_eps, raw[n1:], out[n1:],
+               conv_next, conv_state, ws)
     return ll.linear(sc, "o", w.o, out, m)

@@ -11,7 +11,7 @@ import torch
 from ..ops import channel_rec as R
 from ..ops import gemm as G
 from ..ops import latent as L
-from .channel_delta import pad_key, scan_rows, second_half
+from .channel_delta import block_elems, pad_key, scan_rows, second_half
 from .config import ModelConfig, Wkv
 from .listed import BatchPlan, ListedLayers, ListedScratch, StepRows, pad64
 from .weights import WkvWeights
@@ -69,7 +69,7 @@ def weight_elems(cfg: ModelConfig, a: Wkv) -> int:
 
 def scratch_elems(cfg: ModelConfig, a: Wkv, rows: int, keys: int) -> int:
     g = WkvGeometry.of(a)
-    return rows * (5 * pad64(cfg.hidden) + 9 * g.n + g.kp + g.hd + g.act + 2 * g.hd)
+    return rows * (5 * pad64(cfg.hidden) + 9 * g.n + g.kp + g.hd + g.act + 2 * g.hd) + block_elems(rows, a.heads, g.d, g.d)
 
 
 def page_planes(a: Wkv) -> dict:

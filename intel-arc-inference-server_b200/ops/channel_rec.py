@@ -47,11 +47,19 @@ def wkv_prep(part, s: int, m: int, g, a, w, lr, act):
                                  g.kp, w.second.stride(0), K._p(act), _f32(w.second), K._stream()), "wkv_prep")
 
 
-def scan(act, delta: bool, m: int, hq: int, h: int, dk: int, dv: int, vdim: int, req, pos, segs, n_segs: int, state, norm, eps: float,
-         raw, out, conv_next=None, conv_state=None):
-    """The recurrence over prepared rows, head norm and gate; ``segs`` None: a sequence per run of equal ``req``."""
+def block_bytes(delta: bool, dk: int, dv: int) -> int:
+    """Workspace of the tensor-core form per (16 rows of a segment, head); 0: the sizes are outside it."""
+    return K.lib().b2_channel_block_bytes(int(delta), dk, dv)
+
+
+def scan(act, delta: bool, m: int, hq: int, h: int, dk: int, dv: int, vdim: int, req, pos, t, state, norm, eps: float, raw, out,
+         conv_next=None, conv_state=None, ws=None):
+    """The recurrence over prepared rows, head norm and gate.  ``t``: the rows' segments (``runtime.batch.ChunkPlan``), or None: a
+    sequence per run of equal ``req``; ``ws`` (segments; uint8, ``4 * t.chunks * h`` blocks): on the tensor cores."""
     elems = conv_state[0].numel() if conv_state is not None else 0
-    K._check(K.lib().b2_channel_scan(K._p(act), int(delta), m, hq, h, dk, dv, vdim, K._p(req), K._p(pos), K._p(segs), n_segs, K._p(state),
-                                     K._p(conv_next), K._p(conv_state), elems, K._p(norm), ctypes.c_float(eps), K._p(raw), K._p(out),
-                                     _f32(out), K._stream()), "channel_scan")
-    K.launch_count += int(segs is not None or not fused(dk, dv))
+    K._check(K.lib().b2_channel_scan(K._p(act), int(delta), m, hq, h, dk, dv, vdim, K._p(req), K._p(pos), K._p(t.segs if t else None),
+                                     t.n_segs if t else 0, t.chunks if t else 0, t.most if t else 0, K._p(state), K._p(conv_next),
+                                     K._p(conv_state), elems, K._p(norm), ctypes.c_float(eps), K._p(ws),
+                                     ctypes.c_longlong(ws.numel() if ws is not None else 0), K._p(raw), K._p(out), _f32(out), K._stream()),
+             "channel_scan")
+    K.launch_count += int(t is not None or not fused(dk, dv)) + int(ws is not None)

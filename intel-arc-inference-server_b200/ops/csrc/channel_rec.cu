@@ -9,7 +9,9 @@
 //   wkv_prep_kernel      time mixing: bonus, decays, output gates
 //   channel_rows_kernel  the recurrence, rows one by one; with few value columns a head's whole read-out stays in one CTA, which
 //                        then also norms and gates it
-//   channel_groups_kernel  the recurrence over prompt segments, four rows at a time
+//   channel_groups_kernel  the recurrence over prompt segments in fp32 arithmetic, four rows at a time
+//   channel_pairs_kernel, channel_chunks_kernel  the same on the tensor cores, sixteen rows at a time: what does not involve the
+//                        state for all chunks and heads at once, then the walk over the chunks
 //   channel_out_kernel   head norm and output gate of what the scan left
 //
 // The prep kernels leave fp32 rows
@@ -17,8 +19,8 @@
 // with s1 = beta, s2 = k . q (delta rule) or s1 = bonus (time mixing).  Everything is fp32; models served in 32-bit use the
 // same kernels.  A sequence's first row (position 0) starts from zeros whatever its slot holds.
 //
-// State of one slot: per head and tile of value columns (8, or 4 for more than 256 key dims) the elements in the order in
-// which a warp holds them: [dk / 32][columns per lane][32 lanes][4 key dims].
+// State of one slot: per head and tile of four value columns the elements in the order in which a warp holds them:
+// [dk / 32][32 lanes][4 key dims].
 #include "common.cuh"
 
 using namespace b2;
@@ -407,7 +409,7 @@ struct ScanParams {
 constexpr int kBlockRows = 16;     // rows staged at a time
 constexpr int kGroup = 4;          // rows of a group in the scan of segments
 
-// A warp holds the state of 4 NC value columns: lane = (dim lane dl = lane / 4, cl = lane % 4), columns cl NC + j of its tile, key
+// A warp holds the state of 4 NC value columns: lane = (dim lane dl = lane / 4, cl = lane % 4), column cl of each of its NC tiles, key
 // dims (8 i + dl) 4 .. + 3.  The dim lanes are the upper lane bits: the four lanes that read the same 16 bytes of a shared row
 // are then neighbours, which halves the wavefronts of the load.
 template <int ND, int NC>
@@ -416,14 +418,14 @@ __device__ __forceinline__ void load_state(float4 (&S)[ND / 4][NC], const float*
   for (int i = 0; i < ND / 4; ++i)
 #pragma unroll
     for (int j = 0; j < NC; ++j)
-      S[i][j] = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : __ldcg(reinterpret_cast<const float4*>(st + (i * NC + j) * 128));
+      S[i][j] = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : __ldcg(reinterpret_cast<const float4*>(st + (j * (ND / 4) + i) * 128));
 }
 template <int ND, int NC>
 __device__ __forceinline__ void store_state(const float4 (&S)[ND / 4][NC], float* st) {
 #pragma unroll
   for (int i = 0; i < ND / 4; ++i)
 #pragma unroll
-    for (int j = 0; j < NC; ++j) *reinterpret_cast<float4*>(st + (i * NC + j) * 128) = S[i][j];
+    for (int j = 0; j < NC; ++j) *reinterpret_cast<float4*>(st + (j * (ND / 4) + i) * 128) = S[i][j];
 }
 __device__ __forceinline__ float fdot4(const float4& a, const float4& b, float c) {
   return fmaf(a.w, b.w, fmaf(a.z, b.z, fmaf(a.y, b.y, fmaf(a.x, b.x, c))));
@@ -512,7 +514,7 @@ __global__ void __launch_bounds__(FUSED ? 512 : 128) channel_rows_kernel(const S
   float* st = p.state + (((size_t)slot * p.H + h) * p.dv + c0 + warp * COLS) * dk + lane * 4;
   float4 S[ND / 4][NC];
   load_state<ND, NC>(S, st, p.pos[row0] == 0);
-  const int col = warp * COLS + cl * NC;
+  const int col = warp * COLS + cl;
   for (int b = 0; b < blocks; ++b) {
     if (b + 1 < blocks) {
       fetch(b + 1);
@@ -531,7 +533,7 @@ __global__ void __launch_bounds__(FUSED ? 512 : 128) channel_rows_kernel(const S
       float v[NC], o[NC], a[NC];
 #pragma unroll
       for (int j = 0; j < NC; ++j) {
-        v[j] = row[3 * dk + col + j];
+        v[j] = row[3 * dk + col + 4 * j];
         o[j] = a[j] = 0.f;
       }
 #pragma unroll
@@ -586,11 +588,11 @@ __global__ void __launch_bounds__(FUSED ? 512 : 128) channel_rows_kernel(const S
         const float f = 1.f / sqrtf(tot / (float)p.vdim + p.eps);
         if (dl == 0) {
 #pragma unroll
-          for (int j = 0; j < NC; ++j) put(reinterpret_cast<T*>(p.out) + at + j, o[j] * f * p.norm[h * p.dv + c0 + col + j] * row[3 * dk + vb + col + j]);
+          for (int j = 0; j < NC; ++j) put(reinterpret_cast<T*>(p.out) + at + 4 * j, o[j] * f * p.norm[h * p.dv + c0 + col + 4 * j] * row[3 * dk + vb + col + 4 * j]);
         }
       } else if (dl == 0) {
 #pragma unroll
-        for (int j = 0; j < NC; ++j) p.o[at + j] = o[j];
+        for (int j = 0; j < NC; ++j) p.o[at + 4 * j] = o[j];
       }
     }
     __syncthreads();       // the block's rows are read: the next fetch may overwrite them
@@ -608,11 +610,12 @@ __global__ void __launch_bounds__(FUSED ? 512 : 128) channel_rows_kernel(const S
 //                S  <- a_3 S + sum_s (b_s k_s) v_s^T
 //
 // Every factor is a product of decays (no quotients).  The CTA scales its staged rows in place, a thread per key dim.
-template <int ND, int NC, bool DELTA>
-__global__ void __launch_bounds__(128) channel_groups_kernel(const ScanParams p) {
-  constexpr int LK = 8, CL = 4, dk = ND * LK, COLS = CL * NC, vb = 4 * COLS, G = kBlockRows / kGroup;
+// Eight warps: two halves of a CTA scale two groups at a time, then every warp walks all groups for its four value columns.
+template <int ND, bool DELTA>
+__global__ void __launch_bounds__(256) channel_groups_kernel(const ScanParams p) {
+  constexpr int LK = 8, CL = 4, dk = ND * LK, vb = 8 * CL, G = kBlockRows / kGroup;
   extern __shared__ __align__(16) float sm[];
-  __shared__ __align__(16) float s_pair[G][4][16], s_dots[G][2][16];     // per warp: partial sums; c and d of a group: [t][s]
+  __shared__ __align__(16) float s_pair[G][4][16], s_dots[G][2][16];     // per warp: partial sums; d and c of a group: [t][s]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, dl = lane / CL, cl = lane % CL;
   const int h = blockIdx.y, c0 = blockIdx.x * vb, hq = h / (p.H / p.Hq);
   pdl_launch_dependents();
@@ -630,10 +633,11 @@ __global__ void __launch_bounds__(128) channel_groups_kernel(const ScanParams p)
     stage.fetch(smb + (b & 1) * SB * 4, p, L, act, b * kBlockRows, min(kBlockRows, rows - b * kBlockRows), h, hq, c0);
   };
   fetch(0);
-  float* st = p.state + (((size_t)slot * p.H + h) * p.dv + c0 + warp * COLS) * dk + lane * 4;
-  float4 S[ND / 4][NC];
-  load_state<ND, NC>(S, st, p.pos[row0] == 0);
-  const int col = warp * COLS + cl * NC;
+  float* st = p.state + (((size_t)slot * p.H + h) * p.dv + c0 + warp * CL) * dk + lane * 4;
+  float4 S[ND / 4][1];
+  load_state<ND, 1>(S, st, p.pos[row0] == 0);
+  const int col = warp * CL + cl;
+  float* out = p.o + (size_t)row0 * (p.H * p.dv) + h * p.dv + c0 + col;
   for (int b = 0; b < blocks; ++b) {
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();       // the block's rows are there, the block before is read
@@ -641,12 +645,12 @@ __global__ void __launch_bounds__(128) channel_groups_kernel(const ScanParams p)
     const int n = min(kBlockRows, rows - b * kBlockRows);
     float* base = sm + (b & 1) * SB;
 #pragma unroll 1
-    for (int gr = 0; gr < G; ++gr) {       // scaled rows, and the products of the group's rows with each other
+    for (int gr = warp >> 2; gr < G; gr += 2) {       // scaled rows, and the products of the group's rows with each other
       if (gr * kGroup >= n) break;
       float w[16];
 #pragma unroll
       for (int e = 0; e < 16; ++e) w[e] = 0.f;
-      for (int d = threadIdx.x; d < dk; d += 128) {
+      for (int d = threadIdx.x & 127; d < dk; d += 128) {
         float q[4], k[4], g[4];
         float* x = base + gr * kGroup * SR + d;
 #pragma unroll
@@ -696,10 +700,10 @@ __global__ void __launch_bounds__(128) channel_groups_kernel(const ScanParams p)
             w[e] = keep + __shfl_xor_sync(0xffffffffu, give, x);
           }
       w[0] += __shfl_xor_sync(0xffffffffu, w[0], 1);
-      if (!(lane & 1)) s_pair[gr][warp][lane >> 1] = w[0];
+      if (!(lane & 1)) s_pair[gr][warp & 3][lane >> 1] = w[0];
     }
     __syncthreads();
-    {                     // full 4 x 4 tables: d, then c
+    if (threadIdx.x < 128) {      // full 4 x 4 tables: d, then c
       const int gr = threadIdx.x >> 5, e = threadIdx.x & 31, t = (e >> 2) & 3, s = e & 3;
       const bool is_c = e >= 16;
       const int i = is_c ? 10 + t * (t - 1) / 2 + s : t * (t + 1) / 2 + s;
@@ -709,103 +713,418 @@ __global__ void __launch_bounds__(128) channel_groups_kernel(const ScanParams p)
     __syncthreads();
     for (int gr = 0; gr * kGroup < n; ++gr) {
       const float* row = base + gr * kGroup * SR;
-      float pq[4][NC], u[4][NC];
+      float pq[4], u[4], v[4], beta[4];
 #pragma unroll
-      for (int t = 0; t < 4; ++t)
-#pragma unroll
-        for (int j = 0; j < NC; ++j) pq[t][j] = u[t][j] = 0.f;
+      for (int t = 0; t < 4; ++t) {
+        const bool ok = gr * kGroup + t < n;
+        pq[t] = u[t] = 0.f;
+        v[t] = ok ? row[t * SR + 3 * dk + col] : 0.f;
+        beta[t] = ok ? row[t * SR + SR - 4] : 0.f;          // time mixing: the bonus
+      }
 #pragma unroll
       for (int i = 0; i < ND / 4; ++i)
 #pragma unroll
         for (int t = 0; t < 4; ++t) {
-          const float4 qv = reinterpret_cast<const float4*>(row + t * SR)[i * LK + dl];
-#pragma unroll
-          for (int j = 0; j < NC; ++j) pq[t][j] = fdot4(S[i][j], qv, pq[t][j]);
-          if (DELTA) {
-            const float4 kv = reinterpret_cast<const float4*>(row + t * SR + dk)[i * LK + dl];
-#pragma unroll
-            for (int j = 0; j < NC; ++j) u[t][j] = fdot4(S[i][j], kv, u[t][j]);
-          }
+          if (DELTA) u[t] = fdot4(S[i][0], reinterpret_cast<const float4*>(row + t * SR + dk)[i * LK + dl], u[t]);
+          pq[t] = fdot4(S[i][0], reinterpret_cast<const float4*>(row + t * SR)[i * LK + dl], pq[t]);
         }
-      float v[4][NC];
-#pragma unroll
-      for (int t = 0; t < 4; ++t)
-#pragma unroll
-        for (int j = 0; j < NC; ++j) v[t][j] = gr * kGroup + t < n ? row[t * SR + 3 * dk + col + j] : 0.f;
       if (DELTA) {
 #pragma unroll
         for (int x = CL; x < 32; x <<= 1)
 #pragma unroll
-          for (int t = 0; t < 4; ++t)
-#pragma unroll
-            for (int j = 0; j < NC; ++j) u[t][j] += __shfl_xor_sync(0xffffffffu, u[t][j], x);
+          for (int t = 0; t < 4; ++t) u[t] += __shfl_xor_sync(0xffffffffu, u[t], x);
 #pragma unroll
         for (int t = 0; t < 4; ++t) {
           const float4 c = *reinterpret_cast<const float4*>(&s_dots[gr][1][t * 4]);
-          const float beta = gr * kGroup + t < n ? row[t * SR + SR - 4] : 0.f;
-#pragma unroll
-          for (int j = 0; j < NC; ++j) {
-            float r = v[t][j] - u[t][j];
-            if (t > 0) r = fmaf(-c.x, u[0][j], r);
-            if (t > 1) r = fmaf(-c.y, u[1][j], r);
-            if (t > 2) r = fmaf(-c.z, u[2][j], r);
-            u[t][j] = beta * r;
-          }
+          float r = v[t] - u[t];
+          if (t > 0) r = fmaf(-c.x, u[0], r);
+          if (t > 1) r = fmaf(-c.y, u[1], r);
+          if (t > 2) r = fmaf(-c.z, u[2], r);
+          u[t] = beta[t] * r;
         }
       } else {
 #pragma unroll
-        for (int t = 0; t < 4; ++t)
-#pragma unroll
-          for (int j = 0; j < NC; ++j) u[t][j] = v[t][j];
+        for (int t = 0; t < 4; ++t) u[t] = v[t];
       }
       // the state after the group
       const float4* av = reinterpret_cast<const float4*>(base + kBlockRows * SR + gr * dk);
 #pragma unroll
       for (int i = 0; i < ND / 4; ++i) {
-        const float4 a = av[i * LK + dl];
+        float4 x = mul4(S[i][0], av[i * LK + dl]);
 #pragma unroll
-        for (int j = 0; j < NC; ++j) S[i][j] = mul4(S[i][j], a);
-#pragma unroll
-        for (int t = 0; t < 4; ++t) {
-          const float4 kv = reinterpret_cast<const float4*>(row + t * SR + 2 * dk)[i * LK + dl];
-#pragma unroll
-          for (int j = 0; j < NC; ++j) S[i][j] = axpy4(u[t][j], kv, S[i][j]);
-        }
+        for (int t = 0; t < 4; ++t) x = axpy4(u[t], reinterpret_cast<const float4*>(row + t * SR + 2 * dk)[i * LK + dl], x);
+        S[i][0] = x;
       }
-      // read-outs: summed over the dim lanes so that lane dl ends with row dl & 3 (and column dl >> 2)
-      const int t = dl & 3;
-      float o[NC];
+      // read-outs: summed over the dim lanes so that lane dl ends with row dl & 3
 #pragma unroll
-      for (int j = 0; j < NC; ++j) {
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const float give = dl & 2 ? pq[e][j] : pq[e + 2][j], keep = dl & 2 ? pq[e + 2][j] : pq[e][j];
-          pq[e][j] = keep + __shfl_xor_sync(0xffffffffu, give, 2 * CL);
-        }
-        const float give = dl & 1 ? pq[0][j] : pq[1][j], keep = dl & 1 ? pq[1][j] : pq[0][j];
-        o[j] = keep + __shfl_xor_sync(0xffffffffu, give, CL);
+      for (int e = 0; e < 2; ++e) {
+        const float give = dl & 2 ? pq[e] : pq[e + 2], keep = dl & 2 ? pq[e + 2] : pq[e];
+        pq[e] = keep + __shfl_xor_sync(0xffffffffu, give, 2 * CL);
       }
-      int j = 0;
-      float mine;
-      if constexpr (NC == 2) {
-        j = dl >> 2;
-        mine = (j ? o[1] : o[0]) + __shfl_xor_sync(0xffffffffu, j ? o[0] : o[1], 4 * CL);
-      } else {
-        mine = o[0] + __shfl_xor_sync(0xffffffffu, o[0], 4 * CL);
-      }
+      const float give = dl & 1 ? pq[0] : pq[1], keep = dl & 1 ? pq[1] : pq[0];
+      float o = keep + __shfl_xor_sync(0xffffffffu, give, CL);
+      o += __shfl_xor_sync(0xffffffffu, o, 4 * CL);
+      const int t = dl & 3, r = gr * kGroup + t;
       const float4 d = *reinterpret_cast<const float4*>(&s_dots[gr][0][t * 4]);
-      mine = fmaf(d.x, NC == 2 && j ? u[0][NC - 1] : u[0][0], mine);
-      mine = fmaf(d.y, NC == 2 && j ? u[1][NC - 1] : u[1][0], mine);
-      mine = fmaf(d.z, NC == 2 && j ? u[2][NC - 1] : u[2][0], mine);
-      mine = fmaf(d.w, NC == 2 && j ? u[3][NC - 1] : u[3][0], mine);
-      const int r = gr * kGroup + t;
-      if (r < n && (NC == 2 || dl < 4)) {
-        if (!DELTA) mine = fmaf(row[t * SR + SR - 4], row[t * SR + 3 * dk + col + j], mine);
-        p.o[(size_t)(row0 + b * kBlockRows + r) * (p.H * p.dv) + h * p.dv + c0 + col + j] = mine;
+      o = fmaf(d.x, u[0], o);
+      o = fmaf(d.y, u[1], o);
+      o = fmaf(d.z, u[2], o);
+      o = fmaf(d.w, u[3], o);
+      if (!DELTA) o = fmaf(t == 0 ? beta[0] : t == 1 ? beta[1] : t == 2 ? beta[2] : beta[3], t == 0 ? v[0] : t == 1 ? v[1] : t == 2 ? v[2] : v[3], o);
+      if (r < n && dl < 4) out[(size_t)(b * kBlockRows + r) * (p.H * p.dv)] = o;
+    }
+  }
+  store_state<ND, 1>(S, st);
+}
+
+// ------------------------------------------------------------------ segments on the tensor cores
+// Chunks of sixteen rows, in the notation of the groups above.  With the rows' writes U and the state S0 at the chunk's start
+//   delta rule   (I + diag(beta) C) U = diag(beta) (V - Kp S0),  so  U = Wv - W S0   with  W = (I + diag(beta) C)^-1 diag(beta) Kp
+//                and Wv likewise from V;   Kp, Qp: rows a_t k_t, a_t q_t
+//   time mixing  U = V;  Qp: rows a_{t-1} q_t;  the bonus is the diagonal of D
+//   both         O = Qp S0 + D U,   S <- diag(a_15) S0 + Ks^T U,   Ks: rows b_s k_s
+// W, Qp, Ks and D enter their products as two bf16 limbs, as do the state and U; a product of two such keeps all but the
+// smallest of its four terms.
+constexpr int CR = 16;                                    // rows of a chunk
+constexpr int kLdd = 24, kLdv = 20;                       // row strides of D (bf16) and of Wv^T (fp32)
+
+// operand block of a (chunk, head): [W hi | W lo |] Q hi | Q lo | Ks hi | Ks lo ([16][dk + 8] bf16 each), a_15 [dk] fp32, D hi | lo
+// [16][24] bf16, then Wv^T [dv][20] fp32
+template <int KB, bool DELTA>
+struct Block {
+  static constexpr int dk = KB * 64, LDK = dk + 8, IMG = CR * LDK * 2;
+  static constexpr int W = 0, Q = DELTA ? 2 * IMG : 0, K = Q + 2 * IMG, A = K + 2 * IMG, D = A + dk * 4, V = D + 2 * CR * kLdd * 2;
+  static constexpr int SLICE = 64 * kLdv * 4;             // Wv^T of 64 value columns
+  static constexpr int STAGE = V + SLICE, NST = KB <= 2 ? 4 : 3;
+  static constexpr int SMEM = NST * STAGE + 64 + 128;
+  static_assert(IMG % 16 == 0 && V % 16 == 0 && STAGE % 16 == 0, "bulk copies move multiples of 16 bytes");
+  static_assert(SMEM <= 227 * 1024, "shared memory of one CTA");
+  __host__ __device__ static constexpr size_t bytes(int dv) { return V + (size_t)dv * kLdv * 4; }
+};
+
+struct ChunkParams {
+  ScanParams s;
+  uint8_t* ws;             // [16-row chunks][H] blocks; a segment's first chunk is four times its `first chunk` word
+};
+
+__device__ __forceinline__ void limbs(float x, float y, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16(x, y);
+  lo = pack_bf16(x - bf16_lo(hi), y - bf16_hi(hi));
+}
+
+template <int KB, bool DELTA>
+__global__ void __launch_bounds__(128) channel_pairs_kernel(const ChunkParams cp) {
+  using B = Block<KB, DELTA>;
+  constexpr int dk = KB * 64, NQ = (dk + 127) / 128;
+  extern __shared__ __align__(16) float sm[];             // q | k | decay, [16][dk] each
+  __shared__ __align__(16) float s_c[CR][CR], s_d[CR][CR], s_s1[CR];
+  const ScanParams& p = cp.s;
+  const int h = blockIdx.y, hq = h / (p.H / p.Hq), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int* seg = p.segs + blockIdx.z * 4;
+  const int n = min(CR, seg[1] - (int)blockIdx.x * CR);
+  if (n <= 0) return;
+  const ActLayout L = act_layout(p.Hq, p.H, dk, p.dv);
+  const float* act = p.act + (size_t)(seg[0] + blockIdx.x * CR) * L.n;
+  uint8_t* blk = cp.ws + ((size_t)(4 * seg[3] + blockIdx.x) * p.H + h) * B::bytes(p.dv);
+  float *sq = sm, *sk = sm + CR * dk, *sg = sm + 2 * CR * dk;
+#pragma unroll
+  for (int i = 0; i < 3 * CR * dk / 4 / 128; ++i) {
+    const int e = (i * 128 + tid) * 4, which = e / (CR * dk), r = (e / dk) % CR, d = e % dk;
+    const int col = which == 0 ? L.q + hq * dk : which == 1 ? L.k + hq * dk : L.g + h * dk;
+    const float pad = which == 2 ? 1.f : 0.f;             // rows past the end keep the state
+    *reinterpret_cast<float4*>(sm + e) = r < n ? __ldcg(reinterpret_cast<const float4*>(act + (size_t)r * L.n + col + d))
+                                               : make_float4(pad, pad, pad, pad);
+  }
+  if (tid < CR) s_s1[tid] = tid < n ? act[(size_t)tid * L.n + L.s1 + h] : 0.f;
+  __syncthreads();
+  // products of the rows with each other: a warp takes four rows s, lanes the key dims; sums over the warp leave value l in
+  // lane l (c_ts: t, d_ts: 16 + t)
+  for (int i = 0; i < 4; ++i) {
+    const int s = i == 0 ? warp : i == 1 ? 7 - warp : i == 2 ? 8 + warp : 15 - warp;
+    float v[32];
+#pragma unroll
+    for (int e = 0; e < 32; ++e) v[e] = 0.f;
+#pragma unroll
+    for (int u = 0; u < NQ; ++u) {
+      const int d = (u * 32 + lane) * 4;
+      if (d >= dk) continue;
+      float4 r = *reinterpret_cast<const float4*>(sk + s * dk + d);
+#pragma unroll
+      for (int t = 0; t < CR; ++t) {
+        if (t < s) continue;
+        const float4 g = *reinterpret_cast<const float4*>(sg + t * dk + d);
+        const float4 q = *reinterpret_cast<const float4*>(sq + t * dk + d);
+        if (DELTA) {
+          if (t > s) {
+            r = mul4(r, g);
+            v[t] = fdot4(r, *reinterpret_cast<const float4*>(sk + t * dk + d), v[t]);
+          }
+          v[16 + t] = fdot4(r, q, v[16 + t]);
+        } else if (t > s) {
+          v[16 + t] = fdot4(r, q, v[16 + t]);
+          r = mul4(r, g);
+        }
+      }
+    }
+#pragma unroll
+    for (int x = 16; x >= 1; x >>= 1)
+#pragma unroll
+      for (int e = 0; e < 16; ++e)
+        if (e < x) {
+          const bool up = lane & x;
+          const float give = up ? v[e] : v[e + x], keep = up ? v[e + x] : v[e];
+          v[e] = keep + __shfl_xor_sync(0xffffffffu, give, x);
+        }
+    if (lane < 16) s_c[lane][s] = v[0];
+    else s_d[lane - 16][s] = !DELTA && lane - 16 == s ? s_s1[s] : v[0];
+  }
+  __syncthreads();
+  if (tid < CR * CR / 2) {             // D's limbs
+    const int t = tid >> 3, s = (tid & 7) * 2;
+    uint32_t hi, lo;
+    limbs(s_d[t][s], s_d[t][s + 1], hi, lo);
+    uint32_t* d = reinterpret_cast<uint32_t*>(blk + B::D) + (t * kLdd + s) / 2;
+    d[0] = hi;
+    d[CR * kLdd / 2] = lo;
+  }
+  // two columns per thread: of the keys (scaled rows, W), then of the values
+  for (int c = tid; c < (dk + p.dv) / 2; c += 128) {
+    const bool key = c < dk / 2;
+    const int d = 2 * (key ? c : c - dk / 2);
+    float2 x[CR];
+    if (key) {
+      float2 a = make_float2(1.f, 1.f);
+#pragma unroll
+      for (int t = 0; t < CR; ++t) {
+        const float2 g = *reinterpret_cast<const float2*>(sg + t * dk + d);
+        const float2 q = *reinterpret_cast<const float2*>(sq + t * dk + d), k = *reinterpret_cast<const float2*>(sk + t * dk + d);
+        if (DELTA) a = make_float2(a.x * g.x, a.y * g.y);
+        uint32_t hi, lo;
+        limbs(a.x * q.x, a.y * q.y, hi, lo);
+        uint32_t* o = reinterpret_cast<uint32_t*>(blk + B::Q) + (t * B::LDK + d) / 2;
+        o[0] = hi;
+        o[B::IMG / 4] = lo;
+        x[t] = make_float2(a.x * k.x, a.y * k.y);
+        if (!DELTA) a = make_float2(a.x * g.x, a.y * g.y);
+      }
+      *reinterpret_cast<float2*>(blk + B::A + d * 4) = a;
+      float2 b = make_float2(1.f, 1.f);
+#pragma unroll
+      for (int t = CR - 1; t >= 0; --t) {
+        const float2 g = *reinterpret_cast<const float2*>(sg + t * dk + d), k = *reinterpret_cast<const float2*>(sk + t * dk + d);
+        uint32_t hi, lo;
+        limbs(b.x * k.x, b.y * k.y, hi, lo);
+        uint32_t* o = reinterpret_cast<uint32_t*>(blk + B::K) + (t * B::LDK + d) / 2;
+        o[0] = hi;
+        o[B::IMG / 4] = lo;
+        b = make_float2(b.x * g.x, b.y * g.y);
+      }
+      if (!DELTA) continue;
+    } else {
+#pragma unroll
+      for (int t = 0; t < CR; ++t)
+        x[t] = t < n ? __ldcg(reinterpret_cast<const float2*>(act + (size_t)t * L.n + L.v + h * p.dv + d)) : make_float2(0.f, 0.f);
+    }
+    if (DELTA) {                       // forward substitution
+#pragma unroll
+      for (int t = 0; t < CR; ++t) {
+        float2 y = x[t];
+#pragma unroll
+        for (int s = 0; s < t; ++s) y = make_float2(fmaf(-s_c[t][s], x[s].x, y.x), fmaf(-s_c[t][s], x[s].y, y.y));
+        x[t] = make_float2(s_s1[t] * y.x, s_s1[t] * y.y);
+      }
+    }
+    if (key) {
+#pragma unroll
+      for (int t = 0; t < CR; ++t) {
+        uint32_t hi, lo;
+        limbs(x[t].x, x[t].y, hi, lo);
+        uint32_t* o = reinterpret_cast<uint32_t*>(blk + B::W) + (t * B::LDK + d) / 2;
+        o[0] = hi;
+        o[B::IMG / 4] = lo;
+      }
+    } else {
+      float4* o = reinterpret_cast<float4*>(blk + B::V) + d * (kLdv / 4);
+#pragma unroll
+      for (int t = 0; t < CR; t += 4) {
+        o[t / 4] = make_float4(x[t].x, x[t + 1].x, x[t + 2].x, x[t + 3].x);
+        o[kLdv / 4 + t / 4] = make_float4(x[t].y, x[t + 1].y, x[t + 2].y, x[t + 3].y);
       }
     }
   }
-  store_state<ND, NC>(S, st);
+}
+
+__device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm_x4_trans(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mma_a(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  mma_bf16_16816(c, a[0], a[1], a[2], a[3], b0, b1);
+}
+
+// grid (value blocks of 64, heads, segments), four warps.  A warp keeps S^T of its 16 value columns in MMA accumulators for the whole
+// walk; products have the value dimension as M, so accumulators become A operands in registers and the warps exchange nothing.
+template <int KB, bool DELTA>
+__global__ void __launch_bounds__(128) channel_chunks_kernel(const ChunkParams cp) {
+  using B = Block<KB, DELTA>;
+  constexpr int dk = KB * 64, NST = B::NST;
+  extern __shared__ __align__(128) uint8_t smem_b[];
+  const ScanParams& p = cp.s;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  const int h = blockIdx.y, c0 = blockIdx.x * 64;
+  const uint32_t base = smem_u32(smem_b), bars = base + NST * B::STAGE;
+  if (tid == 0) {
+    for (int i = 0; i < NST; ++i) mbar_init(bars + 8 * i, 1);
+    mbar_fence_init();
+  }
+  __syncthreads();
+  pdl_launch_dependents();
+  pdl_wait();
+  const int* seg = p.segs + blockIdx.z * 4;
+  const int row0 = seg[0], rows = seg[1], slot = seg[2], chunks = (rows + CR - 1) / CR;
+  commit_inputs(p, slot);
+  const uint8_t* ws = cp.ws + ((size_t)4 * seg[3] * p.H + h) * B::bytes(p.dv);
+  const size_t step = (size_t)p.H * B::bytes(p.dv);
+  auto fetch = [&](int c) {
+    const uint32_t dst = base + (c % NST) * B::STAGE, bar = bars + 8 * (c % NST);
+    const uint8_t* src = ws + (size_t)c * step;
+    mbar_expect_tx(bar, B::STAGE);
+    bulk_g2s(dst, src, B::V, bar);
+    bulk_g2s(dst + B::V, src + B::V + (size_t)c0 * kLdv * 4, B::SLICE, bar);
+  };
+  int issued = min(NST, chunks);
+  if (tid == 0)
+    for (int c = 0; c < issued; ++c) fetch(c);
+  // st[j]: key dims 8 j + 2 t, + 1 of value column vc ([0], [1]) and of column vc + 8 ([2], [3])
+  float st[dk / 8][4];
+  const int vc = 16 * warp + g;
+  float* sp = p.state + (((size_t)slot * p.H + h) * p.dv + c0) * dk;
+  auto place = [&](int d, int col) { return (col >> 2) * 4 * dk + (d >> 5) * 128 + (((d >> 2) & 7) * 4 + (col & 3)) * 4 + (d & 3); };
+  const bool fresh = p.pos[row0] == 0;
+#pragma unroll
+  for (int j = 0; j < dk / 8; ++j)
+#pragma unroll
+    for (int hf = 0; hf < 2; ++hf) {
+      const float2 v = fresh ? make_float2(0.f, 0.f) : __ldcg(reinterpret_cast<const float2*>(sp + place(8 * j + 2 * t, vc + 8 * hf)));
+      st[j][2 * hf] = v.x;
+      st[j][2 * hf + 1] = v.y;
+    }
+  // ldmatrix lanes: B rows [n][k] of two n tiles, and rows [k][n] read transposed
+  const uint32_t nk = (uint32_t)((((lane & 7) + ((lane >> 4) << 3)) * B::LDK + (((lane >> 3) & 1) << 3)) * 2);
+  const uint32_t nd = (uint32_t)((((lane & 7) + ((lane >> 4) << 3)) * kLdd + (((lane >> 3) & 1) << 3)) * 2);
+  const uint32_t kn = (uint32_t)((((lane & 7) + (((lane >> 3) & 1) << 3)) * B::LDK + ((lane >> 4) << 3)) * 2);
+  bool ok = true;
+  for (int c = 0; c < chunks; ++c) {
+    const uint32_t sb = base + (c % NST) * B::STAGE;
+    const uint8_t* sbp = smem_b + (c % NST) * B::STAGE;
+    ok = mbar_wait(bars + 8 * (c % NST), (c / NST) & 1, ERR_GDN_WAIT);
+    if (!__syncthreads_and(ok)) {      // a copy gave up: wait (bounded) for those in flight, leave the state alone
+      if (tid == 0)
+        for (int i = c; i < issued; ++i) mbar_wait(bars + 8 * (i % NST), (i / NST) & 1, ERR_GDN_WAIT);
+      return;
+    }
+    // the state against W and Q: [16 value columns][16 rows]; small terms in sums of their own
+    float r1[2][4] = {}, r2[2][4] = {}, e1[2][4] = {}, e2[2][4] = {};
+#pragma unroll
+    for (int kk = 0; kk < dk / 16; ++kk) {
+      uint32_t ah[4], al[4], qh[4], ql[4];
+      limbs(st[2 * kk][0], st[2 * kk][1], ah[0], al[0]);
+      limbs(st[2 * kk][2], st[2 * kk][3], ah[1], al[1]);
+      limbs(st[2 * kk + 1][0], st[2 * kk + 1][1], ah[2], al[2]);
+      limbs(st[2 * kk + 1][2], st[2 * kk + 1][3], ah[3], al[3]);
+      if (DELTA) {
+        uint32_t wh[4], wl[4];
+        ldsm_x4(sb + B::W + nk + 32 * kk, wh);
+        ldsm_x4(sb + B::W + B::IMG + nk + 32 * kk, wl);
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          mma_a(r1[u], ah, wh[2 * u], wh[2 * u + 1]);
+          mma_a(e1[u], al, wh[2 * u], wh[2 * u + 1]);
+        }
+#pragma unroll
+        for (int u = 0; u < 2; ++u) mma_a(e1[u], ah, wl[2 * u], wl[2 * u + 1]);
+      }
+      ldsm_x4(sb + B::Q + nk + 32 * kk, qh);
+      ldsm_x4(sb + B::Q + B::IMG + nk + 32 * kk, ql);
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        mma_a(r2[u], ah, qh[2 * u], qh[2 * u + 1]);
+        mma_a(e2[u], al, qh[2 * u], qh[2 * u + 1]);
+      }
+#pragma unroll
+      for (int u = 0; u < 2; ++u) mma_a(e2[u], ah, ql[2 * u], ql[2 * u + 1]);
+    }
+    // U^T as an A operand over the chunk's rows
+    uint32_t uh[4], ul[4];
+    const float* wv = reinterpret_cast<const float*>(sbp + B::V);
+#pragma unroll
+    for (int u = 0; u < 2; ++u)
+#pragma unroll
+      for (int hf = 0; hf < 2; ++hf) {
+        float2 v = *reinterpret_cast<const float2*>(wv + (vc + 8 * hf) * kLdv + 8 * u + 2 * t);
+        if (DELTA) {
+          v.x -= r1[u][2 * hf] + e1[u][2 * hf];
+          v.y -= r1[u][2 * hf + 1] + e1[u][2 * hf + 1];
+        }
+        limbs(v.x, v.y, uh[2 * u + hf], ul[2 * u + hf]);
+      }
+    {
+      uint32_t dh[4], dl[4];
+      ldsm_x4(sb + B::D + nd, dh);
+      ldsm_x4(sb + B::D + CR * kLdd * 2 + nd, dl);
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        mma_a(r2[u], uh, dh[2 * u], dh[2 * u + 1]);
+        mma_a(e2[u], ul, dh[2 * u], dh[2 * u + 1]);
+      }
+#pragma unroll
+      for (int u = 0; u < 2; ++u) mma_a(e2[u], uh, dl[2 * u], dl[2 * u + 1]);
+    }
+    // the state after the chunk
+    const float* av = reinterpret_cast<const float*>(sbp + B::A);
+#pragma unroll
+    for (int j = 0; j < dk / 8; ++j) {
+      const float2 a = *reinterpret_cast<const float2*>(av + 8 * j + 2 * t);
+      st[j][0] *= a.x; st[j][1] *= a.y; st[j][2] *= a.x; st[j][3] *= a.y;
+    }
+#pragma unroll
+    for (int jj = 0; jj < dk / 16; ++jj) {
+      uint32_t kh[4], kl[4];
+      ldsm_x4_trans(sb + B::K + kn + 32 * jj, kh);
+      ldsm_x4_trans(sb + B::K + B::IMG + kn + 32 * jj, kl);
+#pragma unroll
+      for (int u = 0; u < 2; ++u) mma_a(st[2 * jj + u], ul, kh[2 * u], kh[2 * u + 1]);
+#pragma unroll
+      for (int u = 0; u < 2; ++u) mma_a(st[2 * jj + u], uh, kl[2 * u], kl[2 * u + 1]);
+#pragma unroll
+      for (int u = 0; u < 2; ++u) mma_a(st[2 * jj + u], uh, kh[2 * u], kh[2 * u + 1]);
+    }
+    float* o = p.o + (size_t)(row0 + c * CR) * (p.H * p.dv) + h * p.dv + c0 + vc;
+    const int n = rows - c * CR;
+#pragma unroll
+    for (int u = 0; u < 2; ++u)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int r = 8 * u + 2 * t + (e & 1);
+        if (r < n) o[(size_t)r * (p.H * p.dv) + 8 * (e >> 1)] = r2[u][e] + e2[u][e];
+      }
+    __syncthreads();       // every warp is done with the stage
+    if (c + NST < chunks) {
+      if (tid == 0) fetch(c + NST);
+      issued = c + NST + 1;
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < dk / 8; ++j)
+#pragma unroll
+    for (int hf = 0; hf < 2; ++hf)
+      *reinterpret_cast<float2*>(sp + place(8 * j + 2 * t, vc + 8 * hf)) = make_float2(st[j][2 * hf], st[j][2 * hf + 1]);
 }
 
 // one warp per (row, head)
@@ -837,13 +1156,13 @@ __global__ void __launch_bounds__(256) channel_out_kernel(const float* __restric
 bool dk_ok(int dk) { return dk == 64 || dk == 128 || dk == 192 || dk == 256 || dk == 384 || dk == 512; }
 
 template <typename F>
-int launch_scan_kernel(F kernel, const ScanParams& p, dim3 grid, int threads, int smem, cudaStream_t st) {
+int launch_scan_kernel(F kernel, const ScanParams& p, dim3 grid, int threads, int smem, cudaStream_t st, bool pdl = true) {
   if (smem > 227 * 1024 - 4096) return -6;
   if (smem > 44 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return (int)e;
   }
-  return b2_launch(kernel, grid, dim3(threads), smem, st, true, p);
+  return b2_launch(kernel, grid, dim3(threads), smem, st, pdl, p);
 }
 
 template <int ND, int NC, bool DELTA, bool FUSED, typename T>
@@ -853,10 +1172,41 @@ int launch_rows(const ScanParams& p, int seqs, cudaStream_t st) {
   return launch_scan_kernel(channel_rows_kernel<ND, NC, DELTA, FUSED, T>, p, dim3(p.dv / vb, p.H, seqs), warps * 32, smem, st);
 }
 
-template <int ND, int NC, bool DELTA>
+// not started while the kernel before still runs: its few, long CTAs would gather on the SMs that happen to be free
+template <int ND, bool DELTA>
 int launch_groups(const ScanParams& p, int seqs, cudaStream_t st) {
-  constexpr int vb = 16 * NC, smem = 2 * (kBlockRows * (3 * ND * 8 + vb + 4) + kBlockRows / kGroup * ND * 8) * 4;
-  return launch_scan_kernel(channel_groups_kernel<ND, NC, DELTA>, p, dim3(p.dv / vb, p.H, seqs), 128, smem, st);
+  constexpr int vb = 32, smem = 2 * (kBlockRows * (3 * ND * 8 + vb + 4) + kBlockRows / kGroup * ND * 8) * 4;
+  return launch_scan_kernel(channel_groups_kernel<ND, DELTA>, p, dim3(p.dv / vb, p.H, seqs), 256, smem, st, false);
+}
+
+template <int KB, bool DELTA>
+int launch_chunks(const ChunkParams& p, int n_segs, int most, size_t ws_bytes, int chunks, cudaStream_t st) {
+  using B = Block<KB, DELTA>;
+  if (ws_bytes < (size_t)chunks * p.s.H * B::bytes(p.s.dv)) return -7;
+  constexpr int psm = 3 * CR * KB * 64 * 4;
+  static bool configured[64] = {};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (!configured[dev & 63]) {
+    cudaError_t e = cudaFuncSetAttribute(channel_chunks_kernel<KB, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, B::SMEM);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(channel_pairs_kernel<KB, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, psm);
+    if (e != cudaSuccess) return (int)e;
+    configured[dev & 63] = true;
+  }
+  int rc = b2_launch(channel_pairs_kernel<KB, DELTA>, dim3(most, p.s.H, n_segs), dim3(128), psm, st, true, p);
+  if (rc) return rc;
+  return b2_launch(channel_chunks_kernel<KB, DELTA>, dim3(p.s.dv / 64, p.s.H, n_segs), dim3(128), B::SMEM, st, false, p);     // as launch_groups
+}
+
+template <bool DELTA>
+int launch_chunks_dk(const ChunkParams& p, int n_segs, int most, size_t ws_bytes, int chunks, cudaStream_t st) {
+  switch (p.s.dk) {
+    case 64: return launch_chunks<1, DELTA>(p, n_segs, most, ws_bytes, chunks, st);
+    case 128: return launch_chunks<2, DELTA>(p, n_segs, most, ws_bytes, chunks, st);
+    case 192: return launch_chunks<3, DELTA>(p, n_segs, most, ws_bytes, chunks, st);
+    case 256: return launch_chunks<4, DELTA>(p, n_segs, most, ws_bytes, chunks, st);
+  }
+  return -1;
 }
 
 template <bool DELTA, typename T>
@@ -874,12 +1224,12 @@ template <bool DELTA>
 int launch_scan_dk(const ScanParams& p, int seqs, cudaStream_t st) {
   if (p.segs) {
     switch (p.dk) {
-      case 64: return launch_groups<8, 2, DELTA>(p, seqs, st);
-      case 128: return launch_groups<16, 2, DELTA>(p, seqs, st);
-      case 192: return launch_groups<24, 2, DELTA>(p, seqs, st);
-      case 256: return launch_groups<32, 2, DELTA>(p, seqs, st);
-      case 384: return launch_groups<48, 1, DELTA>(p, seqs, st);
-      case 512: return launch_groups<64, 1, DELTA>(p, seqs, st);
+      case 64: return launch_groups<8, DELTA>(p, seqs, st);
+      case 128: return launch_groups<16, DELTA>(p, seqs, st);
+      case 192: return launch_groups<24, DELTA>(p, seqs, st);
+      case 256: return launch_groups<32, DELTA>(p, seqs, st);
+      case 384: return launch_groups<48, DELTA>(p, seqs, st);
+      case 512: return launch_groups<64, DELTA>(p, seqs, st);
     }
     return -1;
   }
@@ -968,12 +1318,29 @@ extern "C" int b2_channel_state_elems(int H, int dk, int dv) { return H * dk * d
 // 1 when the scan's CTA holds a whole head and writes the finished rows itself
 extern "C" int b2_channel_fused(int dk, int dv) { return dk <= 256 && dv <= 128; }
 
+// bytes of a (16-row chunk, head) operand block of the tensor-core form; 0: the sizes are outside it
+extern "C" int b2_channel_block_bytes(int delta, int dk, int dv) {
+  switch (dk * 2 + (delta ? 1 : 0)) {
+    case 128: return (int)Block<1, false>::bytes(dv);
+    case 129: return (int)Block<1, true>::bytes(dv);
+    case 256: return (int)Block<2, false>::bytes(dv);
+    case 257: return (int)Block<2, true>::bytes(dv);
+    case 384: return (int)Block<3, false>::bytes(dv);
+    case 385: return (int)Block<3, true>::bytes(dv);
+    case 512: return (int)Block<4, false>::bytes(dv);
+    case 513: return (int)Block<4, true>::bytes(dv);
+  }
+  return 0;
+}
+
 // The recurrence over prepared rows.  segs null: rows 0 .. M - 1, a sequence per run of equal `req`; else n_segs x 4 ints
-// (first row, rows, slot, unused).  out [rows][H dv]; raw: fp32 of the same shape, unused where b2_channel_fused says so and
+// (first row, rows, slot, first 64-row chunk; `chunks` such chunks in all, `most` in one segment).  With `ws` (segments; chunks x 4 x
+// H blocks of b2_channel_block_bytes) on the tensor cores.  out [rows][H dv]; raw: fp32 of the same shape, unused where b2_channel_fused says so and
 // segs is null.  delta 1: delta rule, 0: time mixing.
 extern "C" int b2_channel_scan(const float* act, int delta, int M, int Hq, int H, int dk, int dv, int vdim, const int* req, const int* pos,
-                               const int* segs, int n_segs, float* state, const float* conv_next, float* conv_state, int conv_elems,
-                               const float* norm, float eps, float* raw, void* out, int f32, void* stream) {
+                               const int* segs, int n_segs, int chunks, int most, float* state, const float* conv_next, float* conv_state,
+                               int conv_elems, const float* norm, float eps, void* ws, long long ws_bytes, float* raw, void* out, int f32,
+                               void* stream) {
   if (M < 1 || H < 1 || H > 65535 || Hq < 1 || H % Hq || !dk_ok(dk) || dv % 64 || dv < 64 || dv > 512 || conv_elems % 4) return -1;
   const int seqs = segs ? n_segs : M;
   if (seqs < 1 || seqs > 65535) return -2;
@@ -984,10 +1351,20 @@ extern "C" int b2_channel_scan(const float* act, int delta, int M, int Hq, int H
     return f32 ? launch_fused_dk<false, float>(p, seqs, st) : launch_fused_dk<false, __nv_bfloat16>(p, seqs, st);
   }
   if (!raw) return -3;
-  const int rc = delta ? launch_scan_dk<true>(p, seqs, st) : launch_scan_dk<false>(p, seqs, st);
+  int rc;
+  if (segs && ws) {
+    if ((uintptr_t)ws & 15) return -8;
+    const ChunkParams cp{p, (uint8_t*)ws};
+    rc = delta ? launch_chunks_dk<true>(cp, n_segs, 4 * most, (size_t)ws_bytes, 4 * chunks, st)
+               : launch_chunks_dk<false>(cp, n_segs, 4 * most, (size_t)ws_bytes, 4 * chunks, st);
+  } else {
+    rc = delta ? launch_scan_dk<true>(p, seqs, st) : launch_scan_dk<false>(p, seqs, st);
+  }
   if (rc) return rc;
   const ActLayout L = act_layout(Hq, H, dk, dv);
   const dim3 grid((unsigned)(((long long)M * H + 7) / 8));
   return f32 ? b2_launch(channel_out_kernel<float>, grid, dim3(256), 0, st, true, (const float*)raw, act, L.n, L.z, norm, M, H, dv, vdim, eps, (float*)out)
              : b2_launch(channel_out_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, true, (const float*)raw, act, L.n, L.z, norm, M, H, dv, vdim, eps, (__nv_bfloat16*)out);
 }
+
+B2_DEFINE_STATUS(channel)

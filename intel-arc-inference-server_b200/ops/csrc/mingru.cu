@@ -150,6 +150,7 @@ extern "C" int b2_mingru(const float* part, int slices, int M, int N, int col, i
     rc = f32 ? b2_launch(mingru_rows_kernel<float>, dim3((W + 127) / 128, n1), dim3(128), 0, st, true, p)
              : b2_launch(mingru_rows_kernel<__nv_bfloat16>, dim3((W + 127) / 128, n1), dim3(128), 0, st, true, p);
   if (rc || n1 == M) return rc;
-  return f32 ? b2_launch(mingru_segments_kernel<float>, dim3(W / 32, n_segs), dim3(kParts * 32), 0, st, true, p)
-             : b2_launch(mingru_segments_kernel<__nv_bfloat16>, dim3(W / 32, n_segs), dim3(kParts * 32), 0, st, true, p);
+  // not started while the kernel before still runs: its few, long CTAs would gather on the SMs that happen to be free
+  return f32 ? b2_launch(mingru_segments_kernel<float>, dim3(W / 32, n_segs), dim3(kParts * 32), 0, st, false, p)
+             : b2_launch(mingru_segments_kernel<__nv_bfloat16>, dim3(W / 32, n_segs), dim3(kParts * 32), 0, st, false, p);
 }

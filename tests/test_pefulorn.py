@@ -500,7 +500,7 @@ class Cell:
         assert out.shape[1] == self.cols
         return out
 
-    def run(self, runs, dtype, seg, eps=0.02):
+    def run(self, runs, dtype, seg, eps=0.02, tc=False):
         from b200serve.ops import channel_rec as R
         at = runs_rows([(s, p, len(x["q"])) for s, p, x in runs])
         m = len(at)
@@ -508,11 +508,15 @@ class Cell:
         t = segments([(s, p, len(x["q"])) for s, p, x in runs]) if seg else None
         raw = torch.full((m, self.h * self.dv), float("nan"), device=DEV)
         out = torch.full((m, self.h * self.dv), float("nan"), dtype=dtype, device=DEV)
-        R.scan(act, self.delta, m, self.hq, self.h, self.dk, self.dv, self.vdim, i32([s for s, _ in at]), i32([p for _, p in at]),
-               t.segs if t else None, t.n_segs if t else 0, self.state, self.normp, eps, raw, out)
+        R.scan(act, self.delta, m, self.hq, self.h, self.dk, self.dv, self.vdim, i32([s for s, _ in at]), i32([p for _, p in at]), t,
+               self.state, self.normp, eps, raw, out, ws=self.workspace(t) if tc else None)
         v = out.view(m, self.h, self.dv)
         assert torch.all(v[..., self.vdim:] == 0)
         return v[..., : self.vdim]
+
+    def workspace(self, t):
+        from b200serve.ops import channel_rec as R
+        return torch.full((4 * t.chunks * self.h * R.block_bytes(self.delta, self.dk, self.dv),), 0xFF, dtype=torch.uint8, device=DEV)
 
 
 def cut_inputs(x, lo, hi):
@@ -546,6 +550,25 @@ def test_channel_recurrence(shape, delta):
         assert float(row_errors(c.run([(2, 0, again)], BF16, seg), c.reference(again)).max()) < 6e-3
 
 
+@pytest.mark.parametrize("shape", [s for s in CELLS if s[2] <= 256])
+@pytest.mark.parametrize("delta", [True, False])
+def test_channel_recurrence_on_tensor_cores(shape, delta):
+    """Segments in chunks of sixteen rows, the last one cut anywhere, between rows one by one; several sequences."""
+    if not delta:
+        shape = (shape[1],) + shape[1:]
+    for cuts in ((200,), (64, 1, 33, 47, 3, 52), (100, 100), (32, 168)):
+        c = Cell(shape, delta, seed=shape[2])
+        xs = {s: c.inputs(200, s) for s in (0, 3)}
+        ref = {s: c.reference(x) for s, x in xs.items()}
+        at = 0
+        for n in cuts:
+            runs = [(s, at, cut_inputs(x, at, at + n)) for s, x in xs.items()]
+            got = c.run(runs, F32, n >= 32, tc=n >= 32)
+            assert float(row_errors(got, torch.cat([ref[s][at: at + n] for s in xs])).max()) < 2e-4, (cuts, at, n)
+            at += n
+        assert torch.isnan(c.state[1]).all()
+
+
 @pytest.mark.parametrize("delta", [True, False])
 def test_decays_at_their_ends(delta):
     """Decays of nearly one remember a strong early write for hundreds of rows, decays of nearly zero forget it at once, mixed
@@ -561,8 +584,8 @@ def test_decays_at_their_ends(delta):
         x["s1"][5] = 1.0
         x["q"][5:] = x["k"][5]                     # late rows ask for the early write
         ref = c.reference(x)
-        for seg in (False, True):
-            assert float(row_errors(c.run([(1, 0, x)], F32, seg), ref).max()) < 5e-4, (decay, seg)
+        for seg, tc in ((False, False), (True, False), (True, True)):
+            assert float(row_errors(c.run([(1, 0, x)], F32, seg, tc=tc), ref).max()) < 5e-4, (decay, seg, tc)
 
 
 def prep_model(mixer, taps_seed=0):
