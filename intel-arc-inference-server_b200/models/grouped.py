@@ -175,8 +175,8 @@ class Mixer:
         n1 = m if plan is None or not self.tile_rows else plan.n_single
         if n1 and self.rows_form:
             ns, cap = self.nsplit(n1), self.partials(g)
-            op = sc.get("o_part", cap, g.dv, torch.float32) if ns > 1 else None
-            ml = sc.get("ml_part", cap, 2, torch.float32) if ns > 1 else None
+            op = sc.get(f"o_part{cap}", cap, g.dv, torch.float32) if ns > 1 else None      # layers of other heads have their own
+            ml = sc.get(f"ml_part{cap}", cap, 2, torch.float32) if ns > 1 else None
             P.rows(q, k, v, n1, g, rows.req, rows.pos, block_table, ns, a.chunk, a.scale, w.slope2, w.sink2, op, ml, out, **more)
         elif n1:
             P.simple(q, k, v, n1, g, rows.req, rows.pos, block_table, a.chunk, a.scale, w.slope2, w.sink2, out, **more)

@@ -714,11 +714,12 @@ def one_config():
 
 
 def flat_config():
-    """No loop at all; wide heads."""
+    """No loop at all; wide heads; two attention layers with the same value size and other heads."""
     ff = DenseFfn(64, gelu=True, bias=True)
     return listed_config("pefulorn-flat", "Pefulorn", (
         LayerSpec(attention_beside_gru(4, 2, 190, 130, 0.1, 130, 0.6, 20, (0.9, 1.1)), ff), LayerSpec(Wkv(3, 128, 40), ff),
-        LayerSpec(ChannelDelta(2, 1, 256, 128, 3, 40, 24), ff)), 320, 211, 1e-6, PLAIN)
+        LayerSpec(ChannelDelta(2, 1, 256, 128, 3, 40, 24), ff), LayerSpec(attention_beside_gru(3, 3, 64, 150, 0.15, 64, 0.4, 50, (1.0, 0.6)), None)),
+        320, 211, 1e-6, PLAIN)
 
 
 def lively(name, t):
