@@ -101,7 +101,8 @@ __device__ __forceinline__ float4 embedded(const StreamParams& p, int tok, int p
   return v;
 }
 
-template <int S, int CS>
+// EXT: the options at the end of the list above
+template <int S, int CS, bool EXT>
 __global__ void __launch_bounds__(kThreads) streams_kernel(const StreamParams p) {
   extern __shared__ __align__(16) float vals[];            // u of the row at hand, then h of the row before
   __shared__ float red[kThreads / 32], stat, s_mix[S * S], s_out[S], s_in[S];
@@ -111,7 +112,7 @@ __global__ void __launch_bounds__(kThreads) streams_kernel(const StreamParams p)
     s_in[tid] = p.in ? p.in[tid] : 1.f;
   }
   if (tid < S * S) s_mix[tid] = !p.y ? 0.f : p.mix ? p.mix[tid] : tid % (S + 1) == 0 ? 1.f : 0.f;
-  const float g = p.g_cols ? 1.f : p.g[0];
+  const float g = EXT && p.g_cols ? 1.f : p.g[0];
   pdl_launch_dependents();
   pdl_wait();
   __syncthreads();
@@ -126,7 +127,7 @@ __global__ void __launch_bounds__(kThreads) streams_kernel(const StreamParams p)
   auto pass = [&](int m, bool store) -> float {
     float ssq = 0.f;
     int tok = 0, pos = 0;
-    if (!p.y || p.again) {
+    if (!p.y || (EXT && p.again)) {
       tok = p.tokens[m];
       pos = p.pos[m];
       if (tok < 0 || tok >= p.vocab) {
@@ -146,26 +147,26 @@ __global__ void __launch_bounds__(kThreads) streams_kernel(const StreamParams p)
         float4 y = b[0];
 #pragma unroll
         for (int s = 1; s < 8; ++s) y = fma4(1.f, b[s], y);
-        if (p.bias) y = fma4(1.f, *reinterpret_cast<const float4*>(p.bias + c), y);
+        if (EXT && p.bias) y = fma4(1.f, *reinterpret_cast<const float4*>(p.bias + c), y);
         if (p.scale) {
           const float4 w = *reinterpret_cast<const float4*>(p.scale + c);
           y.x *= w.x; y.y *= w.y; y.z *= w.z; y.w *= w.w;
         }
         float4 ahead = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (p.again) ahead = embedded(p, tok, pos, c);
-        if (p.add) ahead = fma4(1.f, *reinterpret_cast<const float4*>(p.add + c), ahead);
+        if (EXT && p.again) ahead = embedded(p, tok, pos, c);
+        if (EXT && p.add) ahead = fma4(1.f, *reinterpret_cast<const float4*>(p.add + c), ahead);
 #pragma unroll
         for (int t = 0; t < S; ++t) {
           float4 v = make_float4(s_out[t] * y.x, s_out[t] * y.y, s_out[t] * y.z, s_out[t] * y.w);
 #pragma unroll
           for (int s = 0; s < S; ++s) v = fma4(s_mix[s * S + t], x[s], v);
-          v = fma4(1.f, ahead, v);
+          if (EXT) v = fma4(1.f, ahead, v);
           if (store && p.x_out) *reinterpret_cast<float4*>(p.x_out + ((size_t)m * S + t) * p.ld + c) = v;
           a = fma4(s_in[t], v, a);
         }
       } else {
         float4 v = embedded(p, tok, pos, c);
-        if (p.add) v = fma4(1.f, *reinterpret_cast<const float4*>(p.add + c), v);
+        if (EXT && p.add) v = fma4(1.f, *reinterpret_cast<const float4*>(p.add + c), v);
 #pragma unroll
         for (int t = 0; t < S; ++t) {
           if (store && p.x_out) *reinterpret_cast<float4*>(p.x_out + ((size_t)m * S + t) * p.ld + c) = v;
@@ -198,7 +199,7 @@ __global__ void __launch_bounds__(kThreads) streams_kernel(const StreamParams p)
         const float r = pass(m - 1, false);
         for (int c = c0 + tid * 4; c < c1; c += kThreads * 4)
 #pragma unroll
-          for (int j = 0; j < 4; ++j) before[c + j] = u[c + j] * r * (p.g_cols ? p.g[c + j] : 1.f);
+          for (int j = 0; j < 4; ++j) before[c + j] = u[c + j] * r * (EXT && p.g_cols ? p.g[c + j] : 1.f);
       }
     }
     const bool last = m + 1 == p.M || p.req[m + 1] != req;
@@ -209,7 +210,7 @@ __global__ void __launch_bounds__(kThreads) streams_kernel(const StreamParams p)
       if (p.commit && last) *reinterpret_cast<float4*>(p.commit + st) = __ldcg(reinterpret_cast<const float4*>(p.next + st));
       float4 h = *reinterpret_cast<const float4*>(u + c);
       h.x *= r; h.y *= r; h.z *= r; h.w *= r;
-      if (p.g_cols) {
+      if (EXT && p.g_cols) {
         const float4 w = *reinterpret_cast<const float4*>(p.g + c);
         h.x *= w.x; h.y *= w.y; h.z *= w.z; h.w *= w.w;
       }
@@ -222,7 +223,7 @@ __global__ void __launch_bounds__(kThreads) streams_kernel(const StreamParams p)
         float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
         if (follows) b = *reinterpret_cast<const float4*>(before + c);
         else if (!first) b = __ldcg(reinterpret_cast<const float4*>(p.prev + st));
-        for (int i = 0; i < p.planes; ++i) {
+        for (int i = 0; i < (EXT ? p.planes : 1); ++i) {
           const float4 w = *reinterpret_cast<const float4*>(p.mu + (size_t)i * p.ld + c);
           store(i, make_float4(fmaf(b.x - h.x, w.x, h.x), fmaf(b.y - h.y, w.y, h.y), fmaf(b.z - h.z, w.z, h.z), fmaf(b.w - h.w, w.w, h.w)));
         }
@@ -236,12 +237,12 @@ __global__ void __launch_bounds__(kThreads) streams_kernel(const StreamParams p)
   }
 }
 
-template <int S, int CS>
-int launch(const StreamParams& p, cudaStream_t st) {
+template <int S, int CS, bool EXT>
+int launch_form(const StreamParams& p, cudaStream_t st) {
   const size_t smem = 2 * (size_t)(((p.ld / 4 + CS - 1) / CS) * 4) * sizeof(float);
   if (smem > 48 * 1024) {
     if (smem > 200 * 1024) return -5;
-    cudaError_t e = cudaFuncSetAttribute(streams_kernel<S, CS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(streams_kernel<S, CS, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
   cudaLaunchConfig_t cfg = {};
@@ -258,7 +259,12 @@ int launch(const StreamParams& p, cudaStream_t st) {
   cfg.attrs = attr;
   static const bool no_pdl = getenv("B2_NO_PDL") != nullptr;  // measurement switch, as in b2_launch
   cfg.numAttrs = no_pdl ? 1 : 2;
-  return (int)cudaLaunchKernelEx(&cfg, streams_kernel<S, CS>, p);
+  return (int)cudaLaunchKernelEx(&cfg, streams_kernel<S, CS, EXT>, p);
+}
+
+template <int S, int CS>
+int launch(const StreamParams& p, cudaStream_t st) {
+  return p.g_cols || p.bias || p.add || p.again || p.planes > 1 ? launch_form<S, CS, true>(p, st) : launch_form<S, CS, false>(p, st);
 }
 
 template <int S>
