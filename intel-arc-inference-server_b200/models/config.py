@@ -7,6 +7,7 @@ is generated from it rather than written per model.
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field, asdict, replace
 from typing import Optional
 
@@ -46,8 +47,32 @@ class LatentAttention:
 
 
 @dataclass(frozen=True)
+class Rotary:
+    """Rotation of the first ``dims`` dimensions of a head, dimension i with i + dims / 2, by position * base^(-2 i / dims); the
+    rest pass.  Angles are divided by ``factor``; with ``original`` (positions of the first training, YaRN) only those that turn
+    less than ``slow`` times over them, those above ``fast`` turns stay, a linear ramp in between, and cosines and sines are
+    multiplied by 0.1 ln(factor) + 1."""
+    dims: int
+    base: float
+    factor: float = 1.0
+    original: float = 0.0
+    fast: float = 32.0
+    slow: float = 1.0
+
+    def frequencies(self) -> tuple:
+        """(angle per position of every pair, factor of cosines and sines), in double precision."""
+        f = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        if not self.original:
+            return [x / self.factor for x in f], 1.0
+        at = lambda turns: self.dims * math.log(self.original / (2 * math.pi * turns)) / (2 * math.log(self.base))     # noqa: E731
+        lo, hi = max(math.floor(at(self.fast)), 0), min(math.ceil(at(self.slow)), self.dims - 1)
+        ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(len(f))]
+        return [x / self.factor * r + x * (1 - r) for x, r in zip(f, ramp)], 0.1 * math.log(self.factor) + 1.0
+
+
+@dataclass(frozen=True)
 class GroupedAttention:
-    """Grouped-query attention without a rotation; the cache holds keys and values per key/value head."""
+    """Grouped-query attention; the cache holds keys and values per key/value head."""
     heads: int
     kv_heads: int
     dim: int
@@ -63,13 +88,30 @@ class GroupedAttention:
     v_norm: bool = False          # values are divided by their root mean square per head
     temp: float = 0.0             # queries at position p times 1 + temp ln(floor((p + 1) / temp_every) + 1)
     temp_every: int = 1
+    rot: Optional[Rotary] = None  # rotation of queries and keys, behind their norms
+    rot_values: bool = False      # values are rotated too (all of vdim, plain angles of rot.base), every head's result is turned back
+    tied: bool = False            # the values are the projected keys, unrotated
+    window: int = 0               # a position sees itself and the window - 1 positions before it (0: all)
+    pool: int = 0                 # beside the window: one mean key and value per block of this many positions that lies wholly before it
+    gate: bool = False            # the heads' results times the sigmoid of a projection
 
     def linear_elems(self, h: int) -> int:
-        return h * (self.heads * (self.dim + self.vdim) + (self.kv_heads * (self.dim + self.vdim) if self.kv_from < 0 else 0))
+        q = self.heads * (self.dim + self.vdim * (2 if self.gate else 1))
+        return h * (q + (self.kv_heads * (self.dim + (0 if self.tied else self.vdim)) if self.kv_from < 0 else 0))
 
     @property
     def kv_elems(self) -> int:
         return self.kv_heads * (self.dim + self.vdim) if self.kv_from < 0 else 0
+
+    @property
+    def pool_slots(self) -> int:
+        """Blocks that end in a page of 16 positions, at most."""
+        return (self.pool + 15) // self.pool if self.pool else 0
+
+    @property
+    def pool_elems(self) -> int:
+        """Cached elements of a page's blocks."""
+        return self.pool_slots * self.kv_elems
 
 
 @dataclass(frozen=True)
@@ -110,12 +152,33 @@ class MinGru:
 
 
 @dataclass(frozen=True)
+class Retention:
+    """Recurrent mixer with a matrix memory per head and a fixed decay: S <- decay S + k v^T, the result is S^T q, divided by its
+    root mean square per head and times SiLU of a projection; queries and keys are rotated."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: tuple
+    rot: Rotary
+    recurrent = True
+
+    def linear_elems(self, h: int) -> int:
+        return h * self.heads * (2 * self.dim + 3 * self.vdim)
+
+    @property
+    def kv_elems(self) -> int:
+        return 0
+
+
+@dataclass(frozen=True)
 class ParallelMixer:
-    """Two mixers side by side on the same input; the result is the sum of theirs, each times its scale."""
+    """Two mixers side by side on the same input; the result is the sum of theirs, each times its scale -- with ``normed`` each
+    one's result divided by its root mean square first, with a weight per column."""
     left: object
     right: object
     left_scale: float
     right_scale: float
+    normed: bool = False
 
     @property
     def heads(self) -> int:
@@ -139,6 +202,10 @@ class ParallelMixer:
     @property
     def kv_elems(self) -> int:
         return self.left.kv_elems + self.right.kv_elems
+
+    @property
+    def pool_elems(self) -> int:
+        return sum(getattr(m, "pool_elems", 0) for m in (self.left, self.right))
 
 
 @dataclass(frozen=True)
@@ -185,16 +252,17 @@ class Wkv:
 @dataclass(frozen=True)
 class DenseFfn:
     """down (f(g) (u + shift)), g = min(gate, limit), u = clamp(up, -limit, limit), f(g) = g sigmoid(alpha g), or the tanh form
-    of GELU; ``bias``: all three projections have one."""
+    of GELU; ``bias``: all three projections have one.  ``relu2``: no gate, down relu(up)^2."""
     ff: int
     limit: float = float("inf")
     alpha: float = 1.0
     shift: float = 0.0
     gelu: bool = False
     bias: bool = False
+    relu2: bool = False
 
     def linear_elems(self, h: int) -> tuple:
-        return (3 * self.ff * h,) * 2
+        return ((2 if self.relu2 else 3) * self.ff * h,) * 2
 
 
 @dataclass(frozen=True)
@@ -214,6 +282,16 @@ class StreamBlock:
 
 
 @dataclass(frozen=True)
+class SandwichBlock:
+    """One residual stream with a norm ahead of every sublayer and one behind it: x + norm_b(f(norm_a(x))).  A norm divides each of
+    ``groups`` equal parts of a row by the part's own root mean square; the stream starts as the embedding row times ``scale``."""
+    groups: int = 1
+    scale: float = 1.0
+    streams = 1
+    shift = mixing = columns = False
+
+
+@dataclass(frozen=True)
 class LayerLoop:
     """Layers ``start`` .. ``stop - 1`` run ``times`` times in a row with the same weights, each pass with its own cache and
     state.  Ahead of a pass a learned vector is added to the residual, and ahead of all but the first the embedding row too."""
@@ -226,7 +304,8 @@ class LayerLoop:
 class ExpertFfn:
     """Routed SwiGLU experts.  ``score``: "softmax" over all experts or a "sigmoid" each; with ``groups`` > 1 only
     experts of the ``keep`` groups with the largest sums of their two best scores can be chosen; ``renorm``: the chosen
-    scores are divided by their sum."""
+    scores are divided by their sum.  ``relu2``: experts without a gate, down relu(up)^2.  ``shared``: width of an expert that
+    every token runs, with weight one (0: none)."""
     experts: int
     top: int
     ff: int
@@ -234,23 +313,33 @@ class ExpertFfn:
     groups: int = 1
     keep: int = 1
     renorm: bool = False
+    relu2: bool = False
+    shared: int = 0
 
     @property
     def rule(self) -> tuple:
         return (int(self.score == "sigmoid"), self.groups, self.keep, int(self.renorm))
 
+    @property
+    def shared_slots(self) -> int:
+        """Experts of the common width that together are the shared one: its hidden columns are cut into as many runs."""
+        ffp = (self.ff + 63) // 64 * 64
+        return (self.shared + ffp - 1) // ffp
+
     def linear_elems(self, h: int) -> tuple:
         """(weights a token's step reads, weights held)."""
-        one = 3 * self.ff * h
-        return self.experts * h + self.top * one, self.experts * (h + one)
+        n = 2 if self.relu2 else 3
+        one, shared = n * self.ff * h, n * self.shared * h
+        return self.experts * h + self.top * one + shared, self.experts * (h + one) + shared
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     """One layer of a model that lists its layers: a mixer and a feed-forward (or none).  How they meet the fp32 residual
     is ``ModelConfig.block``: None adds layer norms of the sublayers' outputs to one stream."""
-    mixer: object                 # LatentAttention, GroupedAttention, MatrixLstm, ParallelMixer, ChannelDelta or Wkv
+    mixer: object                 # LatentAttention, GroupedAttention, MatrixLstm, Retention, ParallelMixer, ChannelDelta or Wkv
     ffn: object                   # ExpertFfn, DenseFfn or None
+    weights_of: int = -1          # layer whose weights (mixer, feed-forward, norms) this one uses, with a cache of its own (-1: its own)
 
 
 @dataclass(frozen=True)
@@ -290,7 +379,7 @@ class ModelConfig:
     # models that list their layers one by one (unquantised weights, fp32 residual); the scalar fields above then hold the
     # largest values over the layers
     layer_specs: tuple = ()
-    block: Optional[StreamBlock] = None
+    block: object = None          # StreamBlock, SandwichBlock or None
     loop: Optional[LayerLoop] = None
 
     @property
@@ -426,7 +515,7 @@ class ModelConfig:
     def param_count(self) -> int:
         h = self.hidden
         if self.layer_specs:
-            return int(sum(self.layer_linears(s)[1] for s in self.layer_specs) + 2 * self.vocab * h)
+            return int(sum(self.layer_linears(s)[1] for s in self.layer_specs if s.weights_of < 0) + 2 * self.vocab * h)
         per = self._mixer_params()
         if self.is_moe:
             per += self.n_experts * 3 * self.expert_ffn * h + self.n_experts * h
@@ -455,7 +544,8 @@ class ModelConfig:
 
     def kv_bytes_per_token(self, kv_dtype: str = "bf16") -> int:
         if self.layer_specs:
-            return sum(s.mixer.kv_elems for s in self.run_specs) * (4 if kv_dtype == "f32" else 2)
+            pooled = sum(getattr(s.mixer, "pool_elems", 0) for s in self.run_specs)      # of a whole page
+            return (sum(s.mixer.kv_elems for s in self.run_specs) + -(-pooled // self.page_size)) * (4 if kv_dtype == "f32" else 2)
         per_head = self.head_dim * (2 if kv_dtype == "bf16" else 1) + (4 if kv_dtype == "int8" else 0)
         return (self.n_layers - self.n_gdn_layers) * 2 * self.n_kv_heads * per_head
 
@@ -525,7 +615,7 @@ class ModelConfig:
 
 
 def listed_config(name: str, architecture: str, specs, hidden: int, vocab: int, eps: float,
-                  block: Optional[StreamBlock] = None, loop: Optional[LayerLoop] = None) -> ModelConfig:
+                  block=None, loop: Optional[LayerLoop] = None) -> ModelConfig:
     """A model given by its layers; the scalar fields other parts of the framework read hold the largest values."""
     specs = tuple(specs)
     ffns = [s.ffn for s in specs if s.ffn is not None]
@@ -689,8 +779,110 @@ def pefulorn_keys(c: ModelConfig) -> dict:
     return out
 
 
-LISTED_ARCHITECTURES = {"Mumusun": mumusun_config, "Napadra": napadra_config, "Pefulorn": pefulorn_config}
-LISTED_WRITERS = {"Mumusun": mumusun_keys, "Napadra": napadra_keys, "Pefulorn": pefulorn_keys}
+def _rotary(r: dict) -> Rotary:
+    s = r.get("scaling") or {}
+    if r["dims"] % 2 or r["dims"] < 0:
+        raise ValueError(f"{r['dims']} rotated dimensions")
+    return Rotary(r["dims"], float(r["base"]), float(s.get("factor", 1.0)), float(s.get("original", 0.0)), float(s.get("fast", 32.0)),
+                  float(s.get("slow", 1.0)))
+
+
+def _rotary_keys(r: Rotary) -> dict:
+    out = {"dims": r.dims, "base": r.base}
+    if r.original:
+        out["scaling"] = {"factor": r.factor, "original": r.original, "fast": r.fast, "slow": r.slow}
+    elif r.factor != 1.0:
+        out["scaling"] = {"factor": r.factor}
+    return out
+
+
+def vogerax_config(d: dict) -> ModelConfig:
+    """``config.json`` of a Vogerax checkpoint: attention over a window and pooled blocks before it whose values are its keys,
+    layers of gated attention with rotated values beside retention, ungated feed-forwards and experts, layers that use another
+    one's weights, a residual with norms on both sides of every sublayer."""
+    specs = []
+    for i, layer in enumerate(d["layers"]):
+        m, f = layer["mixer"], layer["mlp"]
+        if layer["type"] == "attention":
+            mask = m.get("mask") or {}
+            mixer = GroupedAttention(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]), rot=_rotary(m["rot"]), tied=True,
+                                     window=mask.get("size", 0) or 0, pool=mask.get("pool", 0) or 0)
+            if mixer.vdim != mixer.dim:
+                raise ValueError(f"layer {i}: values of {mixer.vdim} dimensions that are keys of {mixer.dim}")
+            if mixer.window < 0 or mixer.pool < 0 or mixer.pool and not mixer.window:
+                raise ValueError(f"layer {i}: mask {mask}")
+            heads = mixer
+        elif layer["type"] == "parallel":
+            a, b = m["left"], m["right"]
+            heads = GroupedAttention(a["heads"], a["kv_heads"], a["dim"], a["vdim"], float(a["scale"]), sink=True, qk_norm=True,
+                                     rot=_rotary(a["rot"]), rot_values=True, gate=True)
+            right = Retention(b["heads"], b["dim"], b["vdim"], tuple(float(x) for x in b["decay"]), _rotary(b["rot"]))
+            if len(right.decay) != right.heads:
+                raise ValueError(f"layer {i}: {len(right.decay)} decays for {right.heads} heads")
+            if max(right.dim, right.vdim) > 512 or right.rot.dims > right.dim:
+                raise ValueError(f"layer {i}: retention heads of {right.dim} x {right.vdim} (512 at most), {right.rot}")
+            if heads.vdim % 2:
+                raise ValueError(f"layer {i}: {heads.vdim} rotated value dimensions")
+            mixer = ParallelMixer(heads, right, 0.5, 0.5, True)
+        else:
+            raise ValueError(f"layer {i}: mixer {layer['type']!r} is not part of Vogerax")
+        if heads.heads % heads.kv_heads or max(heads.dim, heads.vdim) > 1024 or heads.rot.dims > heads.dim:
+            raise ValueError(f"layer {i}: {heads.heads} / {heads.kv_heads} heads of {heads.dim} x {heads.vdim} (1024 at most), {heads.rot}")
+        ffn = None
+        if f is not None:
+            if f["kind"] == "dense":
+                ffn = DenseFfn(f["ff"], relu2=True)
+            elif f["kind"] == "moe":
+                r = f["router"]
+                if not 1 <= r["top"] <= min(r["experts"], 32) or r["experts"] > 512:
+                    raise ValueError(f"layer {i}: {r['top']} of {r['experts']} experts (32 of 512 at most)")
+                ffn = ExpertFfn(r["experts"], r["top"], f["expert"]["ff"], "softmax", relu2=True, shared=(f.get("shared") or {}).get("ff", 0))
+            else:
+                raise ValueError(f"layer {i}: feed-forward {f['kind']!r} is not part of Vogerax")
+        of = layer.get("weights_of")
+        specs.append(LayerSpec(mixer, ffn, -1 if of is None else of))
+    for i, s in enumerate(specs):
+        seen, j = {i}, s.weights_of
+        while j >= 0:
+            if j >= len(specs) or j in seen or (specs[j].mixer, specs[j].ffn) != (s.mixer, s.ffn):
+                raise ValueError(f"layer {i} cannot use the weights of layer {j}")
+            seen.add(j)
+            j = specs[j].weights_of
+    groups = d["norm"].get("groups", 1)
+    if groups < 1 or d["width"] % groups:
+        raise ValueError(f"{groups} norm groups of {d['width']} columns")
+    scale = float((d.get("embedding") or {}).get("scale", 1.0))
+    return listed_config(d.get("name", "vogerax"), "Vogerax", specs, d["width"], d["vocab"], float(d["norm"]["eps"]),
+                         SandwichBlock(groups, scale))
+
+
+def vogerax_keys(c: ModelConfig) -> dict:
+    def layer(s):
+        m, f = s.mixer, s.ffn
+        if isinstance(m, ParallelMixer):
+            a, b = m.left, m.right
+            kind, mixer = "parallel", {
+                "left": {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim, "scale": a.scale, "rot": _rotary_keys(a.rot)},
+                "right": {"heads": b.heads, "dim": b.dim, "vdim": b.vdim, "decay": list(b.decay), "rot": _rotary_keys(b.rot)}}
+        else:
+            kind, mixer = "attention", {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale,
+                                        "rot": _rotary_keys(m.rot)}
+            if m.window:
+                mixer["mask"] = {"size": m.window, **({"pool": m.pool} if m.pool else {})}
+        mlp = None
+        if isinstance(f, DenseFfn):
+            mlp = {"kind": "dense", "ff": f.ff}
+        elif f is not None:
+            mlp = {"kind": "moe", "expert": {"ff": f.ff}, "router": {"experts": f.experts, "top": f.top}}
+            if f.shared:
+                mlp["shared"] = {"ff": f.shared}
+        return {"type": kind, "mixer": mixer, "mlp": mlp, **({"weights_of": s.weights_of} if s.weights_of >= 0 else {})}
+    return {"embedding": {"scale": c.block.scale}, "norm": {"eps": c.rms_eps, "groups": c.block.groups},
+            "layers": [layer(s) for s in c.layer_specs]}
+
+
+LISTED_ARCHITECTURES = {"Mumusun": mumusun_config, "Napadra": napadra_config, "Pefulorn": pefulorn_config, "Vogerax": vogerax_config}
+LISTED_WRITERS = {"Mumusun": mumusun_keys, "Napadra": napadra_keys, "Pefulorn": pefulorn_keys, "Vogerax": vogerax_keys}
 
 
 def tiny_dense() -> ModelConfig:
@@ -816,6 +1008,38 @@ def pefulorn_7b() -> ModelConfig:
     return pefulorn_like("pefulorn-7b", 4096, 32, 32, 8, 11008, 64000)
 
 
+def vogerax_mini() -> ModelConfig:
+    """Small Vogerax: both kinds of layers with unequal sizes, windows and blocks, shared weights, a layer without a feed-forward."""
+    att = lambda h, g, dim, rot, window, pool: GroupedAttention(h, g, dim, dim, 0.9 * dim ** -0.5, rot=rot, tied=True, window=window, pool=pool)  # noqa: E731
+    par = lambda left, right: ParallelMixer(GroupedAttention(*left[:4], left[2] ** -0.5, sink=True, qk_norm=True, rot=left[4],                    # noqa: E731
+                                                             rot_values=True, gate=True), Retention(*right), 0.5, 0.5, True)
+    a = att(6, 2, 40, Rotary(24, 2e4, 2.0), 70, 6)
+    moe = ExpertFfn(12, 3, 80, "softmax", relu2=True, shared=150)
+    return listed_config("vogerax-mini", "Vogerax", (
+        LayerSpec(par((4, 2, 48, 72, Rotary(40, 1e4, 4.0, 128, 16.0, 1.5)), (3, 56, 40, (0.97, 0.9, 0.995), Rotary(32, 3e4))), DenseFfn(176, relu2=True)),
+        LayerSpec(a, moe), LayerSpec(a, moe, 1), LayerSpec(att(4, 4, 72, Rotary(72, 1e4), 33, 20), None),
+        LayerSpec(par((3, 1, 130, 36, Rotary(64, 5e4, 8.0, 64, 32.0, 1.0)), (2, 96, 136, (0.99, 0.8), Rotary(96, 1e4, 3.0))),
+                  ExpertFfn(9, 2, 128, "softmax", relu2=True)), LayerSpec(att(2, 1, 40, Rotary(16, 1e4), 16, 16), DenseFfn(64, relu2=True))),
+        210, 700, 1e-5, SandwichBlock(3, 8.0))
+
+
+def vogerax_like(name: str, width: int, layers: int, heads: int, kv: int, ff: int, experts: int, top: int, vocab: int, window: int = 2048,
+                 pool: int = 16, r_heads: int = 0) -> ModelConfig:
+    """A Vogerax of real layer sizes: groups of three windowed layers and one of attention beside retention, all heads of 128,
+    experts of width ``ff`` and a shared one of twice that in every layer."""
+    f = ExpertFfn(experts, top, ff, "softmax", relu2=True, shared=2 * ff)
+    near = GroupedAttention(heads, kv, 128, 128, 128 ** -0.5, rot=Rotary(64, 1e6, 4.0), tied=True, window=window, pool=pool)
+    r = r_heads or heads
+    both = ParallelMixer(GroupedAttention(heads, kv, 128, 128, 128 ** -0.5, sink=True, qk_norm=True, rot=Rotary(128, 1e6, 4.0, 8192), rot_values=True,
+                                          gate=True), Retention(r, 128, 128, tuple(1 - 2.0 ** (-5 - 7 * i / r) for i in range(r)), Rotary(128, 1e6)), 0.5, 0.5, True)
+    return listed_config(name, "Vogerax", ([LayerSpec(near, f)] * 3 + [LayerSpec(both, f)]) * (layers // 4), width, vocab, 1e-6, SandwichBlock(2, width ** 0.5))
+
+
+def vogerax_16b() -> ModelConfig:
+    """28 layers, hidden 2048, 16 heads of 128 (4 key heads), 64 experts of 2048, 6 per token, a shared one of 4096."""
+    return vogerax_like("vogerax-16b", 2048, 28, 16, 4, 2048, 64, 6, 102400)
+
+
 def dflash_drafter(target: ModelConfig) -> ModelConfig:
     """DFlash-style block drafter: a 2-layer W4A16 decoder at the target's width."""
     return replace(target, name=target.name + "-dflash", n_layers=2, n_experts=0, top_k=0, expert_ffn=0,
@@ -826,7 +1050,7 @@ def dflash_drafter(target: ModelConfig) -> ModelConfig:
 PRESETS = {
     "tiny-dense": tiny_dense, "tiny-moe": tiny_moe, "small-dense": small_dense, "small-windowed": small_windowed, "small-hybrid": small_hybrid, "small-moe": small_moe, "dense-27b": dense_27b, "hybrid-27b": hybrid_27b, "moe-35b-a3b": moe_35b_a3b,
     "mumusun-mini": mumusun_mini, "mumusun-16b": mumusun_16b, "napadra-mini": napadra_mini, "napadra-7b": napadra_7b,
-    "pefulorn-mini": pefulorn_mini, "pefulorn-7b": pefulorn_7b,
+    "pefulorn-mini": pefulorn_mini, "pefulorn-7b": pefulorn_7b, "vogerax-mini": vogerax_mini, "vogerax-16b": vogerax_16b,
 }
 
 

@@ -22,7 +22,7 @@ from typing import Dict, List, Optional
 import torch
 
 from ..ops import lib as K
-from .config import ModelConfig
+from .config import ModelConfig, SandwichBlock
 from .oracle import rope_tables
 from .weights import ModelWeights, LayerWeights, QLinear
 
@@ -100,7 +100,7 @@ class ListedBuffers:
 class KVCache:
     """Paged KV: per layer ``[page][kv_head][16][D]`` for K and for V (bf16 or int8 + fp32 scales).  Models that list their
     layers keep what their mixers ask for, by name and layer run: planes of the page pool (``pages``: ``[page][kv_head][16][d]``,
-    or ``[page][16][d]`` for rows shared by the heads).  ``states``: recurrent state ``[layers][slot]...`` by name, of every
+    or ``[page][16][d]`` for rows shared by the heads; pooled blocks: fewer rows per page).  ``states``: recurrent state ``[layers][slot]...`` by name, of every
     family that has some."""
 
     def __init__(self, cfg: ModelConfig, n_layers: int, num_pages: int, device, kv_dtype: str = "bf16", n_slots: int = 1):
@@ -117,8 +117,9 @@ class KVCache:
                 raise ValueError(f"{cfg.name} keeps a bf16 (or, served in 32-bit, fp32) cache, not {kv_dtype}")
             ldt = torch.float32 if kv_dtype == "f32" else torch.bfloat16
             for li, sp in enumerate(cfg.run_specs):
-                for name, (heads, cols) in kind(sp.mixer).page_planes(sp.mixer).items():
-                    shape = (num_pages, heads, cfg.page_size, cols) if heads else (num_pages, cfg.page_size, cols)
+                for name, (heads, cols, *per) in kind(sp.mixer).page_planes(sp.mixer).items():
+                    rows = per[0] if per else cfg.page_size
+                    shape = (num_pages, heads, rows, cols) if heads else (num_pages, rows, cols)
                     self.pages[f"{name}{li}"] = torch.zeros(shape, dtype=ldt, device=device)
                 for name, shape in kind(sp.mixer).state_shapes(sp.mixer).items():
                     self.states[f"{name}{li}"] = torch.zeros((1, n_slots) + shape, dtype=torch.float32, device=device)
@@ -195,7 +196,10 @@ class DecoderModel:
                 raise ValueError("models that list their layers run on one GPU with an unquantised head")
             self.listed = ListedLayers(weights, max_pos)
             self.streams = None
-            if cfg.block is not None:
+            if isinstance(cfg.block, SandwichBlock):
+                from .sandwich import SandwichWalk
+                self.streams = SandwichWalk(self.listed)
+            elif cfg.block is not None:
                 from .streams import StreamWalk
                 self.streams = StreamWalk(self.listed)
             self.buf = ListedBuffers(cfg, max_rows, self.listed.wp, self.device, self.listed.dtype)
@@ -598,8 +602,8 @@ class DecoderModel:
         ``listed_logits`` selects from.  ``plan``: how a mixed batch's rows are attended (None: every row on its own).
 
         One residual stream (left in ``resid[:m]``), per layer: the mixer's slices, folded by the kernel that norms them and
-        adds them to the residual; the experts' slots, weighted and folded by the same kernel.  Several streams:
-        ``models.streams.StreamWalk``."""
+        adds them to the residual; the experts' slots, weighted and folded by the same kernel.  Several streams, or one with
+        pre-normed sublayers: ``models.streams.StreamWalk``; norms on both sides of a sublayer: ``models.sandwich.SandwichWalk``."""
         from ..ops import latent as L
         ll, cfg = self.listed, self.cfg
         if self.streams is not None:

@@ -1,13 +1,14 @@
 """Models that list their layers: what every such model shares.
 
 A layer is a mixer and a feed-forward (``LayerSpec``).  Each kind of mixer has a module of its own (``latent``, ``grouped``,
-``mlstm``, ``mingru``, ``channel_delta``, ``wkv``; ``parallel``: two of them side by side) with the same functions: ``shapes`` and
+``mlstm``, ``retention``, ``mingru``, ``channel_delta``, ``wkv``; ``parallel``: two of them side by side) with the same functions: ``shapes`` and
 ``assemble`` (checkpoint tensors, kernel-layout weights), ``tensor_sizes`` (sizes that only the tensors give; not every kind has
 some), ``weight_elems`` and ``scratch_elems`` (the planner's figures), ``page_planes`` (what it keeps per position in the page
 pool), ``state_shapes`` (what it keeps per sequence) and ``Mixer``, whose ``run`` enqueues its kernels for the rows of a step and
 whose ``forms`` are the tables it wants of a mixed batch's prompt segments.  Pages and states belong to layer runs
-(``ModelConfig.layer_runs``): a layer that runs several times in a step has several.
-The residual around the sublayers is ``streams.StreamWalk``, or the layer-normed single stream of
+(``ModelConfig.layer_runs``): a layer that runs several times in a step has several, and a layer that uses another one's weights
+(``LayerSpec.weights_of``) has its own.
+The residual around the sublayers is ``streams.StreamWalk``, ``sandwich.SandwichWalk`` or the layer-normed single stream of
 ``DecoderModel.listed_walk``.  ``Engine`` gives both the rows of a decode step (control block, CUDA graphs) or of a mixed
 batch (``runtime/batch.py``).
 
@@ -30,7 +31,7 @@ from ..ops import gemm as G
 from ..ops import latent as L
 from ..ops import moe as M
 from .config import (ChannelDelta, DenseFfn, ExpertFfn, GroupedAttention, LatentAttention, MatrixLstm, MinGru, ModelConfig,
-                     ParallelMixer, Wkv)
+                     ParallelMixer, Retention, Rotary, SandwichBlock, Wkv)
 from .weights import DenseWeights, ExpertStack, LayerWeights, ModelWeights, interleave16
 
 SMS = 148
@@ -45,9 +46,14 @@ def pad64(n: int) -> int:
 
 def kind(mixer):
     """The module of a mixer's kind."""
-    from . import channel_delta, grouped, latent, mingru, mlstm, parallel, wkv
-    return {LatentAttention: latent, GroupedAttention: grouped, MatrixLstm: mlstm, MinGru: mingru, ParallelMixer: parallel,
-            ChannelDelta: channel_delta, Wkv: wkv}[type(mixer)]
+    from . import channel_delta, grouped, latent, mingru, mlstm, parallel, retention, wkv
+    return {LatentAttention: latent, GroupedAttention: grouped, MatrixLstm: mlstm, Retention: retention, MinGru: mingru,
+            ParallelMixer: parallel, ChannelDelta: channel_delta, Wkv: wkv}[type(mixer)]
+
+
+def pair_order(dims: int, size: int) -> list:
+    """Order of a head's dimensions in the kernels, which rotate neighbours: i and i + dims / 2 next to each other, then the rest."""
+    return [i + half for i in range(dims // 2) for half in (0, dims // 2)] + list(range(dims, size))
 
 
 def sizes_in_tensors(cfg: ModelConfig) -> bool:
@@ -68,26 +74,37 @@ def with_tensor_sizes(cfg: ModelConfig, shape: Callable[[str], tuple]) -> ModelC
 def tensor_shapes(cfg: ModelConfig) -> Dict[str, tuple]:
     """Checkpoint tensors of a listed model, by name."""
     from . import streams
-    h = cfg.hidden
-    norm = (h,) if cfg.block is None or cfg.block.columns else ()
+    h, behind = cfg.hidden, isinstance(cfg.block, SandwichBlock)
+    norm = (h,) if cfg.block is None or cfg.block.columns or behind else ()
+
+    def feed(p, ff, gated):
+        out.update({p + "up": (ff, h), p + "down": (h, ff)})
+        if gated:
+            out[p + "gate"] = (ff, h)
     out = {"embed": (cfg.vocab, h), "final.norm": norm, "head": (cfg.vocab, h)}
     for i, s in enumerate(cfg.layer_specs):
         p, f = f"l{i}.", s.ffn
+        if s.weights_of >= 0:
+            continue
         out[p + "norm1"] = norm
         out.update(kind(s.mixer).shapes(cfg, p + "mix.", s.mixer))
-        if cfg.block is not None:
+        if behind:
+            out.update({p + f"norm{q}b": norm for q in ((1,) if f is None else (1, 2))})
+        elif cfg.block is not None:
             out.update(streams.shapes(cfg, p, s))
         if f is None:
             continue
         out[p + "norm2"] = norm
         if isinstance(f, DenseFfn):
-            out.update({p + "mlp.gate": (f.ff, h), p + "mlp.up": (f.ff, h), p + "mlp.down": (h, f.ff)})
+            feed(p + "mlp.", f.ff, not f.relu2)
             if f.bias:
                 out.update({p + "mlp.gate.b": (f.ff,), p + "mlp.up.b": (f.ff,), p + "mlp.down.b": (h,)})
         else:
             out[p + "mlp.router"] = (f.experts, h)
             for e in range(f.experts):
-                out.update({f"{p}mlp.e{e}.gate": (f.ff, h), f"{p}mlp.e{e}.up": (f.ff, h), f"{p}mlp.e{e}.down": (h, f.ff)})
+                feed(f"{p}mlp.e{e}.", f.ff, not f.relu2)
+            if f.shared:
+                feed(p + "mlp.shared.", f.shared, not f.relu2)
     if cfg.loop is not None:
         out["loop.step"] = (cfg.loop.times, h)
     return out
@@ -112,6 +129,8 @@ class Assembler:
 
     def norm(self, name: str) -> torch.Tensor:
         """Norm weights as factors."""
+        if isinstance(self.cfg.block, SandwichBlock):
+            return self.vec(name, self.wp)
         if self.cfg.block is None or not self.cfg.block.columns:
             return self.vec(name)
         return self.vec(name, self.wp) + (torch.arange(self.wp, device=self.device) < self.cfg.hidden)
@@ -133,24 +152,31 @@ class Assembler:
         out[: w.shape[0], : w.shape[1]] = w
         return out
 
-    def heads(self, w: torch.Tensor, n: int, parts, cols: int) -> torch.Tensor:
-        """Head-major rows: each head's parts (true size, padded size) in turn."""
+    def heads(self, w: torch.Tensor, n: int, parts, cols: int, order=None) -> torch.Tensor:
+        """Head-major rows: each head's parts (true size, padded size) in turn; ``order``: of a head's rows."""
         out = self.zeros(n, sum(p for _, p in parts), cols)
         v = w.reshape(n, sum(s for s, _ in parts), w.shape[1])
+        if order is not None:
+            v = v[:, order]
         src = dst = 0
         for size, pad in parts:
             out[:, dst: dst + size, : w.shape[1]] = v[:, src: src + size]
             src, dst = src + size, dst + pad
         return out.reshape(-1, cols)
 
-    def out_proj(self, name: str, heads: int, size: int, pad: int) -> torch.Tensor:
-        """Output projection over concatenated heads: [wp][heads * pad]."""
-        o = self.zeros(self.wp, heads, pad)
-        o[: self.cfg.hidden, :, :size] = self.t(name).reshape(self.cfg.hidden, heads, size)
+    def out_proj(self, name: str, heads: int, size: int, pad: int, order=None) -> torch.Tensor:
+        """Output projection over concatenated heads: [wp][heads * pad]; ``order``: of a head's columns."""
+        o, w = self.zeros(self.wp, heads, pad), self.t(name).reshape(self.cfg.hidden, heads, size)
+        o[: self.cfg.hidden, :, :size] = w if order is None else w[..., order]
         return o.reshape(self.wp, heads * pad)
 
-    def gate_up(self, gate: str, up: str, ffp: int) -> torch.Tensor:
-        return interleave16(self.padded(self.t(gate), ffp, self.wp), self.padded(self.t(up), ffp, self.wp))
+    def gate_up(self, p: str, ffp: int, gated: bool = True, lo: int = 0) -> torch.Tensor:
+        """What a feed-forward's hidden columns ``lo`` .. are made with."""
+        up = self.padded(self.t(p + "up")[lo: lo + ffp], ffp, self.wp)
+        return interleave16(self.padded(self.t(p + "gate")[lo: lo + ffp], ffp, self.wp), up) if gated else up
+
+    def down(self, p: str, ffp: int, lo: int = 0) -> torch.Tensor:
+        return self.padded(self.t(p + "down")[:, lo: lo + ffp], self.wp, ffp)
 
 
 def assemble(cfg: ModelConfig, get: Callable[[str], torch.Tensor], device, dtype=torch.bfloat16) -> ModelWeights:
@@ -160,25 +186,36 @@ def assemble(cfg: ModelConfig, get: Callable[[str], torch.Tensor], device, dtype
     wp, layers = a.wp, []
     for i, s in enumerate(cfg.layer_specs):
         p, f = f"l{i}.", s.ffn
+        if s.weights_of >= 0:
+            layers.append(None)
+            continue
         lw = LayerWeights(input_norm=a.norm(p + "norm1"), post_norm=a.norm(p + "norm2") if f is not None else None, qkv=None, o=None)
         lw.mixer = kind(s.mixer).assemble(a, p + "mix.", s.mixer)
         if cfg.block is not None and cfg.block.mixing:
             lw.streams = streams.assemble(a, p, s)
+        if isinstance(cfg.block, SandwichBlock):
+            lw.behind = (a.norm(p + "norm1b"), a.norm(p + "norm2b") if f is not None else None)
         if isinstance(f, DenseFfn):
             ffp = pad64(f.ff)
-            lw.dense = DenseWeights(a.gate_up(p + "mlp.gate", p + "mlp.up", ffp), a.padded(a.t(p + "mlp.down"), wp, ffp))
+            lw.dense = DenseWeights(a.gate_up(p + "mlp.", ffp, not f.relu2), a.down(p + "mlp.", ffp))
             if f.bias:
                 lw.dense.bias = interleave16(a.vec(p + "mlp.gate.b", ffp)[:, None], a.vec(p + "mlp.up.b", ffp)[:, None]).view(-1).contiguous()
                 lw.dense.down_bias = a.vec(p + "mlp.down.b", wp)
         elif f is not None:
             ffp = pad64(f.ff)
-            gu, dn = a.zeros(f.experts, 2 * ffp, wp), a.zeros(f.experts, wp, ffp)
-            for e in range(f.experts):
-                q = f"{p}mlp.e{e}."
-                gu[e] = a.gate_up(q + "gate", q + "up", ffp)
-                dn[e, : cfg.hidden, : f.ff] = a.t(q + "down")
+            held = f.experts + f.shared_slots
+            gu, dn = a.zeros(held, (1 if f.relu2 else 2) * ffp, wp), a.zeros(held, wp, ffp)
+            for e in range(held):      # a shared expert is as many of the common width as its hidden columns fill
+                q, lo = (f"{p}mlp.e{e}.", 0) if e < f.experts else (p + "mlp.shared.", (e - f.experts) * ffp)
+                gu[e] = a.gate_up(q, ffp, not f.relu2, lo)
+                dn[e] = a.down(q, ffp, lo)
             lw.moe = ExpertStack(a.padded(a.t(p + "mlp.router"), (f.experts + 7) // 8 * 8, wp), gu, dn)
         layers.append(lw)
+    for i, s in enumerate(cfg.layer_specs):
+        j = i
+        while cfg.layer_specs[j].weights_of >= 0:
+            j = cfg.layer_specs[j].weights_of
+        layers[i] = layers[j]
     w = ModelWeights(cfg, a.padded(a.t("embed"), cfg.vocab, wp), a.padded(a.t("head"), cfg.vocab, wp), a.norm("final.norm"), layers)
     if cfg.loop is not None:
         w.loop_step = torch.zeros(cfg.loop.times, wp, dtype=torch.float32, device=device)
@@ -209,11 +246,12 @@ def padded_weight_elems(cfg: ModelConfig) -> int:
     wp, n = pad64(cfg.hidden), 2 * cfg.vocab * pad64(cfg.hidden)
     for s in cfg.layer_specs:
         f = s.ffn
+        if s.weights_of >= 0:
+            continue
         n += kind(s.mixer).weight_elems(cfg, s.mixer)
-        if isinstance(f, DenseFfn):
-            n += 3 * pad64(f.ff) * wp
-        elif f is not None:
-            n += (f.experts + 7) // 8 * 8 * wp + 3 * f.experts * pad64(f.ff) * wp
+        if f is not None:
+            each = (2 if f.relu2 else 3) * pad64(f.ff) * wp
+            n += each if isinstance(f, DenseFfn) else (f.experts + 7) // 8 * 8 * wp + (f.experts + f.shared_slots) * each
     return n
 
 
@@ -238,11 +276,11 @@ def step_scratch_elems(cfg: ModelConfig, rows: int, keys: int = 0) -> int:
         if isinstance(f, DenseFfn):
             one += rows * 3 * pad64(f.ff)
         elif f is not None:
-            slots = rows * f.top + (f.experts + 1) * 128
+            slots = rows * (f.top + f.shared_slots) + (f.experts + f.shared_slots + 1) * 128
             one += slots * (4 * wp + pad64(f.ff)) + rows * f.experts
         n = max(n, one)
     # layers of unequal sizes keep scratch of their own
-    n = n * len(set(cfg.layer_specs)) + rows * wp * 4
+    n = n * len({(s.mixer, s.ffn) for s in cfg.layer_specs}) + rows * wp * 4
     return n + (rows * wp * (2 * cfg.block.streams + 2) if cfg.block is not None else 0)
 
 
@@ -308,6 +346,14 @@ class ListedLayers:
         self.mixers = [kind(self.cfg.layer_specs[i].mixer).Mixer(self, j, self.cfg.layer_specs[i].mixer, weights.layers[i].mixer)
                        for j, (i, _) in enumerate(self.cfg.layer_runs)]
 
+    def rotation(self, rot: Rotary):
+        """(cos, sin) tables ``[positions][pairs]``, angles in double precision."""
+        if rot not in self.shared:
+            freq, amp = rot.frequencies()
+            angle = torch.arange(self.max_pos, dtype=torch.float64)[:, None] * torch.tensor(freq, dtype=torch.float64)[None, :]
+            self.shared[rot] = tuple((f(angle) * amp).float().to(self.device).contiguous() for f in (torch.cos, torch.sin))
+        return self.shared[rot]
+
     def forms(self):
         """Tables the mixers want of a mixed batch's prompt segments."""
         return sorted({f for m in self.mixers for f in m.forms})
@@ -356,9 +402,18 @@ class ListedLayers:
 
     # ---------------------------------------------------------------- feed-forwards
     def dense(self, sc: ListedScratch, f: DenseFfn, w: DenseWeights, m: int):
-        """Gated feed-forward of the step's rows: fp32 slices of its down projection (without its bias)."""
+        """Feed-forward of the step's rows: fp32 slices of its down projection (without its bias)."""
         h = sc.get("h", m, self.wp)
         n = w.gate_up.shape[0]
+        if f.relu2:
+            act = sc.get("ffn_act", m, n)
+            if self.f32:
+                L.linear_f32(h, w.gate_up, act, m, squared=True)
+            elif m <= L.GEMV_ROWS:
+                L.gemv_bf16(w.gate_up, h, act, m, n, self.wp, epi=L.EPI_RELU2)
+            else:
+                G.gemm_bf16(h, w.gate_up, act, epi=G.EPI_RELU2)
+            return self.linear(sc, "ffn_down", w.down, act, m)
         act = sc.get("ffn_act", m, n // 2)
         if self.f32:
             gu = sc.get("gate_up", m, n)
@@ -371,8 +426,10 @@ class ListedLayers:
         return self.linear(sc, "ffn_down", w.down, act, m)
 
     def experts(self, sc: ListedScratch, f: ExpertFfn, w: ExpertStack, m: int):
-        """Routed experts of the step's rows: arguments of ``sublayer_norm`` that describe the weighted slots."""
-        k, wp, er = f.top, self.wp, w.router.shape[0]
+        """Routed experts of the step's rows (and the shared one, as slots with weight one): arguments of ``sublayer_norm`` that
+        describe the weighted slots."""
+        shared = f.shared_slots
+        k, wp, er = f.top + shared, self.wp, w.router.shape[0]
         ffp = w.down.shape[2]
         i32, f32 = torch.int32, torch.float32
         h = sc.get("h", m, wp)
@@ -380,22 +437,22 @@ class ListedLayers:
         idx, wt = sc.get("topk_idx", m, k, i32), sc.get("topk_w", m, k, f32)
         few = m <= EXPERT_GEMV_ROWS
         if not self.f32 and m <= L.GEMV_ROWS:
-            M.router_rows(w.router, h, logits, m, f.experts, wp, er, f.experts, k, False, False, idx, wt,
+            M.router_rows(w.router, h, logits, m, f.experts, wp, er, f.experts, f.top, shared, False, idx, wt,
                           sc.get("ticket", 1, 1, i32), rule=f.rule)
         else:
             if self.f32:
                 L.linear_f32(h, w.router, logits, m)
             else:
                 G.gemm_bf16(h, w.router, logits, epi=G.EPI_F32)
-            M.route(logits, er, m, f.experts, k, idx, wt, rule=f.rule)
+            M.route(logits, er, m, f.experts, f.top, idx, wt, rule=f.rule, shared=shared)
         if self.f32:
             act, y = sc.get("act", m * k, ffp, mult=k), sc.get("y", m * k, wp, mult=k)
-            L.linear_f32_experts(w.gate_up, idx.view(-1), m * k, h, k, act, True)
-            L.linear_f32_experts(w.down, idx.view(-1), m * k, act, 1, y, False)
+            L.linear_f32_experts(w.gate_up, idx.view(-1), m * k, h, k, act, L.ACT_RELU2 if f.relu2 else L.ACT_SILU)
+            L.linear_f32_experts(w.down, idx.view(-1), m * k, act, 1, y, L.ACT_NONE)
             return dict(y=y, slots=k, row_elems=wp, slot_w=wt)
         if few:
             act = sc.get("act", m * k, ffp, mult=k)
-            L.gemv_bf16_experts(w.gate_up, idx, m * k, h, k, act, 2 * ffp, wp, epi=L.EPI_SILU)
+            L.gemv_bf16_experts(w.gate_up, idx, m * k, h, k, act, w.gate_up.shape[1], wp, epi=L.EPI_RELU2 if f.relu2 else L.EPI_SILU)
             s = self._splits.get((wp, ffp, "experts"))
             if s is None:
                 s = self._splits[(wp, ffp, "experts")] = min(2, L.gemv_splits(wp, ffp))
@@ -403,7 +460,7 @@ class ListedLayers:
             L.gemv_bf16_experts(w.down, idx, m * k, act, 1, y, wp, ffp, splits=s)
             return dict(y=y, slots=k, slices=s, row_elems=s * wp, slice_elems=wp, slot_w=wt)
         # expert-sorted rows in blocks of 128 for the grouped GEMMs; counts stay on the device
-        e = f.experts
+        e = f.experts + shared
         blk = (m * k + 127) // 128 + e
         cap = (max(m, sc.fixed) * k + 127) // 128 + e
         meta = sc.get(f"moe_tables_{e}_{k}", 2 * e + 3 * cap + 2, 1, i32).view(-1)
@@ -416,6 +473,6 @@ class ListedLayers:
         M.sort(idx, m, k, e, blk, counts, rank, base, be, br, bn, n_blk, total)
         M.scatter(idx, rank, base, m, k, h, wp, row_of, xs)
         blocks = (be, br, bn, n_blk, blk)
-        G.gemm_grouped_bf16(xs, w.gate_up, act, blocks, epi=G.EPI_SILU_MUL)
+        G.gemm_grouped_bf16(xs, w.gate_up, act, blocks, epi=G.EPI_RELU2 if f.relu2 else G.EPI_SILU_MUL)
         G.gemm_grouped_bf16(act, w.down, y, blocks)
         return dict(y=y, slots=k, row_elems=wp, slot_w=wt, row_of=row_of)

@@ -98,8 +98,9 @@ class LatentWeights:
 
 @dataclass
 class GroupedWeights:
-    """A grouped-query attention mixer, unquantised, heads padded to whole 64s."""
-    qkv: Optional[torch.Tensor]    # [heads * dk + kv_heads * (dk + dv)][Wp], or the queries' rows alone
+    """A grouped-query attention mixer, unquantised, heads padded to whole 64s; rotated pairs are neighbours."""
+    qkv: Optional[torch.Tensor]    # [heads * dk + kv_heads * (dk + dv)][Wp], without values that are the keys and with [heads * dv]
+                                   # rows of a gate behind; or the queries' rows alone
     o: Optional[torch.Tensor]      # [Wp][heads * dv]
     slope2: Optional[torch.Tensor]     # fp32 [heads] distance bias times log2 e
     sink2: Optional[torch.Tensor]      # fp32 [heads] sinks times log2 e
@@ -108,6 +109,14 @@ class GroupedWeights:
     k_norm: Optional[torch.Tensor] = None    # fp32 [dk]
     r1: Optional[torch.Tensor] = None        # fp32 [heads] logarithmic distance bias
     r2: Optional[torch.Tensor] = None
+
+
+@dataclass
+class RetentionWeights:
+    """A retention mixer, unquantised, heads padded to whole 64s; rotated pairs of q and k are neighbours."""
+    proj: Optional[torch.Tensor]   # [heads * 2 (dk + dv)][Wp]: q, k, v, gate
+    o: Optional[torch.Tensor]      # [Wp][heads * dv]
+    decay: torch.Tensor            # fp32 [2][heads]: decays and their log2
 
 
 @dataclass
@@ -130,11 +139,14 @@ class MinGruWeights:
 
 @dataclass
 class ParallelWeights:
-    """Two mixers side by side: their input projections one below the other, their output projections side by side."""
+    """Two mixers side by side: their input projections one below the other, their output projections side by side -- or, where each
+    one's result has a norm of its own, one below the other (equal columns) or apart."""
     proj: torch.Tensor
-    o: torch.Tensor
+    o: Optional[torch.Tensor]
     left: object                   # the two mixers' other weights
     right: object
+    norms: Optional[list] = None   # fp32 [Wp] each
+    outs: Optional[list] = None    # output projections apart
 
 
 @dataclass
@@ -163,8 +175,8 @@ class WkvWeights:
 
 @dataclass
 class DenseWeights:
-    """Unquantised gated feed-forward, padded to whole 64s."""
-    gate_up: torch.Tensor          # [2 * ffp][Wp], interleave16
+    """Unquantised feed-forward, padded to whole 64s."""
+    gate_up: torch.Tensor          # [2 * ffp][Wp], interleave16; without a gate [ffp][Wp]
     down: torch.Tensor             # [Wp][ffp]
     bias: Optional[torch.Tensor] = None          # fp32 [2 * ffp], interleave16
     down_bias: Optional[torch.Tensor] = None     # fp32 [Wp]
@@ -184,8 +196,8 @@ class StreamWeights:
 class ExpertStack:
     """Unquantised routed experts of one layer, padded to whole 64s."""
     router: torch.Tensor           # [E rounded up to 8][Wp]
-    gate_up: torch.Tensor          # [E][2 * ffp][Wp], interleave16
-    down: torch.Tensor             # [E][Wp][ffp]
+    gate_up: torch.Tensor          # [E][2 * ffp][Wp], interleave16; without a gate [E][ffp][Wp]
+    down: torch.Tensor             # [E][Wp][ffp]; runs of a shared expert's columns behind the routed ones
 
 
 @dataclass
@@ -210,6 +222,7 @@ class LayerWeights:
     moe: Optional[ExpertStack] = None
     dense: Optional[DenseWeights] = None
     streams: Optional[StreamWeights] = None
+    behind: Optional[tuple] = None                 # norms behind the mixer and the feed-forward (``SandwichBlock``)
 
 
 @dataclass
@@ -236,7 +249,7 @@ class ModelWeights:
 
     def nbytes(self) -> int:
         tot = self.embed.numel() * 2 + self.lm_head.numel() * 2
-        for lw in self.layers + (self.mtp.layers if self.mtp else []):
+        for lw in {id(x): x for x in self.layers + (self.mtp.layers if self.mtp else [])}.values():      # layers may share weights
             for ql in (lw.qkv, lw.o, lw.gate_up, lw.down):
                 if ql is not None:
                     tot += ql.nbytes
@@ -254,7 +267,9 @@ class ModelWeights:
 
 def part_nbytes(part) -> int:
     """Bytes of a container of tensors and containers."""
-    return sum(t.numel() * t.element_size() if isinstance(t, torch.Tensor) else part_nbytes(t) for t in vars(part).values() if t is not None)
+    def one(t):
+        return t.numel() * t.element_size() if isinstance(t, torch.Tensor) else sum(map(one, t)) if isinstance(t, list) else part_nbytes(t)
+    return sum(one(t) for t in vars(part).values() if t is not None)
 
 
 def _norm_weight(h, device, gen=None):

@@ -1,7 +1,8 @@
 // Causal flash attention for prompt chunks on tcgen05 / TMEM: over the paged KV cache (head_dim 128), over contiguous
 // key / value rows with their own head sizes (latent attention, whose keys and values are expanded before), and over
 // paged keys and values of any sizes for the segments of a mixed batch (tiles that name their sequence; optional distance
-// bias (linear or logarithmic), sink and chunked mask, as in paged.cu).
+// bias (linear or logarithmic), sink, chunked mask, window with pooled blocks before it, values turned back and a gate, as
+// in paged.cu; a batch's pooled blocks come as contiguous rows and are walked ahead of the window's pages).
 //
 //   O[r] = softmax( q[r] . K[0 .. pos(r)]^T / sqrt(D) ) V[0 .. pos(r)]      pos(r) = pos0 + r
 //
@@ -45,6 +46,13 @@ struct AttnPfParams {
   int ldo;             // paged segments: elements of an output row
   float mult;          // paged segments: factor of the result
   int dn;              // columns of a head in the key matrix (a multiple of 64; the shared part fills up the head)
+  // paged segments: the window is p.window; pool > 0: pooled blocks before it, pool_row[tile] the first one's row in map_pk / map_pv
+  int pool;
+  const int* pool_row;
+  const float *turn_cos, *turn_sin;    // [positions][half]: pair i of a result is turned back (half 0: none)
+  int half;
+  const __nv_bfloat16* gate;           // rows of ldg elements [H][DV], or null
+  int ldg;
 };
 constexpr int kTileWords = 4;
 
@@ -120,6 +128,7 @@ template <class F>
 __global__ void __launch_bounds__(kThreads2, 1)
 attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                          const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_r,
+                         const __grid_constant__ CUtensorMap map_pk, const __grid_constant__ CUtensorMap map_pv,
                          const AttnPfParams p) {
   constexpr int KVS = F::KVS, NDK = F::NDK, NDV = F::NDV;
   extern __shared__ uint8_t smem_raw[];
@@ -148,8 +157,10 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     if (F::SEG) block_table += (size_t)krow * p.max_blocks;
   }
   // key tiles each query tile needs, counted from the first tile any of the CTA's rows needs
-  const int t0 = F::SEG ? (p.chunk > 0 ? (pos0 - pos0 % p.chunk) / BK2 : 0)
-                        : p.window > 0 ? max(0, pos0 + row0 - p.window + 1) / BK2 : 0;
+  const int t_first = F::SEG && p.chunk > 0 ? (pos0 - pos0 % p.chunk) / BK2 : p.window > 0 ? max(0, pos0 + row0 - p.window + 1) / BK2 : 0;
+  // pooled blocks the last row sees, in tiles ahead of the others
+  const int n_pool = F::SEG && p.pool > 0 ? (max(0, pos0 + C - p.window) / p.pool + BK2 - 1) / BK2 : 0;
+  const int t0 = t_first - n_pool;
   int n_w[2];
   n_w[0] = (pos0 + min(row0 + BQ, C) - 1) / BK2 + 1 - t0;
   n_w[1] = F::NW > 1 && row0 + BQ < C ? (pos0 + min(row0 + 2 * BQ, C) - 1) / BK2 + 1 - t0 : 0;
@@ -205,8 +216,10 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         // patterns, and 0 * NaN in P V would poison the row.
         constexpr int n_pages = BK2 / 16;
         int rowc[n_pages];
+        const bool pooled = F::SEG && i < n_pool;
+        const int pr = pooled ? __ldg(p.pool_row + blockIdx.x) + i * BK2 : 0;
 #pragma unroll
-        for (int pg = 0; pg < n_pages && F::PAGED; ++pg) {
+        for (int pg = 0; pg < n_pages && F::PAGED && !pooled; ++pg) {
           const int pi = (t0 + i) * n_pages + pg;
           const int page = pi < p.max_blocks ? __ldg(block_table + pi) : 0;
           rowc[pg] = (page * p.n_kv + kh) * 16;
@@ -216,7 +229,10 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         if (i >= KVS) ok = mbar_wait(b_kempty + 8 * s, ph ^ 1, ERR_ATTN_WAIT);
         if (!ok) break;
         mbar_expect_tx(b_kfull + 8 * s, F::K_BYTES);
-        if (F::PAGED) {
+        if (pooled) {          // rows past the batch's last block are zero, those of another segment masked out
+#pragma unroll
+          for (int c = 0; c < NDK; ++c) tma_load_2d(k_s + c * (BK2 * 128), &map_pk, (kh * NDK + c) * 64, pr, b_kfull + 8 * s);
+        } else if (F::PAGED) {
 #pragma unroll
           for (int pg = 0; pg < n_pages; ++pg) {
 #pragma unroll
@@ -236,7 +252,10 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
           break;
         }
         mbar_expect_tx(b_vfull + 8 * s, F::V_BYTES);
-        if (F::PAGED) {
+        if (pooled) {
+#pragma unroll
+          for (int c = 0; c < NDV; ++c) tma_load_2d(v_s + c * (BK2 * 128), &map_pv, (kh * NDV + c) * 64, pr, b_vfull + 8 * s);
+        } else if (F::PAGED) {
 #pragma unroll
           for (int pg = 0; pg < n_pages; ++pg) {
 #pragma unroll
@@ -337,11 +356,14 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const int rowg = row0 + w * BQ + r;   // row inside the chunk
     const int qpos = pos0 + rowg;
     // the row's keys: qlo <= key <= qpos
-    const int qlo = F::SEG ? (p.chunk > 0 ? qpos - qpos % p.chunk : 0) : p.window > 0 ? qpos - p.window + 1 : 0;
+    const int qlo = F::SEG && p.chunk > 0 ? qpos - qpos % p.chunk : p.window > 0 ? qpos - p.window + 1 : 0;
+    const int q_pool = F::SEG && p.pool > 0 ? max(qlo, 0) / p.pool : 0;      // pooled blocks the row sees
     const bool row_ok = rowg < C;
     const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
     const int first_pos = pos0 + row0 + w * BQ;             // position of the tile's first row
-    const int last_lo = !F::SEG || p.chunk <= 0 ? 0 : first_pos + BQ - 1 - (first_pos + BQ - 1) % p.chunk;   // first key of its last row
+    // first key of its last row
+    const int last_lo = F::SEG && p.chunk > 0 ? first_pos + BQ - 1 - (first_pos + BQ - 1) % p.chunk : p.window > 0 ? first_pos + BQ - p.window : 0;
+    const int first_pool = F::SEG && p.pool > 0 ? max(first_pos - p.window + 1, 0) / p.pool : 0;      // blocks its first row sees
     const float slope = !F::SEG ? 0.f : p.r1 ? p.r1[head] : p.slope2 ? p.slope2[head] : 0.f, r2 = F::SEG && p.r1 ? p.r2[head] : 0.f;
     const int nt = n_w[w];
     // float [tile w][tile parity][half][128 rows]: the halves of a row exchange their maxima (and, at the end, sums)
@@ -354,7 +376,8 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       if (ok) ok = mbar_wait(b_sfull(w, sb), (i >> 1) & 1, ERR_ATTN_WAIT);
       tc_fence_after();
       APROF_T(t1_);
-      const int key0 = (t0 + i) * BK2 + half * 32;
+      const bool pooled = F::SEG && i < n_pool;
+      const int key0 = (pooled ? i : t0 + i) * BK2 + half * 32;
       // this thread's 32 scores, once: the score buffer goes back to the tensor pipe as soon as they are in registers
       uint32_t v[32];
       if (ok) {
@@ -388,7 +411,13 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         }
         }
       }
-      if (key0 + 31 > first_pos || (F::SEG ? key0 < last_lo : p.window > 0 && key0 < first_pos + BQ - p.window)) {
+      if (pooled) {
+        if (key0 + 31 >= first_pool) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j)
+            if (key0 + j >= q_pool) v[j] = 0xff800000u;
+        }
+      } else if (key0 + 31 > first_pos || key0 < last_lo) {
 #pragma unroll
         for (int j = 0; j < 32; ++j) {
           const int kj = key0 + j;
@@ -511,6 +540,29 @@ attn_prefill_pair_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         B2_TMEM_LD_32(t_o(w) + lane_addr + c * 32, o);
         tmem_ld_wait();
         if (row_ok) {
+          if (F::SEG && (p.half || p.gate)) {
+            const float *cs = p.turn_cos + (size_t)qpos * p.half + c * 16, *sn = p.turn_sin + (size_t)qpos * p.half + c * 16;
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+              if (c * 16 + j < p.half) {
+                const float x = __uint_as_float(o[2 * j]), y = __uint_as_float(o[2 * j + 1]), a = __ldg(cs + j), b = __ldg(sn + j);
+                o[2 * j] = __float_as_uint(x * a + y * b);
+                o[2 * j + 1] = __float_as_uint(y * a - x * b);
+              }
+            if (p.gate) {
+              const uint4* gt = reinterpret_cast<const uint4*>(p.gate + (size_t)(qrow + rowg) * p.ldg + head * F::DV + c * 32);
+#pragma unroll
+              for (int j = 0; j < 4; ++j) {
+                const uint4 g = __ldg(gt + j);
+                const uint32_t gg[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                  o[8 * j + 2 * e] = __float_as_uint(__uint_as_float(o[8 * j + 2 * e]) * bf16_lo(gg[e]));
+                  o[8 * j + 2 * e + 1] = __float_as_uint(__uint_as_float(o[8 * j + 2 * e + 1]) * bf16_hi(gg[e]));
+                }
+              }
+            }
+          }
 #pragma unroll
           for (int j = 0; j < 4; ++j)
             *reinterpret_cast<uint4*>(dst + c * 32 + 8 * j) = make_uint4(
@@ -560,7 +612,8 @@ int make_map_bf16(CUtensorMap* map, const void* ptr, uint64_t rows, uint64_t col
 
 template <class F>
 int launch_form(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mr,
-                const AttnPfParams& p, int columns, int heads, cudaStream_t st) {
+                const AttnPfParams& p, int columns, int heads, cudaStream_t st, const CUtensorMap* mpk = nullptr,
+                const CUtensorMap* mpv = nullptr) {
   static bool configured[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -569,7 +622,7 @@ int launch_form(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap&
     if (e != cudaSuccess) return (int)e;
     configured[dev & 63] = true;
   }
-  attn_prefill_pair_kernel<F><<<dim3(columns, heads), kThreads2, F::SMEM, st>>>(mq, mk, mv, mr, p);
+  attn_prefill_pair_kernel<F><<<dim3(columns, heads), kThreads2, F::SMEM, st>>>(mq, mk, mv, mr, mpk ? *mpk : mk, mpv ? *mpv : mv, p);
   return (int)cudaGetLastError();
 }
 
@@ -654,44 +707,65 @@ extern "C" int b2_attn_segments_per_tile(int dk, int dv) {
 }
 
 template <int NDK>
-static int launch_segments(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const AttnPfParams& p, int ndv,
-                           int n_tiles, cudaStream_t st) {
+static int launch_segments(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap* mpk,
+                           const CUtensorMap* mpv, const AttnPfParams& p, int ndv, int n_tiles, cudaStream_t st) {
   constexpr int NW = NDK <= 3 ? 2 : 1;
   switch (ndv) {
-    case 1: return launch_form<Form<NDK, 1, NW, NDK <= 2 ? 4 : 3, true, true>>(mq, mk, mv, mv, p, n_tiles, p.n_q, st);
-    case 2: return launch_form<Form<NDK, 2, NW, NDK <= 2 ? 4 : 3, true, true>>(mq, mk, mv, mv, p, n_tiles, p.n_q, st);
-    case 3: return launch_form<Form<NDK, 3, 1, NDK == 4 ? 2 : 3, true, true>>(mq, mk, mv, mv, p, n_tiles, p.n_q, st);
-    case 4: return launch_form<Form<NDK, 4, 1, NDK == 4 ? 2 : 3, true, true>>(mq, mk, mv, mv, p, n_tiles, p.n_q, st);
+    case 1: return launch_form<Form<NDK, 1, NW, NDK <= 2 ? 4 : 3, true, true>>(mq, mk, mv, mv, p, n_tiles, p.n_q, st, mpk, mpv);
+    case 2: return launch_form<Form<NDK, 2, NW, NDK <= 2 ? 4 : 3, true, true>>(mq, mk, mv, mv, p, n_tiles, p.n_q, st, mpk, mpv);
+    case 3: return launch_form<Form<NDK, 3, 1, NDK == 4 ? 2 : 3, true, true>>(mq, mk, mv, mv, p, n_tiles, p.n_q, st, mpk, mpv);
+    case 4: return launch_form<Form<NDK, 4, 1, NDK == 4 ? 2 : 3, true, true>>(mq, mk, mv, mv, p, n_tiles, p.n_q, st, mpk, mpv);
   }
   return -1;
 }
 
 // q: bf16 rows of ldq elements (the first H * dk of each are the queries); k / v caches [num_pages][G][16][dk | dv];
 // block_table [slots][max_blocks]; out: rows of ldo elements, H * dv of them written.  tiles: n_tiles x 4 ints: first row of q, rows, position of that
-// row, slot.
+// row, slot.  extra (host structure, or null): window; pooled blocks as rows pk [pool_rows][G * dk], pv [pool_rows][G * dv], the
+// first one of tile i's sequence at row pool_row[i]; results turned back by tables [positions][half], gates [rows][ldg].
+struct B2SegExtra {
+  int window, pool, pool_rows;
+  const int* pool_row;
+  const void *pk, *pv;
+  const float *cos, *sin;
+  int half;
+  const void* gate;
+  int ldg;
+};
 extern "C" int b2_attn_prefill_segments(const void* q, int ldq, const void* k_cache, const void* v_cache,
                                         const int* block_table, int max_blocks, void* out, const int* tiles, int n_tiles,
                                         int q_rows, int H, int G, int dk, int dv, int num_pages, float scale, int chunk,
                                         const float* slope2, const float* sink2, const float* r1, const float* r2, int ldo,
-                                        float mult, void* stream) {
+                                        float mult, const B2SegExtra* extra, void* stream) {
+  const B2SegExtra x = extra ? *extra : B2SegExtra{};
   if (!b2_attn_segments_per_tile(dk, dv) || n_tiles < 1 || H < 1 || H % G || ldq % 8 || ldq < H * dk || chunk < 0 || ldo % 8 || ldo < H * dv ||
       (r1 && !r2))
     return -1;
-  CUtensorMap mq, mk, mv;
+  if (x.window < 0 || x.pool < 0 || (x.window && chunk) || (x.pool && (!x.window || slope2 || r1)) || x.half < 0 || 2 * x.half > dv ||
+      (x.half && (!x.cos || !x.sin)) || (x.gate && (x.ldg % 8 || x.ldg < H * dv)) ||
+      (x.pool && (x.pool_rows < 0 || (x.pool_rows && (!x.pk || !x.pv || !x.pool_row)))))
+    return -2;
+  CUtensorMap mq, mk, mv, mpk, mpv;
   int rc = make_map_bf16(&mq, q, (uint64_t)q_rows, (uint64_t)H * dk, BQ, (uint64_t)ldq);
   if (!rc) rc = make_map_bf16(&mk, k_cache, (uint64_t)num_pages * G * 16, (uint64_t)dk, 16);
   if (!rc) rc = make_map_bf16(&mv, v_cache, (uint64_t)num_pages * G * 16, (uint64_t)dv, 16);
+  const bool pooled = x.pool && x.pool_rows;      // no rows: no row of the batch sees a block
+  if (!rc && pooled) rc = make_map_bf16(&mpk, x.pk, (uint64_t)x.pool_rows, (uint64_t)G * dk, BK2);
+  if (!rc && pooled) rc = make_map_bf16(&mpv, x.pv, (uint64_t)x.pool_rows, (uint64_t)G * dv, BK2);
   if (rc) return rc;
   AttnPfParams p = {};
   p.block_table = block_table; p.max_blocks = max_blocks; p.n_q = H; p.n_kv = G; p.scale_log2 = scale * 1.4426950408889634f;
   p.out = (__nv_bfloat16*)out; p.tiles = tiles; p.chunk = chunk; p.slope2 = slope2; p.sink2 = sink2;
   p.r1 = r1; p.r2 = r2; p.ldo = ldo; p.mult = mult;
+  p.window = x.window; p.pool = pooled ? x.pool : 0; p.pool_row = x.pool_row;
+  p.turn_cos = x.cos; p.turn_sin = x.sin; p.half = x.half; p.gate = (const __nv_bfloat16*)x.gate; p.ldg = x.ldg;
   cudaStream_t st = (cudaStream_t)stream;
+  const CUtensorMap *a = pooled ? &mpk : nullptr, *b = pooled ? &mpv : nullptr;
   switch (dk / 64) {
-    case 1: return launch_segments<1>(mq, mk, mv, p, dv / 64, n_tiles, st);
-    case 2: return launch_segments<2>(mq, mk, mv, p, dv / 64, n_tiles, st);
-    case 3: return launch_segments<3>(mq, mk, mv, p, dv / 64, n_tiles, st);
-    case 4: return launch_segments<4>(mq, mk, mv, p, dv / 64, n_tiles, st);
+    case 1: return launch_segments<1>(mq, mk, mv, a, b, p, dv / 64, n_tiles, st);
+    case 2: return launch_segments<2>(mq, mk, mv, a, b, p, dv / 64, n_tiles, st);
+    case 3: return launch_segments<3>(mq, mk, mv, a, b, p, dv / 64, n_tiles, st);
+    case 4: return launch_segments<4>(mq, mk, mv, a, b, p, dv / 64, n_tiles, st);
   }
   return -1;
 }

@@ -272,6 +272,7 @@ __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
   __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
   return *reinterpret_cast<uint32_t*>(&v);
 }
+__device__ __forceinline__ float relu2(float x) { return fmaxf(x, 0.f) * fmaxf(x, 0.f); }
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + __expf(-x)); }
 // Gated product of two projections: f(g') (u' + shift) with g' = min(g, limit), u' = clamp(u, -limit, limit);
 // f(x) = x sigmoid(alpha x), or with gelu 1 the tanh form of GELU: x (1 + tanh(y)) / 2 = x / (1 + e^(-2 y)) with

@@ -41,7 +41,7 @@ constexpr int BM = 128;
 constexpr int BKB = 128;  // bytes of K per stage row (64 bf16 or 128 int8)
 constexpr int kThreads = 192;
 
-enum Epi : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SILU_MUL = 2, EPI_RESID_ADD = 3, EPI_RS_PUSH = 4, EPI_EP_RETURN = 5, EPI_GLU = 6 };
+enum Epi : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SILU_MUL = 2, EPI_RESID_ADD = 3, EPI_RS_PUSH = 4, EPI_EP_RETURN = 5, EPI_GLU = 6, EPI_RELU2 = 7 };
 
 struct GemmParams {
   int M, N, K;       // K in elements
@@ -425,6 +425,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
               } else {
                 for (int j = 0; j < 32 && n0 + j < p.N; ++j) f[j] += __bfloat162float(rs[j]);
               }
+            }
+            if (p.epi == EPI_RELU2) {
+#pragma unroll
+              for (int j = 0; j < 32; ++j) f[j] = relu2(f[j]);
             }
             if (n0 + 32 <= p.N) {
 #pragma unroll

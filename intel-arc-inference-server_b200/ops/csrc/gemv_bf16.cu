@@ -6,8 +6,8 @@
 //                      activations as A and the weight rows as B, in a k order chosen so that a lane's 16-byte vector is
 //                      its fragment (as in the lm_head kernel).  The first weight vectors are requested before the
 //                      kernel waits for its predecessor.
-//                      Epilogues: fp32 slices [split][m][N] (the consumer folds them), bf16, or SiLU(gate) * up (or another
-//                      gated product) over interleave16 rows.  Batched form: batch b multiplies activation row b / x_div with the weight of
+//                      Epilogues: fp32 slices [split][m][N] (the consumer folds them), bf16, relu(x)^2 as bf16, or SiLU(gate) *
+//                      up (or another gated product) over interleave16 rows.  Batched form: batch b multiplies activation row b / x_div with the weight of
 //                      expert ids[b] (mixture-of-experts decode rows).
 //   linear_f32_kernel  C[M][N] = A[M][K] B[N][K]^T in fp32 FMA arithmetic (models served in 32-bit)
 //   linear_f32_rows    the batched expert form of it: one warp per output
@@ -20,7 +20,7 @@ using namespace b2;
 
 namespace {
 
-enum Epi : int { EPI_PART = 0, EPI_BF16 = 1, EPI_SILU = 2, EPI_GLU = 3 };
+enum Epi : int { EPI_PART = 0, EPI_BF16 = 1, EPI_SILU = 2, EPI_GLU = 3, EPI_RELU2 = 4 };
 
 struct GemvBfParams {
   const __nv_bfloat16* w;    // [N][K], or [E][N][K] in the batched form
@@ -124,7 +124,7 @@ __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const GemvBfPara
 #pragma unroll
     for (int e = 0; e < 4; ++e) red[(warp * 16 + g + 8 * (e >> 1)) * 33 + 8 * j + 2 * t + (e & 1)] = acc[j][e];
   __syncthreads();
-  if (p.epi >= EPI_SILU) {
+  if (p.epi == EPI_SILU || p.epi == EPI_GLU) {
     for (int i = threadIdx.x; i < M * 16; i += kWarps * 32) {
       const int m = i >> 4, c = i & 15;
       float gt = 0.f, up = 0.f;
@@ -148,8 +148,8 @@ __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const GemvBfPara
 #pragma unroll
     for (int q = 0; q < kWarps; ++q) v += red[(q * 16 + m) * 33 + c];
     if (n0 + c >= p.N) continue;
-    if (p.epi == EPI_BF16)
-      reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)(batched ? batch : m) * p.N + n0 + c] = __float2bfloat16(v);
+    if (p.epi == EPI_BF16 || p.epi == EPI_RELU2)
+      reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)(batched ? batch : m) * p.N + n0 + c] = __float2bfloat16(p.epi == EPI_BF16 ? v : relu2(v));
     else if (batched)
       reinterpret_cast<float*>(p.out)[((size_t)batch * p.splits + split) * p.N + n0 + c] = v;
     else
@@ -160,7 +160,7 @@ __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const GemvBfPara
 // ------------------------------------------------------------------ 32-bit linears
 // 64 x 64 tile, 256 threads, 4 x 4 outputs per thread, K in steps of 16
 __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict__ a, const float* __restrict__ b,
-                                                         float* __restrict__ c, int M, int N, int K, int ldc) {
+                                                         float* __restrict__ c, int M, int N, int K, int ldc, int squared) {
   __shared__ float as[16][68], bs[16][68];
   pdl_wait();
   pdl_launch_dependents();
@@ -191,13 +191,15 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict
   for (int i = 0; i < 4; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j)
-      if (m0 + ty * 4 + i < M && n0 + tx * 4 + j < N) c[(size_t)(m0 + ty * 4 + i) * ldc + n0 + tx * 4 + j] = acc[i][j];
+      if (m0 + ty * 4 + i < M && n0 + tx * 4 + j < N) c[(size_t)(m0 + ty * 4 + i) * ldc + n0 + tx * 4 + j] = squared ? relu2(acc[i][j]) : acc[i][j];
 }
 
-// batch b: out[b][n] = x[b / x_div] . w[ids[b]][n]; one warp per output.  silu: w rows interleave16, out [b][N / 2]
+// batch b: out[b][n] = x[b / x_div] . w[ids[b]][n]; one warp per output.  act 1: SiLU(gate) * up of w rows interleave16, out
+// [b][N / 2]; 2: relu(x)^2
 __global__ void __launch_bounds__(256) linear_f32_rows_kernel(const float* __restrict__ w, const int* __restrict__ ids,
                                                               const float* __restrict__ x, float* __restrict__ out, int N,
-                                                              int K, int ldx, int x_div, int do_silu) {
+                                                              int K, int ldx, int x_div, int act) {
+  const bool do_silu = act == 1;
   pdl_wait();
   pdl_launch_dependents();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, b = blockIdx.y;
@@ -213,7 +215,7 @@ __global__ void __launch_bounds__(256) linear_f32_rows_kernel(const float* __res
   }
   u = warp_sum(u);
   v = warp_sum(v);
-  if (lane == 0) out[(size_t)b * outs + o] = do_silu ? u / (1.f + expf(-u)) * v : u;
+  if (lane == 0) out[(size_t)b * outs + o] = do_silu ? u / (1.f + expf(-u)) * v : act == 2 ? relu2(u) : u;
 }
 
 __global__ void __launch_bounds__(256) glu_rows_f32_kernel(const float* __restrict__ in, float* __restrict__ out, int N, const Glu p) {
@@ -269,11 +271,11 @@ extern "C" int b2_gemv_bf16_splits(int N, int K) {
   return (steps + per - 1) / per;       // no empty slices
 }
 
-// out: epi 0: fp32 [splits][M][N] (batched: [batch][splits][N]); epi 1: bf16 [M][N]; epi 2: bf16 [M][N / 2] (both splits = 1)
+// out: epi 0: fp32 [splits][M][N] (batched: [batch][splits][N]); epi 1, 4: bf16 [M][N]; epi 2: bf16 [M][N / 2] (all splits = 1)
 extern "C" int b2_gemv_bf16(const void* w, const int* ids, int batches, const void* x, int ldx, int x_div, void* out, int M,
                             int N, int K, int splits, int epi, void* stream) {
   if (K % 64 || N < 1 || M < 1 || M > 16 || splits < 1 || ldx % 8 || (epi != EPI_PART && splits != 1)) return -1;
-  if (epi == EPI_SILU && N % 32) return -2;
+  if ((epi == EPI_SILU && N % 32) || epi < EPI_PART || epi > EPI_RELU2 || epi == EPI_GLU) return -2;
   if (ids && (M != 1 || x_div < 1)) return -3;
   GemvBfParams p{(const __nv_bfloat16*)w, ids, (const __nv_bfloat16*)x, out, M, N, K, ldx, splits, epi, x_div, 0, 1, 0, {}};
   return M <= 8 ? launch_gemv<1>(p, ids ? batches : 1, (cudaStream_t)stream)
@@ -306,16 +308,16 @@ extern "C" int b2_glu_rows_f32(const float* in, float* out, int M, int N, float 
                    Glu{limit, alpha, shift, gelu, bias});
 }
 
-extern "C" int b2_linear_f32(const float* a, const float* w, float* c, int M, int N, int K, int ldc, void* stream) {
+extern "C" int b2_linear_f32(const float* a, const float* w, float* c, int M, int N, int K, int ldc, int squared, void* stream) {
   if (K % 16 || M < 1 || N < 1 || ldc < N) return -1;
   return b2_launch(linear_f32_kernel, dim3((N + 63) / 64, (M + 63) / 64), dim3(256), 0, (cudaStream_t)stream, true, a, w, c,
-                   M, N, K, ldc);
+                   M, N, K, ldc, squared);
 }
 
 extern "C" int b2_linear_f32_rows(const float* w, const int* ids, int batches, const float* x, int ldx, int x_div, float* out,
-                                  int N, int K, int do_silu, void* stream) {
-  if (batches < 1 || batches > 65535 || x_div < 1 || (do_silu && N % 32)) return -1;
-  const int outs = do_silu ? N / 2 : N;
+                                  int N, int K, int act, void* stream) {
+  if (batches < 1 || batches > 65535 || x_div < 1 || act < 0 || act > 2 || (act == 1 && N % 32)) return -1;
+  const int outs = act == 1 ? N / 2 : N;
   return b2_launch(linear_f32_rows_kernel, dim3((outs + 7) / 8, batches), dim3(256), 0, (cudaStream_t)stream, true, w, ids, x,
-                   out, N, K, ldx, x_div, do_silu);
+                   out, N, K, ldx, x_div, act);
 }

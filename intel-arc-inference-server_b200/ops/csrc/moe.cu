@@ -131,19 +131,25 @@ __device__ __forceinline__ void route_row(const float* __restrict__ lrow, int E,
 template <bool PLAIN>
 __global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict__ logits, int ld, int T, int E, int k,
                                                         const RouteRule rule, int* __restrict__ topk_idx,
-                                                        float* __restrict__ topk_w) {
+                                                        float* __restrict__ topk_w, int shared) {
   pdl_wait();
   pdl_launch_dependents();
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (warp >= T) return;
-  route_row<PLAIN>(logits + (size_t)warp * ld, E, k, rule, topk_idx + (size_t)warp * k, topk_w + (size_t)warp * k, lane);
+  const size_t at = (size_t)warp * (k + shared);
+  route_row<PLAIN>(logits + (size_t)warp * ld, E, k, rule, topk_idx + at, topk_w + at, lane);
+  for (int i = lane; i < shared; i += 32) {
+    topk_idx[at + k + i] = E + i;
+    topk_w[at + k + i] = 1.f;
+  }
 }
 
 // ---------------------------------------------------------------- decode rows: router logits + routing in one launch
 // logits[m][r] = x[m] . W[r] for the R router rows (E experts, then the shared expert's gate row when there is one):
 // a warp per router row, eight token rows per pass over the weights.  The CTA that finishes last (a ticket) then
 // routes every token row.  With `shared_slot` each row gets one more slot: expert id E (the shared expert, see the
-// batched GEMV's alt weights) with weight sigmoid(gate logit), or 1 without a gate row.
+// batched GEMV's alt weights) with weight sigmoid(gate logit), or 1 without a gate row; with shared_slot n > 1 (no gate
+// row) n more slots, ids E .. E + n - 1 with weight 1: runs of a shared expert's hidden columns.
 struct RouterRowsParams {
   const __nv_bfloat16* w;   // [R][H]
   const __nv_bfloat16* x;   // [M][H]
@@ -218,9 +224,9 @@ __global__ void __launch_bounds__(256) moe_router_rows_kernel(const RouterRowsPa
   for (int m = warp; m < p.M; m += 8) {
     const float* lrow = p.logits + (size_t)m * p.ld;
     route_row<PLAIN>(lrow, p.E, p.k, p.rule, p.topk_idx + (size_t)m * stride, p.topk_w + (size_t)m * stride, lane);
-    if (p.shared_slot && lane == 0) {
-      p.topk_idx[(size_t)m * stride + p.k] = p.E;
-      p.topk_w[(size_t)m * stride + p.k] = p.has_gate ? 1.f / (1.f + __expf(-__ldcg(lrow + p.E))) : 1.f;
+    for (int i = lane; i < p.shared_slot; i += 32) {
+      p.topk_idx[(size_t)m * stride + p.k + i] = p.E + i;
+      p.topk_w[(size_t)m * stride + p.k + i] = p.has_gate ? 1.f / (1.f + __expf(-__ldcg(lrow + p.E))) : 1.f;
     }
   }
 }
@@ -400,20 +406,22 @@ static bool route_ok(int E, int k, const RouteRule& r) {
   return r.groups <= 32 && E % r.groups == 0 && r.keep >= 1 && r.keep <= r.groups && k <= r.keep * (E / r.groups);
 }
 
+// shared: more slots per row, ids E .. with weight 1
 extern "C" int b2_moe_route(const float* logits, int ld, int T, int E, int k, int sigmoid, int groups, int keep, int renorm,
-                            int* topk_idx, float* topk_w, void* stream) {
+                            int* topk_idx, float* topk_w, int shared, void* stream) {
   const RouteRule rule{sigmoid, groups, keep, renorm};
-  if (!route_ok(E, k, rule)) return -1;
+  if (!route_ok(E, k, rule) || shared < 0) return -1;
   const int blocks = (T * 32 + 255) / 256;
   return b2_launch(route_plain(rule) ? moe_route_kernel<true> : moe_route_kernel<false>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, true, logits, ld, T, E, k,
-                   rule, topk_idx, topk_w);
+                   rule, topk_idx, topk_w, shared);
 }
 
 extern "C" int b2_moe_router_rows(const void* w, const void* x, float* logits, int M, int R, int H, int ld, int E, int k,
                                   int shared_slot, int has_gate, int sigmoid, int groups, int keep, int renorm,
                                   int* topk_idx, float* topk_w, int* ticket, void* stream) {
   const RouteRule rule{sigmoid, groups, keep, renorm};
-  if (!route_ok(E, k, rule) || H % 8 || M < 1 || R < E + (has_gate ? 1 : 0) || ld < R) return -1;
+  if (!route_ok(E, k, rule) || H % 8 || M < 1 || R < E + (has_gate ? 1 : 0) || ld < R || shared_slot < 0 || (has_gate && shared_slot > 1))
+    return -1;
   RouterRowsParams p{(const __nv_bfloat16*)w, (const __nv_bfloat16*)x, logits, M, R, H, ld, E, k, shared_slot, has_gate,
                      rule, topk_idx, topk_w, ticket};
   return b2_launch(route_plain(rule) ? moe_router_rows_kernel<true> : moe_router_rows_kernel<false>, dim3((R + 7) / 8), dim3(256), 0, (cudaStream_t)stream, true, p);

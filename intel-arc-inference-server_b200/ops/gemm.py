@@ -9,6 +9,7 @@ import torch
 from . import lib as K
 
 EPI_BF16, EPI_F32, EPI_SILU_MUL, EPI_RESID_ADD, EPI_RS_PUSH, EPI_EP_RETURN = 0, 1, 2, 3, 4, 5
+EPI_RELU2 = 7
 
 
 def _launch(a, b, c, m, n, k, ldc, i8, epi, resid=None, a_scale=None, b_scale=None, blocks=None, n_experts=0, bn=0):
@@ -25,7 +26,7 @@ def _launch(a, b, c, m, n, k, ldc, i8, epi, resid=None, a_scale=None, b_scale=No
 def gemm_bf16(a: torch.Tensor, b: torch.Tensor, c: torch.Tensor, epi: int = EPI_BF16,
               resid: Optional[torch.Tensor] = None, bn: int = 0):
     """``c = a @ b.T`` with ``a`` ``[M][K]``, ``b`` ``[N][K]`` bf16.  ``epi``: bf16 / fp32 store,
-    SiLU(gate)*up over interleave16 columns (``c`` is ``[M][N/2]``), or ``resid + a b^T`` in bf16."""
+    SiLU(gate)*up over interleave16 columns (``c`` is ``[M][N/2]``), ``resid + a b^T`` in bf16, or relu(x)^2 in bf16."""
     m, k = a.shape
     n = b.shape[0]
     _launch(a, b, c, m, n, k, c.stride(0), False, epi, resid=resid, bn=bn)

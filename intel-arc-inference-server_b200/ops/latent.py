@@ -12,7 +12,8 @@ import torch
 from . import lib as K
 
 GEMV_ROWS = 16                       # most rows of the weight-streaming form
-EPI_PART, EPI_BF16, EPI_SILU = 0, 1, 2
+EPI_PART, EPI_BF16, EPI_SILU, EPI_RELU2 = 0, 1, 2, 4
+ACT_NONE, ACT_SILU, ACT_RELU2 = 0, 1, 2
 
 
 def _f32(t: torch.Tensor) -> int:
@@ -26,7 +27,8 @@ def gemv_splits(n: int, k: int) -> int:
 
 
 def gemv_bf16(w, x, out, m: int, n: int, k: int, splits: int = 1, epi: int = EPI_PART):
-    """``x @ w.T`` for ``m`` <= 16 rows: fp32 slices ``[splits][m][n]``, bf16, or SiLU(gate) * up of interleave16 rows."""
+    """``x @ w.T`` for ``m`` <= 16 rows: fp32 slices ``[splits][m][n]``, bf16, relu(x)^2 as bf16, or SiLU(gate) * up of
+    interleave16 rows."""
     K._check(K.lib().b2_gemv_bf16(K._p(w), None, 1, K._p(x), x.stride(0), 1, K._p(out), m, n, k, splits, epi, K._stream()),
              "gemv_bf16")
 
@@ -55,19 +57,20 @@ def gemv_bf16_experts(w, ids, batches: int, x, x_div: int, out, n: int, k: int, 
                                   K._stream()), "gemv_bf16_experts")
 
 
-def linear_f32(a, w, c, m: int):
-    """``c[:m] = a[:m] @ w.T`` in fp32 (``c``: rows of any stride)."""
+def linear_f32(a, w, c, m: int, squared: bool = False):
+    """``c[:m] = a[:m] @ w.T`` in fp32 (``c``: rows of any stride); ``squared``: relu of it, squared."""
     n, k = w.shape
-    K._check(K.lib().b2_linear_f32(K._p(a), K._p(w), K._p(c), m, n, k, c.stride(0), K._stream()), "linear_f32")
+    K._check(K.lib().b2_linear_f32(K._p(a), K._p(w), K._p(c), m, n, k, c.stride(0), int(squared), K._stream()), "linear_f32")
 
 
-def linear_f32_experts(w, ids, batches: int, x, x_div: int, out, silu: bool):
+def linear_f32_experts(w, ids, batches: int, x, x_div: int, out, act: int):
+    """Batch ``b``: row ``b // x_div`` of ``x`` against expert ``ids[b]``; ``act``: ``ACT_SILU`` (of interleave16 rows), ``ACT_RELU2``."""
     e, n, k = w.shape
     for b0 in range(0, batches, 65520 // x_div * x_div):      # grid rows of one launch
         nb = min(batches - b0, 65520 // x_div * x_div)
-        outs = n // 2 if silu else n
+        outs = n // 2 if act == ACT_SILU else n
         K._check(K.lib().b2_linear_f32_rows(K._p(w), K._p(ids[b0:]), nb, K._p(x[b0 // x_div:]), x.stride(0), x_div,
-                                            K._p(out.view(-1)[b0 * outs:]), n, k, int(silu), K._stream()), "linear_f32_rows")
+                                            K._p(out.view(-1)[b0 * outs:]), n, k, act, K._stream()), "linear_f32_rows")
 
 
 # ----------------------------------------------------------------------------- norms and residual rows

@@ -12,11 +12,11 @@ SOFTMAX_RENORM = (0, 1, 1, 1)     # routing rule: (sigmoid scores, expert groups
 
 
 def route(logits: torch.Tensor, ld: int, t: int, e: int, k: int, topk_idx: torch.Tensor, topk_w: torch.Tensor,
-          rule=SOFTMAX_RENORM):
+          rule=SOFTMAX_RENORM, shared: int = 0):
     """Scores of the first ``e`` columns (softmax, or a sigmoid each) -> top-k (ties to the lower id) -> weights.
     ``rule``: (sigmoid, groups, keep, renorm); with ``groups`` > 1 only experts of the ``keep`` groups with the largest
-    sums of their two best scores can be chosen."""
-    K._check(K.lib().b2_moe_route(K._p(logits), ld, t, e, k, *rule, K._p(topk_idx), K._p(topk_w), K._stream()), "moe_route")
+    sums of their two best scores can be chosen.  ``shared``: each row gets as many more slots, ids ``e`` .. with weight 1."""
+    K._check(K.lib().b2_moe_route(K._p(logits), ld, t, e, k, *rule, K._p(topk_idx), K._p(topk_w), shared, K._stream()), "moe_route")
 
 
 def sort(topk_idx, t, k, e, max_blk, counts, rank, expert_base, blk_expert, blk_row0, blk_rows, n_blk, total_rows):
@@ -56,7 +56,8 @@ def router_rows(w, x, logits, m, r, h, ld, e, k, shared_slot, has_gate, topk_idx
                 rule=SOFTMAX_RENORM):
     """Decode rows: router logits (``r`` rows of ``w``: the experts, then the shared expert's gate row) and the
     routing of every row in one launch.  ``shared_slot``: each row gets slot k = (expert id ``e``, sigmoid(gate logit)
-    or 1), so ``topk_idx`` / ``topk_w`` hold k + 1 entries per row.  ``ticket``: one zeroed int32 word."""
+    or 1), so ``topk_idx`` / ``topk_w`` hold k + 1 entries per row; a number above 1: that many more slots, ids ``e`` .. with
+    weight 1.  ``ticket``: one zeroed int32 word."""
     K._check(K.lib().b2_moe_router_rows(K._p(w), K._p(x), K._p(logits), m, r, h, ld, e, k, int(shared_slot), int(has_gate), *rule,
                                         K._p(topk_idx), K._p(topk_w), K._p(ticket), K._stream()), "moe_router_rows")
 

@@ -7,7 +7,9 @@ row by row, longer ones as prompt segments; both kinds share every linear and ev
 ``DecoderModel.listed_walk``, as in decode steps.
 
 Forms: ``("keys", window, rows per tile)`` lists the cache rows the segments see, to be expanded, and query tiles over them;
-``("tiles", chunk, rows per tile)`` query tiles over the pages; ``("chunks",)`` the segments of a recurrence.
+``("tiles", chunk, rows per tile)`` query tiles over the pages; ``("pooled", window, pool, rows per tile)`` query tiles and the pooled
+blocks that rows of a segment see before their window; ``("chunks",)`` the segments of a recurrence, in chunks of 64 rows or
+``("chunks", rows)``.
 
 Takes the place of the reference's chunk walk (src/runtime/prefill/step.cc:102-319) for models that list their layers.
 """
@@ -45,6 +47,18 @@ class TilePlan:
 
 
 @dataclass
+class PoolPlan:
+    """Query tiles over a window of the pages and the pooled blocks before it: slots and blocks of the segments' pooled rows, one
+    segment after another, and the first row of every tile's segment."""
+    n_tiles: int
+    tiles: torch.Tensor
+    n_pool: int
+    preq: torch.Tensor
+    block: torch.Tensor
+    first: torch.Tensor
+
+
+@dataclass
 class ChunkPlan:
     """Segments of a recurrence: [n][4] (first row, rows, slot, first chunk); chunks in total and in the longest one."""
     n_segs: int
@@ -71,14 +85,31 @@ def segment_tiles(segments: Sequence[Tuple[int, int, int]], chunk: int, per: int
     return tiles
 
 
-def segment_chunks(segments: Sequence[Tuple[int, int, int]]):
+def segment_chunks(segments: Sequence[Tuple[int, int, int]], per: int = CHUNK):
     """Prompt segments of a recurrence as (first row, rows, slot, first chunk), and the number of chunks."""
     out, row, chunks = [], 0, 0
     for slot, _, n in segments:
         out.append((row, n, slot, chunks))
         row += n
-        chunks += (n + CHUNK - 1) // CHUNK
+        chunks += (n + per - 1) // per
     return out, chunks
+
+
+def segment_blocks(segments: Sequence[Tuple[int, int, int]], window: int, pool: int, per: int):
+    """Query tiles as in ``segment_tiles``, every tile's first pooled row, and the slots and numbers of the blocks that the segments'
+    last rows see, one segment after another."""
+    preq, block, tiles = [], [], []
+    qrow = rows = 0
+    for slot, p, n in segments:
+        blocks = max(0, p + n - window) // pool if pool else 0
+        preq.append(np.full(blocks, slot))
+        block.append(np.arange(blocks))
+        tiles += [(qrow + r, min(per, n - r), p + r, slot, rows) for r in range(0, n, per)]
+        qrow += n
+        rows += blocks
+    cost = lambda t: min(t[2], window) + t[1] + (max(0, t[2] + t[1] - window) // pool if pool else 0)      # noqa: E731
+    tiles.sort(key=lambda t: -cost(t))                     # tiles with many keys first
+    return [t[:4] for t in tiles], [t[4] for t in tiles], np.concatenate(preq), np.concatenate(block)
 
 
 def segment_keys(segments: Sequence[Tuple[int, int, int]], window: int, per: int):
@@ -131,9 +162,14 @@ class BatchRunner:
             elif form[0] == "tiles":
                 tiles = segment_tiles(segs, form[1], form[2])
                 tables[form] = lambda cut, nt=len(tiles), t=add(tiles): TilePlan(nt, cut(t))
+            elif form[0] == "pooled":
+                tiles, first, preq, block = segment_blocks(segs, *form[1:])
+                where = add(tiles), add(preq), add(block), add(first)
+                tables[form] = lambda cut, nt=len(tiles), n=len(block), w=where: PoolPlan(nt, cut(w[0]), n, cut(w[1]), cut(w[2]), cut(w[3]))
             else:
-                rows, chunks = segment_chunks(segs)
-                most = max((n + CHUNK - 1) // CHUNK for _, _, n in segs)
+                per = form[1] if len(form) > 1 else CHUNK
+                rows, chunks = segment_chunks(segs, per)
+                most = max((n + per - 1) // per for _, _, n in segs)
                 tables[form] = lambda cut, n=len(rows), t=add(rows), c=chunks, most=most: ChunkPlan(n, cut(t), c, most)
         return np.concatenate(parts), spans, tables
 

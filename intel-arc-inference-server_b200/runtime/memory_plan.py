@@ -68,7 +68,8 @@ def kv_bytes_per_page(cfg: ModelConfig, kv_dtype: str, tp: int = 1) -> int:
     if cfg.layer_specs:
         from ..models.listed import kind
         planes = [pl for s in cfg.run_specs for pl in kind(s.mixer).page_planes(s.mixer).values()]
-        return sum(max(1, heads) * cols for heads, cols in planes) * cfg.page_size * (4 if kv_dtype == "f32" else 2)
+        rows = lambda pl: pl[2] if len(pl) > 2 else cfg.page_size        # noqa: E731
+        return sum(max(1, pl[0]) * pl[1] * rows(pl) for pl in planes) * (4 if kv_dtype == "f32" else 2)
     per_tok_head = cfg.head_dim * (1 if kv_dtype == "int8" else 2) + (4 if kv_dtype == "int8" else 0)
     return (cfg.n_layers - cfg.n_gdn_layers + cfg.mtp_layers) * 2 * (cfg.n_kv_heads // tp) * per_tok_head * cfg.page_size
 
