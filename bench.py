@@ -101,7 +101,7 @@ def main():
     ap.add_argument("--model", default="dense-27b")
     ap.add_argument("--depth", type=int, default=4096, help="context length the decode steps run at")
     ap.add_argument("--prefill-len", type=int, default=4096)
-    ap.add_argument("--what", default="all", help="decode | prefill | prefill32k | moe | w4 | spec | spec65k | batch32k | prefix | hybrid | mumusun | napadra | pefulorn | tp | ep | pp | replica | all")
+    ap.add_argument("--what", default="all", help="decode | prefill | prefill32k | moe | w4 | spec | spec65k | batch32k | prefix | hybrid | mumusun | napadra | pefulorn | vogerax | tp | ep | pp | replica | all")
     ap.add_argument("--kv-cache", default="bf16")
     ap.add_argument("--int8-head", action="store_true")
     ap.add_argument("--prefill-backend", default="auto")
@@ -213,7 +213,7 @@ def main():
             return {"ms_per_step": r["ms_per_step"], "tokens_per_s": 1e3 / r["ms_per_step"],
                     "e2e_tokens_per_s": 1e3 / r["e2e_ms_per_step"], "depth": a.depth, "config": r["config"]}
         guarded("moe_decode", moe_decode)
-    if world == 1 and args.what in ("mumusun", "napadra", "pefulorn"):
+    if world == 1 and args.what in ("mumusun", "napadra", "pefulorn", "vogerax"):
         # models that list their layers beside the closest other model at equal size (not part of "all")
         from b200serve.utils import bench_listed
         guarded(args.what, lambda: bench_listed.run(release, args.what))

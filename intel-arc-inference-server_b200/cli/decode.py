@@ -106,14 +106,14 @@ def _profile(eng, f, first):
     targets = [(n, K, n) for n in names]        # label, module, function
     if eng.cfg.layer_specs:
         from ..ops import latent as L, moe as M
-        from ..ops import channel_rec as C, mingru as U, mlstm as R, paged as P, streams as S
+        from ..ops import channel_rec as C, mingru as U, mlstm as R, paged as P, retention as T, sandwich as B, streams as S
         targets += [(n, L, n) for n in ("embed_rows", "gemv_bf16", "prep", "absorb", "rows", "simple", "merge", "sublayer_norm",
                                         "gemv_bf16_experts", "layer_norm_rows", "linear_f32", "linear_f32_experts", "gemv_bf16_glu",
                                         "gemv_bf16_planes", "glu_rows_f32")]
         targets += [("router_rows", M, "router_rows"), ("streams_embed", S, "embed"), ("streams_boundary", S, "boundary"),
                     ("kv_append", P, "append"), ("paged_rows", P, "rows"), ("paged_simple", P, "simple"), ("mlstm_step", R, "step"),
                     ("kv_norm", P, "norm"), ("mingru", U, "scan"), ("delta_prep", C, "delta_prep"), ("wkv_prep", C, "wkv_prep"),
-                    ("channel_scan", C, "scan")]
+                    ("channel_scan", C, "scan"), ("retention_step", T, "step"), ("sandwich_boundary", B, "boundary")]
     pending = []
 
     def wrap(name, fn):

@@ -176,28 +176,52 @@ struct Chunk {
   static_assert(SMEM <= 227 * 1024, "shared memory of one CTA");
 };
 
-// keys (rotated, scaled, times decay^(rows - 1 - row) with `lg`) and values of a chunk into shared tiles; rows past it are zero
+// `cols` columns from `src` (rows `ld` apart) of `rows_all` rows into a shared tile; rows from `rows` on are zero.  ROT: rotated by
+// the rows' positions from `pos` on, times `scale`, and with DECAY times decay^(rows - 1 - row).  Several loads in flight.
+template <int LIMBS, bool ROT, bool DECAY>
+__device__ __forceinline__ void stage(const RetentionParams& p, uint8_t* tile, uint32_t lo_off, const float* src, size_t ld, int rows_all, int cols,
+                                      int rows, int pos, float scale, float lg) {
+  constexpr int U = ROT ? 4 : 8;
+  const int quads = cols / 4, n = rows_all * quads;
+  for (int i0 = threadIdx.x; i0 < n; i0 += U * kThreads) {
+    float4 x[U];
+    float t[ROT ? U : 1][4];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + u * kThreads, r = i / quads, c = (i - r * quads) * 4;
+      x[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < n && r < rows) x[u] = __ldcg(reinterpret_cast<const float4*>(src + r * ld + c));
+      if constexpr (ROT) {
+        t[u][0] = t[u][2] = 1.f;
+        t[u][1] = t[u][3] = 0.f;
+        const int k = c >> 1;
+        const size_t at = (size_t)(pos + min(r, rows - 1)) * p.half + k;
+        if (k < p.half) { t[u][0] = p.cos[at]; t[u][1] = p.sin[at]; }
+        if (k + 1 < p.half) { t[u][2] = p.cos[at + 1]; t[u][3] = p.sin[at + 1]; }
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + u * kThreads, r = i / quads, c = (i - r * quads) * 4;
+      if (i >= n) break;
+      if constexpr (ROT) {
+        const float f = DECAY ? scale * decayed(lg, rows - 1 - r) : scale;
+        x[u] = make_float4((x[u].x * t[u][0] - x[u].y * t[u][1]) * f, (x[u].y * t[u][0] + x[u].x * t[u][1]) * f,
+                           (x[u].z * t[u][2] - x[u].w * t[u][3]) * f, (x[u].w * t[u][2] + x[u].z * t[u][3]) * f);
+      }
+      put4<LIMBS>(tile, lo_off, rows_all, r, c, x[u]);
+    }
+  }
+}
+
+// keys and values of a chunk
 template <int KB, int VB, bool DECAY>
 __device__ __forceinline__ void stage_kv(const RetentionParams& p, uint8_t* k_s, uint8_t* v_s, int row0, int rows, int h, int vb, float lg) {
   using C = Chunk<KB, VB>;
   const int Hk = p.H * C::dk;
-  for (int i = threadIdx.x; i < CH * (C::dk / 4); i += kThreads) {
-    const int r = i / (C::dk / 4), c = (i - r * (C::dk / 4)) * 4;
-    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (r < rows) {
-      x = __ldcg(reinterpret_cast<const float4*>(p.part + (size_t)(row0 + r) * p.N + p.col + Hk + h * C::dk + c));
-      x = rotated(p, x, p.pos[row0 + r], c);
-      const float f = p.k_scale * (DECAY ? decayed(lg, rows - 1 - r) : 1.f);
-      x = make_float4(x.x * f, x.y * f, x.z * f, x.w * f);
-    }
-    put4<2>(k_s, C::K_LIMB, CH, r, c, x);
-  }
-  for (int i = threadIdx.x; i < CH * (C::DVB / 4); i += kThreads) {
-    const int r = i / (C::DVB / 4), c = (i - r * (C::DVB / 4)) * 4;
-    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (r < rows) x = __ldcg(reinterpret_cast<const float4*>(p.part + (size_t)(row0 + r) * p.N + p.col + 2 * Hk + h * p.dv + vb * C::DVB + c));
-    put4<1>(v_s, 0, CH, r, c, x);
-  }
+  const float* row = p.part + (size_t)row0 * p.N + p.col;
+  stage<2, true, DECAY>(p, k_s, C::K_LIMB, row + Hk + h * C::dk, p.N, CH, C::dk, rows, p.pos[row0], p.k_scale, lg);
+  stage<1, false, false>(p, v_s, 0, row + 2 * Hk + h * p.dv + vb * C::DVB, p.N, CH, C::DVB, rows, 0, 1.f, 0.f);
 }
 
 // grid (chunks of the longest segment, heads x value blocks, segments)
@@ -292,33 +316,23 @@ __global__ void __launch_bounds__(kThreads) retention_chunk_kernel(const Retenti
   const int row0 = seg[0] + blockIdx.x * CH, rows = min(CH, seg[1] - (int)blockIdx.x * CH);
   const float lg = p.decay[p.H + h];
   const uint32_t base = smem_u32(sp);
+  // this warp's queries as operand fragments, two limbs, through the shared tile
+  const int lo_row = warp * 16;
+  uint32_t q[2][KB * 4][4];
+  stage<2, true, false>(p, sp, C::K_LIMB, p.part + (size_t)row0 * p.N + p.col + h * C::dk, p.N, CH, C::dk, rows, p.pos[row0], 1.f, 0.f);
+  __syncthreads();
+#pragma unroll
+  for (int k = 0; k < KB * 4; ++k) {
+    const int r = lo_row + 8 * (mi & 1) + (lane & 7);
+    const uint32_t at = base + (k >> 2) * CH * 128 + r * 128 + (((2 * (k & 3) + (mi >> 1)) ^ (r & 7)) << 4);
+    ldsm_x4(at, q[0][k]);
+    ldsm_x4(at + C::K_LIMB, q[1][k]);
+  }
+  __syncthreads();
   // the state ahead of the chunk, two limbs
   const float* kv = p.kv + ((size_t)(seg[3] + blockIdx.x) * p.H + h) * C::dk * p.dv + vb * C::DVB;
   const bool zero = blockIdx.x == 0 && p.pos[seg[0]] == 0;
-  if (!zero)
-    for (int i = threadIdx.x; i < C::dk * (C::DVB / 4); i += kThreads) {
-      const int r = i / (C::DVB / 4), c = (i - r * (C::DVB / 4)) * 4;
-      put4<2>(sp, C::S_LIMB, C::dk, r, c, __ldcg(reinterpret_cast<const float4*>(kv + (size_t)r * p.dv + c)));
-    }
-  // this warp's queries as operand fragments, two limbs: a register holds a rotated pair
-  const int lo_row = warp * 16;
-  uint32_t q[2][KB * 4][4];
-#pragma unroll
-  for (int k = 0; k < KB * 4; ++k)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int r = lo_row + g + 8 * (e & 1), c = k * 16 + 2 * t + 8 * (e >> 1);
-      float2 x = make_float2(0.f, 0.f);
-      if (r < rows) {
-        x = __ldcg(reinterpret_cast<const float2*>(p.part + (size_t)(row0 + r) * p.N + p.col + h * C::dk + c));
-        if ((c >> 1) < p.half) {
-          const size_t at = (size_t)p.pos[row0 + r] * p.half + (c >> 1);
-          const float a = p.cos[at], b = p.sin[at];
-          x = make_float2(x.x * a - x.y * b, x.y * a + x.x * b);
-        }
-      }
-      split2(x.x, x.y, q[0][k][e], q[1][k][e]);
-    }
+  if (!zero) stage<2, false, false>(p, sp, C::S_LIMB, kv, p.dv, C::dk, C::DVB, C::dk, 0, 1.f, 0.f);
   __syncthreads();
   float o[VB * 8][4];
 #pragma unroll

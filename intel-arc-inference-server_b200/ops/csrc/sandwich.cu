@@ -9,8 +9,9 @@
 // its source (`vocab` > 0: value rows are tokens), no residual and no post norm; the last one leaves the head's input and no
 // residual.
 //
-// A row is handled by one CTA, or by a cluster of up to 8 CTAs that share the columns and exchange their sums of squares through
-// distributed shared memory (few rows).
+// Two forms.  Groups of whole 128s: a CTA keeps a row in registers, every warp a run of 128 columns at a time, and meets once per
+// norm; few rows get a thread per four columns.  Any other size goes through shared memory; few rows are then shared by a cluster
+// of up to 8 CTAs, which exchange their sums of squares through distributed shared memory.
 #include "common.cuh"
 
 #include <cooperative_groups.h>
@@ -241,8 +242,187 @@ __global__ void __launch_bounds__(kThreads) sandwich_kernel(const SandwichParams
   if (CS > 1) cg::this_cluster().sync();    // no CTA leaves while another may still read its statistics
 }
 
+// ------------------------------------------------------------------ groups of whole 128s
+constexpr int kRuns = 64;       // runs of 128 columns of a row
+
+// The sum of `per` neighbouring runs from `first`
+__device__ __forceinline__ float run_sums(const float* stat, int first, int per) {
+  float a = 0.f;
+  for (int i = threadIdx.x & 31; i < per; i += 32) a += stat[first + i];
+  return warp_sum(a);
+}
+
+// NT threads; Q: runs of a warp; TF: values of a column in flight; MB: CTAs per SM
+template <bool TWO, int NT, int Q, int TF, int MB>
+__global__ void __launch_bounds__(NT, MB) sandwich_runs_kernel(const SandwichParams p) {
+  constexpr int NS = TWO ? 2 : 1, NW = NT / 32;
+  __shared__ float stat[4][kRuns];           // sums of squares of the runs: of the two results, of y, of x'
+  const int m = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int runs = p.ld / 128, group = p.size / 128;      // runs of the row, of a group
+  pdl_launch_dependents();
+  pdl_wait();
+  auto squares = [&](const float4 (&v)[Q], float* to) {
+#pragma unroll
+    for (int u = 0; u < Q; ++u) {
+      const float s = warp_sum(v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w);
+      if (lane == 0 && u * NW + warp < runs) to[u * NW + warp] = s;
+    }
+  };
+  // 1 / root mean square of the group of every run of this warp
+  auto factors = [&](float* of, float (&inv)[Q]) {
+    int have = -1;
+    float last = 0.f;
+#pragma unroll
+    for (int u = 0; u < Q; ++u) {
+      const int g = min(u * NW + warp, runs - 1) / group;
+      if (g != have) last = 1.f / sqrtf(run_sums(of, g * group, group) / (float)p.size + p.eps);
+      have = g;
+      inv[u] = last;
+    }
+  };
+  float4 y[NS][Q], x[Q];
+#pragma unroll
+  for (int u = 0; u < Q; ++u) {
+    const bool in = u * NW + warp < runs && p.x_in;
+    const int c = (u * NW + warp) * 128 + lane * 4;
+    x[u] = in ? __ldcg(reinterpret_cast<const float4*>(p.x_in + (size_t)m * p.ld + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+#pragma unroll
+  for (int s = 0; s < NS; ++s) {
+    const B2Source& q = p.src[s];
+    const int terms = q.slots * q.slices;
+#pragma unroll
+    for (int u = 0; u < Q; ++u) y[s][u] = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int t0 = 0; t0 < terms; t0 += TF) {       // slots in order, slices of a slot in order
+      long long off[TF];
+      float wt[TF];
+#pragma unroll
+      for (int i = 0; i < TF; ++i) {
+        const int t = min(t0 + i, terms - 1), slot = q.slices > 1 ? t / q.slices : t;
+        long long r = q.row_of ? q.row_of[m * q.slots + slot] : (long long)m * q.slots + slot;
+        if (p.vocab > 0 && (r < 0 || r >= p.vocab)) {
+          if (threadIdx.x == 0 && p.flag) p.flag[0] = 1;
+          r = 0;
+        }
+        off[i] = r * q.row + (t - slot * q.slices) * q.slice;
+        wt[i] = t0 + i < terms ? (q.slot_w ? q.slot_w[m * q.slots + slot] : 1.f) : 0.f;
+      }
+#pragma unroll
+      for (int u = 0; u < Q; ++u) {
+        if (u * NW + warp >= runs) break;
+        const int c = (u * NW + warp) * 128 + lane * 4;
+        float4 v[TF];
+#pragma unroll
+        for (int i = 0; i < TF; ++i) v[i] = t0 + i < terms ? value4(q, off[i] + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < TF; ++i) {
+          y[s][u].x = fmaf(wt[i], v[i].x, y[s][u].x);
+          y[s][u].y = fmaf(wt[i], v[i].y, y[s][u].y);
+          y[s][u].z = fmaf(wt[i], v[i].z, y[s][u].z);
+          y[s][u].w = fmaf(wt[i], v[i].w, y[s][u].w);
+        }
+      }
+    }
+  }
+  if (TWO) {
+#pragma unroll
+    for (int s = 0; s < NS; ++s) squares(y[s], stat[s]);
+    __syncthreads();
+    float f[NS];
+#pragma unroll
+    for (int s = 0; s < NS; ++s) {
+      f[s] = p.src[s].factor;
+      if (p.src[s].norm) f[s] /= sqrtf(run_sums(stat[s], 0, runs) / (float)p.width + p.eps);
+    }
+#pragma unroll
+    for (int u = 0; u < Q; ++u) {
+      if (u * NW + warp >= runs) break;
+      const int c = (u * NW + warp) * 128 + lane * 4;
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int s = 0; s < NS; ++s) {
+        const float4 w = p.src[s].norm ? *reinterpret_cast<const float4*>(p.src[s].norm + c) : make_float4(1.f, 1.f, 1.f, 1.f);
+        a.x = fmaf(y[s][u].x * f[s], w.x, a.x);
+        a.y = fmaf(y[s][u].y * f[s], w.y, a.y);
+        a.z = fmaf(y[s][u].z * f[s], w.z, a.z);
+        a.w = fmaf(y[s][u].w * f[s], w.w, a.w);
+      }
+      y[0][u] = a;
+    }
+  } else {
+    const float f = p.src[0].factor;
+#pragma unroll
+    for (int u = 0; u < Q; ++u) y[0][u] = make_float4(y[0][u].x * f, y[0][u].y * f, y[0][u].z * f, y[0][u].w * f);
+  }
+  float inv[Q];
+  if (p.post) {
+    squares(y[0], stat[2]);
+    __syncthreads();
+    factors(stat[2], inv);
+  }
+#pragma unroll
+  for (int u = 0; u < Q; ++u) {
+    if (u * NW + warp >= runs) break;
+    const int c = (u * NW + warp) * 128 + lane * 4;
+    float4 v = y[0][u];
+    if (p.post) {
+      const float4 w = *reinterpret_cast<const float4*>(p.post + c);
+      v = make_float4(v.x * inv[u] * w.x, v.y * inv[u] * w.y, v.z * inv[u] * w.z, v.w * inv[u] * w.w);
+    }
+    x[u] = make_float4(v.x + x[u].x, v.y + x[u].y, v.z + x[u].z, v.w + x[u].w);
+    if (p.x_out) *reinterpret_cast<float4*>(p.x_out + (size_t)m * p.ld + c) = x[u];
+  }
+  squares(x, stat[3]);
+  __syncthreads();
+  factors(stat[3], inv);
+#pragma unroll
+  for (int u = 0; u < Q; ++u) {
+    if (u * NW + warp >= runs) break;
+    const int c = (u * NW + warp) * 128 + lane * 4;
+    const float4 w = *reinterpret_cast<const float4*>(p.next + c);
+    const float4 v = make_float4(x[u].x * inv[u] * w.x, x[u].y * inv[u] * w.y, x[u].z * inv[u] * w.z, x[u].w * inv[u] * w.w);
+    const size_t at = ((size_t)m * p.ld + c) / 4;
+    if (p.h_f32) reinterpret_cast<float4*>(p.h)[at] = v;
+    else reinterpret_cast<uint2*>(p.h)[at] = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+  }
+}
+
+int launch_kernel(void (*kernel)(SandwichParams), const SandwichParams& p, int cs, int threads, size_t smem, cudaStream_t st) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(p.M * cs);
+  cfg.blockDim = dim3(threads);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = st;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = cs;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  static const bool no_pdl = getenv("B2_NO_PDL") != nullptr;  // measurement switch, as in b2_launch
+  cfg.numAttrs = no_pdl ? 1 : 2;
+  return (int)cudaLaunchKernelEx(&cfg, kernel, p);
+}
+
+template <bool TWO>
+int launch_runs(const SandwichParams& p, cudaStream_t st) {
+  // measured: threads and values in flight that fill the SMs with many rows, and the shortest chain for few
+  if (p.M > 64) {
+    if (p.ld <= 1024) return launch_kernel(sandwich_runs_kernel<TWO, 128, 2, 2, 8>, p, 1, 128, 0, st);
+    if (p.ld <= 2048) return launch_kernel(sandwich_runs_kernel<TWO, 128, 4, 2, 8>, p, 1, 128, 0, st);
+    if (p.ld <= 4096) return launch_kernel(sandwich_runs_kernel<TWO, 256, 4, 4, 4>, p, 1, 256, 0, st);
+    return launch_kernel(sandwich_runs_kernel<TWO, 256, 8, 4, 1>, p, 1, 256, 0, st);
+  }
+  if (p.ld <= 1024) return launch_kernel(sandwich_runs_kernel<TWO, 256, 1, 4, 4>, p, 1, 256, 0, st);
+  if (p.ld <= 2048) return launch_kernel(sandwich_runs_kernel<TWO, 512, 1, 4, 2>, p, 1, 512, 0, st);
+  if (p.ld <= 4096) return launch_kernel(sandwich_runs_kernel<TWO, 1024, 1, 4, 1>, p, 1, 1024, 0, st);
+  return launch_kernel(sandwich_runs_kernel<TWO, 1024, 2, 4, 1>, p, 1, 1024, 0, st);
+}
+
 template <int CS, bool TWO>
 int launch_form(const SandwichParams& p, cudaStream_t st) {
+  if (p.width == p.ld && p.size % 128 == 0 && p.ld <= 128 * kRuns) return launch_runs<TWO>(p, st);
   const int per = ((p.ld / 4 + CS - 1) / CS) * 4;
   const size_t smem = ((size_t)(TWO ? 2 : 1) * per + 4 * p.groups) * sizeof(float);
   if (smem > 200 * 1024) return -5;
@@ -250,21 +430,7 @@ int launch_form(const SandwichParams& p, cudaStream_t st) {
     cudaError_t e = cudaFuncSetAttribute(sandwich_kernel<CS, TWO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3(p.M * CS);
-  cfg.blockDim = dim3(kThreads);
-  cfg.dynamicSmemBytes = smem;
-  cfg.stream = st;
-  cudaLaunchAttribute attr[2];
-  attr[0].id = cudaLaunchAttributeClusterDimension;
-  attr[0].val.clusterDim.x = CS;
-  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
-  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  attr[1].val.programmaticStreamSerializationAllowed = 1;
-  cfg.attrs = attr;
-  static const bool no_pdl = getenv("B2_NO_PDL") != nullptr;  // measurement switch, as in b2_launch
-  cfg.numAttrs = no_pdl ? 1 : 2;
-  return (int)cudaLaunchKernelEx(&cfg, sandwich_kernel<CS, TWO>, p);
+  return launch_kernel(sandwich_kernel<CS, TWO>, p, CS, kThreads, smem, st);
 }
 
 template <int CS>

@@ -21,7 +21,9 @@ def source(y, row_elems: int, *, slices: int = 1, slice_elems: int = 0, slots: i
     row is the sum of its slots weighted by ``slot_w`` (slot ``s`` of row ``i``: value row ``row_of[i * slots + s]``, or
     ``i * slots + s``), times ``factor``; ``norm``: weight of an RMS norm ahead of the factor (two sources only)."""
     ptr = lambda t: 0 if t is None else t.data_ptr()        # noqa: E731
-    return _Source(ptr(y), ptr(row_of), ptr(slot_w), slice_elems, row_elems, slots, slices, int(y.dtype == torch.bfloat16), factor, ptr(norm))
+    s = _Source(ptr(y), ptr(row_of), ptr(slot_w), slice_elems, row_elems, slots, slices, int(y.dtype == torch.bfloat16), factor, ptr(norm))
+    s.tensors = (y, row_of, slot_w, norm)       # alive as long as the source
+    return s
 
 
 def boundary(sources, *, m: int, width: int, groups: int, eps: float, post, next, x_in, x_out, h, vocab: int = 0, flag=None):

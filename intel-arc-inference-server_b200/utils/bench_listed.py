@@ -11,7 +11,7 @@ import dataclasses
 import torch
 
 from ..models.config import (DenseFfn, GroupedAttention, LayerSpec, MatrixLstm, ModelConfig, listed_config, pefulorn_like,
-                             preset)
+                             preset, vogerax_like)
 from ..models.weights import random_weights
 from ..ops import lib as K
 from ..runtime.engine import Engine
@@ -70,7 +70,22 @@ def pefulorn_sizes():
     return out
 
 
-SIZES = {"mumusun": mumusun_sizes, "napadra": napadra_sizes, "pefulorn": pefulorn_sizes}
+def vogerax_sizes():
+    """(windowed attention with pooled blocks, gated attention beside retention and ungated experts; grouped-query mixture of
+    experts) pairs: the same width, layers, query and key heads, window, experts, experts per token and weights per expert (two
+    matrices here, three there); every fourth layer sees the whole context."""
+    out = []
+    for cfg in (preset("vogerax-16b"), vogerax_like("vogerax-2b", 1024, 24, 8, 2, 768, 32, 4, 65536, 1024),
+                vogerax_like("vogerax-wide-12l", 4096, 12, 32, 8, 1536, 64, 6, 102400)):
+        a, f = cfg.layer_specs[0].mixer, cfg.layer_specs[0].ffn
+        ff = f.ff * 2 // 3 // 64 * 64
+        out.append((cfg, ModelConfig(f"gqa-moe-like-{cfg.name}", cfg.n_layers, cfg.hidden, a.heads, a.kv_heads, 128, 0, cfg.vocab,
+                                     n_experts=f.experts, top_k=f.top, expert_ffn=ff, shared_ffn=2 * ff, sliding_window=a.window,
+                                     full_attn_every=4, architecture="B200MoeForCausalLM")))
+    return out
+
+
+SIZES = {"mumusun": mumusun_sizes, "napadra": napadra_sizes, "pefulorn": pefulorn_sizes, "vogerax": vogerax_sizes}
 
 
 def _timed(fn, warm: int, reps: int) -> float:

@@ -110,8 +110,11 @@ def attention(w, p, m, eps, h):
     t, pos = len(h), torch.arange(len(h))
     q, k = ((h @ w[p + n].T).reshape(t, c, -1) for n, c in (("q", m["heads"]), ("k", m["kv_heads"])))
     freq, amp = rotation(m["rot"])
-    o = pooled_window_attend(rotate(q, pos, freq, amp), rotate(k, pos, freq, amp), k, pos, m["mask"]["size"], m["mask"]["pool"],
-                             m["scale"])
+    mask, qr, kr = m.get("mask"), rotate(q, pos, freq, amp), rotate(k, pos, freq, amp)
+    if mask and mask.get("pool"):
+        o = pooled_window_attend(qr, kr, k, pos, mask["size"], mask["pool"], m["scale"])
+    else:
+        o = attend(qr, kr, k, window_and_blocks(pos, t, mask["size"], t)[0] if mask else causal(pos, t), m["scale"])
     return o.reshape(t, -1) @ w[p + "o"].T
 
 
