@@ -172,8 +172,8 @@ class Assembler:
 
     def gate_up(self, p: str, ffp: int, gated: bool = True, lo: int = 0) -> torch.Tensor:
         """What a feed-forward's hidden columns ``lo`` .. are made with."""
-        up = self.padded(self.t(p + "up")[lo: lo + ffp], ffp, self.wp)
-        return interleave16(self.padded(self.t(p + "gate")[lo: lo + ffp], ffp, self.wp), up) if gated else up
+        gate, up = (self.padded(self.t(p + n)[lo: lo + ffp], ffp, self.wp) if n == "up" or gated else None for n in ("gate", "up"))
+        return interleave16(gate, up) if gated else up
 
     def down(self, p: str, ffp: int, lo: int = 0) -> torch.Tensor:
         return self.padded(self.t(p + "down")[:, lo: lo + ffp], self.wp, ffp)
